@@ -45,6 +45,7 @@ class BlockPhase(C.Structure):
     ]
 
 
+ACT_SILU, ACT_GELU_TANH = 0, 1
 PHASE_GEMM, PHASE_GEMM_SILU_MUL, PHASE_ADD_RMSNORM, PHASE_QKV_ROPE_STORE = 1, 2, 3, 4
 
 # name -> (restype, argtypes); must list every symbol include/fk_b200.h declares
@@ -108,9 +109,38 @@ PROTOTYPES = {
                                      _vp, _vp]),
     "fk_decode_block_workspace_bytes": (_sz, [_i64]),
     "fk_decode_block": (_i32, [C.POINTER(BlockPhase), _i32, _i64, _vp, _sz, _vp, _vp]),
+    "fk_embed_f32": (_i32, [_vp, _i32, _i64, _vp, _vp, _i64, _i32, _vp, _vp]),
+    "fk_norm_shift": (_i32, [_vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _i32, _vp, _i32, _vp, _vp,
+                             _vp, _i32, _i64, _i32, _i32, _f32, _vp, _vp]),
+    "fk_branch_combine": (_i32, [_vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _i32, _i64, _i32,
+                                 _i32, _f32, _vp]),
+    "fk_rope_rms_store": (_i32, [_vp, _vp, _i64, _i32, _vp, _vp, _vp, _vp, _i64, _vp, _vp, _i64,
+                                 _i32, _i32, _i32, _i32, _i32, _i32, _f32, _i64, _vp, _vp]),
+    "fk_act_and_mul": (_i32, [_vp, _i64, _vp, _i64, _i32, _i64, _i64, _i32, _vp]),
+    "fk_gemm_bf16_act_mul": (_i32, [_vp, _i64, _vp, _vp, _vp, _i64, _i64, _i64, _i64, _i32, _vp,
+                                    _sz, _vp, _vp]),
+    "fk_delta_padded_dim": (_i32, [_i32]),
+    "fk_delta_prepare": (_i32, [_vp, _vp, _vp, _vp, _vp, _i64, _i32, _vp, _i64, _vp, _vp, _vp,
+                                _i64, _i32, _i32, _i32, _f32, _f32, _vp]),
+    "fk_delta_scan": (_i32, [_vp, _vp, _vp, _i32, _vp, _i32, _vp, _vp, _i64, _i32, _i32, _vp,
+                             _vp]),
+    "fk_delta_output": (_i32, [_vp, _vp, _i64, _vp, _vp, _i64, _i32, _i64, _i32, _i32, _f32,
+                               _vp]),
+    "fk_gemm_f32": (_i32, [_vp, _i64, _vp, _vp, _i64, _i64, _i64, _i64, _vp]),
+    "fk_paged_attn_any": (_i32, [_vp, _i64, _vp, _i64, _vp, _vp, _i32, _i64, _i32, _vp, _vp, _vp,
+                                 _i64, _i32, _i64, _i32, _i32, _i32, _f32, _vp, _vp]),
+    "fk_argmax_f32": (_i32, [_vp, _i64, _i64, _i64, _vp, _vp, _vp]),
     "fk_gemm_bf16_static": (_i32, [_vp, _i64, _vp, _vp, _vp, _i64, _i64, _i64, _i64, _vp, _vp]),
     "fk_gemm_bf16": (_i32, [_vp, _i64, _vp, _vp, _vp, _i64, _i64, _i64, _i64, _vp, _sz,
                             _vp, _vp]),
+}
+
+
+# Parts of the library that a partial build may leave out (build.COMPONENT_SOURCES),
+# by the symbols they export; a part is there with all of them or not at all.
+COMPONENTS = {
+    "comm": [n for n in PROTOTYPES if n.startswith(("fk_comm_", "fk_allreduce_"))],
+    "block": ["fk_decode_block_workspace_bytes", "fk_decode_block"],
 }
 
 
@@ -124,7 +154,10 @@ def _load() -> C.CDLL:
             f"{LIB_PATH} not found: build it with `python -m fastkernels_b200.build` "
             "(there is no CPU or library fallback)")
     lib = C.CDLL(str(LIB_PATH))
+    absent = {n for names in COMPONENTS.values() if not hasattr(lib, names[0]) for n in names}
     for name, (res, args) in PROTOTYPES.items():
+        if name in absent:      # left out of this build: AttributeError when it is called
+            continue
         fn = getattr(lib, name)  # AttributeError if the symbol is missing
         fn.restype = res
         fn.argtypes = args

@@ -19,9 +19,13 @@ from pathlib import Path
 PKG = Path(__file__).resolve().parent
 CSRC = PKG / "csrc"
 LIB = PKG / "libfk_b200.so"
-SOURCES = ["fk_host.cu", "fk_elementwise.cu", "fk_attn.cu", "fk_gemm.cu", "fk_comm.cu",
-           "fk_prefill.cu", "fk_gemm_large.cu", "fk_block.cu"]
+# what every model needs, and the parts only some runs do (see _lib.COMPONENTS)
+CORE_SOURCES = ["fk_host.cu", "fk_elementwise.cu", "fk_attn.cu", "fk_gemm.cu", "fk_prefill.cu",
+                "fk_gemm_large.cu", "fk_mixer.cu", "fk_delta.cu", "fk_plain.cu"]
+COMPONENT_SOURCES = {"comm": ["fk_comm.cu"], "block": ["fk_block.cu"]}
+SOURCES = CORE_SOURCES + [s for c in COMPONENT_SOURCES.values() for s in c]
 HEADERS = [CSRC / "fk_common.cuh", CSRC / "fk_tcgen05.cuh", CSRC / "fk_rowops.cuh",
+           CSRC / "fk_types.cuh",
            CSRC / "fk_gemm_shared.cuh", PKG.parent / "include" / "fk_b200.h"]
 
 NVCC_FLAGS = [
@@ -57,12 +61,18 @@ def _compile(src: Path, obj: Path, verbose: bool, defines=()) -> str:
     return r.stdout + r.stderr
 
 
-def build(force: bool = False, verbose: bool = False, defines=(), out: Path | None = None) -> Path:
+def build(force: bool = False, verbose: bool = False, defines=(), out: Path | None = None,
+          components=None) -> Path:
     """Default: the library proper, objects next to the sources.  With `defines`
     (e.g. FK_GEMM_TRACE, FK_BLOCK_TRACE: per-CTA time stamps for
     `microbench timeline`) a diagnostic copy is built into `out`'s directory and
-    loaded by setting FK_B200_LIB to it."""
-    srcs = [CSRC / s for s in SOURCES if (CSRC / s).exists()]
+    loaded by setting FK_B200_LIB to it.  `components` limits a first build to the core
+    and the named parts; parts that are built already stay in the library."""
+    names = list(SOURCES)
+    if components is not None:
+        names = CORE_SOURCES + [s for c, ss in COMPONENT_SOURCES.items() for s in ss
+                                if c in components or (CSRC / s).with_suffix(".o").exists()]
+    srcs = [CSRC / s for s in names if (CSRC / s).exists()]
     lib = LIB
     if defines or out is not None:
         lib = Path(out) if out is not None else PKG.parent / "build" / "libfk_b200_diag.so"

@@ -137,6 +137,25 @@ __device__ __forceinline__ uint32_t silu_mul2(uint32_t g, uint32_t u) {
   return pack_bf16(a0 * bf16lo(u), a1 * bf16hi(u));
 }
 
+// Tanh-form GELU, 0.5 g (1 + tanh(a)) = g sigmoid(2 a) with
+// a = sqrt(2 / pi) (g + 0.044715 g^3).
+__device__ __forceinline__ float gelu_tanh_arg(float g) {
+  return 1.5957691216057308f * (g + 0.044715f * g * g * g);   // 2 a
+}
+__device__ __forceinline__ float gelu_tanh_f32(float g) {
+  return g / (1.0f + expf(-gelu_tanh_arg(g)));
+}
+// The same on packed bf16 pairs times `u`, rounded once at the end.
+__device__ __forceinline__ uint32_t gelu_mul2(uint32_t g, uint32_t u) {
+  const float g0 = bf16lo(g), g1 = bf16hi(g);
+  const float a0 = __fdividef(g0, 1.0f + __expf(-gelu_tanh_arg(g0)));
+  const float a1 = __fdividef(g1, 1.0f + __expf(-gelu_tanh_arg(g1)));
+  return pack_bf16(a0 * bf16lo(u), a1 * bf16hi(u));
+}
+__device__ __forceinline__ uint32_t act_mul2(uint32_t g, uint32_t u, int act) {
+  return act == FK_ACT_GELU_TANH ? gelu_mul2(g, u) : silu_mul2(g, u);
+}
+
 // No-ops when the kernel was launched without the programmatic attribute.
 __device__ __forceinline__ void pdl_launch_dependents() {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");

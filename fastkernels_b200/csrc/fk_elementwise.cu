@@ -8,6 +8,7 @@
 // the order of the fp32 row reduction.
 #include "fk_common.cuh"
 #include "fk_rowops.cuh"
+#include "fk_types.cuh"
 
 namespace fk {
 
@@ -386,17 +387,18 @@ __device__ __forceinline__ void amax_take(float& bv, int64_t& bi, float v,
   if (v > bv || (v == bv && i < bi)) { bv = v; bi = i; }
 }
 
+template <typename T>
 __global__ void __launch_bounds__(1024) argmax_rows_kernel(
-    const uint16_t* __restrict__ x, int64_t x_stride, int64_t cols,
+    const T* __restrict__ x, int64_t x_stride, int64_t cols,
     float* __restrict__ out_val, int64_t* __restrict__ out_idx) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float sv[32];
   __shared__ int64_t si[32];
-  const uint16_t* row = x + (int64_t)blockIdx.x * x_stride;
+  const T* row = x + (int64_t)blockIdx.x * x_stride;
   float bv = -INFINITY;
   int64_t bi = 0x7fffffffffffffffll;
-  const bool vec = (cols % 8 == 0) && (x_stride % 8 == 0) &&
+  const bool vec = sizeof(T) == 2 && (cols % 8 == 0) && (x_stride % 8 == 0) &&
                    ((reinterpret_cast<uintptr_t>(x) & 15u) == 0);
   if (vec) {
     const uint4* r4 = reinterpret_cast<const uint4*>(row);
@@ -411,7 +413,7 @@ __global__ void __launch_bounds__(1024) argmax_rows_kernel(
     }
   } else {
     for (int64_t c = threadIdx.x; c < cols; c += blockDim.x)
-      amax_take(bv, bi, bf16_bits_to_float(row[c]), c);
+      amax_take(bv, bi, Elem<T>::load(row + c), c);
   }
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) {
@@ -846,8 +848,23 @@ int fk_argmax_bf16(const void* x, int64_t x_stride, int64_t rows, int64_t cols,
   FK_REQUIRE(x && out_idx, FK_ERR_INVALID_ARG, "fk_argmax_bf16: null pointer");
   FK_REQUIRE(x_stride >= cols && rows < (1ll << 31), FK_ERR_INVALID_ARG,
              "fk_argmax_bf16: bad stride or row count");
-  FK_LAUNCH((argmax_rows_kernel), dim3((int)rows), dim3(1024), 0, static_cast<cudaStream_t>(stream), 
-      (const uint16_t*)x, x_stride, cols, out_val, out_idx);
+  FK_LAUNCH((argmax_rows_kernel<uint16_t>), dim3((int)rows), dim3(1024), 0,
+            static_cast<cudaStream_t>(stream), (const uint16_t*)x, x_stride, cols, out_val,
+            out_idx);
+  count_launch();
+  FK_CUDA_OK(cudaGetLastError());
+  return FK_OK;
+}
+
+int fk_argmax_f32(const float* x, int64_t x_stride, int64_t rows, int64_t cols,
+                  float* out_val, int64_t* out_idx, fk_stream_t stream) {
+  FK_REQUIRE(rows >= 0 && cols > 0, FK_ERR_INVALID_ARG, "fk_argmax_f32: bad sizes");
+  if (rows == 0) return FK_OK;
+  FK_REQUIRE(x && out_idx, FK_ERR_INVALID_ARG, "fk_argmax_f32: null pointer");
+  FK_REQUIRE(x_stride >= cols && rows < (1ll << 31), FK_ERR_INVALID_ARG,
+             "fk_argmax_f32: bad stride or row count");
+  FK_LAUNCH((argmax_rows_kernel<float>), dim3((int)rows), dim3(1024), 0,
+            static_cast<cudaStream_t>(stream), x, x_stride, cols, out_val, out_idx);
   count_launch();
   FK_CUDA_OK(cudaGetLastError());
   return FK_OK;

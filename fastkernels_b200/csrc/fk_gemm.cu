@@ -70,6 +70,7 @@ struct GemmParams {
   int num_ctas;
   int splits, kb_per_split;  // cluster mode: k-blocks per CTA of a cluster
   int half_n;              // SILU: rows of the gate block (= rows of the up block)
+  int act;                 // SILU: FK_ACT_SILU or FK_ACT_GELU_TANH
   float* part;             // [GEMM_MAX_CTAS][MPAD][128] fp32 partial tiles
   int* flags;              // [GEMM_MAX_CTAS], zero when idle
   int32_t* status;
@@ -469,8 +470,8 @@ __global__ void __launch_bounds__(GEMM_THREADS, 1) gemm_bf16_kernel(
               const uint4 g = *reinterpret_cast<const uint4*>(st + r * GEMM_BN + ch * 8);
               const uint4 u = *reinterpret_cast<const uint4*>(st + r * GEMM_BN + 64 + ch * 8);
               uint4 o;
-              o.x = silu_mul2(g.x, u.x); o.y = silu_mul2(g.y, u.y);
-              o.z = silu_mul2(g.z, u.z); o.w = silu_mul2(g.w, u.w);
+              o.x = act_mul2(g.x, u.x, p.act); o.y = act_mul2(g.y, u.y, p.act);
+              o.z = act_mul2(g.z, u.z, p.act); o.w = act_mul2(g.w, u.w, p.act);
               uint16_t* yrow = p.y + (int64_t)(c + r) * p.y_stride + n0 + ch * 8;
               if (vec_store) {
                 *reinterpret_cast<uint4*>(yrow) = o;
@@ -1008,10 +1009,12 @@ int fk_gemm_bf16_silu_mul_fusable(int64_t m, int64_t n, int64_t k) {
   return plan_gemm(mpad_for(m), n_tiles, (int)(k / GEMM_BK)).splits == 0 ? 1 : 0;
 }
 
-int fk_gemm_bf16_silu_mul(const void* x, int64_t x_stride, const void* w,
-                          const void* bias, void* y, int64_t y_stride, int64_t m,
-                          int64_t n, int64_t k, void* workspace,
-                          size_t workspace_bytes, int32_t* status, fk_stream_t stream) {
+int fk_gemm_bf16_act_mul(const void* x, int64_t x_stride, const void* w,
+                         const void* bias, void* y, int64_t y_stride, int64_t m,
+                         int64_t n, int64_t k, int act, void* workspace,
+                         size_t workspace_bytes, int32_t* status, fk_stream_t stream) {
+  FK_REQUIRE(act == FK_ACT_SILU || act == FK_ACT_GELU_TANH, FK_ERR_INVALID_ARG,
+             "fk_gemm_bf16_act_mul: unknown activation %d", act);
   FK_REQUIRE(m >= 0 && n >= 0 && k > 0, FK_ERR_INVALID_ARG, "fk_gemm_bf16_silu_mul: bad sizes");
   if (m == 0 || n == 0) return FK_OK;
   FK_REQUIRE(x && w && y, FK_ERR_INVALID_ARG, "fk_gemm_bf16_silu_mul: null pointer");
@@ -1043,6 +1046,7 @@ int fk_gemm_bf16_silu_mul(const void* x, int64_t x_stride, const void* w,
   p.y = (uint16_t*)y; p.y_stride = y_stride;
   p.m = (int)m; p.n = (int)n; p.k = (int)k;
   p.half_n = (int)half;
+  p.act = act;
   p.n_tiles = (int)(half / 64); p.kb_total = (int)(k / GEMM_BK);
   const GemmPlan plan = plan_gemm(mpad, p.n_tiles, p.kb_total);   // stream-K (checked above)
   p.splits = 0; p.kb_per_split = 0; p.num_ctas = plan.num_ctas;
@@ -1057,6 +1061,14 @@ int fk_gemm_bf16_silu_mul(const void* x, int64_t x_stride, const void* w,
     case 128: return launch_gemm<128>(mw, mx, p, s);
     default: return launch_gemm<256>(mw, mx, p, s);
   }
+}
+
+int fk_gemm_bf16_silu_mul(const void* x, int64_t x_stride, const void* w,
+                          const void* bias, void* y, int64_t y_stride, int64_t m,
+                          int64_t n, int64_t k, void* workspace,
+                          size_t workspace_bytes, int32_t* status, fk_stream_t stream) {
+  return fk_gemm_bf16_act_mul(x, x_stride, w, bias, y, y_stride, m, n, k, FK_ACT_SILU,
+                              workspace, workspace_bytes, status, stream);
 }
 
 #ifdef FK_GEMM_TRACE

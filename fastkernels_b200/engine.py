@@ -1,5 +1,6 @@
-"""Decode-step engine: paged KV pool, block manager, CUDA-graph decode, greedy
-sampling, tensor parallelism (one process per GPU, NCCL).
+"""Serving engine: paged KV pools, recurrent-state slots, prefill in portions,
+CUDA-graph decode, greedy sampling, tensor parallelism (one process per GPU, NCCL).
+The model behind it is chosen by its configuration (models.registry).
 
 Mirror of the decode path of the reference engine (fastkernels/infra/engine.py):
   BlockManager.maybe_append_pages            engine.py:530-537
@@ -9,10 +10,11 @@ Mirror of the decode path of the reference engine (fastkernels/infra/engine.py):
   ModelRunner.capture_cudagraph              engine.py:6701-7025  (graph body, graph_vars)
   ModelRunner._greedy_from_hidden            engine.py:5711-5746  (argmax, tp all-gather)
 plus the prefill side of ModelRunner.run (engine.py:4902-4990, 6048-6063): whole
-or chunked prompts fill their KV pages and join the running batch.  Scheduling
-of mixed prefill + decode batches, HTTP serving and checkpoint loading are
-outside this build; sequences may also enter with their context already in the
-cache (synthetic contexts for the benchmark, or whatever the caller wrote).
+or chunked prompts fill their KV pages and join the running batch.  `feed` runs
+given tokens of any mix of sequences (portions of prompts and single tokens) and
+returns logits.  HTTP serving is outside this build; sequences may also enter with
+their context already in the cache (synthetic contexts for the benchmark, or
+whatever the caller wrote).
 
 Every rank of a tensor-parallel group runs this same host code on the same
 inputs (deterministic scheduling), so no control-plane exchange is needed; the
@@ -23,92 +25,34 @@ all captured in the CUDA graph.
 from __future__ import annotations
 
 import os
-from dataclasses import dataclass, field
 
 import numpy as np
 import torch
 
 from . import ops
-from .candidate.L4.llama import LlamaConfig, LlamaForCausalLM
-from .infra.context import get_context, reset_context, set_context
+from .cache import BlockManager, Sequence, StateSlots, pack_prefill_chunk
+from .infra.context import SpanBatch, get_context, reset_context, set_context
 from .infra.tp import _tp_rank, _tp_size
+from .models.registry import load_folder, model_class
 
 # FK_B200_PREPARE_AHEAD=0: stage every step's host arrays only when the step is
 # called (for A/B timing of the look-ahead in DecodeEngine.step)
 _NO_PREPARE_AHEAD = os.environ.get("FK_B200_PREPARE_AHEAD", "1") == "0"
 
 
-@dataclass
-class Sequence:
-    """One running request: `num_tokens` counts the tokens whose K/V are (or, for
-    the newest one, are about to be) in the cache; `block_table` lists its pages."""
-    seq_id: int
-    num_tokens: int
-    block_table: list[int] = field(default_factory=list)
-    last_token: int = 0
-    output: list[int] = field(default_factory=list)
-
-
-def pack_prefill_chunk(prompt_lens, done, budget):
-    """Next prefill forward: walk the sequences in order and take as many of each
-    one's remaining prompt tokens as the token budget allows (None = no limit).
-    Returns [(sequence index, first token, count)]; every sequence appears at most
-    once, so a forward holds at most one chunk per sequence."""
-    left = budget if budget is not None else 1 << 62
-    part = []
-    for i, n in enumerate(prompt_lens):
-        take = min(n - done[i], left)
-        if take > 0:
-            part.append((i, done[i], take))
-            left -= take
-        if left == 0:
-            break
-    return part
-
-
-class BlockManager:
-    """Free-list page allocator (decode subset of engine.py:380-586)."""
-
-    def __init__(self, num_blocks: int, block_size: int):
-        self.block_size = block_size
-        self.free = list(range(num_blocks - 1, -1, -1))
-
-    def allocate(self, seq: Sequence) -> None:
-        need = (seq.num_tokens + self.block_size - 1) // self.block_size
-        while len(seq.block_table) < need:
-            seq.block_table.append(self._pop())
-
-    def maybe_append_page(self, seq: Sequence) -> bool:
-        """Called with num_tokens INCLUDING the token sampled last step: a new
-        page is needed when that token is the first of a page (engine.py:530-533)."""
-        if seq.num_tokens % self.block_size == 1 and \
-                len(seq.block_table) * self.block_size < seq.num_tokens:
-            seq.block_table.append(self._pop())
-            return True
-        return False
-
-    def _pop(self) -> int:
-        if not self.free:
-            raise RuntimeError("KV pool exhausted")
-        return self.free.pop()
-
-    def release(self, seq: Sequence) -> None:
-        self.free.extend(reversed(seq.block_table))
-        seq.block_table.clear()
-
-
 class DecodeEngine:
-    def __init__(self, config: LlamaConfig, *, max_num_seqs: int, max_model_len: int,
-                 num_kv_blocks: int, device="cuda", seed: int = 0,
-                 enforce_eager: bool = False, init_scale: float = 0.02,
+    def __init__(self, config, *, max_num_seqs: int, max_model_len: int,
+                 num_kv_blocks: int | list[int], device="cuda", seed: int = 0,
+                 enforce_eager: bool = False, init_scale: float | None = 0.02,
                  attn_max_splits: int | None = None):
+        """num_kv_blocks: pages of the KV pool, one number for every span of the model
+        or one per span.  init_scale None leaves the weights for load_weights."""
         self.config = config
         self.device = torch.device(device)
         self.tp, self.rank = _tp_size(), _tp_rank()
         self.block_size = config.kv_block_size
         self.max_num_seqs = max_num_seqs
         self.max_model_len = max_model_len
-        self.max_num_blocks = (max_model_len + self.block_size - 1) // self.block_size
         self.enforce_eager = enforce_eager
         self.h2d_bytes = 0
         self.d2h_bytes = 0
@@ -117,14 +61,14 @@ class DecodeEngine:
         torch.set_default_dtype(config.dtype)
         try:
             with torch.device(self.device):
-                self.model = LlamaForCausalLM(config)
+                self.model = model_class(config)(config)
         finally:
             torch.set_default_dtype(prev)
-        self.init_random_weights(seed, init_scale)
+        if init_scale is not None:
+            self.init_random_weights(seed, init_scale)
         if attn_max_splits is None:
             attn_max_splits = ops.max_splits_for(max_model_len)
-        for layer in self.model.model.layers:
-            layer.self_attn.attn.decode_op._max_splits = attn_max_splits
+        self._attn_max_splits = attn_max_splits
 
         # tensor parallel: fused all-reduce + add + RMSNorm over peer memory unless
         # FK_B200_NCCL_ALLREDUCE=1 asks for the plain NCCL path
@@ -137,118 +81,116 @@ class DecodeEngine:
             if max_num_seqs > 512:
                 raise ValueError("tensor-parallel decode batches are limited to 512 sequences "
                                  "by the fused all-reduce (set FK_B200_NCCL_ALLREDUCE=1 for more)")
-            self.comm = TpComm(512, config.hidden_size, self.device)
+            self.comm = TpComm(512, self.model.hidden_columns, self.device)
             algo = os.environ.get("FK_B200_ALLREDUCE_ALGO", "auto")
             if algo not in ("auto", "one_stage", "two_stage", "push"):
                 raise ValueError("FK_B200_ALLREDUCE_ALGO must be auto, one_stage, two_stage "
                                  "or push")
             self.comm.algo = algo
             set_tp_comm(self.comm)
-        self.allocate_kv_cache(num_kv_blocks)
-        self.blocks = BlockManager(num_kv_blocks, self.block_size)
+        spans = self.model.kv_spans
+        per_span = list(num_kv_blocks) if isinstance(num_kv_blocks, (list, tuple)) \
+            else [num_kv_blocks] * len(spans)
+        self.span_blocks = [BlockManager(nb, self.block_size, g, chunk)
+                            for g, (nb, chunk) in enumerate(zip(per_span, spans))]
+        self.blocks = self.span_blocks[0]
+        self.max_num_blocks = [b.max_blocks(max_model_len) for b in self.span_blocks]
+        self.allocate_kv_cache(per_span)
+        self.state_slots = StateSlots(max_num_seqs) if self.model.uses_state else None
+        if self.state_slots is not None:
+            self.model.allocate_state(max_num_seqs, self.device)
         self.seqs: list[Sequence] = []
+        self._next_id = 0
         self._init_buffers()
         self.graphs: dict[int, torch.cuda.CUDAGraph] = {}
         self.graph_pool = None
         self._bt_dirty = True
+        self._staged_for = None     # ids of the sequences the device tables belong to
+
+    @classmethod
+    def from_folder(cls, folder, dtype=torch.bfloat16, **kw):
+        """Engine for the model in a folder (config.json, safetensors)."""
+        config, source = load_folder(folder, dtype)
+        eng = cls(config, init_scale=None, **kw)
+        eng.load_weights(source)
+        return eng
 
     # ------------------------------------------------------------------ weights
-    @torch.no_grad()
     def init_random_weights(self, seed: int, scale: float) -> None:
-        """Random-init every parameter (randn * scale; norm weights 1.0).  Shards
-        are drawn per rank: statistically the same model at every tp degree."""
-        g = torch.Generator(device=self.device).manual_seed(seed * 1000003 + self.rank)
-        for name, p in self.model.named_parameters():
-            if "norm" in name or "layernorm" in name:
-                p.fill_(1.0)
-            else:
-                p.normal_(0.0, scale, generator=g)
+        self.model.init_random(seed, scale, self.rank)
 
     @torch.no_grad()
+    def load_weights(self, source) -> None:
+        """Weights from a models.weights.TensorSource."""
+        self.model.load_tensors(source)
+
     def load_full_weights(self, w: dict) -> None:
-        """Load UNSHARDED weights (dict of tensors in the layout of
-        tests/cases.py:decoder_weights) through each parameter's weight_loader,
-        which takes this rank's shard exactly as the reference loaders do."""
-        m, c = self.model, self.config
-        dev = self.device
-
-        def t(a):
-            return torch.as_tensor(a).to(device=dev, dtype=c.dtype)
-
-        emb = m.model.embed_tokens.embedding_op.emb.weight
-        emb.weight_loader(emb, t(w["embed"]))
-        lm = m.lm_head.embedding_op.emb.weight
-        lm.weight_loader(lm, t(w["lm_head"]))
-        m.model.norm.weight.copy_(t(w["norm"]))
-        hq, hkv, d = c.num_attention_heads, c.num_key_value_heads, c.head_dim
-        for li, layer in enumerate(m.model.layers):
-            p = f"l{li}."
-            layer.input_layernorm.weight.copy_(t(w[p + "ln1"]))
-            layer.post_attention_layernorm.weight.copy_(t(w[p + "ln2"]))
-            qkv = t(w[p + "qkv"])
-            qp = layer.self_attn.qkv_proj.weight
-            qp.weight_loader(qp, qkv[:hq * d], "q")
-            qp.weight_loader(qp, qkv[hq * d:(hq + hkv) * d], "k")
-            qp.weight_loader(qp, qkv[(hq + hkv) * d:], "v")
-            op = layer.self_attn.o_proj.weight
-            op.weight_loader(op, t(w[p + "o"]))
-            gu = layer.mlp.gate_up_proj.weight
-            gu.weight_loader(gu, t(w[p + "gate_up"]))
-            dn = layer.mlp.down_proj.weight
-            dn.weight_loader(dn, t(w[p + "down"]))
-            if c.qk_norm:
-                layer.self_attn.q_norm.weight.copy_(t(w[p + "qn"]))
-                layer.self_attn.k_norm.weight.copy_(t(w[p + "kn"]))
+        """UNSHARDED Llama / Qwen3 weights in the merged layout of ServedLlama.load_full."""
+        self.model.load_full(w)
 
     # ----------------------------------------------------------------- KV cache
-    def allocate_kv_cache(self, num_blocks: int) -> None:
-        """Pool [2, layers, num_blocks, BLOCK, Hkv/tp, D] (NHD) or
-        [2, layers, num_blocks, Hkv/tp, BLOCK, D] (HND); every attention layer gets
-        its K and V views (engine.py:1783-1793)."""
-        c = self.config
-        hkv = max(c.num_key_value_heads // self.tp, 1)
-        self.num_kv_blocks = num_blocks
-        shape = (num_blocks, hkv, self.block_size, c.head_dim) if c.kv_layout == "HND" \
-            else (num_blocks, self.block_size, hkv, c.head_dim)
-        self.kv_cache = torch.zeros((2, c.num_hidden_layers, *shape), dtype=c.dtype,
-                                    device=self.device)
-        for li, layer in enumerate(self.model.model.layers):
-            layer.self_attn.attn.k_cache = self.kv_cache[0, li]
-            layer.self_attn.attn.v_cache = self.kv_cache[1, li]
+    def allocate_kv_cache(self, num_blocks) -> None:
+        """Page pools of all spans, installed into the attention layers; kv_cache is
+        what the model returns (one tensor [2, layers, ...] where all layers share a
+        shape)."""
+        per_span = list(num_blocks) if isinstance(num_blocks, (list, tuple)) \
+            else [num_blocks] * len(self.span_blocks)
+        self.num_kv_blocks = per_span[0]
+        self.kv_cache = self.model.allocate_kv(per_span, self.block_size, self.device)
 
     @torch.no_grad()
     def fill_kv_random(self, seed: int, scale: float = 0.5) -> None:
         """Synthetic contexts: fill the whole pool with randn * scale."""
         g = torch.Generator(device=self.device).manual_seed(seed * 7919 + self.rank)
-        for li in range(self.config.num_hidden_layers):
-            self.kv_cache[:, li].normal_(0.0, scale, generator=g)
+        pools = self.kv_cache if isinstance(self.kv_cache, (list, tuple)) \
+            else [self.kv_cache[:, li] for li in range(self.kv_cache.shape[1])]
+        for pool in pools:
+            pool.normal_(0.0, scale, generator=g)
 
     # ------------------------------------------------------------------ buffers
     def _init_buffers(self) -> None:
         n, dev, c = self.max_num_seqs, self.device, self.config
-        vocab_local = c.vocab_size // self.tp
+        nsp = len(self.span_blocks)
         # The per-step inputs live in ONE buffer, [input_ids i64 | positions i64 |
-        # slot_mapping i32 | context_lens i32], so that a step stages them with a
-        # single host-to-device copy (all four, or the last three when the token ids
-        # stay on the device).
-        def packed_views(buf):
-            return dict(input_ids=buf[:8 * n].view(torch.int64),
-                        positions=buf[8 * n:16 * n].view(torch.int64),
-                        slot_mapping=buf[16 * n:20 * n].view(torch.int32),
-                        context_lens=buf[20 * n:24 * n].view(torch.int32))
+        # (slot_mapping i32 | context_lens i32) per span | state slots i32], so that a
+        # step stages them with a single host-to-device copy (all of it, or all but the
+        # token ids when those stay on the device).
+        self._packed_bytes = n * (16 + 8 * nsp + (4 if self.state_slots is not None else 0))
 
-        self._packed_dev = torch.zeros(24 * n, dtype=torch.uint8, device=dev)
-        self._packed_dev[16 * n:20 * n].view(torch.int32).fill_(-1)   # slot_mapping: no slot
+        def packed_views(buf):
+            v = dict(input_ids=buf[:8 * n].view(torch.int64),
+                     positions=buf[8 * n:16 * n].view(torch.int64))
+            slots, lens, o = [], [], 16 * n
+            for _ in range(nsp):
+                slots.append(buf[o:o + 4 * n].view(torch.int32))
+                lens.append(buf[o + 4 * n:o + 8 * n].view(torch.int32))
+                o += 8 * n
+            v.update(slot_mapping=slots[0], context_lens=lens[0], span_slots=slots,
+                     span_lens=lens)
+            if self.state_slots is not None:
+                v["state_slots"] = buf[o:o + 4 * n].view(torch.int32)
+            return v
+
+        def clear(v):
+            for t in v["span_slots"]:
+                t.fill_(-1)                     # no slot
+            if "state_slots" in v:
+                v["state_slots"].fill_(-1)
+
+        self._packed_dev = torch.zeros(self._packed_bytes, dtype=torch.uint8, device=dev)
+        tables = [torch.full((n, cols), -1, dtype=torch.int32, device=dev)
+                  for cols in self.max_num_blocks]
         self.graph_vars = dict(
             **packed_views(self._packed_dev),
-            block_tables=torch.full((n, self.max_num_blocks), -1, dtype=torch.int32,
-                                    device=dev),
-            outputs=torch.zeros((n, c.hidden_size), dtype=c.dtype, device=dev),
-            lm_logits=torch.zeros((n, vocab_local), dtype=c.dtype, device=dev),
+            block_tables=tables[0], span_tables=tables,
+            outputs=torch.zeros((n, self.model.hidden_columns), dtype=c.dtype, device=dev),
+            lm_logits=torch.zeros((n, self.model.logit_columns), dtype=c.dtype, device=dev),
             lm_max_vals=torch.zeros(n, dtype=torch.float32, device=dev),
             lm_max_idxs=torch.zeros(n, dtype=torch.int64, device=dev),
             token_ids=torch.zeros(n, dtype=torch.int64, device=dev),
+            cu_rows=torch.arange(n + 1, dtype=torch.int32, device=dev),
         )
+        clear(self.graph_vars)
 
         def pinned(shape, dtype):
             return torch.zeros(shape, dtype=dtype).pin_memory() if dev.type == "cuda" \
@@ -261,32 +203,36 @@ class DecodeEngine:
         self.RING = 4
         self._ring = []
         for _ in range(self.RING):
-            packed = pinned(24 * n, torch.uint8)
-            packed[16 * n:20 * n].view(torch.int32).fill_(-1)   # slot_mapping: no slot
-            self._ring.append(dict(
-                **packed_views(packed), packed=packed,
-                block_tables=pinned((n, self.max_num_blocks), torch.int32),
-                token_ids=pinned(n, torch.int64)))
-        self._ring_np = [{k: v.numpy() for k, v in slot.items()} for slot in self._ring]
+            packed = pinned(self._packed_bytes, torch.uint8)
+            tables = [pinned((n, cols), torch.int32) for cols in self.max_num_blocks]
+            slot = dict(**packed_views(packed), packed=packed, block_tables=tables[0],
+                        span_tables=tables, token_ids=pinned(n, torch.int64))
+            clear(slot)
+            self._ring.append(slot)
+        self._ring_np = [{k: [t.numpy() for t in v] if isinstance(v, list) else v.numpy()
+                          for k, v in slot.items()} for slot in self._ring]
         self._ring_events = [None] * self.RING
         self._ring_pos = 0
         # (sequence-set version, count) the staging slot was prepared ahead for, or None
         self._ahead = None
         self._seq_epoch = 0
         self.host, self.host_np = self._ring[0], self._ring_np[0]
-        # one split-KV workspace serves every layer (they run back to back on
-        # one stream)
-        first = self.model.model.layers[0].self_attn.attn.decode_op
-        first.preallocate(n, dev)
-        ws_attr = "_fk_workspace" if hasattr(first, "_fk_workspace") else "_workspace"
-        for layer in self.model.model.layers[1:]:
-            op = layer.self_attn.attn.decode_op
-            setattr(op, ws_attr, getattr(first, ws_attr))
-            op._ws_batch, op._status = first._ws_batch, first._status
-        self.attn_workspace = getattr(first, ws_attr)
-        self.status = first._status
+        self.status = self.model.preallocate(n, self.max_model_len, dev, self._attn_max_splits)
+        self.attn_workspace = getattr(self.model, "attn_workspace", None)
 
     # ---------------------------------------------------------------- sequences
+    def _new_sequence(self, num_tokens: int, last_token: int = 0) -> Sequence:
+        s = Sequence(self._next_id, num_tokens, last_token=last_token)
+        self._next_id += 1
+        if self.state_slots is not None:
+            self.state_slots.allocate(s)
+        return s
+
+    def _running_set_changed(self) -> None:
+        self._bt_dirty = True
+        self._seq_epoch += 1
+        self._ahead = None
+
     def add_sequences(self, context_lens, first_tokens) -> list[Sequence]:
         """Register running sequences whose first `L - 1` tokens are already in
         the cache and whose L-th token (`first_tokens[i]`) is the next input."""
@@ -296,13 +242,100 @@ class DecodeEngine:
                 raise RuntimeError("max_num_seqs exceeded")
             if L < 1 or L > self.max_model_len:
                 raise ValueError(f"context length {L} outside [1, {self.max_model_len}]")
-            s = Sequence(len(self.seqs), int(L), last_token=int(tok))
-            self.blocks.allocate(s)
+            s = self._new_sequence(int(L), int(tok))
+            for blocks in self.span_blocks:
+                blocks.allocate(s)
             self.seqs.append(s)
             out.append(s)
-        self._bt_dirty = True
-        self._seq_epoch += 1
+        self._running_set_changed()
         return out
+
+    def open_sequence(self) -> Sequence:
+        """A running sequence without tokens; they come through feed()."""
+        if len(self.seqs) >= self.max_num_seqs:
+            raise RuntimeError("max_num_seqs exceeded")
+        s = self._new_sequence(0)
+        self.seqs.append(s)
+        self._running_set_changed()
+        return s
+
+    def finish(self, seq: Sequence) -> None:
+        """End a sequence: its pages and its state slot go back."""
+        self.seqs.remove(seq)
+        for blocks in self.span_blocks:
+            blocks.release(seq)
+        if self.state_slots is not None:
+            self.state_slots.release(seq)
+        self._running_set_changed()
+
+    @torch.no_grad()
+    def _forward_portions(self, portions, use_block_tables: bool = True):
+        """Run portions [(sequence, first position, token ids)], at most one per
+        sequence, through the model; hidden rows in the order of the tokens.  Metadata
+        as in prepare_prefill (fastkernels/infra/engine.py:4902-4990): cu_seqlens,
+        per-token slots and block tables, so attention reads the pages the store has
+        just written.  In a chunked span a portion falls into one segment per chunk."""
+        dev = self.device
+        ids = np.concatenate([np.asarray(t, dtype=np.int64) for _, _, t in portions])
+        pos = np.concatenate([np.arange(a, a + len(t), dtype=np.int64) for _, a, t in portions])
+        i32 = []                           # all int32 metadata travels in one copy
+
+        def put(a):
+            a = np.ascontiguousarray(a, dtype=np.int32)
+            i32.append(a.reshape(-1))
+            return a.shape
+
+        layout = []
+        for blocks in self.span_blocks:
+            segs, slots = [], []
+            for s, a, t in portions:
+                seg, sl = blocks.extend(s, a, len(t))
+                segs += seg
+                slots.append(sl)
+            q = np.array([c for c, _, _ in segs])
+            kv = np.array([k for _, k, _ in segs])
+            bt = np.full((len(segs), max(len(pg) for _, _, pg in segs)), -1, dtype=np.int32)
+            for j, (_, _, pg) in enumerate(segs):
+                bt[j, :len(pg)] = pg
+            layout.append((put(np.concatenate(slots)), put(bt), put(kv),
+                           put(np.concatenate([[0], np.cumsum(q)])),
+                           put(np.concatenate([[0], np.cumsum(kv)])), int(q.max()),
+                           int(kv.max())))
+        state_shape = cu_shape = None
+        if self.state_slots is not None:
+            state_shape = put(np.repeat([s.state_slot for s, _, _ in portions],
+                                        [len(t) for _, _, t in portions]))
+            cu_shape = put(np.concatenate([[0], np.cumsum([len(t) for _, _, t in portions])]))
+        flat = torch.from_numpy(np.concatenate(i32)).to(dev)
+        at = 0
+
+        def take(shape):
+            nonlocal at
+            n = int(np.prod(shape))
+            v = flat[at:at + n].view(*shape)
+            at += n
+            return v
+
+        spans = []
+        for slots, bt, kv, cq, ck, max_q, max_k in layout:
+            spans.append(SpanBatch(take(slots), take(bt), take(kv), take(cq), take(ck), max_q,
+                                   max_k))
+        first = spans[0]
+        set_context(True, cu_seqlens_q=first.cu_seqlens_q, cu_seqlens_k=first.cu_seqlens_k,
+                    max_seqlen_q=first.max_seqlen_q, max_seqlen_k=first.max_seqlen_k,
+                    slot_mapping=first.slot_mapping,
+                    block_tables=first.block_tables if use_block_tables else None, spans=spans,
+                    state_slots=take(state_shape) if state_shape is not None else None,
+                    cu_portions=take(cu_shape) if cu_shape is not None else None)
+        try:
+            hidden = self.model(torch.from_numpy(ids).to(dev), torch.from_numpy(pos).to(dev))
+        finally:
+            reset_context()
+        for blocks in self.span_blocks:
+            blocks.flush()
+        self._bt_dirty = True          # the page tables have grown
+        self._ahead = None
+        return hidden
 
     @torch.no_grad()
     def prefill(self, prompts, chunk_tokens: int | None = None,
@@ -310,65 +343,40 @@ class DecodeEngine:
         """Run whole prompts through the model, fill their KV pages and sample the
         first new token of each (greedy); the sequences then join the running
         batch, ready for step().  Prefill side of ModelRunner.run
-        (fastkernels/infra/engine.py:6048-6063) with the metadata of
-        prepare_prefill (engine.py:4902-4990): cu_seqlens, per-token slots and the
-        block tables, so attention reads the pages the store has just written.
+        (fastkernels/infra/engine.py:6048-6063).
 
         chunk_tokens=C splits the work into forwards of at most C tokens; a chunk
         attends over the pages written by earlier chunks plus itself (the
         reference's chunked prefill).  With a tensor-parallel communicator the
         chunk defaults to its row capacity.  use_block_tables=False (whole prompts
-        only) attends over the batch's own dense K/V instead, the reference's
-        path when no block table exists (its warm-up)."""
+        of a model with one whole-context span only) attends over the batch's own
+        dense K/V instead, the reference's path when no block table exists (its
+        warm-up)."""
         from .comm import get_tp_comm
         comm = get_tp_comm()
         if chunk_tokens is None and comm is not None and comm.world > 1:
             chunk_tokens = comm.max_rows
-        dev, bs_ = self.device, self.block_size
-        new = []
         for prompt in prompts:
             n = len(prompt)
             if n < 1 or n + 1 > self.max_model_len:
                 raise ValueError(f"prompt length {n} outside [1, {self.max_model_len - 1}]")
-            if len(self.seqs) + len(new) >= self.max_num_seqs:
-                raise RuntimeError("max_num_seqs exceeded")
-            s = Sequence(len(self.seqs) + len(new), n)
-            self.blocks.allocate(s)
-            new.append(s)
+        if len(self.seqs) + len(prompts) > self.max_num_seqs:
+            raise RuntimeError("max_num_seqs exceeded")
+        new = [self._new_sequence(len(prompt)) for prompt in prompts]
         done = [0] * len(new)
         first = np.zeros(len(new), dtype=np.int64)
         while any(d < len(pr) for d, pr in zip(done, prompts)):
             part = pack_prefill_chunk([len(pr) for pr in prompts], done, chunk_tokens)
-            ids = np.concatenate([np.asarray(prompts[i][a:a + c], dtype=np.int64)
-                                  for i, a, c in part])
-            pos = np.concatenate([np.arange(a, a + c, dtype=np.int64) for i, a, c in part])
-            tabs = [np.asarray(new[i].block_table, dtype=np.int64) for i, a, c in part]
-            slots = np.concatenate([tabs[j][np.arange(a, a + c) // bs_] * bs_
-                                    + np.arange(a, a + c) % bs_
-                                    for j, (i, a, c) in enumerate(part)]).astype(np.int32)
-            cu_q = np.concatenate([[0], np.cumsum([c for _, _, c in part])]).astype(np.int32)
-            cu_k = np.concatenate([[0], np.cumsum([a + c for _, a, c in part])]).astype(np.int32)
-            paged = use_block_tables or chunk_tokens is not None
-            bt = None
-            if paged:
-                cols = max(len(t) for t in tabs)
-                bt_np = np.full((len(part), cols), -1, dtype=np.int32)
-                for j, t in enumerate(tabs):
-                    bt_np[j, :len(t)] = t
-                bt = torch.from_numpy(bt_np).to(dev)
-            set_context(True, cu_seqlens_q=torch.from_numpy(cu_q).to(dev),
-                        cu_seqlens_k=torch.from_numpy(cu_k).to(dev),
-                        max_seqlen_q=max(c for _, _, c in part),
-                        max_seqlen_k=max(a + c for _, a, c in part),
-                        slot_mapping=torch.from_numpy(slots).to(dev), block_tables=bt)
-            hidden = self.model(torch.from_numpy(ids).to(dev), torch.from_numpy(pos).to(dev))
-            reset_context()
+            hidden = self._forward_portions(
+                [(new[i], a, prompts[i][a:a + c]) for i, a, c in part],
+                use_block_tables or chunk_tokens is not None)
+            row_end = np.cumsum([c for _, _, c in part])
             ends = [(j, i) for j, (i, a, c) in enumerate(part) if a + c == len(prompts[i])]
             if ends:
-                rows = torch.from_numpy(cu_q[[j + 1 for j, _ in ends]].astype(np.int64) - 1).to(dev)
-                logits = self.model.lm_head.project(hidden.index_select(0, rows))
+                rows = torch.from_numpy(row_end[[j for j, _ in ends]].astype(np.int64) - 1)
+                logits = self.model.project(hidden.index_select(0, rows.to(self.device)))
                 vals, idxs = ops.argmax_rows(logits)
-                tok = self.model.lm_head.greedy_pairs(vals, idxs).cpu().numpy()
+                tok = self.model.greedy(vals, idxs).cpu().numpy()
                 for (j, i), t in zip(ends, tok):
                     first[i] = int(t)
             for i, a, c in part:
@@ -378,9 +386,61 @@ class DecodeEngine:
             s.last_token = int(t)
             s.output.append(int(t))
             self.seqs.append(s)
-        self._bt_dirty = True
-        self._seq_epoch += 1
+        self._running_set_changed()
         return first
+
+    @torch.no_grad()
+    def feed(self, entries, want=None) -> list[torch.Tensor]:
+        """Run the next tokens of open sequences, [(sequence, token ids)], and return
+        for each entry the logits (fp32, on the host) at the places `want[i]` among its
+        tokens (default: the last one).  Single tokens of sequences that already have
+        some take the decode step, everything else goes through in portions; nothing
+        is sampled.  Sequences fed here have no pending token: step() and feed() are
+        not mixed on one sequence."""
+        if want is None:
+            want = [[len(t) - 1] for _, t in entries]
+        if len({id(s) for s, _ in entries}) != len(entries):
+            raise ValueError("at most one entry per sequence")
+        for s, t in entries:
+            if len(t) < 1 or s.num_tokens + len(t) > self.max_model_len:
+                raise ValueError(f"sequence of {s.num_tokens} + {len(t)} tokens outside "
+                                 f"[1, {self.max_model_len}]")
+        single = [i for i, (s, t) in enumerate(entries) if len(t) == 1 and s.num_tokens > 0]
+        rest = [i for i in range(len(entries)) if i not in set(single)]
+        empty = torch.empty((0, self.model.logit_columns))
+        out = [empty] * len(entries)
+        if rest:
+            hidden = self._forward_portions([(entries[i][0], entries[i][0].num_tokens,
+                                              entries[i][1]) for i in rest])
+            rows, o = [], 0
+            for i in rest:
+                rows += [o + int(w) for w in want[i]]
+                o += len(entries[i][1])
+                entries[i][0].num_tokens += len(entries[i][1])
+            if rows:
+                idx = torch.tensor(rows, dtype=torch.int64, device=self.device)
+                logits = self.model.project(hidden.index_select(0, idx)).float().cpu()
+                o = 0
+                for i in rest:
+                    out[i] = logits[o:o + len(want[i])]
+                    o += len(want[i])
+        if single:
+            seqs = [entries[i][0] for i in single]
+            for i in single:
+                s, t = entries[i]
+                s.num_tokens += 1
+                s.last_token = int(t[0])
+            self._ahead = None
+            n = self.prepare_decode(True, seqs)
+            bs = self.graph_batch_size(n)
+            self.stage_inputs(n, bs, True)
+            self.run_step_device(bs)
+            self._mark_slot_in_flight()
+            if any(len(want[i]) for i in single):
+                logits = self.graph_vars["lm_logits"][:n].float().cpu()
+                for j, i in enumerate(single):
+                    out[i] = logits[j:j + 1].expand(len(want[i]), -1)
+        return out
 
     def graph_batch_size(self, n: int) -> int:
         for bs in sorted(self.graphs):
@@ -389,20 +449,21 @@ class DecodeEngine:
         return n
 
     # ----------------------------------------------------------- host-side prep
-    def prepare_decode(self, use_host_ids: bool) -> int:
-        """Fill the pinned staging arrays for this step (engine.py:5793-5798):
-        position = n - 1, context_len = n,
-        slot = block_table[-1] * BLOCK + ((n % BLOCK) - 1 if n % BLOCK else BLOCK - 1).
+    def prepare_decode(self, use_host_ids: bool, seqs=None) -> int:
+        """Fill the pinned staging arrays for this step (engine.py:5793-5798) of the
+        running sequences, or of `seqs`: position = n - 1 and, per span, context_len =
+        keys visible from there and slot = place of the newest token in its pages.
         Everything but the token ids may already have been written while the previous
         step ran on the device (`_prepare_ahead`)."""
-        if self._ahead is not None and self._ahead == (self._seq_epoch, len(self.seqs)):
+        if seqs is None and self._ahead is not None and \
+                self._ahead == (self._seq_epoch, len(self.seqs)):
             n = len(self.seqs)
         else:
-            n = self._prepare_layout()
+            n = self._prepare_layout(seqs)
         self._ahead = None
         if use_host_ids:
             ids = self.host_np["input_ids"]
-            for i, s in enumerate(self.seqs):
+            for i, s in enumerate(self.seqs if seqs is None else seqs):
                 ids[i] = s.last_token
         return n
 
@@ -414,39 +475,44 @@ class DecodeEngine:
         empty), so that such errors are still raised by the step they belong to."""
         if not self.seqs or _NO_PREPARE_AHEAD:
             return
-        bs_, pages = self.block_size, 0
-        for s in self.seqs:
-            if s.num_tokens > self.max_model_len:
-                return
-            if s.num_tokens % bs_ == 1 and len(s.block_table) * bs_ < s.num_tokens:
-                pages += 1
-        if pages > len(self.blocks.free):
+        if any(s.num_tokens > self.max_model_len for s in self.seqs):
             return
+        for blocks in self.span_blocks:
+            if sum(blocks.pages_missing(s) for s in self.seqs) > len(blocks.free):
+                return
         self._prepare_layout()
         self._ahead = (self._seq_epoch, len(self.seqs))
 
-    def _prepare_layout(self) -> int:
+    def _prepare_layout(self, seqs=None) -> int:
+        seqs = self.seqs if seqs is None else seqs
         self._ring_pos = (self._ring_pos + 1) % self.RING
         ev = self._ring_events[self._ring_pos]
         if ev is not None:
             ev.synchronize()            # copies issued from this slot have landed
         self.host, self.host_np = self._ring[self._ring_pos], self._ring_np[self._ring_pos]
-        h, bs_ = self.host_np, self.block_size
-        n = len(self.seqs)
-        for i, s in enumerate(self.seqs):
-            if self.blocks.maybe_append_page(s):
-                self._bt_dirty = True
+        h = self.host_np
+        n = len(seqs)
+        staged_for = tuple(s.seq_id for s in seqs)
+        if staged_for != self._staged_for:
+            self._bt_dirty = True
+            self._staged_for = staged_for
+        for i, s in enumerate(seqs):
             if s.num_tokens > self.max_model_len:
                 raise RuntimeError("sequence exceeds max_model_len")
-            m = s.num_tokens % bs_
-            h["positions"][i] = s.num_tokens - 1
-            h["context_lens"][i] = s.num_tokens
-            h["slot_mapping"][i] = s.block_table[-1] * bs_ + (m - 1 if m else bs_ - 1)
+            pos = s.num_tokens - 1
+            h["positions"][i] = pos
+            for g, blocks in enumerate(self.span_blocks):
+                if blocks.maybe_append_page(s):
+                    self._bt_dirty = True
+                h["span_lens"][g][i] = pos - blocks.base(pos) + 1
+                h["span_slots"][g][i] = blocks.slot(s, pos)
+            if self.state_slots is not None:
+                h["state_slots"][i] = s.state_slot
         if self._bt_dirty:
-            bt = h["block_tables"]
-            bt[:n].fill(-1)
-            for i, s in enumerate(self.seqs):
-                bt[i, :len(s.block_table)] = s.block_table
+            for g, bt in enumerate(h["span_tables"]):
+                bt[:n].fill(-1)
+                for i, s in enumerate(seqs):
+                    bt[i, :len(s.table(g))] = s.table(g)
         return n
 
     def _mark_slot_in_flight(self) -> None:
@@ -461,43 +527,46 @@ class DecodeEngine:
         rows get slot -1 / context_len 0 (engine.py:5404-5406)."""
         gv, h = self.graph_vars, self.host
         if bs > n:
-            h["slot_mapping"][n:bs] = -1
-            h["context_lens"][n:bs] = 0
+            for slots, lens in zip(h["span_slots"], h["span_lens"]):
+                slots[n:bs] = -1
+                lens[n:bs] = 0
+            if self.state_slots is not None:
+                h["state_slots"][n:bs] = -1
             h["positions"][n:bs] = 0
         first = 0 if use_host_ids else 8 * self.max_num_seqs
         self._packed_dev[first:].copy_(h["packed"][first:], non_blocking=True)
         self.h2d_bytes += h["packed"].numel() - first
         if self._bt_dirty:
-            gv["block_tables"][:bs].copy_(h["block_tables"][:bs], non_blocking=True)
-            self.h2d_bytes += h["block_tables"][:bs].numel() * 4
+            for dst, src in zip(gv["span_tables"], h["span_tables"]):
+                dst[:bs].copy_(src[:bs], non_blocking=True)
+                self.h2d_bytes += src[:bs].numel() * 4
             self._bt_dirty = False
 
     # -------------------------------------------------------------- graph body
     def _forward(self, bs: int) -> None:
         gv = self.graph_vars
-        # one split-KV schedule per step, shared by every layer
-        ctx = get_context()
-        att = self.model.model.layers[0].self_attn.attn
-        op = att.decode_op
-        ops.paged_decode_attn_plan(ctx.context_lens, ctx.block_tables, self.block_size,
-                                   att.num_heads, att.num_kv_heads, att.head_size,
-                                   self.attn_workspace, op._max_splits, status=op._status)
-        ctx.attn_plan_ready = True
+        self.model.begin_decode(get_context())
         hidden = self.model(gv["input_ids"][:bs], gv["positions"][:bs])
         gv["outputs"][:bs] = hidden
-        logits = self.model.lm_head.project(hidden)
+        logits = self.model.project(hidden)
         gv["lm_logits"][:bs] = logits
         ops.argmax_rows(gv["lm_logits"][:bs], gv["lm_max_vals"][:bs], gv["lm_max_idxs"][:bs])
-        ids = self.model.lm_head.greedy_pairs(gv["lm_max_vals"][:bs], gv["lm_max_idxs"][:bs])
+        ids = self.model.greedy(gv["lm_max_vals"][:bs], gv["lm_max_idxs"][:bs])
         gv["token_ids"][:bs] = ids
         # hand the sampled ids to the next step on the device (engine.py:5689-5705)
         gv["input_ids"][:bs] = ids
 
     def _set_context(self, bs: int, max_ctx: int) -> None:
         gv = self.graph_vars
+        cu = gv["cu_rows"][:bs + 1]
+        spans = [SpanBatch(slots[:bs], tables[:bs], lens[:bs], cu)
+                 for slots, lens, tables in zip(gv["span_slots"], gv["span_lens"],
+                                                gv["span_tables"])]
         set_context(False, slot_mapping=gv["slot_mapping"][:bs],
                     context_lens=gv["context_lens"][:bs],
-                    block_tables=gv["block_tables"][:bs], max_context_len=max_ctx)
+                    block_tables=gv["block_tables"][:bs], max_context_len=max_ctx, spans=spans,
+                    state_slots=gv["state_slots"][:bs] if self.state_slots is not None else None,
+                    cu_portions=cu if self.state_slots is not None else None)
 
     @torch.no_grad()
     def capture_cudagraph(self, batch_sizes) -> None:
@@ -505,11 +574,14 @@ class DecodeEngine:
         inputs; max_context_len is max_model_len at capture (engine.py:6832-6836)
         and the real lengths are read on the device at replay."""
         gv = self.graph_vars
-        saved = {k: gv[k].clone() for k in ("input_ids", "positions", "slot_mapping",
-                                             "context_lens", "block_tables")}
-        gv["slot_mapping"].fill_(-1)
-        gv["context_lens"].fill_(1)
-        gv["block_tables"].fill_(0)
+        inputs = [self._packed_dev, *gv["span_tables"]]
+        saved = [t.clone() for t in inputs]
+        for slots, lens, tables in zip(gv["span_slots"], gv["span_lens"], gv["span_tables"]):
+            slots.fill_(-1)
+            lens.fill_(1)
+            tables.fill_(0)
+        if self.state_slots is not None:
+            gv["state_slots"].fill_(-1)
         gv["positions"].zero_()
         gv["input_ids"].zero_()
         for bs in sorted(batch_sizes, reverse=True):
@@ -525,8 +597,8 @@ class DecodeEngine:
             self.graphs[bs] = graph
             torch.cuda.synchronize()
             reset_context()
-        for k, v in saved.items():
-            gv[k].copy_(v)
+        for t, v in zip(inputs, saved):
+            t.copy_(v)
 
     # -------------------------------------------------------------------- steps
     @torch.no_grad()

@@ -24,6 +24,21 @@ _REFERENCE_CONTEXT_MODULE = "fastkernels.infra.context"
 
 
 @dataclass
+class SpanBatch:
+    """Attention metadata of one span (the layers that see the same part of a
+    sequence).  Prefill: one row of cu_seqlens / block_tables per segment, a run of
+    queries that see the same pages; kv_lens = keys per segment.  Decode: one row per
+    sequence, kv_lens = context_lens."""
+    slot_mapping: torch.Tensor
+    block_tables: torch.Tensor | None
+    kv_lens: torch.Tensor
+    cu_seqlens_q: torch.Tensor
+    cu_seqlens_k: torch.Tensor | None = None
+    max_seqlen_q: int = 1
+    max_seqlen_k: int = 0
+
+
+@dataclass
 class Context:
     is_prefill: bool = False
     cu_seqlens_q: torch.Tensor | None = None    # [num_seqs + 1] int32 (prefill)
@@ -37,6 +52,10 @@ class Context:
     # set by the engine once it has computed the step's split-KV schedule into the
     # attention workspace all layers share; layers then skip their own plan launch
     attn_plan_ready: bool = False
+    # models with several spans or recurrent state
+    spans: list[SpanBatch] | None = None
+    state_slots: torch.Tensor | None = None     # [N] int32 state slot per token, -1 padded
+    cu_portions: torch.Tensor | None = None     # [portions + 1] int32: token ranges
 
 
 _CONTEXT = Context()
@@ -68,7 +87,7 @@ def reference_attn_backend():
 
 def set_context(is_prefill, cu_seqlens_q=None, cu_seqlens_k=None, max_seqlen_q=0,
                 max_seqlen_k=0, slot_mapping=None, context_lens=None, block_tables=None,
-                max_context_len=0) -> None:
+                max_context_len=0, spans=None, state_slots=None, cu_portions=None) -> None:
     """Same argument order as the reference's set_context (context.py:411-440,
     the fields this path reads).  Prefill: cu_seqlens / max_seqlen, slot_mapping
     and, when a prefix is already cached, block_tables.  Decode: slot_mapping,
@@ -77,7 +96,8 @@ def set_context(is_prefill, cu_seqlens_q=None, cu_seqlens_k=None, max_seqlen_q=0
     _OWN_CONTEXT_SET = True
     _CONTEXT = Context(bool(is_prefill), cu_seqlens_q, cu_seqlens_k, int(max_seqlen_q),
                        int(max_seqlen_k), slot_mapping, context_lens, block_tables,
-                       max_context_len)
+                       max_context_len, spans=spans, state_slots=state_slots,
+                       cu_portions=cu_portions)
 
 
 def reset_context() -> None:

@@ -391,8 +391,10 @@ def xor_u32(t: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
 
 # -------------------------------------------------------------------------- argmax
 def argmax_rows(x, out_val=None, out_idx=None):
-    """(max as fp32, lowest index of the max) per row of a bf16 [rows, cols] matrix."""
-    _need(x, BF16, "x")
+    """(max as fp32, lowest index of the max) per row of a bf16 or fp32 [rows, cols]
+    matrix."""
+    if x.dtype != torch.float32:
+        _need(x, BF16, "x")
     if x.dim() != 2 or x.stride(1) != 1:
         raise _lib.FkError("argmax_rows needs a 2-D row-dense input")
     rows, cols = x.shape
@@ -400,8 +402,9 @@ def argmax_rows(x, out_val=None, out_idx=None):
         out_val = torch.empty(rows, dtype=torch.float32, device=x.device)
     if out_idx is None:
         out_idx = torch.empty(rows, dtype=torch.int64, device=x.device)
-    check(lib.fk_argmax_bf16(_ptr(x), x.stride(0) if rows else cols, rows, cols,
-                             _ptr(out_val), _ptr(out_idx), _stream()), "fk_argmax_bf16")
+    fn = lib.fk_argmax_f32 if x.dtype == torch.float32 else lib.fk_argmax_bf16
+    check(fn(_ptr(x), x.stride(0) if rows else cols, rows, cols,
+             _ptr(out_val), _ptr(out_idx), _stream()), "fk_argmax")
     return out_val, out_idx
 
 
@@ -492,6 +495,262 @@ def gemm_silu_mul(x, w, bias=None, out=None, workspace=None, status=None):
                                     _ptr(workspace),
                                     workspace.numel() * workspace.element_size(),
                                     _status_ptr(status, x), _stream()), "fk_gemm_bf16_silu_mul")
+    return out
+
+
+def gemm_act_mul(x, w, act, out=None, workspace=None, status=None):
+    """act(x @ wg.T) * (x @ wu.T), w = [wg; wu] rows: one launch where the shape has
+    one (see gemm_silu_mul_fusable), else the projection followed by act_and_mul."""
+    m, k = x.shape
+    half = w.shape[0] // 2
+    if x.dtype == BF16 and gemm_silu_mul_fusable(m, 2 * half, k):
+        _need(x, BF16, "x")
+        _need(w, BF16, "w")
+        if x.stride(1) != 1 or not w.is_contiguous():
+            raise _lib.FkError("gemm_act_mul needs row-dense x and contiguous w")
+        if out is None:
+            out = torch.empty((m, half), dtype=BF16, device=x.device)
+        if workspace is None:
+            workspace = gemm_workspace(x.device)
+        check(lib.fk_gemm_bf16_act_mul(
+            _ptr(x), x.stride(0) if m else k, _ptr(w), None, _ptr(out),
+            out.stride(0) if m else half, m, 2 * half, k, int(act), _ptr(workspace),
+            workspace.numel() * workspace.element_size(), _status_ptr(status, x), _stream()),
+            "fk_gemm_bf16_act_mul")
+        return out
+    return act_and_mul(gemm(x, w, workspace=workspace, status=status), act, out=out)
+
+
+def gemm(x, w, out=None, workspace=None, status=None):
+    """x @ w.T in the type of its operands: bf16 (tensor cores, fp32 accumulation) or
+    true fp32."""
+    if x.dtype != torch.float32:
+        return gemm_bf16(x, w, out=out, workspace=workspace, status=status)
+    _need(x, torch.float32, "x")
+    _need(w, torch.float32, "w")
+    if x.dim() != 2 or x.stride(1) != 1 or not w.is_contiguous():
+        raise _lib.FkError("gemm needs row-dense x and contiguous w")
+    m, k = x.shape
+    n = w.shape[0]
+    if out is None:
+        out = torch.empty((m, n), dtype=torch.float32, device=x.device)
+    check(lib.fk_gemm_f32(_ptr(x), x.stride(0) if m else k, _ptr(w), _ptr(out),
+                          out.stride(0) if m else n, m, n, k, _stream()), "fk_gemm_f32")
+    return out
+
+
+# ------------------------------------- fp32 residual stream, linear-attention mixers
+def _is_f32(t: torch.Tensor, name: str) -> int:
+    if not t.is_cuda:
+        raise _lib.FkError(f"{name} must be a CUDA tensor (no CPU path exists)")
+    if t.dtype not in (BF16, torch.float32):
+        raise _lib.FkError(f"{name} must be bf16 or fp32, got {t.dtype}")
+    return int(t.dtype == torch.float32)
+
+
+def embed_f32(table, ids, out=None, status=None):
+    """fp32 residual rows table[ids]; table [vocab, stride] bf16 or fp32."""
+    f32 = _is_f32(table, "table")
+    _need(ids, torch.int64, "ids")
+    if not table.is_contiguous():
+        raise _lib.FkError("table must be contiguous")
+    n, stride = ids.shape[0], table.shape[1]
+    if out is None:
+        out = torch.empty((n, stride), dtype=torch.float32, device=table.device)
+    check(lib.fk_embed_f32(_ptr(table), f32, table.shape[0], _ptr(ids), _ptr(out), n, stride,
+                           _status_ptr(status, table), _stream()), "fk_embed_f32")
+    return out
+
+
+def norm_shift(x, gain, width, eps, dtype, y=None, y_gain=None, x_out=None, shift=None,
+               state=None, slots=None, positions=None, cu_portions=None, out=None, status=None):
+    """x' = x + rms(y) * y_gain; h = rms(x') * gain; token shift of h (see
+    fk_norm_shift).  x fp32 [T, stride]; returns (x', out of `dtype`)."""
+    _need(x, torch.float32, "x")
+    if x.dim() != 2 or not x.is_contiguous():
+        raise _lib.FkError("norm_shift needs a contiguous [T, stride] residual")
+    rows, stride = x.shape
+    if out is None:
+        out = torch.empty((rows, stride), dtype=dtype, device=x.device)
+    f32 = _is_f32(out, "out")
+    if y is not None:
+        _need(y, out.dtype, "y")
+        if y.shape != x.shape or y.stride(1) != 1:
+            raise _lib.FkError("norm_shift: y must be row-dense with the residual's shape")
+        if x_out is None:
+            x_out = torch.empty_like(x) if shift is not None else x
+    n_port = 0
+    if shift is not None:
+        _need(state, torch.float32, "state")
+        _need(slots, torch.int32, "slots")
+        _need(positions, torch.int64, "positions")
+        _need(cu_portions, torch.int32, "cu_portions")
+        if state.dim() != 2 or state.shape[1] != stride or not state.is_contiguous():
+            raise _lib.FkError("norm_shift: state must be a contiguous [slots, stride]")
+        n_port = cu_portions.numel() - 1
+    check(lib.fk_norm_shift(
+        _ptr(x), _ptr(x_out), _ptr(y), y.stride(0) if y is not None and rows else stride,
+        _ptr(y_gain), _ptr(gain), _ptr(shift), _ptr(out), f32, _ptr(state),
+        state.shape[0] if state is not None else 0, _ptr(slots), _ptr(positions),
+        _ptr(cu_portions), n_port, rows, stride, int(width), float(eps),
+        _status_ptr(status, x), _stream()), "fk_norm_shift")
+    return (x if x_out is None else x_out), out
+
+
+def branch_combine(a, b, weight_a, weight_b, gain_out, x, width, eps, gain=None, out=None):
+    """x += rms((rms(a) * weight_a + rms(b) * weight_b) / 2) * gain_out in place;
+    returns rms(x) * gain in the type of a (None when gain is None)."""
+    f32 = _is_f32(a, "a")
+    _need(b, a.dtype, "b")
+    _need(x, torch.float32, "x")
+    rows, stride = x.shape
+    if a.shape != x.shape or b.shape != x.shape or a.stride(1) != 1 or \
+            (rows and b.stride() != a.stride()) or not x.is_contiguous():
+        raise _lib.FkError("branch_combine needs row-dense operands of one shape")
+    if gain is not None and out is None:
+        out = torch.empty((rows, stride), dtype=a.dtype, device=x.device)
+    check(lib.fk_branch_combine(
+        _ptr(a), _ptr(b), a.stride(0) if rows else stride, _ptr(weight_a), _ptr(weight_b),
+        _ptr(gain_out), _ptr(gain), _ptr(x), _ptr(out), f32, rows, stride, int(width),
+        float(eps), _stream()), "fk_branch_combine")
+    return out
+
+
+def rope_rms_store(q, k, q_out, k_cache, v_cache, slots, positions, cos_sin, rot_dims,
+                   num_q_heads, num_kv_heads, head_dim, eps, status=None) -> None:
+    """Interleaved partial rotation + weight-less RMS norm of q and k heads; k (and k
+    as projected, as the value) to the paged pool [blocks, page, Hkv, padded_dim].
+    q / k are column ranges of the packed projection rows; q_out is
+    [T, Hkv * padded_group, padded_dim]."""
+    f32 = _is_f32(q, "q")
+    for name, t in (("k", k), ("q_out", q_out), ("k_cache", k_cache), ("v_cache", v_cache)):
+        _need(t, q.dtype, name)
+    _need(slots, torch.int32, "slots")
+    _need(positions, torch.int64, "positions")
+    _need(cos_sin, torch.float32, "cos_sin")
+    rows = q.shape[0]
+    if q.stride(1) != 1 or k.stride(1) != 1 or (rows and q.stride(0) != k.stride(0)):
+        raise _lib.FkError("q and k must be column ranges of the same rows")
+    if not (q_out.is_contiguous() and k_cache.is_contiguous() and v_cache.is_contiguous()
+            and cos_sin.is_contiguous()):
+        raise _lib.FkError("q_out, caches and cos_sin must be contiguous")
+    if q_out.shape[1] % num_kv_heads or k_cache.shape[2:] != (num_kv_heads, q_out.shape[2]) or \
+            cos_sin.shape[1] != max(rot_dims, 1):
+        raise _lib.FkError("rope_rms_store: shape mismatch")
+    check(lib.fk_rope_rms_store(
+        _ptr(q), _ptr(k), q.stride(0) if rows else 0, f32, _ptr(q_out), _ptr(k_cache),
+        _ptr(v_cache), _ptr(slots), k_cache.shape[0] * k_cache.shape[1], _ptr(positions),
+        _ptr(cos_sin), cos_sin.shape[0], rot_dims, num_q_heads, num_kv_heads, head_dim,
+        q_out.shape[1] // num_kv_heads, q_out.shape[2], float(eps), rows,
+        _status_ptr(status, q), _stream()), "fk_rope_rms_store")
+
+
+def act_and_mul(x, act, out=None):
+    """act(x[:, :d]) * x[:, d:], bf16 or fp32."""
+    f32 = _is_f32(x, "x")
+    if x.dim() != 2 or x.stride(1) != 1:
+        raise _lib.FkError("act_and_mul needs a 2-D row-dense input")
+    rows, d = x.shape[0], x.shape[1] // 2
+    if out is None:
+        out = torch.empty((rows, d), dtype=x.dtype, device=x.device)
+    check(lib.fk_act_and_mul(_ptr(x), x.stride(0) if rows else 2 * d, _ptr(out),
+                             out.stride(0) if rows else d, f32, rows, d, int(act), _stream()),
+          "fk_act_and_mul")
+    return out
+
+
+def delta_padded_dim(dim: int) -> int:
+    """Key channels per head in the delta rule's packed operands and state."""
+    n = int(lib.fk_delta_padded_dim(int(dim)))
+    if n <= 0:
+        raise _lib.FkError(f"delta rule: head size {dim} unsupported")
+    return n
+
+
+def delta_prepare(r, k, v, a, y1, w2, w0, a_bias, heads, dim, decay_scale, unit_eps,
+                  packed=None):
+    """Per-token operands of the delta rule, packed [heads, T, 6, padded_dim] fp32.
+    r, k, v, a [T, heads * dim] and y1 [T, rank] are column ranges of the same rows;
+    w2 [heads * dim, padded rank]."""
+    f32 = _is_f32(k, "k")
+    rows, rank = y1.shape
+    for name, t in (("r", r), ("v", v), ("a", a), ("y1", y1), ("w2", w2)):
+        _need(t, k.dtype, name)
+        if t is not w2 and (t.stride(1) != 1 or (rows and t.stride(0) != k.stride(0))):
+            raise _lib.FkError(f"{name} must be a column range of the packed rows")
+    _need(w0, torch.float32, "w0")
+    _need(a_bias, torch.float32, "a_bias")
+    if not w2.is_contiguous() or w2.shape[0] != heads * dim:
+        raise _lib.FkError("w2 must be contiguous [heads * dim, padded rank]")
+    if packed is None:
+        packed = torch.empty((heads, rows, 6, delta_padded_dim(dim)), dtype=torch.float32,
+                             device=k.device)
+    check(lib.fk_delta_prepare(
+        _ptr(r), _ptr(k), _ptr(v), _ptr(a), _ptr(y1), k.stride(0) if rows else 0, f32, _ptr(w2),
+        w2.shape[1], _ptr(w0), _ptr(a_bias), _ptr(packed), rows, heads, dim, rank,
+        float(decay_scale), float(unit_eps), _stream()), "fk_delta_prepare")
+    return packed
+
+
+def delta_scan(packed, state, cu_portions, slots, positions, dim, out=None, status=None):
+    """The recurrence over packed operands; state [slots, heads, dim, padded_dim] fp32
+    is read and replaced.  Returns o [T, heads * dim] fp32."""
+    _need(packed, torch.float32, "packed")
+    _need(state, torch.float32, "state")
+    _need(cu_portions, torch.int32, "cu_portions")
+    _need(slots, torch.int32, "slots")
+    _need(positions, torch.int64, "positions")
+    heads, rows = packed.shape[0], packed.shape[1]
+    if not packed.is_contiguous() or not state.is_contiguous() or \
+            tuple(state.shape[1:]) != (heads, dim, packed.shape[3]):
+        raise _lib.FkError("delta_scan: packed or state has the wrong shape")
+    if out is None:
+        out = torch.empty((rows, heads * dim), dtype=torch.float32, device=packed.device)
+    check(lib.fk_delta_scan(
+        _ptr(packed), _ptr(out), _ptr(state), state.shape[0], _ptr(cu_portions),
+        cu_portions.numel() - 1, _ptr(slots), _ptr(positions), rows, heads, dim,
+        _status_ptr(status, packed), _stream()), "fk_delta_scan")
+    return out
+
+
+def delta_output(o, gate, weight, heads, dim, eps, out):
+    """out = rms(o per head) * weight * sigmoid(gate); columns of out beyond
+    heads * dim are zeroed."""
+    _need(o, torch.float32, "o")
+    f32 = _is_f32(gate, "gate")
+    _need(out, gate.dtype, "out")
+    _need(weight, torch.float32, "weight")
+    rows = o.shape[0]
+    if not o.is_contiguous() or not out.is_contiguous() or gate.stride(1) != 1:
+        raise _lib.FkError("delta_output needs dense operands")
+    check(lib.fk_delta_output(_ptr(o), _ptr(gate), gate.stride(0) if rows else heads * dim,
+                              _ptr(weight), _ptr(out), out.shape[1], f32, rows, heads, dim,
+                              float(eps), _stream()), "fk_delta_output")
+    return out
+
+
+def paged_attn_any(q, k_cache, v_cache, cu_seqlens_q, kv_lens, block_tables, softmax_scale,
+                   out=None, status=None):
+    """Causal attention over the NHD pool without shape restrictions (bf16 or fp32):
+    the path for fp32 and for head sizes / GQA ratios the tensor-core kernels lack."""
+    f32 = _is_f32(q, "q")
+    _need(k_cache, q.dtype, "k_cache")
+    _need(v_cache, q.dtype, "v_cache")
+    for name, t in (("cu_seqlens_q", cu_seqlens_q), ("kv_lens", kv_lens),
+                    ("block_tables", block_tables)):
+        _need(t, torch.int32, name)
+    rows, hq, d = q.shape
+    nb, bs, hkv, d2 = k_cache.shape
+    if d2 != d or v_cache.shape != k_cache.shape or not k_cache.is_contiguous() or \
+            not v_cache.is_contiguous() or not q.is_contiguous() or block_tables.stride(1) != 1:
+        raise _lib.FkError("paged_attn_any: shape or stride mismatch")
+    if out is None:
+        out = torch.empty((rows, hq, d), dtype=q.dtype, device=q.device)
+    check(lib.fk_paged_attn_any(
+        _ptr(q), hq * d, _ptr(out), out.stride(0) if rows else hq * d, _ptr(k_cache),
+        _ptr(v_cache), f32, nb, bs, _ptr(cu_seqlens_q), _ptr(kv_lens), _ptr(block_tables),
+        block_tables.stride(0), cu_seqlens_q.numel() - 1, rows, hq, hkv, d,
+        float(softmax_scale), _status_ptr(status, q), _stream()), "fk_paged_attn_any")
     return out
 
 

@@ -52,6 +52,12 @@ enum fk_device_status {
   FK_DEV_TMEM_BASE = 16    /* tensor memory was not handed out from column 0  */
 };
 
+/* Activation of a gated feed-forward, act(gate) * up. */
+enum fk_activation {
+  FK_ACT_SILU = 0,
+  FK_ACT_GELU_TANH = 1     /* 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))) */
+};
+
 /* Library version: major*10000 + minor*100 + patch. */
 int fk_version(void);
 
@@ -569,6 +575,105 @@ int fk_merge_attn_states(void* out, int64_t out_stride_token, int64_t out_stride
                          const float* suffix_lse, int64_t num_tokens, int num_heads,
                          int head_dim, int64_t prefill_tokens_with_context,
                          fk_stream_t stream);
+
+/* ------------------------------------------------------------------------
+ * Decoders with an fp32 residual stream and linear-attention mixers.
+ *
+ * `is_f32` picks the activation type (0: bf16, 1: fp32); weights of norms, biases
+ * and everything that enters the recurrence are fp32 in both.  Rows are padded to
+ * `stride` elements with a zero tail.  A batch is a list of portions, each a run of
+ * consecutive tokens of one sequence: cu_portions [num_portions + 1] int32 row
+ * ranges, slots [rows] int32 = the sequence's state slot (-1: padded row),
+ * positions [rows] int64 inside the sequence (0: the state starts at zero).
+ * ------------------------------------------------------------------------ */
+
+/* x[i] = float(table[ids[i]]), table [vocab, stride]. */
+int fk_embed_f32(const void* table, int is_f32, int64_t vocab, const int64_t* ids, float* x,
+                 int64_t rows, int stride, int32_t* status, fk_stream_t stream);
+
+/* x' = x + rms(y) * y_gain (y null: x' = x), stored to x_out when given;
+ * h = rms(x') * gain with ONE gain each; out = h + (h_prev - h) * shift with h_prev
+ * the sequence's previous h (`state` [num_slots, stride] fp32 across calls, updated),
+ * or out = h when shift is null.  With a shift x_out must not be x_in. */
+int fk_norm_shift(const float* x_in, float* x_out, const void* y, int64_t y_stride,
+                  const float* y_gain, const float* gain, const float* shift, void* out,
+                  int is_f32, float* state, int num_slots, const int32_t* slots,
+                  const int64_t* positions, const int32_t* cu_portions, int num_portions,
+                  int64_t rows, int stride, int width, float eps, int32_t* status,
+                  fk_stream_t stream);
+
+/* m = (rms(a) * weight_a + rms(b) * weight_b) / 2; x += rms(m) * gain_out;
+ * out = rms(x) * gain (out null: not computed). */
+int fk_branch_combine(const void* a, const void* b, int64_t ab_stride, const float* weight_a,
+                      const float* weight_b, const float* gain_out, const float* gain, float* x,
+                      void* out, int is_f32, int64_t rows, int stride, int width, float eps,
+                      fk_stream_t stream);
+
+/* Per head: interleaved rotation (pair 2e, 2e+1) of the first rot_dims channels with
+ * cos_sin [max_position, rot_dims] = (cos | sin) fp32, then division by the root mean
+ * square over head_dim.  q -> q_out [rows, num_kv_heads * padded_group, padded_dim]
+ * (query heads of a KV head padded to padded_group, zeros), k -> k_cache, and k as
+ * projected -> v_cache, both NHD [slots, num_kv_heads, padded_dim]. */
+int fk_rope_rms_store(const void* q, const void* k, int64_t in_stride, int is_f32, void* q_out,
+                      void* k_cache, void* v_cache, const int32_t* slots, int64_t num_slots,
+                      const int64_t* positions, const float* cos_sin, int64_t max_position,
+                      int rot_dims, int num_q_heads, int num_kv_heads, int head_dim,
+                      int padded_group, int padded_dim, float eps, int64_t rows,
+                      int32_t* status, fk_stream_t stream);
+
+/* out[i, c] = act(x[i, c]) * x[i, d + c] (act: enum fk_activation). */
+int fk_act_and_mul(const void* x, int64_t x_stride, void* out, int64_t out_stride, int is_f32,
+                   int64_t rows, int64_t d, int act, fk_stream_t stream);
+
+/* fk_gemm_bf16_silu_mul with a choice of activation; same single-launch shapes. */
+int fk_gemm_bf16_act_mul(const void* x, int64_t x_stride, const void* w, const void* bias,
+                         void* y, int64_t y_stride, int64_t m, int64_t n, int64_t k, int act,
+                         void* workspace, size_t workspace_bytes, int32_t* status,
+                         fk_stream_t stream);
+
+/* Generalized delta rule, per head with key channels c and value channels v:
+ *   S_t = diag(w_t) S_{t-1} - (a_t * u_t) (u_t^T S_{t-1}) + k_t v_t^T,  o_t = S_t^T r_t
+ *   w_t = exp(-decay_scale * sigmoid(w2 tanh(y1) + w0)), a_t = sigmoid(a + a_bias),
+ *   u_t = k_t / sqrt(sum k_t^2 + unit_eps)
+ * fk_delta_padded_dim: key channels per head in `packed` and `state` (0: unsupported,
+ * head size above 256).  fk_delta_prepare writes packed [heads][rows][6][padded_dim]
+ * fp32 (w, u, a * u, k, r, v) from packed projection rows; w2 [heads * dim, w2_stride]
+ * in the activation type, rows zero-padded to a multiple of 4 (rank <= 512).
+ * fk_delta_scan runs the recurrence for every portion from and to
+ * state [num_slots][heads][dim (value)][padded_dim (key)] fp32 and writes
+ * o [rows, heads * dim] fp32.  fk_delta_output: out = rms(o per head) * weight *
+ * sigmoid(gate), columns beyond heads * dim zeroed. */
+int fk_delta_padded_dim(int dim);
+int fk_delta_prepare(const void* r, const void* k, const void* v, const void* a, const void* y1,
+                     int64_t in_stride, int is_f32, const void* w2, int64_t w2_stride,
+                     const float* w0, const float* a_bias, float* packed, int64_t rows,
+                     int heads, int dim, int rank, float decay_scale, float unit_eps,
+                     fk_stream_t stream);
+int fk_delta_scan(const float* packed, float* o, float* state, int num_slots,
+                  const int32_t* cu_portions, int num_portions, const int32_t* slots,
+                  const int64_t* positions, int64_t rows, int heads, int dim, int32_t* status,
+                  fk_stream_t stream);
+int fk_delta_output(const float* o, const void* gate, int64_t gate_stride, const float* weight,
+                    void* out, int64_t out_stride, int is_f32, int64_t rows, int heads, int dim,
+                    float eps, fk_stream_t stream);
+
+/* y[m, n] = x[m, k] w[n, k]^T in fp32 (no tensor cores); k % 4 == 0. */
+int fk_gemm_f32(const float* x, int64_t x_stride, const float* w, float* y, int64_t y_stride,
+                int64_t m, int64_t n, int64_t k, fk_stream_t stream);
+
+/* Causal attention over the NHD pool for any head size up to 512 (multiple of 4), any
+ * query / KV head ratio, bf16 or fp32: sequence i brings query rows cu_seqlens_q[i] ..
+ * cu_seqlens_q[i + 1] that end at its kv_lens[i]-th key. */
+int fk_paged_attn_any(const void* q, int64_t q_stride, void* out, int64_t out_stride,
+                      const void* k_cache, const void* v_cache, int is_f32, int64_t num_blocks,
+                      int block_size, const int32_t* cu_seqlens_q, const int32_t* kv_lens,
+                      const int32_t* block_tables, int64_t block_table_stride, int num_seqs,
+                      int64_t rows, int num_q_heads, int num_kv_heads, int head_dim,
+                      float softmax_scale, int32_t* status, fk_stream_t stream);
+
+/* fk_argmax_bf16 on fp32 rows. */
+int fk_argmax_f32(const float* x, int64_t x_stride, int64_t rows, int64_t cols, float* out_val,
+                  int64_t* out_idx, fk_stream_t stream);
 
 #ifdef __cplusplus
 }
