@@ -41,23 +41,29 @@ struct NormShiftParams {
   int32_t* status;
 };
 
-// x' = x + rms(y) * y_gain; returns h = rms(x') * gain and, when asked, stores x'.
+// The loads of one row.
 template <typename T, int VPT>
-__device__ __forceinline__ void norm_row(const NormShiftParams& p, int64_t t, bool store_x,
-                                         Row<VPT>& h, float* red, int& flip) {
+__device__ __forceinline__ void load_row(const NormShiftParams& p, int64_t t, Row<VPT>& x,
+                                         Row<VPT>& y) {
   const int groups = p.stride >> 2;
-  const float inv_w = 1.0f / (float)p.width;
-  Row<VPT> y;
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int g = threadIdx.x + i * blockDim.x;
-    h.v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-    y.v[i] = h.v[i];
+    x.v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    y.v[i] = x.v[i];
     if (g < groups) {
-      h.v[i] = *reinterpret_cast<const float4*>(p.x_in + t * p.stride + g * 4);
+      x.v[i] = *reinterpret_cast<const float4*>(p.x_in + t * p.stride + g * 4);
       if (p.y) y.v[i] = Elem<T>::load4(static_cast<const T*>(p.y) + t * p.y_stride + g * 4);
     }
   }
+}
+
+// x' = x + rms(y) * y_gain, stored when asked; h (in: x) = rms(x') * gain.
+template <typename T, int VPT>
+__device__ __forceinline__ void norm_row(const NormShiftParams& p, int64_t t, bool store_x,
+                                         Row<VPT>& h, const Row<VPT>& y, float* red, int& flip) {
+  const int groups = p.stride >> 2;
+  const float inv_w = 1.0f / (float)p.width;
   if (p.y) {
     float s[1] = {0.f};
 #pragma unroll
@@ -83,6 +89,14 @@ __device__ __forceinline__ void norm_row(const NormShiftParams& p, int64_t t, bo
   for (int i = 0; i < VPT; ++i) h.v[i] = h.v[i] * sc;
 }
 
+template <typename T, int VPT>
+__device__ __forceinline__ void one_row(const NormShiftParams& p, int64_t t, Row<VPT>& h,
+                                        float* red, int& flip) {
+  Row<VPT> y;
+  load_row<T, VPT>(p, t, h, y);
+  norm_row<T, VPT>(p, t, false, h, y, red, flip);
+}
+
 // A CTA walks `rows_per_cta` consecutive rows and carries the normed row from one
 // to the next.  The row ahead of its first one is computed once more (from x_in,
 // which this kernel does not change), or comes from the sequence's state when a
@@ -98,21 +112,25 @@ __global__ void __launch_bounds__(512) norm_shift_kernel(const NormShiftParams p
   const int groups = p.stride >> 2;
   const int64_t t0 = (int64_t)blockIdx.x * p.rows_per_cta;
   const int64_t t1 = min(t0 + p.rows_per_cta, p.rows);
-  Row<VPT> prev;
-  bool have_prev = false;
+  Row<VPT> prev, nx, ny;
+  load_row<T, VPT>(p, t0, nx, ny);
   for (int64_t t = t0; t < t1; ++t) {
-    Row<VPT> h;
-    if (!p.shift) {
-      norm_row<T, VPT>(p, t, true, h, red, flip);
-    } else {
-      const int slot = p.slots[t];
-      const bool first = slot < 0 || t == 0 || p.slots[t - 1] != slot;
+    // the next row's loads are in flight during this row's reductions
+    Row<VPT> h = nx;
+    const Row<VPT> y = ny;
+    if (t + 1 < t1) load_row<T, VPT>(p, t + 1, nx, ny);
+    bool first = false, in_range = false;
+    int slot = -1;
+    float* st = nullptr;
+    if (p.shift) {
+      slot = p.slots[t];
+      first = slot < 0 || t == 0 || p.slots[t - 1] != slot;
       if (first) {
-        const bool in_range = slot >= 0 && slot < p.num_slots;
+        in_range = slot >= 0 && slot < p.num_slots;
         if (slot >= p.num_slots && threadIdx.x == 0 && p.status)
           atomicOr(p.status, FK_DEV_BAD_SLOT);
         const bool from_state = in_range && p.positions[t] > 0;
-        float* st = p.state + (int64_t)(in_range ? slot : 0) * p.stride;
+        st = p.state + (int64_t)(in_range ? slot : 0) * p.stride;
 #pragma unroll
         for (int i = 0; i < VPT; ++i) {
           const int g = threadIdx.x + i * blockDim.x;
@@ -120,28 +138,26 @@ __global__ void __launch_bounds__(512) norm_shift_kernel(const NormShiftParams p
           if (from_state && g < groups)
             prev.v[i] = *reinterpret_cast<const float4*>(st + g * 4);
         }
-        norm_row<T, VPT>(p, t, true, h, red, flip);
-        if (in_range) {
-          // last row of the portion that starts here
-          int lo = 0, hi = p.num_portions;
-          while (hi - lo > 1) {
-            const int mid = (lo + hi) >> 1;
-            if (p.cu[mid] <= t) lo = mid; else hi = mid;
-          }
-          const int64_t last = (int64_t)p.cu[lo + 1] - 1;
-          Row<VPT> z = h;
-          if (last > t && last < p.rows) norm_row<T, VPT>(p, last, false, z, red, flip);
-#pragma unroll
-          for (int i = 0; i < VPT; ++i) {
-            const int g = threadIdx.x + i * blockDim.x;
-            if (g < groups) *reinterpret_cast<float4*>(st + g * 4) = z.v[i];
-          }
-        }
-      } else {
-        if (!have_prev) norm_row<T, VPT>(p, t - 1, false, prev, red, flip);
-        norm_row<T, VPT>(p, t, true, h, red, flip);
+      } else if (t == t0) {
+        one_row<T, VPT>(p, t - 1, prev, red, flip);
       }
-      have_prev = true;
+    }
+    norm_row<T, VPT>(p, t, true, h, y, red, flip);
+    if (in_range) {
+      // last row of the portion that starts here
+      int lo = 0, hi = p.num_portions;
+      while (hi - lo > 1) {
+        const int mid = (lo + hi) >> 1;
+        if (p.cu[mid] <= t) lo = mid; else hi = mid;
+      }
+      const int64_t last = (int64_t)p.cu[lo + 1] - 1;
+      Row<VPT> z = h;
+      if (last > t && last < p.rows) one_row<T, VPT>(p, last, z, red, flip);
+#pragma unroll
+      for (int i = 0; i < VPT; ++i) {
+        const int g = threadIdx.x + i * blockDim.x;
+        if (g < groups) *reinterpret_cast<float4*>(st + g * 4) = z.v[i];
+      }
     }
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
@@ -339,6 +355,128 @@ __global__ void __launch_bounds__(256) rope_rms_store_kernel(const RopeRmsParams
   }
 }
 
+// bf16, d and dp multiples of 8: LPH = dp / 8 lanes per head, 8 channels (4 pairs) a
+// lane, two tokens in flight.
+template <int LPH>
+__global__ void __launch_bounds__(256) rope_rms_store_vec_kernel(const RopeRmsParams p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  constexpr int TOK = 2;
+  const int j = threadIdx.x % LPH;
+  const int qheads = p.hkv * p.gp;
+  const int heads = qheads + p.hkv;
+  const int h = blockIdx.x * (256 / LPH) + threadIdx.x / LPH;
+  const bool is_q = h < qheads;
+  const int kvh = is_q ? h / p.gp : h - qheads;
+  const int in_group = is_q ? h - kvh * p.gp : 0;
+  const bool live = h < heads;
+  const bool real = live && (!is_q || in_group < p.g) && j * 8 < p.d;
+  const uint16_t* src = static_cast<const uint16_t*>(is_q ? p.q : p.k) +
+                        (is_q ? (int64_t)(kvh * p.g + in_group) : (int64_t)kvh) * p.d + j * 8;
+  const int half = p.rot >> 1;
+  const bool vec_cs = (half & 3) == 0;
+  const float inv_d = 1.0f / (float)p.d;
+  for (int64_t t0 = (int64_t)blockIdx.y * TOK; t0 < p.rows; t0 += (int64_t)gridDim.y * TOK) {
+    uint4 raw[TOK];
+    int64_t slot[TOK], pos[TOK];
+    float4 cs[TOK], sn[TOK];
+#pragma unroll
+    for (int i = 0; i < TOK; ++i) {
+      raw[i] = make_uint4(0u, 0u, 0u, 0u);
+      slot[i] = -1;
+      pos[i] = 0;
+      if (t0 + i < p.rows) {
+        if (real) raw[i] = *reinterpret_cast<const uint4*>(src + (t0 + i) * p.in_stride);
+        pos[i] = p.positions[t0 + i];
+        if (!is_q) slot[i] = p.slots[t0 + i];
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < TOK; ++i) {
+      if (pos[i] < 0 || pos[i] >= p.max_position) {
+        if (threadIdx.x == 0 && p.status) atomicOr(p.status, FK_DEV_BAD_POSITION);
+        pos[i] = 0;
+      }
+      const float* c = p.cos_sin + pos[i] * p.rot;
+      cs[i] = make_float4(1.f, 1.f, 1.f, 1.f);
+      sn[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      const int e = j * 4;
+      if (vec_cs) {
+        if (e < half) {
+          cs[i] = __ldg(reinterpret_cast<const float4*>(c + e));
+          sn[i] = __ldg(reinterpret_cast<const float4*>(c + half + e));
+        }
+      } else {
+        float* cf = reinterpret_cast<float*>(&cs[i]);
+        float* sf = reinterpret_cast<float*>(&sn[i]);
+#pragma unroll
+        for (int x = 0; x < 4; ++x)
+          if (e + x < half) {
+            cf[x] = __ldg(c + e + x);
+            sf[x] = __ldg(c + half + e + x);
+          }
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < TOK; ++i) {
+      const float u[4] = {bf16lo(raw[i].x), bf16lo(raw[i].y), bf16lo(raw[i].z), bf16lo(raw[i].w)};
+      const float v[4] = {bf16hi(raw[i].x), bf16hi(raw[i].y), bf16hi(raw[i].z), bf16hi(raw[i].w)};
+      const float c4[4] = {cs[i].x, cs[i].y, cs[i].z, cs[i].w};
+      const float s4[4] = {sn[i].x, sn[i].y, sn[i].z, sn[i].w};
+      float a[4], b[4], ss = 0.f;
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        a[x] = u[x] * c4[x] - v[x] * s4[x];
+        b[x] = v[x] * c4[x] + u[x] * s4[x];
+        ss += a[x] * a[x] + b[x] * b[x];
+      }
+#pragma unroll
+      for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      const float rs = rsqrtf(ss * inv_d + p.eps);
+      if (!live || t0 + i >= p.rows) continue;
+      const uint4 r = make_uint4(pack_bf16(a[0] * rs, b[0] * rs), pack_bf16(a[1] * rs, b[1] * rs),
+                                 pack_bf16(a[2] * rs, b[2] * rs), pack_bf16(a[3] * rs, b[3] * rs));
+      if (is_q) {
+        *reinterpret_cast<uint4*>(static_cast<uint16_t*>(p.q_out) +
+                                  ((t0 + i) * qheads + h) * p.dp + j * 8) = r;
+      } else if (slot[i] >= p.num_slots) {
+        if (p.status) atomicOr(p.status, FK_DEV_BAD_SLOT);
+      } else if (slot[i] >= 0) {
+        const int64_t off = (slot[i] * p.hkv + kvh) * p.dp + j * 8;
+        *reinterpret_cast<uint4*>(static_cast<uint16_t*>(p.k_cache) + off) = r;
+        *reinterpret_cast<uint4*>(static_cast<uint16_t*>(p.v_cache) + off) = raw[i];
+      }
+    }
+  }
+}
+
+// act(gate) * up on 8 bf16 at a time
+__global__ void __launch_bounds__(256) act_and_mul_bf16x8_kernel(
+    const uint16_t* __restrict__ x, int64_t x_stride, uint16_t* __restrict__ out,
+    int64_t out_stride, int64_t rows, int packs, int half, int kind) {
+  pdl_launch_dependents();
+  pdl_wait();
+  constexpr int TOK = 4;
+  const int c = blockIdx.x * blockDim.x + threadIdx.x;
+  if (c >= packs) return;
+  for (int64_t t0 = (int64_t)blockIdx.y * TOK; t0 < rows; t0 += (int64_t)gridDim.y * TOK) {
+    uint4 g[TOK], u[TOK];
+#pragma unroll
+    for (int i = 0; i < TOK; ++i)
+      if (t0 + i < rows) {
+        const uint16_t* row = x + (t0 + i) * x_stride + c * 8;
+        g[i] = *reinterpret_cast<const uint4*>(row);
+        u[i] = *reinterpret_cast<const uint4*>(row + half);
+      }
+#pragma unroll
+    for (int i = 0; i < TOK; ++i)
+      if (t0 + i < rows)
+        *reinterpret_cast<uint4*>(out + (t0 + i) * out_stride + c * 8) =
+            make_uint4(act_mul2(g[i].x, u[i].x, kind), act_mul2(g[i].y, u[i].y, kind),
+                       act_mul2(g[i].z, u[i].z, kind), act_mul2(g[i].w, u[i].w, kind));
+  }
+}
+
 __device__ __forceinline__ float act_f32(float g, int kind) {
   return kind == FK_ACT_SILU ? g * sigmoid_f32(g) : gelu_tanh_f32(g);
 }
@@ -525,6 +663,22 @@ int fk_rope_rms_store(const void* q, const void* k, int64_t in_stride, int is_f3
   const int64_t ny = rows < 8192 ? rows : 8192;
   const dim3 grid((unsigned)((heads + 7) / 8), (unsigned)ny);
   cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const bool vec = !is_f32 && head_dim % 8 == 0 && (padded_dim == 64 || padded_dim == 128) &&
+                   in_stride % 8 == 0 && aligned16(q) && aligned16(k) && aligned16(q_out) &&
+                   aligned16(k_cache) && aligned16(v_cache) && aligned16(cos_sin);
+  if (vec) {
+    const int per = 256 / (padded_dim / 8);
+    const int gx = (heads + per - 1) / per;
+    const int64_t pairs = (rows + 1) / 2;
+    int64_t gy = (int64_t)sm_count() * 16 / gx;
+    gy = gy < 1 ? 1 : gy < pairs ? gy : pairs;
+    const dim3 vgrid((unsigned)gx, (unsigned)gy);
+    FK_CUDA_OK(padded_dim == 64
+                   ? launch_kernel(rope_rms_store_vec_kernel<8>, vgrid, dim3(256), 0, s, p)
+                   : launch_kernel(rope_rms_store_vec_kernel<16>, vgrid, dim3(256), 0, s, p));
+    count_launch();
+    return FK_OK;
+  }
   FK_CUDA_OK(is_f32 ? launch_rope_rms<float>(p, grid, s) : launch_rope_rms<uint16_t>(p, grid, s));
   count_launch();
   return FK_OK;
@@ -542,15 +696,20 @@ int fk_act_and_mul(const void* x, int64_t x_stride, void* out, int64_t out_strid
              FK_ERR_ALIGNMENT, "fk_act_and_mul: rows must be 16-byte aligned");
   FK_REQUIRE(d < (1ll << 30) && x_stride >= 2 * d && out_stride >= d, FK_ERR_INVALID_ARG,
              "fk_act_and_mul: bad stride");
-  const int groups = (int)(d / 4);
-  const dim3 grid((unsigned)((groups + 255) / 256), (unsigned)(rows < 16384 ? rows : 16384));
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  cudaError_t e =
-      is_f32 ? launch_kernel(act_and_mul_kernel<float>, grid, dim3(256), 0, s, (const float*)x,
-                             x_stride, (float*)out, out_stride, rows, groups, (int)d, act)
-             : launch_kernel(act_and_mul_kernel<uint16_t>, grid, dim3(256), 0, s,
-                             (const uint16_t*)x, x_stride, (uint16_t*)out, out_stride, rows,
-                             groups, (int)d, act);
+  cudaError_t e;
+  if (is_f32) {
+    const int groups = (int)(d / 4);
+    const dim3 grid((unsigned)((groups + 255) / 256), (unsigned)(rows < 16384 ? rows : 16384));
+    e = launch_kernel(act_and_mul_kernel<float>, grid, dim3(256), 0, s, (const float*)x, x_stride,
+                      (float*)out, out_stride, rows, groups, (int)d, act);
+  } else {
+    const int packs = (int)(d / 8);
+    const int64_t quads = (rows + 3) / 4;
+    const dim3 grid((unsigned)((packs + 255) / 256), (unsigned)(quads < 16384 ? quads : 16384));
+    e = launch_kernel(act_and_mul_bf16x8_kernel, grid, dim3(256), 0, s, (const uint16_t*)x,
+                      x_stride, (uint16_t*)out, out_stride, rows, packs, (int)d, act);
+  }
   FK_CUDA_OK(e);
   count_launch();
   return FK_OK;
