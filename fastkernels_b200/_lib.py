@@ -120,9 +120,10 @@ PROTOTYPES = {
     "fk_gemm_bf16_act_mul": (_i32, [_vp, _i64, _vp, _vp, _vp, _i64, _i64, _i64, _i64, _i32, _vp,
                                     _sz, _vp, _vp]),
     "fk_delta_padded_dim": (_i32, [_i32]),
+    "fk_delta_packed_floats": (_i64, [_i64, _i32, _i32, _i32, _i32]),
     "fk_delta_prepare": (_i32, [_vp, _vp, _vp, _vp, _vp, _i64, _i32, _vp, _i64, _vp, _vp, _vp,
-                                _i64, _i32, _i32, _i32, _f32, _f32, _vp]),
-    "fk_delta_scan": (_i32, [_vp, _vp, _vp, _i32, _vp, _i32, _vp, _vp, _i64, _i32, _i32, _vp,
+                                _i32, _vp, _i32, _i64, _i32, _i32, _i32, _f32, _f32, _vp]),
+    "fk_delta_scan": (_i32, [_vp, _i32, _vp, _vp, _i32, _vp, _i32, _vp, _vp, _i64, _i32, _i32, _vp,
                              _vp]),
     "fk_delta_output": (_i32, [_vp, _vp, _i64, _vp, _vp, _i64, _i32, _i64, _i32, _i32, _f32,
                                _vp]),

@@ -135,9 +135,10 @@ class GeneralizedDelta:
         ctx = get_context()
         packed = ops.delta_prepare(cols["r"], cols["k"], cols["v"], cols["a"], cols["w1"],
                                    self.w2, self.w0, self.a_bias, self.heads, self.dim,
-                                   self.DECAY_SCALE, self.UNIT_EPS)
+                                   self.DECAY_SCALE, self.UNIT_EPS,
+                                   cu_portions=ctx.cu_portions if ctx.is_prefill else None)
         o = ops.delta_scan(packed, self.states[run], ctx.cu_portions, ctx.state_slots, positions,
-                           self.dim, status=self.status)
+                           ctx.is_prefill, status=self.status)
         out = torch.empty((positions.shape[0], self.out_columns), dtype=self.dtype,
                           device=positions.device)
         return ops.delta_output(o, cols["g"], self.norm, self.heads, self.dim, self.eps, out)

@@ -668,10 +668,10 @@ def delta_padded_dim(dim: int) -> int:
 
 
 def delta_prepare(r, k, v, a, y1, w2, w0, a_bias, heads, dim, decay_scale, unit_eps,
-                  packed=None):
-    """Per-token operands of the delta rule, packed [heads, T, 6, padded_dim] fp32.
-    r, k, v, a [T, heads * dim] and y1 [T, rank] are column ranges of the same rows;
-    w2 [heads * dim, padded rank]."""
+                  cu_portions=None, packed=None):
+    """Operands of the delta rule (fp32, opaque): in blocks of 8 tokens of the portions
+    when cu_portions is given, else token by token.  r, k, v, a [T, heads * dim] and
+    y1 [T, rank] are column ranges of the same rows; w2 [heads * dim, padded rank]."""
     f32 = _is_f32(k, "k")
     rows, rank = y1.shape
     for name, t in (("r", r), ("v", v), ("a", a), ("y1", y1), ("w2", w2)):
@@ -682,33 +682,42 @@ def delta_prepare(r, k, v, a, y1, w2, w0, a_bias, heads, dim, decay_scale, unit_
     _need(a_bias, torch.float32, "a_bias")
     if not w2.is_contiguous() or w2.shape[0] != heads * dim:
         raise _lib.FkError("w2 must be contiguous [heads * dim, padded rank]")
+    n_port = 0
+    if cu_portions is not None:
+        _need(cu_portions, torch.int32, "cu_portions")
+        n_port = cu_portions.numel() - 1
+    delta_padded_dim(dim)
     if packed is None:
-        packed = torch.empty((heads, rows, 6, delta_padded_dim(dim)), dtype=torch.float32,
-                             device=k.device)
+        n = int(lib.fk_delta_packed_floats(rows, n_port, heads, dim, int(n_port > 0)))
+        packed = torch.empty(n, dtype=torch.float32, device=k.device)
     check(lib.fk_delta_prepare(
         _ptr(r), _ptr(k), _ptr(v), _ptr(a), _ptr(y1), k.stride(0) if rows else 0, f32, _ptr(w2),
-        w2.shape[1], _ptr(w0), _ptr(a_bias), _ptr(packed), rows, heads, dim, rank,
-        float(decay_scale), float(unit_eps), _stream()), "fk_delta_prepare")
+        w2.shape[1], _ptr(w0), _ptr(a_bias), _ptr(packed), int(n_port > 0), _ptr(cu_portions),
+        n_port, rows, heads, dim, rank, float(decay_scale), float(unit_eps), _stream()),
+        "fk_delta_prepare")
     return packed
 
 
-def delta_scan(packed, state, cu_portions, slots, positions, dim, out=None, status=None):
-    """The recurrence over packed operands; state [slots, heads, dim, padded_dim] fp32
-    is read and replaced.  Returns o [T, heads * dim] fp32."""
+def delta_scan(packed, state, cu_portions, slots, positions, blocked, out=None, status=None):
+    """The recurrence over prepared operands (`blocked`: prepared with cu_portions);
+    state [slots, heads, dim, padded_dim] fp32 is read and replaced.  Returns
+    o [T, heads * dim] fp32."""
     _need(packed, torch.float32, "packed")
     _need(state, torch.float32, "state")
     _need(cu_portions, torch.int32, "cu_portions")
     _need(slots, torch.int32, "slots")
     _need(positions, torch.int64, "positions")
-    heads, rows = packed.shape[0], packed.shape[1]
+    rows, heads, dim = positions.shape[0], state.shape[1], state.shape[2]
+    n_port = cu_portions.numel() - 1
     if not packed.is_contiguous() or not state.is_contiguous() or \
-            tuple(state.shape[1:]) != (heads, dim, packed.shape[3]):
+            state.shape[3] != delta_padded_dim(dim) or packed.numel() < \
+            int(lib.fk_delta_packed_floats(rows, n_port, heads, dim, int(bool(blocked)))):
         raise _lib.FkError("delta_scan: packed or state has the wrong shape")
     if out is None:
         out = torch.empty((rows, heads * dim), dtype=torch.float32, device=packed.device)
     check(lib.fk_delta_scan(
-        _ptr(packed), _ptr(out), _ptr(state), state.shape[0], _ptr(cu_portions),
-        cu_portions.numel() - 1, _ptr(slots), _ptr(positions), rows, heads, dim,
+        _ptr(packed), int(bool(blocked)), _ptr(out), _ptr(state), state.shape[0],
+        _ptr(cu_portions), n_port, _ptr(slots), _ptr(positions), rows, heads, dim,
         _status_ptr(status, packed), _stream()), "fk_delta_scan")
     return out
 

@@ -636,20 +636,25 @@ int fk_gemm_bf16_act_mul(const void* x, int64_t x_stride, const void* w, const v
  *   w_t = exp(-decay_scale * sigmoid(w2 tanh(y1) + w0)), a_t = sigmoid(a + a_bias),
  *   u_t = k_t / sqrt(sum k_t^2 + unit_eps)
  * fk_delta_padded_dim: key channels per head in `packed` and `state` (0: unsupported,
- * head size above 256).  fk_delta_prepare writes packed [heads][rows][6][padded_dim]
- * fp32 (w, u, a * u, k, r, v) from packed projection rows; w2 [heads * dim, w2_stride]
- * in the activation type, rows zero-padded to a multiple of 4 (rank <= 512).
+ * head size above 256).  fk_delta_prepare writes the operands of the scan from packed
+ * projection rows; w2 [heads * dim, w2_stride] in the activation type, rows zero-padded
+ * to a multiple of 4 (rank <= 512).  blocked 0: per token, packed
+ * [heads][rows][6][padded_dim] fp32 (w, u, a * u, k, r, v), for single tokens;
+ * blocked 1: blocks of 8 tokens of a portion (layout: csrc/fk_delta.cu), for portions.
+ * fk_delta_packed_floats: size of `packed` in floats.
  * fk_delta_scan runs the recurrence for every portion from and to
  * state [num_slots][heads][dim (value)][padded_dim (key)] fp32 and writes
  * o [rows, heads * dim] fp32.  fk_delta_output: out = rms(o per head) * weight *
  * sigmoid(gate), columns beyond heads * dim zeroed. */
 int fk_delta_padded_dim(int dim);
+int64_t fk_delta_packed_floats(int64_t rows, int num_portions, int heads, int dim, int blocked);
 int fk_delta_prepare(const void* r, const void* k, const void* v, const void* a, const void* y1,
                      int64_t in_stride, int is_f32, const void* w2, int64_t w2_stride,
-                     const float* w0, const float* a_bias, float* packed, int64_t rows,
+                     const float* w0, const float* a_bias, float* packed, int blocked,
+                     const int32_t* cu_portions, int num_portions, int64_t rows,
                      int heads, int dim, int rank, float decay_scale, float unit_eps,
                      fk_stream_t stream);
-int fk_delta_scan(const float* packed, float* o, float* state, int num_slots,
+int fk_delta_scan(const float* packed, int blocked, float* o, float* state, int num_slots,
                   const int32_t* cu_portions, int num_portions, const int32_t* slots,
                   const int64_t* positions, int64_t rows, int heads, int dim, int32_t* status,
                   fk_stream_t stream);

@@ -396,7 +396,7 @@ def test_delta_rule_in_portions(heads, dim, rank, dtype):
     slots, at = [4, 0, 2], [0, 0, 0]
     st = ops.new_status("cuda")
 
-    def run(portions):
+    def run(portions, blocked=True):
         z = np.concatenate([rows[i][at[i]:at[i] + n] for i, n in portions] + [rows[0][:1]])
         cu = np.concatenate([[0], np.cumsum([n for _, n in portions] + [1])])
         pos = np.concatenate([np.arange(at[i], at[i] + n) for i, n in portions] + [[0]])
@@ -405,9 +405,10 @@ def test_delta_rule_in_portions(heads, dim, rank, dtype):
         col = {n: zd[:, o:o + w] for n, o, w in zip(names + ["y1"], offs, widths)}
         packed = ops.delta_prepare(col["r"], col["k"], col["v"], col["a"], col["y1"],
                                    dev(w2p, dtype), dev(w0), dev(ab), heads, dim,
-                                   float(np.exp(-0.5)), 1e-6)
+                                   float(np.exp(-0.5)), 1e-6,
+                                   cu_portions=i32(cu) if blocked else None)
         o = torch.zeros((len(z), hd), device="cuda")
-        ops.delta_scan(packed, state, i32(cu), i32(sl), i64(pos), dim, out=o, status=st)
+        ops.delta_scan(packed, state, i32(cu), i32(sl), i64(pos), blocked, out=o, status=st)
         out = torch.full((len(z), (hd + 63) // 64 * 64), 9.0, dtype=dtype, device="cuda")
         ops.delta_output(o, col["g"], dev(norm), heads, dim, eps, out)
         row = 0
@@ -422,11 +423,12 @@ def test_delta_rule_in_portions(heads, dim, rank, dtype):
     run([(0, 1), (1, 40)])
     run([(0, 2), (2, 9)])
     run([(2, 1), (0, 40), (1, 1)])
-    for _ in range(5):
-        run([(0, 1), (1, 1), (2, 1)])
+    for x in range(5):
+        run([(0, 1), (1, 1), (2, 1)], blocked=x % 2 == 0)
     run([(2, 17)])
+    run([(2, 5)], blocked=False)
     while at[1] < total or at[0] < total:
-        run([(i, 1) for i in (0, 1) if at[i] < total])
+        run([(i, 1) for i in (0, 1) if at[i] < total], blocked=False)
     assert int(st.item()) == 0
     for i in (0, 1):
         got = state[slots[i], :, :, :dim].permute(0, 2, 1)
@@ -435,30 +437,47 @@ def test_delta_rule_in_portions(heads, dim, rank, dtype):
 
 
 def test_delta_rule_long_run_does_not_drift():
-    """1500 tokens with slow decay in one portion and in portions of 7 give the same
-    state, close to the plain recurrence."""
+    """1500 tokens with slow decay in one portion, in portions of 7 and of 64, and token
+    by token give the same state, close to the plain recurrence; many heads and
+    sequences as few."""
     from fastkernels_b200 import ops
     rs = np.random.RandomState(9)
-    t, dim = 1500, 24
-    r, k, v = (rs.randn(t, 1, dim) for _ in range(3))
-    decay, rate = rs.uniform(0.97, 1, (t, 1, dim)), rs.uniform(0, 1, (t, 1, dim))
-    dp = ops.delta_padded_dim(dim)
-    u = k / np.sqrt((k * k).sum(-1, keepdims=True) + 1e-6)
-    packed = np.zeros((1, t, 6, dp))
-    for f, a in enumerate((decay, u, rate * u, k, r, v)):
-        packed[0, :, f, :dim] = a[:, 0]
-    want, s = P.delta_rule(r, k, v, decay, rate)
+    t, dim, rank = 1500, 24, 4
+    z = P.bf16(rs.randn(t, 4 * dim + 8))
+    w2, w0, ab = P.bf16(rs.randn(dim, rank)), np.full(dim, -4.0), rs.randn(dim)
+    r, k, v, a = (z[:, i * dim:(i + 1) * dim].reshape(t, 1, dim) for i in range(4))
+    decay = P.delta_decay(z[:, 4 * dim:4 * dim + rank], w2, w0).reshape(t, 1, dim)
+    want, s = P.delta_rule(r, k, v, decay, P.sigmoid(a + ab))
     outs = []
-    for step in (t, 7):
-        state = torch.zeros((1, 1, dim, dp), device="cuda")
+    for step, blocked, copies in ((t, True, 1), (t, True, 700), (7, True, 1), (64, True, 1),
+                                  (50, False, 1)):
+        zd = dev(z)
+        col = [zd[:, i * dim:(i + 1) * dim] for i in range(4)] + [zd[:, 4 * dim:4 * dim + rank]]
+        state = torch.zeros((copies, 1, dim, ops.delta_padded_dim(dim)), device="cuda")
         o = []
-        for a in range(0, t, step):
-            n = min(step, t - a)
-            o.append(ops.delta_scan(dev(packed[:, a:a + n]), state, i32([0, n]), i32([0] * n),
-                                    i64(np.arange(a, a + n)), dim))
-        outs.append(torch.cat(o))
-        close(outs[-1], want[:, 0], F32, scale=np.abs(want).max())
-    torch.testing.assert_close(outs[0], outs[1], rtol=1e-5, atol=1e-4)
+        for at in range(0, t, step):
+            n = min(step, t - at)
+            cols = [c[at:at + n] for c in col]
+            if copies > 1:               # the same sequence many times over
+                big = zd[:200].repeat(copies, 1)
+                cols = [big[:, i * dim:(i + 1) * dim] for i in range(4)] + \
+                    [big[:, 4 * dim:4 * dim + rank]]
+                n = 200
+            cu = i32(np.arange(copies + 1) * n)
+            packed = ops.delta_prepare(*cols, dev(w2), dev(w0), dev(ab), 1, dim,
+                                       float(np.exp(-0.5)), 1e-6, cu_portions=cu if blocked else None)
+            o.append(ops.delta_scan(packed, state, cu, i32(np.repeat(np.arange(copies), n)),
+                                    i64(np.tile(np.arange(at, at + n), copies)), blocked))
+        o = torch.cat(o)
+        if copies > 1:
+            ref = dev(want[:200, 0]).repeat(copies, 1)
+            torch.testing.assert_close(o, ref, rtol=1e-4, atol=1e-4 * float(ref.abs().max()))
+            continue
+        outs.append(o)
+        close(o, want[:, 0], F32, scale=2 * np.abs(want).max())
+        close(state[0, :, :, :dim].permute(0, 2, 1), s, F32, scale=2 * np.abs(s).max())
+    for o in outs[1:]:
+        torch.testing.assert_close(outs[0], o, rtol=1e-4, atol=1e-3)
 
 
 # ------------------------------------------------------------------- the whole decoder
