@@ -130,6 +130,12 @@ PROTOTYPES = {
     "fk_gemm_f32": (_i32, [_vp, _i64, _vp, _vp, _i64, _i64, _i64, _i64, _vp]),
     "fk_paged_attn_any": (_i32, [_vp, _i64, _vp, _i64, _vp, _vp, _i32, _i64, _i32, _vp, _vp, _vp,
                                  _i64, _i32, _i64, _i32, _i32, _i32, _f32, _vp, _vp]),
+    "fk_paged_decode_attn_2p": (_i32, [_i32, _vp, _i64, _vp, _i64, _vp, _vp, _i64, _i32, _i64,
+                                       _i32, _vp, _vp, _i64, _i32, _i32, _i32, _i32, _f32, _i32,
+                                       _vp, _sz, _vp, _vp]),
+    "fk_prefill_attn_2p": (_i32, [_vp, _i64, _vp, _i64, _vp, _vp, _vp, _i64, _i64, _i32, _i32,
+                                  _vp, _vp, _vp, _i64, _i32, _i64, _i64, _i32, _i32, _i32, _i32,
+                                  _f32, _i32, _vp, _vp]),
     "fk_argmax_f32": (_i32, [_vp, _i64, _i64, _i64, _vp, _vp, _vp]),
     "fk_gemm_bf16_static": (_i32, [_vp, _i64, _vp, _vp, _vp, _i64, _i64, _i64, _i64, _vp, _vp]),
     "fk_gemm_bf16": (_i32, [_vp, _i64, _vp, _vp, _vp, _i64, _i64, _i64, _i64, _vp, _sz,

@@ -227,7 +227,9 @@ __global__ void __launch_bounds__(1024) attn_plan_kernel(
 // ---------------------------------------------------------------------------
 // main kernel
 // ---------------------------------------------------------------------------
-template <bool G16>
+// SPLIT: the softmax weights enter P V as two bf16 parts (16 significant bits) instead
+// of one.
+template <bool G16, bool SPLIT>
 __global__ void __launch_bounds__(ATT_THREADS, 1) attn_decode_kernel(
     const __grid_constant__ CUtensorMap tmap_k,
     const __grid_constant__ CUtensorMap tmap_v, const AttnParams p) {
@@ -541,6 +543,17 @@ __global__ void __launch_bounds__(ATT_THREADS, 1) attn_decode_kernel(
         pa[1] = 0u;
         pa[3] = 0u;
       }
+      uint32_t pl[4] = {0u, 0u, 0u, 0u};
+      if (SPLIT) {
+#pragma unroll
+        for (int h = 0; h < (G16 ? 2 : 1); ++h)
+#pragma unroll
+          for (int nt = 0; nt < 2; ++nt) {
+            const uint32_t hi2 = pa[h + 2 * nt];
+            pl[h + 2 * nt] = pack_bf16(pa_f[nt][2 * h] - bf16lo(hi2),
+                                       pa_f[nt][2 * h + 1] - bf16hi(hi2));
+          }
+      }
 
       // ---- O += P V (16 x 128 per warp) ----
       {
@@ -555,6 +568,10 @@ __global__ void __launch_bounds__(ATT_THREADS, 1) attn_decode_kernel(
                                 (((c & 7) ^ sw) << 4);
           uint32_t b0, b1, b2, b3;
           ldmatrix_x4_trans(addr, b0, b1, b2, b3);
+          if (SPLIT) {
+            mma_bf16_16816(o[2 * pr], pl, b0, b1);
+            mma_bf16_16816(o[2 * pr + 1], pl, b2, b3);
+          }
           mma_bf16_16816(o[2 * pr], pa, b0, b1);
           mma_bf16_16816(o[2 * pr + 1], pa, b2, b3);
         }
@@ -815,7 +832,24 @@ size_t fk_paged_decode_attn_workspace_bytes(int batch, int num_q_heads,
          parts * sizeof(float2);
 }
 
-static int attn_impl(int mode, const void* q, int64_t q_stride_token, void* out,
+// launch of the main kernel: 16 query heads per KV head or fewer, weights in one part
+// or two
+static cudaError_t launch_decode(bool g16, bool split, int grid, const CUtensorMap& mk,
+                                 const CUtensorMap& mv, const AttnParams& p, cudaStream_t s) {
+  static PerDeviceOnce once[4];
+  auto go = [&](PerDeviceOnce& o, auto kernel) {
+    const cudaError_t e = set_max_dynamic_smem(o, kernel, AttnSmem::kAlloc);
+    if (e != cudaSuccess) return e;
+    return launch_kernel(kernel, dim3(grid), dim3(ATT_THREADS), (size_t)AttnSmem::kAlloc, s, mk,
+                         mv, p);
+  };
+  if (g16) return split ? go(once[3], attn_decode_kernel<true, true>)
+                        : go(once[1], attn_decode_kernel<true, false>);
+  return split ? go(once[2], attn_decode_kernel<false, true>)
+               : go(once[0], attn_decode_kernel<false, false>);
+}
+
+static int attn_impl(int mode, bool split, const void* q, int64_t q_stride_token, void* out,
                          int64_t out_stride_token, const void* k_cache,
                          const void* v_cache, int64_t num_blocks,
                          int block_size, int64_t kv_block_stride, int kv_layout,
@@ -927,20 +961,11 @@ static int attn_impl(int mode, const void* q, int64_t q_stride_token, void* out,
   p.status = status;
 
   const int grid = sm_count();
-  static PerDeviceOnce attr_nhd, attr_hnd;
-  FK_CUDA_OK(set_max_dynamic_smem(attr_nhd, attn_decode_kernel<false>, AttnSmem::kAlloc));
-  FK_CUDA_OK(set_max_dynamic_smem(attr_hnd, attn_decode_kernel<true>, AttnSmem::kAlloc));
 
   if (direct) {
     const int dgrid = batch * num_kv_heads;
-    if (g > 8)
-      FK_LAUNCH(attn_decode_kernel<true>, dim3(dgrid), dim3(ATT_THREADS),
-                (size_t)AttnSmem::kAlloc, s, mk, mv, p);
-    else
-      FK_LAUNCH(attn_decode_kernel<false>, dim3(dgrid), dim3(ATT_THREADS),
-                (size_t)AttnSmem::kAlloc, s, mk, mv, p);
+    FK_CUDA_OK(launch_decode(g > 8, split, dgrid, mk, mv, p, s));
     count_launch(1);
-    FK_CUDA_OK(cudaGetLastError());
     return FK_OK;
   }
   if (mode != 2) {
@@ -953,12 +978,7 @@ static int attn_impl(int mode, const void* q, int64_t q_stride_token, void* out,
     FK_CUDA_OK(cudaGetLastError());
     return FK_OK;
   }
-  if (g > 8)
-    FK_LAUNCH(attn_decode_kernel<true>, dim3(grid), dim3(ATT_THREADS),
-              (size_t)AttnSmem::kAlloc, s, mk, mv, p);
-  else
-    FK_LAUNCH(attn_decode_kernel<false>, dim3(grid), dim3(ATT_THREADS),
-              (size_t)AttnSmem::kAlloc, s, mk, mv, p);
+  FK_CUDA_OK(launch_decode(g > 8, split, grid, mk, mv, p, s));
   const int warps = batch * num_q_heads;
   FK_LAUNCH(attn_merge_kernel, dim3((warps * 32 + 255) / 256), dim3(256), 0, s, p);
   count_launch(2);
@@ -977,7 +997,7 @@ int fk_paged_decode_attn(const void* q, int64_t q_stride_token, void* out,
                          float softmax_scale, int max_splits, void* workspace,
                          size_t workspace_bytes, int32_t* status,
                          fk_stream_t stream) {
-  return attn_impl(0, q, q_stride_token, out, out_stride_token, k_cache, v_cache,
+  return attn_impl(0, false, q, q_stride_token, out, out_stride_token, k_cache, v_cache,
                    num_blocks, block_size, kv_block_stride, kv_layout, context_lens,
                    block_tables,
                    block_table_stride, batch, num_q_heads, num_kv_heads, head_dim,
@@ -991,7 +1011,7 @@ int fk_paged_decode_attn_plan(const int32_t* context_lens,
                               int max_splits, void* workspace,
                               size_t workspace_bytes, int32_t* status,
                               fk_stream_t stream) {
-  return attn_impl(1, nullptr, (int64_t)num_q_heads * head_dim, nullptr,
+  return attn_impl(1, false, nullptr, (int64_t)num_q_heads * head_dim, nullptr,
                    (int64_t)num_q_heads * head_dim, nullptr, nullptr, 1, block_size,
                    (int64_t)block_size * num_kv_heads * head_dim, 0, context_lens,
                    block_tables, block_table_stride, batch, num_q_heads, num_kv_heads,
@@ -1010,10 +1030,28 @@ int fk_paged_decode_attn_planned(const void* q, int64_t q_stride_token, void* ou
                                  float softmax_scale, int max_splits,
                                  void* workspace, size_t workspace_bytes,
                                  int32_t* status, fk_stream_t stream) {
-  return attn_impl(2, q, q_stride_token, out, out_stride_token, k_cache, v_cache,
+  return attn_impl(2, false, q, q_stride_token, out, out_stride_token, k_cache, v_cache,
                    num_blocks, block_size, kv_block_stride, kv_layout, context_lens,
                    block_tables,
                    block_table_stride, batch, num_q_heads, num_kv_heads, head_dim,
+                   softmax_scale, max_splits, workspace, workspace_bytes, status, stream);
+}
+
+int fk_paged_decode_attn_2p(int planned, const void* q, int64_t q_stride_token, void* out,
+                            int64_t out_stride_token, const void* k_cache,
+                            const void* v_cache, int64_t num_blocks,
+                            int block_size, int64_t kv_block_stride,
+                            int kv_layout,
+                            const int32_t* context_lens,
+                            const int32_t* block_tables,
+                            int64_t block_table_stride, int batch,
+                            int num_q_heads, int num_kv_heads, int head_dim,
+                            float softmax_scale, int max_splits,
+                            void* workspace, size_t workspace_bytes,
+                            int32_t* status, fk_stream_t stream) {
+  return attn_impl(planned ? 2 : 0, true, q, q_stride_token, out, out_stride_token, k_cache,
+                   v_cache, num_blocks, block_size, kv_block_stride, kv_layout, context_lens,
+                   block_tables, block_table_stride, batch, num_q_heads, num_kv_heads, head_dim,
                    softmax_scale, max_splits, workspace, workspace_bytes, status, stream);
 }
 

@@ -48,8 +48,8 @@ inline bool aligned16(const void* p) {
 bool pdl_enabled();
 
 template <typename... KArgs, typename... Args>
-inline cudaError_t launch_kernel(void (*kernel)(KArgs...), dim3 grid, dim3 block,
-                                 size_t smem, cudaStream_t stream, Args... args) {
+inline cudaError_t launch_kernel_pdl(bool early, void (*kernel)(KArgs...), dim3 grid, dim3 block,
+                                     size_t smem, cudaStream_t stream, Args... args) {
   cudaLaunchConfig_t cfg{};
   cfg.gridDim = grid;
   cfg.blockDim = block;
@@ -59,8 +59,20 @@ inline cudaError_t launch_kernel(void (*kernel)(KArgs...), dim3 grid, dim3 block
   attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
   attr[0].val.programmaticStreamSerializationAllowed = 1;
   cfg.attrs = attr;
-  cfg.numAttrs = pdl_enabled() ? 1 : 0;
+  cfg.numAttrs = early && pdl_enabled() ? 1 : 0;
   return cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...);
+}
+template <typename... KArgs, typename... Args>
+inline cudaError_t launch_kernel(void (*kernel)(KArgs...), dim3 grid, dim3 block,
+                                 size_t smem, cudaStream_t stream, Args... args) {
+  return launch_kernel_pdl(true, kernel, grid, block, smem, stream, args...);
+}
+// For a kernel whose CTAs should find empty SMs: it starts when its predecessors have
+// ended.
+template <typename... KArgs, typename... Args>
+inline cudaError_t launch_kernel_after(void (*kernel)(KArgs...), dim3 grid, dim3 block,
+                                       size_t smem, cudaStream_t stream, Args... args) {
+  return launch_kernel_pdl(false, kernel, grid, block, smem, stream, args...);
 }
 
 #define FK_LAUNCH(kernel, ...) (void)::fk::launch_kernel(kernel, __VA_ARGS__)

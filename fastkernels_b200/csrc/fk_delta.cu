@@ -62,6 +62,16 @@ struct DeltaPrepParams {
   float decay_scale, unit_eps;
 };
 
+// fp32 exponential and sigmoid: the hardware approximations (relative error around
+// 1e-6) beside bf16 operands, the accurate functions beside fp32 ones.
+template <typename T>
+struct Gate {
+  static __device__ __forceinline__ float exp(float x) { return sizeof(T) == 2 ? __expf(x) : expf(x); }
+  static __device__ __forceinline__ float sigmoid(float z) {
+    return sizeof(T) == 2 ? __fdividef(1.0f, 1.0f + __expf(-z)) : sigmoid_f32(z);
+  }
+};
+
 // CTA = 16 tokens, some heads in turn.
 template <typename T, int DP, bool BLOCKED>
 __global__ void __launch_bounds__(DL_THREADS) delta_prepare_kernel(const DeltaPrepParams p) {
@@ -91,7 +101,8 @@ __global__ void __launch_bounds__(DL_THREADS) delta_prepare_kernel(const DeltaPr
   uint16_t* lo = hi + DL_UNIT * ld;
   float* th = reinterpret_cast<float*>(dl_prep_smem);            // fp32: [16][rank_p]
   float* vec = reinterpret_cast<float*>(dl_prep_smem) + DL_UNIT * ld;   // [6][16][DP]
-  float* unit = vec + DL_FIELDS * DL_UNIT * DP;                  // [16]
+  float* part = vec + DL_FIELDS * DL_UNIT * DP;                  // [16][DP / 32]
+  float* unit = part + DL_UNIT * (DP / 32);                      // [16]
   for (int i = threadIdx.x; i < DL_UNIT * rank_p; i += DL_THREADS) {
     const int t = i / rank_p, r = i - t * rank_p;
     float z = 0.f;
@@ -116,6 +127,50 @@ __global__ void __launch_bounds__(DL_THREADS) delta_prepare_kernel(const DeltaPr
   for (int h = blockIdx.y * p.heads_per_cta; h < h1; ++h) {
     __syncthreads();       // tanh written; vec and unit of the last head consumed
     const int64_t ch0 = (int64_t)h * p.d;
+    // this thread's elements of the head's [16][DP] tile.  Single tokens: requested before
+    // the decay projection so that their latency passes behind it; blocks: as they are
+    // needed, many CTAs share an SM
+    constexpr int F = DL_UNIT * DP;                      // floats of one field
+    constexpr int NIT = F / DL_THREADS;
+    constexpr int PASS = BLOCKED ? 4 : NIT < 16 ? NIT : 16;
+    constexpr int SL = DP / 32;                          // warps that hold one token
+    // element x: token tok(x), channel chan(x); one channel per thread up to DP = 128
+    constexpr int TSTEP = DP <= DL_THREADS ? DL_THREADS / DP : 1;
+    constexpr int CPT = DP <= DL_THREADS ? 1 : DP / DL_THREADS;
+    const int c_first = DP <= DL_THREADS ? (int)(threadIdx.x % DP) : (int)threadIdx.x;
+    const int t_first = DP <= DL_THREADS ? (int)(threadIdx.x / DP) : 0;
+    auto tok = [&](int x) { return t_first + x / CPT * TSTEP; };
+    auto chan = [&](int x) { return c_first + x % CPT * DL_THREADS; };
+    const int64_t base = (t0 + t_first) * p.in_stride + ch0 + c_first;
+    const T* pk = static_cast<const T*>(p.k) + base;
+    const T* pa = static_cast<const T*>(p.a) + base;
+    const T* pr = static_cast<const T*>(p.r) + base;
+    const T* pv = static_cast<const T*>(p.v) + base;
+    auto offset = [&](int x) {
+      return (int64_t)(x / CPT * TSTEP) * p.in_stride + x % CPT * DL_THREADS;
+    };
+    float w0c[CPT], abc[CPT];
+#pragma unroll
+    for (int x = 0; x < CPT; ++x) {
+      const bool on = chan(x) < p.d;
+      w0c[x] = on ? __ldg(p.w0 + ch0 + chan(x)) : 0.f;
+      abc[x] = on ? __ldg(p.a_bias + ch0 + chan(x)) : 0.f;
+    }
+    T kx[PASS], ax[PASS], rx[PASS], vx[PASS];
+    auto fetch = [&](int x0) {
+#pragma unroll
+      for (int x = 0; x < PASS; ++x) {
+        kx[x] = ax[x] = rx[x] = vx[x] = T(0);
+        if (tok(x0 + x) < nt && chan(x0 + x) < p.d) {
+          const int64_t o = offset(x0 + x);
+          kx[x] = __ldg(pk + o);
+          ax[x] = __ldg(pa + o);
+          rx[x] = __ldg(pr + o);
+          vx[x] = __ldg(pv + o);
+        }
+      }
+    };
+    if (!BLOCKED) fetch(0);
     // decay projection into field 0
     if (MMA) {
       const int kq = (lane & 3) * 2, r0 = lane >> 2;
@@ -124,24 +179,33 @@ __global__ void __launch_bounds__(DL_THREADS) delta_prepare_kernel(const DeltaPr
         const int ch = n0 + r0;
         const bool on = ch < p.d;
         const uint16_t* w2 = static_cast<const uint16_t*>(p.w2) + (ch0 + (on ? ch : 0)) * p.w2_stride;
-#pragma unroll 4
-        for (int k0 = 0; k0 < rank_p; k0 += 16) {
-          uint32_t b0 = 0, b1 = 0;
-          if (on && k0 + kq < p.w2_stride) b0 = *reinterpret_cast<const uint32_t*>(w2 + k0 + kq);
-          if (on && k0 + kq + 8 < p.w2_stride)
-            b1 = *reinterpret_cast<const uint32_t*>(w2 + k0 + kq + 8);
-          const uint16_t* ah = hi + r0 * ld + k0 + kq;
-          const uint16_t* al = lo + r0 * ld + k0 + kq;
-          const uint32_t fh[4] = {*reinterpret_cast<const uint32_t*>(ah),
-                                  *reinterpret_cast<const uint32_t*>(ah + 8 * ld),
-                                  *reinterpret_cast<const uint32_t*>(ah + 8),
-                                  *reinterpret_cast<const uint32_t*>(ah + 8 * ld + 8)};
-          const uint32_t fl[4] = {*reinterpret_cast<const uint32_t*>(al),
-                                  *reinterpret_cast<const uint32_t*>(al + 8 * ld),
-                                  *reinterpret_cast<const uint32_t*>(al + 8),
-                                  *reinterpret_cast<const uint32_t*>(al + 8 * ld + 8)};
-          mma_bf16_16816(c, fl, b0, b1);
-          mma_bf16_16816(c, fh, b0, b1);
+        for (int k1 = 0; k1 < rank_p; k1 += 128) {
+          uint32_t b0[8], b1[8];
+#pragma unroll
+          for (int x = 0; x < 8; ++x) {
+            const int k0 = k1 + x * 16 + kq;
+            b0[x] = b1[x] = 0u;
+            if (on && k0 < p.w2_stride) b0[x] = __ldg(reinterpret_cast<const uint32_t*>(w2 + k0));
+            if (on && k0 + 8 < p.w2_stride)
+              b1[x] = __ldg(reinterpret_cast<const uint32_t*>(w2 + k0 + 8));
+          }
+#pragma unroll
+          for (int x = 0; x < 8; ++x) {
+            const int k0 = k1 + x * 16;
+            if (k0 >= rank_p) break;
+            const uint16_t* ah = hi + r0 * ld + k0 + kq;
+            const uint16_t* al = lo + r0 * ld + k0 + kq;
+            const uint32_t fh[4] = {*reinterpret_cast<const uint32_t*>(ah),
+                                    *reinterpret_cast<const uint32_t*>(ah + 8 * ld),
+                                    *reinterpret_cast<const uint32_t*>(ah + 8),
+                                    *reinterpret_cast<const uint32_t*>(ah + 8 * ld + 8)};
+            const uint32_t fl[4] = {*reinterpret_cast<const uint32_t*>(al),
+                                    *reinterpret_cast<const uint32_t*>(al + 8 * ld),
+                                    *reinterpret_cast<const uint32_t*>(al + 8),
+                                    *reinterpret_cast<const uint32_t*>(al + 8 * ld + 8)};
+            mma_bf16_16816(c, fl, b0[x], b1[x]);
+            mma_bf16_16816(c, fh, b0[x], b1[x]);
+          }
         }
         *reinterpret_cast<float2*>(vec + r0 * DP + n0 + kq) = make_float2(c[0], c[1]);
         *reinterpret_cast<float2*>(vec + (r0 + 8) * DP + n0 + kq) = make_float2(c[2], c[3]);
@@ -157,50 +221,56 @@ __global__ void __launch_bounds__(DL_THREADS) delta_prepare_kernel(const DeltaPr
         vec[i] = z;
       }
     }
-    // 1 / |k|: warp w takes tokens w, w + 4, ...
-#pragma unroll
-    for (int x = 0; x < DL_UNIT / NW; ++x) {
-      const int t = warp + x * NW;
-      float ss = 0.f;
-      for (int c = lane; c < DP; c += 32) {
-        const float k = t < nt && c < p.d ? Elem<T>::load(static_cast<const T*>(p.k) +
-                                                          (t0 + t) * p.in_stride + ch0 + c) : 0.f;
-        ss = fmaf(k, k, ss);
-      }
-      ss = warp_sum(ss);
-      if (lane == 0) unit[t] = 1.0f / sqrtf(ss + p.unit_eps);
+    // sums of k^2 per token: [16][SL] partial sums, one per warp that holds some of it
+#pragma unroll(BLOCKED ? 4 : NIT)
+    for (int x = 0; x < NIT; ++x) {
+      float k = 0.f;
+      if (!BLOCKED && NIT <= PASS)
+        k = Elem<T>::load(&kx[x < PASS ? x : 0]);
+      else if (tok(x) < nt && chan(x) < p.d)
+        k = Elem<T>::load(pk + offset(x));
+      const float ss = warp_sum(k * k);
+      if (lane == 0) part[tok(x) * SL + chan(x) / 32] = ss;
     }
     __syncthreads();
-    constexpr int F = DL_UNIT * DP;      // floats of one field
-#pragma unroll 4
-    for (int i = threadIdx.x; i < F; i += DL_THREADS) {
-      const int t = i / DP, c = i % DP;
-      float w = 1.f, u = 0.f, b = 0.f, k = 0.f, r = 0.f, v = 0.f;
-      if (t < nt && c < p.d) {
-        const int64_t row = (t0 + t) * p.in_stride + ch0 + c;
-        k = Elem<T>::load(static_cast<const T*>(p.k) + row);
-        const float a = Elem<T>::load(static_cast<const T*>(p.a) + row);
-        r = Elem<T>::load(static_cast<const T*>(p.r) + row);
-        v = Elem<T>::load(static_cast<const T*>(p.v) + row);
-        w = expf(-p.decay_scale * sigmoid_f32(vec[i] + p.w0[ch0 + c]));
-        u = k * unit[t];
-        b = u * sigmoid_f32(a + p.a_bias[ch0 + c]);
-      }
-      if (BLOCKED) {
-        vec[i] = w;
-        vec[F + i] = u;
-        vec[2 * F + i] = b;
-        vec[3 * F + i] = k;
-        vec[4 * F + i] = r;
-        vec[5 * F + i] = v;
-      } else if (t < nt) {
-        float* dst = p.packed + (((int64_t)h * p.rows + t0 + t) * DL_FIELDS) * DP + c;
-        dst[0] = w;
-        dst[DP] = u;
-        dst[2 * DP] = b;
-        dst[3 * DP] = k;
-        dst[4 * DP] = r;
-        dst[5 * DP] = v;
+    if (threadIdx.x < DL_UNIT) {
+      float ss = 0.f;
+#pragma unroll
+      for (int y = 0; y < SL; ++y) ss += part[threadIdx.x * SL + y];
+      unit[threadIdx.x] = 1.0f / sqrtf(ss + p.unit_eps);
+    }
+    __syncthreads();
+#pragma unroll(BLOCKED ? 1 : NIT / PASS)
+    for (int x0 = 0; x0 < NIT; x0 += PASS) {
+      if (BLOCKED || x0 > 0) fetch(x0);
+#pragma unroll
+      for (int x = 0; x < PASS; ++x) {
+        const int t = tok(x0 + x), c = chan(x0 + x), i = t * DP + c;
+        const bool on = t < nt && c < p.d;
+        float w = 1.f, u = 0.f, b = 0.f;
+        const float k = Elem<T>::load(&kx[x]), r = Elem<T>::load(&rx[x]);
+        const float v = Elem<T>::load(&vx[x]);
+        if (on) {
+          w = Gate<T>::exp(-p.decay_scale * Gate<T>::sigmoid(vec[i] + w0c[x % CPT]));
+          u = k * unit[t];
+          b = u * Gate<T>::sigmoid(Elem<T>::load(&ax[x]) + abc[x % CPT]);
+        }
+        if (BLOCKED) {
+          vec[i] = w;
+          vec[F + i] = u;
+          vec[2 * F + i] = b;
+          vec[3 * F + i] = k;
+          vec[4 * F + i] = r;
+          vec[5 * F + i] = v;
+        } else if (t < nt) {
+          float* dst = p.packed + (((int64_t)h * p.rows + t0 + t) * DL_FIELDS) * DP + c;
+          dst[0] = w;
+          dst[DP] = u;
+          dst[2 * DP] = b;
+          dst[3 * DP] = k;
+          dst[4 * DP] = r;
+          dst[5 * DP] = v;
+        }
       }
     }
     if (!BLOCKED) continue;
@@ -709,9 +779,10 @@ static int delta_padded(int d) { return d <= 32 ? 32 : d <= 64 ? 64 : d <= 128 ?
 template <typename T, int DP, bool BLOCKED>
 static int launch_prepare_one(const DeltaPrepParams& p, unsigned gx, cudaStream_t s) {
   const size_t smem = (size_t)DL_UNIT * (p.rank_p + 8) * 4 +
-                      (size_t)DL_FIELDS * DL_UNIT * DP * 4 + DL_UNIT * 4;
+                      (size_t)DL_FIELDS * DL_UNIT * DP * 4 + DL_UNIT * (DP / 32 + 1) * 4;
   static PerDeviceOnce once;
-  constexpr int kMaxSmem = DL_UNIT * 520 * 4 + DL_FIELDS * DL_UNIT * DP * 4 + DL_UNIT * 4;
+  constexpr int kMaxSmem = DL_UNIT * 520 * 4 + DL_FIELDS * DL_UNIT * DP * 4 +
+                           DL_UNIT * (DP / 32 + 1) * 4;
   FK_CUDA_OK(set_max_dynamic_smem(once, delta_prepare_kernel<T, DP, BLOCKED>, kMaxSmem));
   const dim3 grid(gx, (unsigned)((p.heads + p.heads_per_cta - 1) / p.heads_per_cta));
   FK_CUDA_OK(launch_kernel(delta_prepare_kernel<T, DP, BLOCKED>, grid, dim3(DL_THREADS), smem, s,
@@ -744,8 +815,10 @@ static int launch_scan_blocked(DeltaScanParams& p, cudaStream_t s) {
   FK_CUDA_OK(set_max_dynamic_smem(once, delta_scan_blocked_kernel<LANES, CPL, NC>, (int)kSmem));
   const dim3 grid((unsigned)((p.d + COLS - 1) / COLS), (unsigned)p.heads,
                   (unsigned)p.num_portions);
-  FK_CUDA_OK(launch_kernel(delta_scan_blocked_kernel<LANES, CPL, NC>, grid, dim3(DL_THREADS),
-                           kSmem, s, p));
+  // not ahead of its predecessor's end: CTAs that squeeze in beside the last ones of it
+  // pile up on a few SMs and stay there
+  FK_CUDA_OK(launch_kernel_after(delta_scan_blocked_kernel<LANES, CPL, NC>, grid,
+                                 dim3(DL_THREADS), kSmem, s, p));
   count_launch();
   return FK_OK;
 }

@@ -183,6 +183,9 @@ __device__ __forceinline__ PfItem pf_load_item(const PrefillParams& p, int idx) 
   return it;
 }
 
+// SPLIT: P enters P V as two bf16 parts (16 significant bits): the high parts in the
+// first 64 columns of S_t, the low parts in the other 64, two products per K/V tile.
+template <bool SPLIT>
 __global__ void __launch_bounds__(PF_THREADS, 1)
 prefill_attn_kernel(const __grid_constant__ CUtensorMap tmap_q,
                     const __grid_constant__ CUtensorMap tmap_k,
@@ -346,6 +349,10 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmap_q,
         tc_mma_bf16_ts_elect(tmem_base + 2 * PF_BN + t * PF_D, a + kk * 8,
                              smem_desc_sw128_mn(b + kk * 2048, PF_HALF_BYTES, 1024),
                              idesc_pv, (acc || kk > 0) ? 1u : 0u);
+        if (SPLIT)
+          tc_mma_bf16_ts_elect(tmem_base + 2 * PF_BN + t * PF_D, a + 64 + kk * 8,
+                               smem_desc_sw128_mn(b + kk * 2048, PF_HALF_BYTES, 1024),
+                               idesc_pv, 1u);
       }
     };
     int kv_base = 0;               // slot uses before this item
@@ -512,7 +519,10 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmap_q,
         const uint64_t nm2 = pf_pack2(neg_mu, neg_mu);
         uint64_t sum2[2] = {0ull, 0ull};
 #pragma unroll
-        for (int c = 0; c < 64; c += 2) {
+        for (int half = 0; half < 2; ++half) {
+          uint32_t lo[SPLIT ? 32 : 1];
+#pragma unroll
+        for (int c = half * 32; c < half * 32 + 32; c += 2) {
           float t0, t1, t2, t3;
           pf_unpack2(pf_fma2(pf_pack2(__uint_as_float(sr[2 * c]), __uint_as_float(sr[2 * c + 1])),
                              sc2, nm2), t0, t1);
@@ -524,6 +534,13 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmap_q,
           sum2[1] = pf_add2(sum2[1], pf_pack2(e2, e3));
           sr[c] = pack_bf16(e0, e1);
           sr[c + 1] = pack_bf16(e2, e3);
+          if (SPLIT) {
+            lo[SPLIT ? c & 31 : 0] = pack_bf16(e0 - bf16lo(sr[c]), e1 - bf16hi(sr[c]));
+            lo[SPLIT ? (c & 31) + 1 : 0] =
+                pack_bf16(e2 - bf16lo(sr[c + 1]), e3 - bf16hi(sr[c + 1]));
+          }
+        }
+          if (SPLIT) tc_st32(s_addr + 64 + half * 32, lo);
         }
         {
           float a0, a1, a2, a3;
@@ -744,7 +761,7 @@ using namespace fk;
 
 extern "C" {
 
-int fk_prefill_attn(const void* q, int64_t q_stride_token, void* out,
+static int prefill_impl(bool split, const void* q, int64_t q_stride_token, void* out,
                     int64_t out_stride_token, float* out_lse, const void* k,
                     const void* v, int64_t kv_stride, int64_t num_blocks,
                     int block_size, int kv_layout, const int32_t* cu_seqlens_q,
@@ -847,12 +864,15 @@ int fk_prefill_attn(const void* q, int64_t q_stride_token, void* out,
   static cudaError_t attr_err = cudaSuccess;
   static int launch_regs = 0;
   static PerDeviceOnce smem_once;
-  FK_CUDA_OK(set_max_dynamic_smem(smem_once, prefill_attn_kernel, PF_SMEM_ALLOC));
+  static PerDeviceOnce smem_once2;
+  FK_CUDA_OK(set_max_dynamic_smem(smem_once, prefill_attn_kernel<false>, PF_SMEM_ALLOC));
+  FK_CUDA_OK(set_max_dynamic_smem(smem_once2, prefill_attn_kernel<true>, PF_SMEM_ALLOC));
   // registers per thread of the compiled kernel: the same on every device
   std::call_once(once, [] {
-    cudaFuncAttributes fa;
-    attr_err = cudaFuncGetAttributes(&fa, prefill_attn_kernel);
-    if (attr_err == cudaSuccess) launch_regs = fa.numRegs;
+    cudaFuncAttributes fa, fb;
+    attr_err = cudaFuncGetAttributes(&fa, prefill_attn_kernel<false>);
+    if (attr_err == cudaSuccess) attr_err = cudaFuncGetAttributes(&fb, prefill_attn_kernel<true>);
+    if (attr_err == cudaSuccess) launch_regs = fa.numRegs < fb.numRegs ? fa.numRegs : fb.numRegs;
   });
   FK_CUDA_OK(attr_err);
   FK_REQUIRE(launch_regs * PF_THREADS >= PF_REGS_NEEDED, FK_ERR_UNSUPPORTED,
@@ -865,10 +885,41 @@ int fk_prefill_attn(const void* q, int64_t q_stride_token, void* out,
   p.q_blocks = q_blocks;
   const int ctas = (int)(items < sm_count() ? items : sm_count());
   dim3 grid((unsigned)ctas);
-  FK_CUDA_OK(launch_kernel(prefill_attn_kernel, grid, dim3(PF_THREADS), (size_t)PF_SMEM_ALLOC,
+  FK_CUDA_OK(launch_kernel(split ? prefill_attn_kernel<true> : prefill_attn_kernel<false>, grid,
+                           dim3(PF_THREADS), (size_t)PF_SMEM_ALLOC,
                            static_cast<cudaStream_t>(stream), mq, mk, mv, p));
   count_launch(1);
   return FK_OK;
+}
+
+int fk_prefill_attn(const void* q, int64_t q_stride_token, void* out,
+                    int64_t out_stride_token, float* out_lse, const void* k,
+                    const void* v, int64_t kv_stride, int64_t num_blocks,
+                    int block_size, int kv_layout, const int32_t* cu_seqlens_q,
+                    const int32_t* cu_seqlens_k, const int32_t* block_tables,
+                    int64_t block_table_stride, int num_seqs, int64_t total_q,
+                    int64_t total_k, int max_seqlen_q, int num_q_heads,
+                    int num_kv_heads, int head_dim, float softmax_scale, int causal,
+                    int32_t* status, fk_stream_t stream) {
+  return prefill_impl(false, q, q_stride_token, out, out_stride_token, out_lse, k, v, kv_stride,
+                      num_blocks, block_size, kv_layout, cu_seqlens_q, cu_seqlens_k, block_tables,
+                      block_table_stride, num_seqs, total_q, total_k, max_seqlen_q, num_q_heads,
+                      num_kv_heads, head_dim, softmax_scale, causal, status, stream);
+}
+
+int fk_prefill_attn_2p(const void* q, int64_t q_stride_token, void* out,
+                    int64_t out_stride_token, float* out_lse, const void* k,
+                    const void* v, int64_t kv_stride, int64_t num_blocks,
+                    int block_size, int kv_layout, const int32_t* cu_seqlens_q,
+                    const int32_t* cu_seqlens_k, const int32_t* block_tables,
+                    int64_t block_table_stride, int num_seqs, int64_t total_q,
+                    int64_t total_k, int max_seqlen_q, int num_q_heads,
+                    int num_kv_heads, int head_dim, float softmax_scale, int causal,
+                    int32_t* status, fk_stream_t stream) {
+  return prefill_impl(true, q, q_stride_token, out, out_stride_token, out_lse, k, v, kv_stride,
+                      num_blocks, block_size, kv_layout, cu_seqlens_q, cu_seqlens_k, block_tables,
+                      block_table_stride, num_seqs, total_q, total_k, max_seqlen_q, num_q_heads,
+                      num_kv_heads, head_dim, softmax_scale, causal, status, stream);
 }
 
 int fk_merge_attn_states(void* out, int64_t out_stride_token, int64_t out_stride_head,

@@ -35,7 +35,8 @@ class RotaryAttention:
     rotation and a weight-less RMS norm of q and k, over the paged pool of one span.
 
     bf16 with head sizes up to 128 runs on the tensor-core kernels, heads padded to
-    128 channels and query groups to a power of two (zeros); fp32 and everything else
+    128 channels and query groups to a power of two (zeros), the fp32 softmax weights in
+    two bf16 parts; fp32 and everything else
     on fk_paged_attn_any.  The output weight is packed with the same padding."""
 
     def __init__(self, heads, kv_heads, dim, scale, rot_dims, rot_base, span, eps, dtype):
@@ -98,11 +99,11 @@ class RotaryAttention:
         elif get_context().is_prefill:
             ops.prefill_attn(q, kc, vc, span.cu_seqlens_q, span.cu_seqlens_k, span.max_seqlen_q,
                              self.scale, block_table=span.block_tables, out=heads,
-                             status=self.status)
+                             status=self.status, split_weights=True)
         else:
             ops.paged_decode_attn(q, kc, vc, span.kv_lens, span.block_tables, self.scale,
                                   self.workspace, self.max_splits, out=heads,
-                                  status=self.status, planned=self.plan)
+                                  status=self.status, planned=self.plan, split_weights=True)
         return out
 
 

@@ -13,6 +13,8 @@ modules can still read one word per device after a step.
 """
 from __future__ import annotations
 
+import functools
+
 import torch
 
 from . import _lib
@@ -135,9 +137,10 @@ def paged_decode_attn_plan(context_lens, block_tables, block_size, num_q_heads, 
 
 def paged_decode_attn(q, k_cache, v_cache, context_lens, block_tables, softmax_scale,
                       workspace, max_splits, out=None, status=None, planned=False,
-                      kv_layout="NHD"):
+                      kv_layout="NHD", split_weights=False):
     """out[i,h] = softmax(scale q[i,h] K_i^T) V_i over the paged cache:
-    NHD [blocks, block, Hkv, D] or HND [blocks, Hkv, block, D]."""
+    NHD [blocks, block, Hkv, D] or HND [blocks, Hkv, block, D].  split_weights: the
+    fp32 weights enter P V as two bf16 parts instead of one."""
     _need(q, BF16, "q")
     _need(k_cache, BF16, "k_cache")
     _need(v_cache, BF16, "v_cache")
@@ -163,6 +166,8 @@ def paged_decode_attn(q, k_cache, v_cache, context_lens, block_tables, softmax_s
     if out is None:
         out = torch.empty((b, hq, d), dtype=BF16, device=q.device)
     fn = lib.fk_paged_decode_attn_planned if planned else lib.fk_paged_decode_attn
+    if split_weights:
+        fn = functools.partial(lib.fk_paged_decode_attn_2p, int(planned))
     check(fn(
         _ptr(q), q.stride(0) if b else hq * d, _ptr(out), out.stride(0) if b else hq * d,
         _ptr(k_cache), _ptr(v_cache), nb, bs, k_cache.stride(0), int(kv_layout == "HND"),
@@ -175,7 +180,7 @@ def paged_decode_attn(q, k_cache, v_cache, context_lens, block_tables, softmax_s
 
 def prefill_attn(q, k, v, cu_seqlens_q, cu_seqlens_k, max_seqlen_q, softmax_scale,
                  causal=True, block_table=None, kv_layout="NHD", out=None,
-                 return_lse=False, status=None):
+                 return_lse=False, status=None, split_weights=False):
     """Variable-length prefill attention on q [total_q, Hq, 128].
 
     Without block_table, k / v are dense [total_k, Hkv, 128] (token-strided views
@@ -184,8 +189,9 @@ def prefill_attn(q, k, v, cu_seqlens_q, cu_seqlens_k, max_seqlen_q, softmax_scal
     [blocks, page, Hkv, 128] or HND [blocks, Hkv, page, 128]) and only the
     per-sequence key counts of cu_seqlens_k are used.  Causal masking is aligned
     to the END of each sequence's keys (a chunk of q_len queries after a cached
-    prefix sees the prefix plus its own past).  Returns out, or (out, lse) with
-    lse fp32 [Hq, total_q]."""
+    prefix sees the prefix plus its own past).  split_weights: the fp32 weights enter
+    P V as two bf16 parts instead of one.  Returns out, or (out, lse) with lse fp32
+    [Hq, total_q]."""
     _need(q, BF16, "q")
     _need(k, BF16, "k")
     _need(v, BF16, "v")
@@ -223,7 +229,8 @@ def prefill_attn(q, k, v, cu_seqlens_q, cu_seqlens_k, max_seqlen_q, softmax_scal
         if k.stride()[1:] != dense or v.stride() != k.stride():
             raise _lib.FkError("caches must be dense within a block")
         total_k, kv_stride, bt_stride = 0, k.stride(0), block_table.stride(0)
-    check(lib.fk_prefill_attn(
+    fn = lib.fk_prefill_attn_2p if split_weights else lib.fk_prefill_attn
+    check(fn(
         _ptr(q), q.stride(0) if total_q else hq * d, _ptr(out),
         out.stride(0) if total_q else hq * d, _ptr(lse), _ptr(k), _ptr(v), kv_stride, nb, bs,
         int(kv_layout == "HND"), _ptr(cu_seqlens_q), _ptr(cu_seqlens_k), _ptr(block_table),

@@ -676,6 +676,26 @@ int fk_paged_attn_any(const void* q, int64_t q_stride, void* out, int64_t out_st
                       int64_t rows, int num_q_heads, int num_kv_heads, int head_dim,
                       float softmax_scale, int32_t* status, fk_stream_t stream);
 
+/* fk_paged_decode_attn (planned 0) / _planned (planned 1) and fk_prefill_attn with the
+ * fp32 softmax weights taken into P V as two bf16 parts (16 significant bits) instead of
+ * being rounded to one. */
+int fk_paged_decode_attn_2p(int planned, const void* q, int64_t q_stride_token, void* out,
+                            int64_t out_stride_token, const void* k_cache, const void* v_cache,
+                            int64_t num_blocks, int block_size, int64_t kv_block_stride,
+                            int kv_layout, const int32_t* context_lens,
+                            const int32_t* block_tables, int64_t block_table_stride, int batch,
+                            int num_q_heads, int num_kv_heads, int head_dim,
+                            float softmax_scale, int max_splits, void* workspace,
+                            size_t workspace_bytes, int32_t* status, fk_stream_t stream);
+int fk_prefill_attn_2p(const void* q, int64_t q_stride_token, void* out,
+                       int64_t out_stride_token, float* out_lse, const void* k, const void* v,
+                       int64_t kv_stride, int64_t num_blocks, int block_size, int kv_layout,
+                       const int32_t* cu_seqlens_q, const int32_t* cu_seqlens_k,
+                       const int32_t* block_tables, int64_t block_table_stride, int num_seqs,
+                       int64_t total_q, int64_t total_k, int max_seqlen_q, int num_q_heads,
+                       int num_kv_heads, int head_dim, float softmax_scale, int causal,
+                       int32_t* status, fk_stream_t stream);
+
 /* fk_argmax_bf16 on fp32 rows. */
 int fk_argmax_f32(const float* x, int64_t x_stride, int64_t rows, int64_t cols, float* out_val,
                   int64_t* out_idx, fk_stream_t stream);

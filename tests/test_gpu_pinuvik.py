@@ -682,3 +682,34 @@ def test_trace_runner_end_to_end(tmp_path, dtype):
     got = np.concatenate([np.fromfile(tmp_path / "o" / f"{i}.f32", "<f4").reshape(-1, cfg["vocab"])
                           for i in range(7)])
     check_logits(torch.from_numpy(got), want[1][:61], getattr(torch, dtype))
+
+
+@pytest.mark.parametrize("decode", [False, True])
+def test_softmax_weights_in_two_parts(decode):
+    """Weights that bf16 cannot hold: the two-part form stays within the rounding of its
+    bf16 output, where a sum of many weights of both signs lands near zero."""
+    from fastkernels_b200 import ops
+    rs = np.random.RandomState(0)
+    n, d, page = 640, 128, 64
+    q = P.bf16(rs.randn(n, 1, d) * 0.3)
+    k, v = P.bf16(rs.randn(n, 1, d) * 0.3), np.ones((n, 1, d))
+    v[:, :, ::2] = np.where(np.arange(n) % 3 == 0, 1.0, -0.5)[:, None, None]
+    s = np.array([q[-1, 0] @ k[j, 0] for j in range(n)]) * 0.2
+    w = np.exp(s - s.max())
+    want = (w / w.sum()) @ v[:, 0]
+    kc, vc = dev(k, BF16).view(-1, page, 1, d), dev(v, BF16).view(-1, page, 1, d)
+    bt = torch.zeros((1, 16), dtype=torch.int32, device="cuda")
+    bt[0, :n // page] = torch.arange(n // page)
+    errs = []
+    for split in (True, False):
+        if decode:
+            ws = torch.empty(ops.attn_workspace_bytes(1, 1, d, 4), dtype=torch.uint8, device="cuda")
+            out = ops.paged_decode_attn(dev(q[-1:], BF16), kc, vc, i32([n]), bt, 0.2, ws, 4,
+                                        split_weights=split)[0, 0]
+        else:
+            out = ops.prefill_attn(dev(q, BF16), kc, vc, i32([0, n]), i32([0, n]), n, 0.2,
+                                   block_table=bt, split_weights=split)[-1, 0]
+        got = out.double().cpu().numpy()
+        np.testing.assert_allclose(got, want, atol=5e-3)
+        errs.append(np.abs(got - want)[::2].max())
+    assert errs[0] <= 2.0 ** -8 * np.abs(want[::2]).max() + 1e-5, errs
