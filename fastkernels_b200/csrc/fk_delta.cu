@@ -822,7 +822,7 @@ static int launch_scan_blocked(DeltaScanParams& p, cudaStream_t s) {
   count_launch();
   return FK_OK;
 }
-// LANES x CPL for single tokens, BL x BC for blocks (fewer lanes to sum over)
+// LANES x CPL for single tokens, BL x BC for blocks
 template <int LANES, int CPL, int BL, int BC>
 static int launch_scan(DeltaScanParams& p, bool blocked, cudaStream_t s) {
   if (!blocked) {
@@ -834,10 +834,10 @@ static int launch_scan(DeltaScanParams& p, bool blocked, cudaStream_t s) {
     return FK_OK;
   }
   // four columns per thread read a stage's vectors half as often as two; two make a
-  // block's instructions fewer where heads and sequences do not fill the SMs
+  // block's instructions fewer where small heads and few sequences do not fill the SMs
   constexpr int COLS4 = DL_THREADS / BL * 4;
-  if (p.d > COLS4 / 2 && (int64_t)p.heads * p.num_portions * ((p.d + COLS4 - 1) / COLS4) >=
-                             2 * sm_count())
+  if (p.d > 64 || (p.d > COLS4 / 2 && (int64_t)p.heads * p.num_portions *
+                                              ((p.d + COLS4 - 1) / COLS4) >= 2 * sm_count()))
     return launch_scan_blocked<BL, BC, 4>(p, s);
   return launch_scan_blocked<BL, BC, 2>(p, s);
 }
@@ -915,8 +915,8 @@ int fk_delta_scan(const float* packed, int blocked, float* o, float* state, int 
   switch (delta_padded(dim)) {
     case 32: return launch_scan<4, 8, 4, 8>(p, blocked != 0, s);
     case 64: return launch_scan<8, 8, 8, 8>(p, blocked != 0, s);
-    case 128: return launch_scan<16, 8, 8, 16>(p, blocked != 0, s);
-    default: return launch_scan<32, 8, 16, 16>(p, blocked != 0, s);
+    case 128: return launch_scan<16, 8, 16, 8>(p, blocked != 0, s);
+    default: return launch_scan<32, 8, 32, 8>(p, blocked != 0, s);
   }
 }
 

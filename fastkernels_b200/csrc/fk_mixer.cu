@@ -17,7 +17,7 @@
 
 namespace fk {
 
-constexpr int MX_MAX_VPT = 8;   // float4 groups of a row per thread
+constexpr int MX_MAX_VPT = 4;   // float4 groups of a row per thread
 
 // One row as registers: group i of thread t is float4 number t + i * blockDim.
 template <int VPT>
@@ -59,19 +59,40 @@ __device__ __forceinline__ void load_row(const NormShiftParams& p, int64_t t, Ro
 }
 
 // x' = x + rms(y) * y_gain, stored when asked; h (in: x) = rms(x') * gain.
+//
+// One reduction for both norms: with c = rms scale of y times its gain,
+// sum x'^2 = sum x^2 + 2 c sum x y + c^2 sum y^2.  Where x and c y cancel to less than a
+// hundredth that would lose digits, and sum x'^2 is taken from x' itself.
 template <typename T, int VPT>
 __device__ __forceinline__ void norm_row(const NormShiftParams& p, int64_t t, bool store_x,
                                          Row<VPT>& h, const Row<VPT>& y, float* red, int& flip) {
   const int groups = p.stride >> 2;
   const float inv_w = 1.0f / (float)p.width;
+  float s[3] = {0.f, 0.f, 0.f};
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    s[0] += sumsq(h.v[i]);
+    if (p.y) {
+      const float4 xy = h.v[i] * y.v[i];
+      s[1] += (xy.x + xy.y) + (xy.z + xy.w);
+      s[2] += sumsq(y.v[i]);
+    }
+  }
+  block_sums<3>(s, red, flip);
+  float ss = s[0];
   if (p.y) {
-    float s[1] = {0.f};
+    const float c = rsqrtf(s[2] * inv_w + p.eps) * *p.y_gain;
 #pragma unroll
-    for (int i = 0; i < VPT; ++i) s[0] += sumsq(y.v[i]);
-    block_sums<1>(s, red, flip);
-    const float sc = rsqrtf(s[0] * inv_w + p.eps) * *p.y_gain;
+    for (int i = 0; i < VPT; ++i) h.v[i] = h.v[i] + y.v[i] * c;
+    const float all = s[0] + c * c * s[2];
+    ss = all + 2.0f * c * s[1];
+    if (ss < 0.01f * all) {
+      float e[3] = {0.f, 0.f, 0.f};
 #pragma unroll
-    for (int i = 0; i < VPT; ++i) h.v[i] = h.v[i] + y.v[i] * sc;
+      for (int i = 0; i < VPT; ++i) e[0] += sumsq(h.v[i]);
+      block_sums<3>(e, red, flip);
+      ss = e[0];
+    }
   }
   if (store_x && p.x_out) {
 #pragma unroll
@@ -80,98 +101,99 @@ __device__ __forceinline__ void norm_row(const NormShiftParams& p, int64_t t, bo
       if (g < groups) *reinterpret_cast<float4*>(p.x_out + t * p.stride + g * 4) = h.v[i];
     }
   }
-  float s[1] = {0.f};
-#pragma unroll
-  for (int i = 0; i < VPT; ++i) s[0] += sumsq(h.v[i]);
-  block_sums<1>(s, red, flip);
-  const float sc = rsqrtf(s[0] * inv_w + p.eps) * *p.gain;
+  const float sc = rsqrtf(ss * inv_w + p.eps) * *p.gain;
 #pragma unroll
   for (int i = 0; i < VPT; ++i) h.v[i] = h.v[i] * sc;
 }
 
-template <typename T, int VPT>
-__device__ __forceinline__ void one_row(const NormShiftParams& p, int64_t t, Row<VPT>& h,
-                                        float* red, int& flip) {
-  Row<VPT> y;
-  load_row<T, VPT>(p, t, h, y);
-  norm_row<T, VPT>(p, t, false, h, y, red, flip);
-}
-
-// A CTA walks `rows_per_cta` consecutive rows and carries the normed row from one
-// to the next.  The row ahead of its first one is computed once more (from x_in,
-// which this kernel does not change), or comes from the sequence's state when a
-// portion starts there.  The state of a portion is read AND replaced by the CTA
-// that owns the portion's first row (it computes the portion's last row for that),
+// A CTA walks `rows_per_cta` consecutive rows and carries the normed row from one to
+// the next.  The row ahead of its first one is computed once more (from x_in, which this
+// kernel does not change), or comes from the sequence's state when a portion starts
+// there.  The state of a portion is read AND replaced by the CTA that owns the portion's
+// first row (for that it computes the portion's last row, if it is not one of its own),
 // so no other CTA touches it.
-template <typename T, int VPT>
-__global__ void __launch_bounds__(512) norm_shift_kernel(const NormShiftParams p) {
+template <typename T, int VPT, bool SHIFT>
+__global__ void __launch_bounds__(512, VPT == 1 ? 4 : VPT == 2 ? 3 : VPT == 4 ? 2 : 1)
+norm_shift_kernel(const NormShiftParams p) {
   pdl_launch_dependents();
   pdl_wait();
-  __shared__ float red[64];
+  __shared__ float red[192];
   int flip = 0;
   const int groups = p.stride >> 2;
   const int64_t t0 = (int64_t)blockIdx.x * p.rows_per_cta;
-  const int64_t t1 = min(t0 + p.rows_per_cta, p.rows);
-  Row<VPT> prev, nx, ny;
-  load_row<T, VPT>(p, t0, nx, ny);
-  for (int64_t t = t0; t < t1; ++t) {
-    // the next row's loads are in flight during this row's reductions
-    Row<VPT> h = nx;
-    const Row<VPT> y = ny;
-    if (t + 1 < t1) load_row<T, VPT>(p, t + 1, nx, ny);
-    bool first = false, in_range = false;
-    int slot = -1;
-    float* st = nullptr;
-    if (p.shift) {
-      slot = p.slots[t];
-      first = slot < 0 || t == 0 || p.slots[t - 1] != slot;
-      if (first) {
-        in_range = slot >= 0 && slot < p.num_slots;
+  const int n = (int)min((int64_t)p.rows_per_cta, p.rows - t0);
+  // the previous normed row: a thread only ever touches its own entries
+  __shared__ float4 prev[SHIFT ? VPT * 512 : 1];
+  float* pend = nullptr;        // state that waits for row pend_row
+  int64_t pend_row = -1;
+  int it = 0;
+  if (SHIFT && t0 > 0) {
+    const int slot = p.slots[t0];
+    if (slot >= 0 && p.slots[t0 - 1] == slot) it = -1;
+  }
+  for (; it < n || (SHIFT && pend != nullptr); ++it) {
+    const bool own = it >= 0 && it < n;
+    const int64_t t = it < n ? t0 + it : pend_row;
+    Row<VPT> h, y;
+    load_row<T, VPT>(p, t, h, y);
+    if (SHIFT && own) {
+      const int slot = p.slots[t];
+      if (slot < 0 || t == 0 || p.slots[t - 1] != slot) {
+        const bool in_range = slot >= 0 && slot < p.num_slots;
         if (slot >= p.num_slots && threadIdx.x == 0 && p.status)
           atomicOr(p.status, FK_DEV_BAD_SLOT);
         const bool from_state = in_range && p.positions[t] > 0;
-        st = p.state + (int64_t)(in_range ? slot : 0) * p.stride;
+        float* st = p.state + (int64_t)(in_range ? slot : 0) * p.stride;
 #pragma unroll
         for (int i = 0; i < VPT; ++i) {
           const int g = threadIdx.x + i * blockDim.x;
-          prev.v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-          if (from_state && g < groups)
-            prev.v[i] = *reinterpret_cast<const float4*>(st + g * 4);
+          if (g < groups)
+            prev[g] = from_state ? *reinterpret_cast<const float4*>(st + g * 4)
+                                 : make_float4(0.f, 0.f, 0.f, 0.f);
         }
-      } else if (t == t0) {
-        one_row<T, VPT>(p, t - 1, prev, red, flip);
+        pend = nullptr;
+        if (in_range) {
+          // last row of the portion that starts here
+          int lo = 0, hi = p.num_portions;
+          while (hi - lo > 1) {
+            const int mid = (lo + hi) >> 1;
+            if (p.cu[mid] <= t) lo = mid; else hi = mid;
+          }
+          pend = st;
+          pend_row = max(t, min((int64_t)p.cu[lo + 1], p.rows) - 1);
+        }
       }
     }
-    norm_row<T, VPT>(p, t, true, h, y, red, flip);
-    if (in_range) {
-      // last row of the portion that starts here
-      int lo = 0, hi = p.num_portions;
-      while (hi - lo > 1) {
-        const int mid = (lo + hi) >> 1;
-        if (p.cu[mid] <= t) lo = mid; else hi = mid;
-      }
-      const int64_t last = (int64_t)p.cu[lo + 1] - 1;
-      Row<VPT> z = h;
-      if (last > t && last < p.rows) one_row<T, VPT>(p, last, z, red, flip);
+    norm_row<T, VPT>(p, t, own, h, y, red, flip);
+    if (SHIFT && pend != nullptr && t == pend_row) {
 #pragma unroll
       for (int i = 0; i < VPT; ++i) {
         const int g = threadIdx.x + i * blockDim.x;
-        if (g < groups) *reinterpret_cast<float4*>(st + g * 4) = z.v[i];
+        if (g < groups) *reinterpret_cast<float4*>(pend + g * 4) = h.v[i];
       }
+      pend = nullptr;
     }
+    if (own) {
 #pragma unroll
-    for (int i = 0; i < VPT; ++i) {
-      const int g = threadIdx.x + i * blockDim.x;
-      if (g < groups) {
-        float4 o = h.v[i];
-        if (p.shift) {
-          const float4 sh = __ldg(reinterpret_cast<const float4*>(p.shift + g * 4));
-          o = o + (prev.v[i] - o) * sh;
+      for (int i = 0; i < VPT; ++i) {
+        const int g = threadIdx.x + i * blockDim.x;
+        if (g < groups) {
+          float4 o = h.v[i];
+          if (SHIFT) {
+            const float4 sh = __ldg(reinterpret_cast<const float4*>(p.shift + g * 4));
+            o = o + (prev[g] - o) * sh;
+          }
+          Elem<T>::store4(static_cast<T*>(p.out) + t * p.stride + g * 4, o);
         }
-        Elem<T>::store4(static_cast<T*>(p.out) + t * p.stride + g * 4, o);
       }
     }
-    prev = h;
+    if (SHIFT) {
+#pragma unroll
+      for (int i = 0; i < VPT; ++i) {
+        const int g = threadIdx.x + i * blockDim.x;
+        if (g < groups) prev[g] = h.v[i];
+      }
+    }
   }
 }
 
@@ -500,24 +522,23 @@ __global__ void __launch_bounds__(256) act_and_mul_kernel(
 
 // threads and float4 groups per thread for a row of `groups` float4
 static bool row_shape(int groups, int* threads, int* vpt) {
-  int th = ((groups + 31) / 32) * 32;
+  int v = (groups + 511) / 512;
+  v = v <= 1 ? 1 : v <= 2 ? 2 : 4;
+  int th = ((groups + v - 1) / v + 31) / 32 * 32;   // no more threads than the row needs
   if (th > 512) th = 512;
-  if (th < 32) th = 32;
-  int v = (groups + th - 1) / th;
-  v = v <= 1 ? 1 : v <= 2 ? 2 : v <= 4 ? 4 : 8;
   *threads = th;
   *vpt = v;
   return groups <= th * MX_MAX_VPT;
 }
 
-template <typename T>
+template <typename T, bool SHIFT>
 static cudaError_t launch_norm_shift(const NormShiftParams& p, int grid, int threads, int vpt,
                                      cudaStream_t s) {
+  const dim3 g(grid), b(threads);
   switch (vpt) {
-    case 1: return launch_kernel(norm_shift_kernel<T, 1>, dim3(grid), dim3(threads), 0, s, p);
-    case 2: return launch_kernel(norm_shift_kernel<T, 2>, dim3(grid), dim3(threads), 0, s, p);
-    case 4: return launch_kernel(norm_shift_kernel<T, 4>, dim3(grid), dim3(threads), 0, s, p);
-    default: return launch_kernel(norm_shift_kernel<T, 8>, dim3(grid), dim3(threads), 0, s, p);
+    case 1: return launch_kernel(norm_shift_kernel<T, 1, SHIFT>, g, b, 0, s, p);
+    case 2: return launch_kernel(norm_shift_kernel<T, 2, SHIFT>, g, b, 0, s, p);
+    default: return launch_kernel(norm_shift_kernel<T, 4, SHIFT>, g, b, 0, s, p);
   }
 }
 template <typename T>
@@ -526,8 +547,7 @@ static cudaError_t launch_combine(const CombineParams& p, int threads, int vpt, 
   switch (vpt) {
     case 1: return launch_kernel(branch_combine_kernel<T, 1>, grid, dim3(threads), 0, s, p);
     case 2: return launch_kernel(branch_combine_kernel<T, 2>, grid, dim3(threads), 0, s, p);
-    case 4: return launch_kernel(branch_combine_kernel<T, 4>, grid, dim3(threads), 0, s, p);
-    default: return launch_kernel(branch_combine_kernel<T, 8>, grid, dim3(threads), 0, s, p);
+    default: return launch_kernel(branch_combine_kernel<T, 4>, grid, dim3(threads), 0, s, p);
   }
 }
 template <typename T>
@@ -602,8 +622,11 @@ int fk_norm_shift(const float* x_in, float* x_out, const void* y, int64_t y_stri
   const int64_t grid = (rows + rpc - 1) / rpc;
   FK_REQUIRE(grid <= 0x7fffffff, FK_ERR_UNSUPPORTED, "fk_norm_shift: too many rows");
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  FK_CUDA_OK(is_f32 ? launch_norm_shift<float>(p, (int)grid, threads, vpt, s)
-                    : launch_norm_shift<uint16_t>(p, (int)grid, threads, vpt, s));
+  const int g = (int)grid;
+  FK_CUDA_OK(shift ? (is_f32 ? launch_norm_shift<float, true>(p, g, threads, vpt, s)
+                             : launch_norm_shift<uint16_t, true>(p, g, threads, vpt, s))
+                   : (is_f32 ? launch_norm_shift<float, false>(p, g, threads, vpt, s)
+                             : launch_norm_shift<uint16_t, false>(p, g, threads, vpt, s)));
   count_launch();
   return FK_OK;
 }

@@ -35,6 +35,7 @@ VOCAB = 32768
 PREFILLS = [(1, 8192), (8, 1024)]
 DECODES = [1, 16, 64]
 CONTEXT = 1500
+FP32_TFLOPS = 148 * 128 * 2 * 1.965e-3      # nominal fp32 rate outside the tensor cores
 
 
 def peaks():
@@ -124,8 +125,12 @@ def _work(name, args, kw, out):
     if name == "qkv_rope_store":
         return 2 * _nbytes(args[0]), 0
     if name == "delta_scan":
-        packed, state, cu = args[0], args[1], args[2]
-        return _nbytes(packed, out) + 2 * (cu.numel() - 1) * _nbytes(state[0]), 0
+        packed, state, cu, positions = args[0], args[1], args[2], args[4]
+        # 4.25 fp32 multiply-adds per state element and token, on the fp32 pipes (not
+        # tensor FLOPs: scaled so that the tensor peak below turns them into their time)
+        fma = 4.25 * positions.numel() * state[0].numel()
+        return _nbytes(packed, out) + 2 * (cu.numel() - 1) * _nbytes(state[0]), \
+            2 * fma * peaks()["bf16_tflops"] / FP32_TFLOPS
     if name == "norm_shift":
         return _nbytes(args[0], kw.get("y"), out[1]) + \
             (_nbytes(args[0]) if kw.get("y") is not None else 0), 0
@@ -133,8 +138,12 @@ def _work(name, args, kw, out):
         return _nbytes(args[0], args[1], out) + 2 * _nbytes(args[5]), 0
     if name == "fused_add_rmsnorm":
         return 2 * _nbytes(args[0], args[1]), 0
-    if name in ("delta_prepare", "delta_output"):
-        return _nbytes(*[x for x in t if torch.is_tensor(x) and x.dim() >= 2]), 0
+    if name == "delta_prepare":
+        return _nbytes(*args[:6], out), 0
+    if name == "delta_output":
+        return _nbytes(args[0], args[1], out), 0
+    if name == "embed_f32":
+        return 2 * _nbytes(out), 0
     return _nbytes(*t), 0
 
 
@@ -258,6 +267,7 @@ def run(args, sampler=None):
                 r[f"decode batch {b}"] = {"ms": round(ms, 4), "tok_s": round(b / ms * 1e3)}
             if args.kernels:
                 r["kernels prefill 1x8192"] = kernel_table(eng, 1, 8192)
+                r["kernels prefill 8x1024"] = kernel_table(eng, 8, 1024)
                 r["kernels decode batch 64"] = kernel_table(eng, 64, 1)
             r["device_status_word"] = eng.device_status()
             res[kind] = r

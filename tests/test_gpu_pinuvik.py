@@ -107,6 +107,23 @@ def test_norm_shift_many_rows(dtype):
     close(st, h[cu[1:] - 1], F32)
 
 
+def test_norm_shift_where_the_sum_cancels():
+    """x + c y of one row is a thousandth of x: the norm is taken from the sum itself."""
+    from fastkernels_b200 import ops
+    rs = np.random.RandomState(6)
+    width, eps = 256, 1e-9
+    y = P.bf16(rs.randn(3, width))
+    x = -P.rms(y, eps) * 1.5 + 1e-3 * rs.randn(3, width)
+    x[1] = rs.randn(width)
+    x = x.astype(np.float32).astype(np.float64)
+    xo, out = ops.norm_shift(dev(x), dev([1.0]), width, eps, F32, y=dev(y), y_gain=dev([1.5]))
+    want = x + P.rms(y, eps) * 1.5
+    close(xo, want, F32)
+    # rounding of x and c y is a thousand times larger beside their sum
+    np.testing.assert_allclose(out.double().cpu().numpy(), P.rms(want, eps), atol=2e-3)
+    close(out[1:2], P.rms(want, eps)[1:2], F32)
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("width,rows", [(40, 3), (576, 37), (3000, 5)])
 def test_branch_combine(width, rows, dtype):
