@@ -107,11 +107,24 @@ class DecodeEngine:
         self._bt_dirty = True
         self._staged_for = None     # ids of the sequences the device tables belong to
 
+    @staticmethod
+    def pages_for(config, max_tokens: int, max_num_seqs: int) -> list[int]:
+        """Pages per span that hold max_tokens tokens of up to max_num_seqs sequences:
+        whole pages, and one more for the last page of every sequence and of every chunk
+        (a portion keeps all the pages it touches until it has run)."""
+        return [-(-max_tokens // config.kv_block_size) + max_num_seqs
+                + (0 if chunk is None else max_tokens // chunk + 1)
+                for chunk in model_class(config).spans_of(config)]
+
     @classmethod
-    def from_folder(cls, folder, dtype=torch.bfloat16, **kw):
-        """Engine for the model in a folder (config.json, safetensors)."""
+    def from_folder(cls, folder, *, max_tokens: int, max_num_seqs: int, dtype=torch.bfloat16,
+                    **kw):
+        """Engine for the model in a folder (config.json, safetensors), with pages for
+        max_tokens live tokens in all."""
         config, source = load_folder(folder, dtype)
-        eng = cls(config, init_scale=None, **kw)
+        eng = cls(config, init_scale=None, max_num_seqs=max_num_seqs,
+                  max_model_len=max_tokens + 1,
+                  num_kv_blocks=cls.pages_for(config, max_tokens, max_num_seqs), **kw)
         eng.load_weights(source)
         return eng
 
@@ -262,11 +275,15 @@ class DecodeEngine:
     def finish(self, seq: Sequence) -> None:
         """End a sequence: its pages and its state slot go back."""
         self.seqs.remove(seq)
+        self._release(seq)
+        self._running_set_changed()
+
+    def _release(self, seq: Sequence) -> None:
         for blocks in self.span_blocks:
             blocks.release(seq)
+            blocks.flush()
         if self.state_slots is not None:
             self.state_slots.release(seq)
-        self._running_set_changed()
 
     @torch.no_grad()
     def _forward_portions(self, portions, use_block_tables: bool = True):
@@ -363,6 +380,21 @@ class DecodeEngine:
         if len(self.seqs) + len(prompts) > self.max_num_seqs:
             raise RuntimeError("max_num_seqs exceeded")
         new = [self._new_sequence(len(prompt)) for prompt in prompts]
+        try:
+            first = self._prefill_new(new, prompts, chunk_tokens, use_block_tables)
+        except BaseException:
+            for s in new:              # nothing joined: what they hold goes back
+                self._release(s)
+            raise
+        for s, t in zip(new, first):
+            s.num_tokens += 1          # the sampled token is the next step's input
+            s.last_token = int(t)
+            s.output.append(int(t))
+            self.seqs.append(s)
+        self._running_set_changed()
+        return first
+
+    def _prefill_new(self, new, prompts, chunk_tokens, use_block_tables) -> np.ndarray:
         done = [0] * len(new)
         first = np.zeros(len(new), dtype=np.int64)
         while any(d < len(pr) for d, pr in zip(done, prompts)):
@@ -381,12 +413,6 @@ class DecodeEngine:
                     first[i] = int(t)
             for i, a, c in part:
                 done[i] = a + c
-        for s, t in zip(new, first):
-            s.num_tokens += 1          # the sampled token is the next step's input
-            s.last_token = int(t)
-            s.output.append(int(t))
-            self.seqs.append(s)
-        self._running_set_changed()
         return first
 
     @torch.no_grad()

@@ -18,7 +18,6 @@ import sys
 import torch
 
 from .engine import DecodeEngine
-from .models.registry import load_folder, model_class
 
 MAX_SEQS = 64
 
@@ -34,16 +33,8 @@ def parse_args(argv=None):
 
 
 def make_engine(folder, dtype, max_tokens) -> DecodeEngine:
-    config, source = load_folder(folder, dtype)
-    # whole pages, and one more for the last page of every request and of every chunk
-    # (a portion holds all the pages it touches until it has run)
-    block = config.kv_block_size
-    pages = [(max_tokens + block - 1) // block + MAX_SEQS
-             + (0 if chunk is None else max_tokens // chunk + 1)
-             for chunk in model_class(config).spans_of(config)]
-    eng = DecodeEngine(config, max_num_seqs=MAX_SEQS, max_model_len=max_tokens + 1,
-                       num_kv_blocks=pages, init_scale=None)
-    eng.load_weights(source)
+    eng = DecodeEngine.from_folder(folder, dtype=dtype, max_tokens=max_tokens,
+                                   max_num_seqs=MAX_SEQS)
     eng.capture_cudagraph([1])
     return eng
 

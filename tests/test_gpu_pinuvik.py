@@ -730,3 +730,21 @@ def test_softmax_weights_in_two_parts(decode):
         np.testing.assert_allclose(got, want, atol=5e-3)
         errs.append(np.abs(got - want)[::2].max())
     assert errs[0] <= 2.0 ** -8 * np.abs(want[::2]).max() + 1e-5, errs
+
+
+def test_generate_command_line(tmp_path):
+    import io
+    from fastkernels_b200 import generate
+    cfg, w, seqs, want = model("plain")
+    P.write_folder(tmp_path, cfg, w)
+    out = io.StringIO()
+    prompts = [seqs[1][:40].tolist(), seqs[2].tolist()]
+    args = ["--model", str(tmp_path), "--max-new-tokens", "12", "--dtype", "float32"]
+    for p in prompts:
+        args += ["--prompt", ",".join(map(str, p))]
+    assert generate.main(args, stdout=out) == 0
+    for p, line in zip(prompts, out.getvalue().splitlines()):
+        got = [int(t) for t in line.split(",")]
+        lg = P.logits(cfg, w, np.array(p + got[:-1]))[len(p) - 1:]
+        assert len(got) == 12
+        assert (lg.max(1) - lg[np.arange(12), got]).max() <= 1e-4

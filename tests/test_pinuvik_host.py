@@ -336,3 +336,24 @@ def test_mistakes_show_in_the_logits(name):
         assert err(P.logits(c, w, s), want) > 0.3
     assert err(P.logits(cfg, {**w, "l0.shift": w["l0.shift"] * 0}, s), want) > 0.3
     assert err(P.logits(cfg, w, s[70:])[:20], want[70:90]) > 0.3
+
+
+def test_a_prefill_that_does_not_fit_gives_everything_back(tmp_path, monkeypatch):
+    small(tmp_path)
+    config, source = registry.load_folder(tmp_path, torch.float32)
+    config.kv_block_size = 8
+    eng = DecodeEngine(config, max_num_seqs=2, max_model_len=300, num_kv_blocks=[6, 6],
+                       device="cpu", init_scale=None)
+    eng.load_weights(source)
+    monkeypatch.setattr(type(eng.model), "forward",
+                        lambda self, ids, pos: torch.zeros(len(ids), self.stride))
+    with pytest.raises(RuntimeError, match="exhausted"):
+        eng.prefill([list(range(50)), list(range(40))])
+    assert not eng.seqs and len(eng.state_slots.free) == 2
+    assert all(len(b.free) == 6 for b in eng.span_blocks)
+    # the sizes the engine works out for itself do hold that many tokens
+    pages = DecodeEngine.pages_for(config, 90, 2)
+    for (chunk, n) in zip((24, 40), pages):
+        bm = BlockManager(n, 8, 0, chunk)
+        for i, t in enumerate((50, 40)):
+            bm.extend(Sequence(i, 0), 0, t)
