@@ -174,9 +174,9 @@ MODELS = {
                              layer_config(heads=4, kv_heads=4, dim=32, rot=(0, 1.0), chunk=17)],
                             width=72, vocab=131, eps=1e-3, loop=(1, 2, 3)), 5),
     "wide": (model_config([layer_config(heads=4, kv_heads=2, dim=128, rot=(64, 1e5), chunk=90,
-                                            delta=(2, 64), ff=192, scale=0.2),
+                                            delta=(3, 64), ff=192, scale=0.2),
                              layer_config(heads=1, kv_heads=1, dim=136, rot=(136, 1e3), chunk=128,
-                                            delta=(2, 72), ff=64)], width=256, vocab=500,
+                                            delta=(2, 72), ff=64)], width=320, vocab=500,
                             loop=(0, 2, 2)), 24),
 }
 
