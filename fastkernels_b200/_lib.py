@@ -125,9 +125,9 @@ PROTOTYPES = {
                                 _i32, _vp, _i32, _i64, _i32, _i32, _i32, _f32, _f32, _vp]),
     "fk_delta_scan": (_i32, [_vp, _i32, _vp, _vp, _i32, _vp, _i32, _vp, _vp, _i64, _i32, _i32, _vp,
                              _vp]),
-    "fk_delta_output": (_i32, [_vp, _vp, _i64, _vp, _vp, _i64, _i32, _i64, _i32, _i32, _f32,
+    "fk_head_norm_gate": (_i32, [_vp, _vp, _i64, _vp, _vp, _i64, _i32, _i64, _i32, _i32, _f32,
                                _vp]),
-    "fk_gemm_f32": (_i32, [_vp, _i64, _vp, _vp, _i64, _i64, _i64, _i64, _vp]),
+    "fk_gemm_f32": (_i32, [_vp, _i64, _vp, _vp, _vp, _i64, _i64, _i64, _i64, _vp]),
     "fk_paged_attn_any": (_i32, [_vp, _i64, _vp, _i64, _vp, _vp, _i32, _i64, _i32, _vp, _vp, _vp,
                                  _i64, _i32, _i64, _i32, _i32, _i32, _f32, _vp, _vp]),
     "fk_paged_decode_attn_2p": (_i32, [_i32, _vp, _i64, _vp, _i64, _vp, _vp, _i64, _i32, _i64,
@@ -135,7 +135,37 @@ PROTOTYPES = {
                                        _vp, _sz, _vp, _vp]),
     "fk_prefill_attn_2p": (_i32, [_vp, _i64, _vp, _i64, _vp, _vp, _vp, _i64, _i64, _i32, _i32,
                                   _vp, _vp, _vp, _i64, _i32, _i64, _i64, _i32, _i32, _i32, _i32,
-                                  _f32, _i32, _vp, _vp]),
+                                  _i32, _f32, _i32, _vp, _vp]),
+    "fk_embed_pair_f32": (_i32, [_vp, _vp, _i32, _i64, _i64, _i64, _i64, _vp, _vp, _i32, _vp, _vp,
+                                 _vp, _i32, _vp, _vp, _i64, _i64, _i32, _vp, _vp]),
+    "fk_add_layernorm": (_i32, [_vp, _vp, _vp, _i64, _vp, _i64, _vp, _i64, _i64, _vp, _vp, _i32,
+                                _vp, _vp, _vp, _i64, _vp, _vp, _vp, _i64, _i32, _i64, _i32, _i32,
+                                _f32, _vp, _vp]),
+    "fk_softcap": (_i32, [_vp, _i64, _i32, _i64, _i64, _f32, _vp]),
+    "fk_group_gemm": (_i32, [_vp, _i64, _i64, _i64, _vp, _vp, _vp, _i64, _i64, _i32, _i32, _vp,
+                             _vp, _i64, _i64, _i32, _i64, _i64, _i32, _vp, _vp]),
+    "fk_moe_route_counts": (_i64, [_i64, _i32, _i32]),
+    "fk_moe_route": (_i32, [_vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i32, _i32, _vp]),
+    "fk_gather_rows": (_i32, [_vp, _i64, _i64, _vp, _vp, _i64, _i64, _vp, _vp]),
+    "fk_latent_prepare": (_i32, [_vp, _vp, _i64, _i32, _i32, _vp, _vp, _i64, _vp, _vp, _vp, _i64,
+                                 _i32, _vp, _i32, _i32, _i32, _i64, _i32, _i32, _i32, _i32, _f32,
+                                 _vp, _vp]),
+    "fk_latent_gather": (_i32, [_vp, _i64, _i64, _i32, _vp, _i64, _vp, _i32, _vp, _i64, _vp,
+                                _vp]),
+    "fk_latent_attn_splits": (_i32, [_i32, _i64, _i32, _i32, _i64]),
+    "fk_latent_attn_workspace_floats": (_i64, [_i64, _i32, _i32, _i32]),
+    "fk_latent_attn": (_i32, [_vp, _i64, _vp, _i64, _i32, _i32, _vp, _i64, _vp, _vp, _vp, _i64,
+                              _i32, _i64, _i64, _i32, _i32, _i32, _f32, _i32, _vp, _i64, _vp,
+                              _vp]),
+    "fk_mlstm_state_cols": (_i32, [_i32]),
+    "fk_mlstm_norm_cols": (_i32, [_i32]),
+    "fk_mlstm_step": (_i32, [_vp, _vp, _vp, _i64, _i32, _vp, _i64, _vp, _i64, _vp, _vp, _vp, _i32,
+                             _vp, _vp, _vp, _i64, _i64, _i32, _i32, _i32, _f32, _f32, _f32, _vp,
+                             _vp]),
+    "fk_mlstm_workspace_floats": (_i64, [_i64, _i32, _i32, _i32, _i32]),
+    "fk_mlstm_portions": (_i32, [_vp, _vp, _vp, _i64, _i32, _vp, _i64, _vp, _vp, _i32, _vp, _i32,
+                                 _vp, _vp, _vp, _i64, _i32, _i32, _i32, _f32, _f32, _vp, _i64,
+                                 _i64, _vp, _vp]),
     "fk_argmax_f32": (_i32, [_vp, _i64, _i64, _i64, _vp, _vp, _vp]),
     "fk_gemm_bf16_static": (_i32, [_vp, _i64, _vp, _vp, _vp, _i64, _i64, _i64, _i64, _vp, _vp]),
     "fk_gemm_bf16": (_i32, [_vp, _i64, _vp, _vp, _vp, _i64, _i64, _i64, _i64, _vp, _sz,
@@ -146,6 +176,11 @@ PROTOTYPES = {
 # Parts of the library that a partial build may leave out (build.COMPONENT_SOURCES),
 # by the symbols they export; a part is there with all of them or not at all.
 COMPONENTS = {
+    "decode_attn": [n for n in PROTOTYPES if n.startswith("fk_paged_decode_attn")],
+    "delta": [n for n in PROTOTYPES if n.startswith("fk_delta_")],
+    "latent": [n for n in PROTOTYPES if n.startswith("fk_latent_")],
+    "mlstm": [n for n in PROTOTYPES if n.startswith("fk_mlstm_")],
+    "experts": ["fk_moe_route", "fk_moe_route_counts", "fk_gather_rows"],
     "comm": [n for n in PROTOTYPES if n.startswith(("fk_comm_", "fk_allreduce_"))],
     "block": ["fk_decode_block_workspace_bytes", "fk_decode_block"],
 }

@@ -20,9 +20,11 @@ PKG = Path(__file__).resolve().parent
 CSRC = PKG / "csrc"
 LIB = PKG / "libfk_b200.so"
 # what every model needs, and the parts only some runs do (see _lib.COMPONENTS)
-CORE_SOURCES = ["fk_host.cu", "fk_elementwise.cu", "fk_attn.cu", "fk_gemm.cu", "fk_prefill.cu",
-                "fk_gemm_large.cu", "fk_mixer.cu", "fk_delta.cu", "fk_plain.cu"]
-COMPONENT_SOURCES = {"comm": ["fk_comm.cu"], "block": ["fk_block.cu"]}
+CORE_SOURCES = ["fk_host.cu", "fk_elementwise.cu", "fk_gemm.cu", "fk_prefill.cu",
+                "fk_gemm_large.cu", "fk_mixer.cu", "fk_residual.cu", "fk_group.cu", "fk_plain.cu"]
+COMPONENT_SOURCES = {"decode_attn": ["fk_attn.cu"], "delta": ["fk_delta.cu"],
+                     "latent": ["fk_latent.cu"], "mlstm": ["fk_mlstm.cu"],
+                     "experts": ["fk_moe.cu"], "comm": ["fk_comm.cu"], "block": ["fk_block.cu"]}
 SOURCES = CORE_SOURCES + [s for c in COMPONENT_SOURCES.values() for s in c]
 HEADERS = [CSRC / "fk_common.cuh", CSRC / "fk_tcgen05.cuh", CSRC / "fk_rowops.cuh",
            CSRC / "fk_types.cuh",

@@ -14,7 +14,6 @@
 //   delta_scan_kernel           the recurrence, token by token: single tokens, bound by
 //                               the state's bytes
 //   delta_scan_blocked_kernel   the recurrence over blocks, for portions
-//   delta_output_kernel         per-head RMS norm of o, weight, output gate
 //
 // The columns of S (value channels) are independent, so a column lives in the registers
 // of LANES threads; a CTA owns some columns of one head of one sequence.  The state comes
@@ -677,103 +676,6 @@ __global__ void __launch_bounds__(DL_THREADS) delta_scan_blocked_kernel(const De
     if (col_on[j]) dl_store<LANES, CPL>(st[j], q, s[j]);
 }
 
-struct DeltaOutParams {
-  const float* o;                     // [rows][heads * d]
-  const void* g; int64_t g_stride;    // gate projection
-  const float* weight;                // [heads * d]
-  void* out; int64_t out_stride;      // [rows, out_stride], tail beyond heads * d zeroed
-  int64_t rows; int heads, d;
-  float eps;
-};
-
-// d a multiple of 4: LPH lanes per (token, head), four channels a lane.
-template <typename T, int LPH>
-__global__ void __launch_bounds__(256) delta_output_vec_kernel(const DeltaOutParams p) {
-  pdl_launch_dependents();
-  pdl_wait();
-  constexpr int PER = 256 / LPH;                 // (token, head) pairs per CTA and pass
-  const int j = threadIdx.x % LPH;
-  const int h = blockIdx.x * PER + threadIdx.x / LPH;
-  const int64_t hd = (int64_t)p.heads * p.d;
-  const bool on = h < p.heads && j * 4 < p.d;
-  const int64_t c0 = (int64_t)h * p.d + j * 4;
-  const float4 wt = on ? __ldg(reinterpret_cast<const float4*>(p.weight + c0))
-                       : make_float4(0.f, 0.f, 0.f, 0.f);
-  for (int64_t t = blockIdx.y; t < p.rows; t += gridDim.y) {
-    float4 x = make_float4(0.f, 0.f, 0.f, 0.f), g = x;
-    if (on) {
-      x = *reinterpret_cast<const float4*>(p.o + t * hd + c0);
-      g = Elem<T>::load4(static_cast<const T*>(p.g) + t * p.g_stride + c0);
-    }
-    float ss = sumsq(x);
-#pragma unroll
-    for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-    const float rs = rsqrtf(ss / (float)p.d + p.eps);
-    T* out = static_cast<T*>(p.out) + t * p.out_stride;
-    if (on)
-      Elem<T>::store4(out + c0, (x * rs) * wt * make_float4(sigmoid_f32(g.x), sigmoid_f32(g.y),
-                                                            sigmoid_f32(g.z), sigmoid_f32(g.w)));
-    if (blockIdx.x == 0 && hd + threadIdx.x < p.out_stride && threadIdx.x < 64)
-      Elem<T>::store(out + hd + threadIdx.x, 0.f);
-  }
-}
-
-// One warp per (token, head), any d.
-template <typename T>
-__global__ void __launch_bounds__(256) delta_output_kernel(const DeltaOutParams p) {
-  pdl_launch_dependents();
-  pdl_wait();
-  const int lane = threadIdx.x & 31;
-  const int h = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-  const int64_t hd = (int64_t)p.heads * p.d;
-  if (h > p.heads) return;
-  for (int64_t t = blockIdx.y; t < p.rows; t += gridDim.y) {
-    T* out = static_cast<T*>(p.out) + t * p.out_stride;
-    if (h == p.heads) {
-      for (int64_t c = hd + lane; c < p.out_stride; c += 32) Elem<T>::store(out + c, 0.f);
-      continue;
-    }
-    const float* o = p.o + t * hd + (int64_t)h * p.d;
-    const T* g = static_cast<const T*>(p.g) + t * p.g_stride + (int64_t)h * p.d;
-    float x[DL_MAX_DIM / 32];
-    float ss = 0.f;
-#pragma unroll
-    for (int i = 0; i < DL_MAX_DIM / 32; ++i) {
-      const int c = lane + i * 32;
-      x[i] = c < p.d ? o[c] : 0.f;
-      ss += x[i] * x[i];
-    }
-    ss = warp_sum(ss);
-    const float rs = rsqrtf(ss / (float)p.d + p.eps);
-#pragma unroll
-    for (int i = 0; i < DL_MAX_DIM / 32; ++i) {
-      const int c = lane + i * 32;
-      if (c < p.d)
-        Elem<T>::store(out + (int64_t)h * p.d + c,
-                       x[i] * rs * p.weight[(int64_t)h * p.d + c] *
-                           sigmoid_f32(Elem<T>::load(g + c)));
-    }
-  }
-}
-
-template <typename T, int LPH>
-static cudaError_t launch_output_vec(const DeltaOutParams& p, cudaStream_t s) {
-  constexpr int PER = 256 / LPH;
-  const int gx = (p.heads + PER - 1) / PER;
-  int64_t gy = (int64_t)sm_count() * 8 / gx;       // CTAs resident at once, tokens strided
-  gy = gy < 1 ? 1 : gy < p.rows ? gy : p.rows;
-  return launch_kernel(delta_output_vec_kernel<T, LPH>, dim3((unsigned)gx, (unsigned)gy),
-                       dim3(256), 0, s, p);
-}
-template <typename T>
-static cudaError_t launch_output(const DeltaOutParams& p, bool vec, cudaStream_t s) {
-  if (vec && p.d <= 32) return launch_output_vec<T, 8>(p, s);
-  if (vec && p.d <= 64) return launch_output_vec<T, 16>(p, s);
-  if (vec) return launch_output_vec<T, 32>(p, s);
-  const dim3 grid((unsigned)(p.heads / 8 + 1), (unsigned)(p.rows < 8192 ? p.rows : 8192));
-  return launch_kernel(delta_output_kernel<T>, grid, dim3(256), 0, s, p);
-}
-
 static int delta_padded(int d) { return d <= 32 ? 32 : d <= 64 ? 64 : d <= 128 ? 128 : 256; }
 
 template <typename T, int DP, bool BLOCKED>
@@ -918,29 +820,6 @@ int fk_delta_scan(const float* packed, int blocked, float* o, float* state, int 
     case 128: return launch_scan<16, 8, 16, 8>(p, blocked != 0, s);
     default: return launch_scan<32, 8, 32, 8>(p, blocked != 0, s);
   }
-}
-
-int fk_delta_output(const float* o, const void* gate, int64_t gate_stride, const float* weight,
-                    void* out, int64_t out_stride, int is_f32, int64_t rows, int heads, int dim,
-                    float eps, fk_stream_t stream) {
-  FK_REQUIRE(rows >= 0 && heads > 0 && dim > 0, FK_ERR_INVALID_ARG,
-             "fk_delta_output: bad sizes");
-  if (rows == 0) return FK_OK;
-  FK_REQUIRE(o && gate && weight && out, FK_ERR_INVALID_ARG, "fk_delta_output: null pointer");
-  FK_REQUIRE(dim <= DL_MAX_DIM, FK_ERR_UNSUPPORTED, "fk_delta_output: head size %d too large",
-             dim);
-  FK_REQUIRE(out_stride >= (int64_t)heads * dim && gate_stride >= (int64_t)heads * dim,
-             FK_ERR_INVALID_ARG, "fk_delta_output: bad stride");
-  DeltaOutParams p{};
-  p.o = o; p.g = gate; p.g_stride = gate_stride; p.weight = weight; p.out = out;
-  p.out_stride = out_stride; p.rows = rows; p.heads = heads; p.d = dim; p.eps = eps;
-  cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const bool vec = dim % 4 == 0 && dim <= 128 && gate_stride % 4 == 0 && out_stride % 4 == 0 &&
-                   out_stride - (int64_t)heads * dim <= 64 && aligned16(o) && aligned16(gate) &&
-                   aligned16(weight) && aligned16(out);
-  FK_CUDA_OK(is_f32 ? launch_output<float>(p, vec, s) : launch_output<uint16_t>(p, vec, s));
-  count_launch();
-  return FK_OK;
 }
 
 }  // extern "C"

@@ -1,0 +1,655 @@
+// Grouped projections y = act(x w_g^T + bias), g = 0 .. groups - 1, in two forms:
+//
+//   column groups   every group takes all rows, its own columns of x and of y
+//                   (x + g x_group, y + g y_group): per-head products, and with one
+//                   group a plain projection with fp32 output
+//   row groups      group g takes the rows offsets[g] .. offsets[g + 1] of y (x rows the
+//                   same, or gather[row]): experts of a mixture
+//
+// act >= 0: w_g has 2 n rows [gate; up] and y = act(x gate^T) * (x up^T).
+// bf16 operands with fp32 accumulation and bf16 or fp32 results, or true fp32.
+//
+//   group_any_kernel     fp32 FMA, any sizes (fp32 operands)
+//   group_skinny_kernel  few rows: streams the weights straight into mma.sync fragments.
+//                        A product may take its k in any order as long as both operands
+//                        do, so a lane's 16 contiguous bytes of a row serve as the k's of
+//                        two instructions: no shared memory, no shuffles.
+//   group_large_kernel   many rows: tcgen05, 128 rows x 256 weight rows, TMA-fed,
+//                        accumulators double-buffered in tensor memory
+#include "fk_tcgen05.cuh"
+#include "fk_types.cuh"
+
+#include <mutex>
+#include <unordered_map>
+
+namespace fk {
+
+struct GroupParams {
+  const void* x; int64_t x_stride, x_group;
+  const void* w; int64_t w_rows;               // weight rows per group (n, or 2 n)
+  const float* bias;                           // [n] or null
+  void* y; int64_t y_stride, y_group;
+  const int32_t* offsets; const int32_t* gather;
+  int64_t rows;                                // column groups: rows; row groups: all rows
+  int64_t x_rows;                              // rows of x (bounds of gather)
+  int groups, n, k, act;
+  int32_t* status;
+};
+
+__device__ __forceinline__ float group_act(float g, int kind) {
+  return kind == FK_ACT_SILU ? g * sigmoid_f32(g) : gelu_tanh_f32(g);
+}
+
+// Row range of a group inside y; empty or clamped when the offsets are not a partition.
+__device__ __forceinline__ void group_range(const GroupParams& p, int g, int64_t* first,
+                                            int64_t* count) {
+  if (!p.offsets) { *first = 0; *count = p.rows; return; }
+  int64_t a = p.offsets[g], b = p.offsets[g + 1];
+  if (a < 0 || b < a || b > p.rows) {
+    if (p.status && threadIdx.x == 0) atomicOr(p.status, FK_DEV_BAD_SLOT);
+    a = b = 0;
+  }
+  *first = a;
+  *count = b - a;
+}
+__device__ __forceinline__ int64_t group_x_row(const GroupParams& p, int64_t row) {
+  if (!p.gather) return row;
+  const int64_t r = p.gather[row];
+  if (r < 0 || r >= p.x_rows) {
+    if (p.status) atomicOr(p.status, FK_DEV_BAD_SLOT);
+    return 0;
+  }
+  return r;
+}
+
+// ------------------------------------------------------------------------- any size
+constexpr int GA_M = 64, GA_N = 64, GA_K = 16;
+
+template <bool ACT>
+__global__ void __launch_bounds__(256) group_any_kernel(const GroupParams p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  constexpr int NB = ACT ? 2 : 1;
+  __shared__ float xs[GA_K][GA_M + 4], ws[NB][GA_K][GA_N + 4];
+  const int g = blockIdx.z;
+  int64_t first, count;
+  group_range(p, g, &first, &count);
+  const int n0 = blockIdx.x * GA_N;
+  const int64_t m0 = (int64_t)blockIdx.y * GA_M;
+  if (m0 >= count) return;
+  const float* x = static_cast<const float*>(p.x) + (p.offsets ? 0 : g * p.x_group);
+  const float* w = static_cast<const float*>(p.w) + (int64_t)g * p.w_rows * p.k;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  const int lr = threadIdx.x >> 2, lc = (threadIdx.x & 3) * 4;
+  const bool x_on = m0 + lr < count, w_on = n0 + lr < p.n;
+  const float* xr = x + (x_on ? group_x_row(p, first + m0 + lr) : 0) * p.x_stride;
+  float acc[NB][4][4] = {};
+  for (int k0 = 0; k0 < p.k; k0 += GA_K) {
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f), b[NB];
+#pragma unroll
+    for (int e = 0; e < NB; ++e) b[e] = a;
+    if (k0 + lc < p.k) {
+      if (x_on) a = *reinterpret_cast<const float4*>(xr + k0 + lc);
+#pragma unroll
+      for (int e = 0; e < NB; ++e)
+        if (w_on)
+          b[e] = *reinterpret_cast<const float4*>(w + ((int64_t)e * p.n + n0 + lr) * p.k + k0 + lc);
+    }
+    __syncthreads();
+    xs[lc][lr] = a.x; xs[lc + 1][lr] = a.y; xs[lc + 2][lr] = a.z; xs[lc + 3][lr] = a.w;
+#pragma unroll
+    for (int e = 0; e < NB; ++e) {
+      ws[e][lc][lr] = b[e].x; ws[e][lc + 1][lr] = b[e].y;
+      ws[e][lc + 2][lr] = b[e].z; ws[e][lc + 3][lr] = b[e].w;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int kk = 0; kk < GA_K; ++kk) {
+      const float4 av = *reinterpret_cast<const float4*>(&xs[kk][ty * 4]);
+      const float aa[4] = {av.x, av.y, av.z, av.w};
+#pragma unroll
+      for (int e = 0; e < NB; ++e) {
+        const float4 bv = *reinterpret_cast<const float4*>(&ws[e][kk][tx * 4]);
+        const float bb[4] = {bv.x, bv.y, bv.z, bv.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) acc[e][i][j] = fmaf(aa[i], bb[j], acc[e][i][j]);
+      }
+    }
+  }
+  float* y = static_cast<float*>(p.y) + (p.offsets ? 0 : g * p.y_group);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int64_t r = m0 + ty * 4 + i;
+    if (r >= count) break;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int c = n0 + tx * 4 + j;
+      if (c >= p.n) continue;
+      float v = acc[0][i][j] + (p.bias ? p.bias[c] : 0.f);
+      if (ACT) v = group_act(v, p.act) * acc[NB - 1][i][j];
+      y[(first + r) * p.y_stride + c] = v;
+    }
+  }
+}
+
+// ------------------------------------------------------------------------- few rows
+// CTA = 16 MT weight rows (of gate and of up with ACT) of one group; its warps share the
+// k range.  Rows go 8 NT at a time.
+template <int MT, int NT, bool ACT, typename OUT>
+__global__ void __launch_bounds__(256) group_skinny_kernel(const GroupParams p) {
+  extern __shared__ float gs_red[];            // [warps][NB MT 16][8 NT]
+  pdl_launch_dependents();
+  constexpr int NB = ACT ? 2 : 1;
+  constexpr int TILES = NB * MT;
+  constexpr int COLS = 8 * NT;
+  const int g = blockIdx.y;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  const int gr = lane >> 2, tq = lane & 3;
+  const int n0 = blockIdx.x * (16 * MT);
+  const uint16_t* w = static_cast<const uint16_t*>(p.w) + (int64_t)g * p.w_rows * p.k;
+  const uint16_t* wr[TILES][2];
+#pragma unroll
+  for (int e = 0; e < TILES; ++e)
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      int r = n0 + (e % MT) * 16 + h * 8 + gr;
+      if (r >= p.n) r = p.n - 1;               // computed, not stored
+      wr[e][h] = w + ((int64_t)(e / MT) * p.n + r) * p.k + tq * 8;
+    }
+  pdl_wait();
+  int64_t first, count;
+  group_range(p, g, &first, &count);
+  if (count == 0) return;
+  const uint16_t* x = static_cast<const uint16_t*>(p.x) + (p.offsets ? 0 : g * p.x_group);
+  const int chunks = (p.k + 31) >> 5;
+  for (int64_t t0 = 0; t0 < count; t0 += COLS) {
+    const uint16_t* xr[NT];
+    bool on[NT];
+#pragma unroll
+    for (int j = 0; j < NT; ++j) {
+      const int64_t t = t0 + j * 8 + gr;
+      on[j] = t < count;
+      xr[j] = x + (on[j] ? group_x_row(p, first + t) : 0) * p.x_stride + tq * 8;
+    }
+    float acc[TILES][NT][4];
+#pragma unroll
+    for (int e = 0; e < TILES; ++e)
+#pragma unroll
+      for (int j = 0; j < NT; ++j)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) acc[e][j][i] = 0.f;
+    constexpr int UN = TILES * 2 + NT <= 4 ? 4 : TILES * 2 + NT <= 8 ? 2 : 1;
+    for (int c0 = warp; c0 < chunks; c0 += warps * UN) {
+      uint4 a[UN][TILES][2], b[UN][NT];
+#pragma unroll
+      for (int u = 0; u < UN; ++u) {
+        const int c = c0 + u * warps;
+        const bool in = c * 32 + tq * 8 < p.k;
+#pragma unroll
+        for (int e = 0; e < TILES; ++e)
+#pragma unroll
+          for (int h = 0; h < 2; ++h)
+            a[u][e][h] = in ? __ldg(reinterpret_cast<const uint4*>(wr[e][h] + c * 32))
+                            : make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll
+        for (int j = 0; j < NT; ++j)
+          b[u][j] = in && on[j] ? *reinterpret_cast<const uint4*>(xr[j] + c * 32)
+                                : make_uint4(0u, 0u, 0u, 0u);
+      }
+#pragma unroll
+      for (int u = 0; u < UN; ++u)
+#pragma unroll
+        for (int e = 0; e < TILES; ++e) {
+          const uint32_t lo[4] = {a[u][e][0].x, a[u][e][1].x, a[u][e][0].y, a[u][e][1].y};
+          const uint32_t hi[4] = {a[u][e][0].z, a[u][e][1].z, a[u][e][0].w, a[u][e][1].w};
+#pragma unroll
+          for (int j = 0; j < NT; ++j) {
+            mma_bf16_16816(acc[e][j], lo, b[u][j].x, b[u][j].y);
+            mma_bf16_16816(acc[e][j], hi, b[u][j].z, b[u][j].w);
+          }
+        }
+    }
+    __syncthreads();
+    float* mine = gs_red + (int64_t)warp * TILES * 16 * COLS;
+#pragma unroll
+    for (int e = 0; e < TILES; ++e)
+#pragma unroll
+      for (int j = 0; j < NT; ++j)
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          mine[(e * 16 + gr + (i >> 1) * 8) * COLS + j * 8 + tq * 2 + (i & 1)] = acc[e][j][i];
+    __syncthreads();
+    OUT* y = static_cast<OUT*>(p.y) + (p.offsets ? 0 : g * p.y_group);
+    for (int i = threadIdx.x; i < MT * 16 * COLS; i += blockDim.x) {
+      const int r = i % (MT * 16), t = i / (MT * 16);
+      const int c = n0 + r;
+      if (c >= p.n || t0 + t >= count) continue;
+      float v = p.bias ? p.bias[c] : 0.f, up = 0.f;
+      for (int q = 0; q < warps; ++q) {
+        v += gs_red[((int64_t)q * TILES * 16 + r) * COLS + t];
+        if (ACT) up += gs_red[((int64_t)q * TILES * 16 + MT * 16 + r) * COLS + t];
+      }
+      if (ACT) v = group_act(v, p.act) * up;
+      Elem<OUT>::store(y + (first + t0 + t) * p.y_stride + c, v);
+    }
+  }
+}
+
+// ------------------------------------------------------------------------ many rows
+constexpr int GG_BM = 128, GG_BN = 256, GG_BK = 64, GG_STAGES = 4;
+constexpr int GG_A_BYTES = GG_BM * GG_BK * 2, GG_B_BYTES = GG_BN * GG_BK * 2;
+constexpr int GG_STAGE_BYTES = GG_A_BYTES + GG_B_BYTES;
+constexpr int GG_MAX_GROUPS = 1024;
+constexpr int GG_OFF_TILES = GG_STAGES * GG_STAGE_BYTES;       // first tile of every group
+constexpr int GG_OFF_BAR = GG_OFF_TILES + (GG_MAX_GROUPS + 8) * 4;
+constexpr int GG_SMEM_ALLOC = GG_OFF_BAR + 256 + 1024;
+constexpr int GG_THREADS = 192;
+static_assert(GG_SMEM_ALLOC <= 232448, "shared memory budget");
+
+__device__ __forceinline__ uint64_t gg_ns() {
+  uint64_t t;
+  asm volatile("mov.u64 %0, %globaltimer;" : "=l"(t));
+  return t;
+}
+__device__ __forceinline__ bool gg_wait(uint64_t* bar, uint32_t parity, volatile int* abort_flag,
+                                        int32_t* status) {
+  if (mbar_try_wait(bar, parity)) return true;
+  const uint64_t t0 = gg_ns();
+  for (;;) {
+    for (int i = 0; i < 128; ++i)
+      if (mbar_try_wait(bar, parity)) return true;
+    if (*abort_flag) return false;
+    if (gg_ns() - t0 > 2000000000ull) {
+      *abort_flag = 1;
+      if (status) atomicOr(status, FK_DEV_WAIT_TIMEOUT);
+      return false;
+    }
+  }
+}
+__device__ __forceinline__ bool gg_wait_warp(uint64_t* bar, uint32_t parity,
+                                             volatile int* abort_flag, int32_t* status) {
+  return __all_sync(0xffffffffu, gg_wait(bar, parity, abort_flag, status) ? 1 : 0) != 0;
+}
+
+struct GgTile {
+  int g, nt;
+  int64_t row0, rows_left;   // first row (of y and x), rows of the group from there on
+};
+
+// Tiles of a group lie together, rows fastest.
+__device__ __forceinline__ GgTile gg_tile(const GroupParams& p, const int* first_tile, int ti,
+                                          int n_tiles) {
+  int lo = 0, hi = p.groups;
+  while (hi - lo > 1) {
+    const int mid = (lo + hi) >> 1;
+    if (first_tile[mid] <= ti) lo = mid; else hi = mid;
+  }
+  const int in_g = ti - first_tile[lo];
+  const int mts = (first_tile[lo + 1] - first_tile[lo]) / n_tiles;
+  const int mt = in_g % mts;
+  GgTile t;
+  t.g = lo;
+  t.nt = in_g / mts;
+  int64_t a = 0, b = p.rows;
+  if (p.offsets) { a = p.offsets[lo]; b = p.offsets[lo + 1]; }
+  t.row0 = a + (int64_t)mt * GG_BM;
+  t.rows_left = b - t.row0;
+  return t;
+}
+
+template <bool ACT, typename OUT>
+__global__ void __launch_bounds__(GG_THREADS, 1)
+group_large_kernel(const __grid_constant__ CUtensorMap tmap_x,
+                   const __grid_constant__ CUtensorMap tmap_w, const GroupParams p) {
+  extern __shared__ uint8_t gg_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(gg_raw) + 1023) &
+                                             ~uintptr_t(1023));
+  int* first_tile = reinterpret_cast<int*>(smem + GG_OFF_TILES);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + GG_OFF_BAR);
+  uint64_t* full = bars;
+  uint64_t* empty = bars + GG_STAGES;
+  uint64_t* acc_full = bars + 2 * GG_STAGES;       // [2]
+  uint64_t* acc_empty = acc_full + 2;              // [2]
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(acc_empty + 2);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(acc_empty + 3);
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  constexpr int TN = ACT ? GG_BN / 2 : GG_BN;      // outputs per tile
+  const int n_tiles = (p.n + TN - 1) / TN;
+  const int kb_total = (p.k + GG_BK - 1) / GG_BK;
+
+  pdl_launch_dependents();
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < GG_STAGES; ++i) {
+      mbar_init(&full[i], 1);
+      mbar_init(&empty[i], 1);
+    }
+    for (int b = 0; b < 2; ++b) {
+      mbar_init(&acc_full[b], 1);
+      mbar_init(&acc_empty[b], 4);
+    }
+    *abort_flag = 0;
+    mbar_fence_init();
+    tma_prefetch_desc(&tmap_x);
+    tma_prefetch_desc(&tmap_w);
+  }
+  if (warp == 1) tmem_alloc(tmem_slot, 512);
+  pdl_wait();
+  // running tile count of the groups
+  if (warp == 0) {
+    int base = 0;
+    for (int g0 = 0; g0 < p.groups; g0 += 32) {
+      int64_t f = 0, c = 0;
+      const int g = g0 + lane;
+      if (g < p.groups) {
+        if (p.offsets) {
+          f = p.offsets[g];
+          c = p.offsets[g + 1] - f;
+          if (f < 0 || c < 0 || f + c > p.rows) {
+            if (p.status) atomicOr(p.status, FK_DEV_BAD_SLOT);
+            c = 0;
+          }
+        } else {
+          c = p.rows;
+        }
+      }
+      const int mine = (int)((c + GG_BM - 1) / GG_BM) * n_tiles;
+      int run = mine;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int up = __shfl_up_sync(0xffffffffu, run, o);
+        if (lane >= o) run += up;
+      }
+      if (g < p.groups) first_tile[g] = base + run - mine;
+      base += __shfl_sync(0xffffffffu, run, 31);
+    }
+    if (lane == 0) first_tile[p.groups] = base;
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_got = *tmem_slot;
+  if (tmem_got != 0) {        // all 512 columns: the allocation starts at column 0
+    if (threadIdx.x == 0 && p.status) atomicOr(p.status, FK_DEV_TMEM_BASE);
+    __syncthreads();
+    if (warp == 1) tmem_dealloc(tmem_got, 512);
+    return;
+  }
+  const int total = first_tile[p.groups];
+
+  if (warp == 0) {
+    if (lane == 0) {
+      int stage = 0;
+      uint32_t phase = 0;
+      bool ok = true;
+      for (int ti = blockIdx.x; ti < total && ok; ti += gridDim.x) {
+        const GgTile t = gg_tile(p, first_tile, ti, n_tiles);
+        const int xc = p.offsets ? 0 : (int)(t.g * p.x_group);
+        const int wrow = (int)(t.g * p.w_rows) + t.nt * TN;
+        for (int kb = 0; kb < kb_total; ++kb) {
+          if (!gg_wait(&empty[stage], phase ^ 1, abort_flag, p.status)) { ok = false; break; }
+          uint8_t* dst = smem + stage * GG_STAGE_BYTES;
+          mbar_arrive_expect_tx(&full[stage], (uint32_t)GG_STAGE_BYTES);
+          tma_load_2d(dst, &tmap_x, &full[stage], xc + kb * GG_BK, (int)t.row0);
+          if (ACT) {
+            tma_load_2d(dst + GG_A_BYTES, &tmap_w, &full[stage], kb * GG_BK, wrow);
+            tma_load_2d(dst + GG_A_BYTES + GG_B_BYTES / 2, &tmap_w, &full[stage], kb * GG_BK,
+                        wrow + p.n);
+          } else {
+            tma_load_2d(dst + GG_A_BYTES, &tmap_w, &full[stage], kb * GG_BK, wrow);
+          }
+          if (++stage == GG_STAGES) { stage = 0; phase ^= 1; }
+        }
+      }
+    }
+  } else if (warp == 1) {
+    constexpr uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) |
+                               ((uint32_t)(GG_BN >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
+    int stage = 0;
+    uint32_t phase = 0, done = 0;
+    bool ok = true;
+    for (int ti = blockIdx.x; ti < total && ok; ti += gridDim.x) {
+      const uint32_t buf = done & 1u, use = done >> 1;
+      if (use > 0) ok = gg_wait_warp(&acc_empty[buf], (use - 1) & 1u, abort_flag, p.status);
+      if (!ok) break;
+      tc_fence_after();
+      for (int kb = 0; kb < kb_total; ++kb) {
+        ok = gg_wait_warp(&full[stage], phase, abort_flag, p.status);
+        if (!ok) break;
+        tc_fence_after();
+        const uint32_t a = smem_u32(smem + stage * GG_STAGE_BYTES);
+        const uint32_t b = a + GG_A_BYTES;
+#pragma unroll
+        for (int kk = 0; kk < GG_BK / 16; ++kk)
+          tc_mma_bf16_elect(buf * GG_BN, smem_desc_sw128(a + kk * 32),
+                            smem_desc_sw128(b + kk * 32), idesc, (kb > 0 || kk > 0) ? 1u : 0u);
+        tc_commit_elect(&empty[stage]);
+        if (++stage == GG_STAGES) { stage = 0; phase ^= 1; }
+      }
+      if (!ok) break;
+      tc_commit_elect(&acc_full[buf]);
+      ++done;
+    }
+  } else {
+    const int q = warp & 3, row = q * 32 + lane;
+    const uint32_t lane_addr = (uint32_t)(q * 32) << 16;
+    uint32_t done = 0;
+    for (int ti = blockIdx.x; ti < total; ti += gridDim.x) {
+      const GgTile t = gg_tile(p, first_tile, ti, n_tiles);
+      const uint32_t buf = done & 1u, use = done >> 1;
+      if (!gg_wait(&acc_full[buf], use & 1u, abort_flag, p.status)) break;
+      tc_fence_after();
+      const bool live = row < t.rows_left;
+      OUT* y = static_cast<OUT*>(p.y) + (p.offsets ? 0 : t.g * p.y_group) +
+               (t.row0 + (live ? row : 0)) * p.y_stride;
+      const int n0 = t.nt * TN;
+#pragma unroll 1
+      for (int c = 0; c < TN / 32; ++c) {
+        uint32_t v[32], u[ACT ? 32 : 1];
+        tc_ld32(lane_addr + buf * GG_BN + c * 32, v);
+        if (ACT) tc_ld32(lane_addr + buf * GG_BN + GG_BN / 2 + c * 32, u);
+        tc_wait_ld();
+        if (!live || n0 + c * 32 >= p.n) continue;
+        float f[32];
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          f[i] = __uint_as_float(v[i]);
+          if (ACT) {
+            const float up = __uint_as_float(u[ACT ? i : 0]);
+            f[i] = (p.act == FK_ACT_SILU ? silu_f32(f[i])
+                                         : __fdividef(f[i], 1.0f + __expf(-gelu_tanh_arg(f[i])))) *
+                   up;
+          } else if (p.bias && n0 + c * 32 + i < p.n) {
+            f[i] += p.bias[n0 + c * 32 + i];
+          }
+        }
+        OUT* dst = y + n0 + c * 32;
+        constexpr int PER = 16 / (int)sizeof(OUT);
+#pragma unroll
+        for (int i = 0; i < 32; i += PER) {
+          if (n0 + c * 32 + i + PER <= p.n) {
+            if (sizeof(OUT) == 2)
+              *reinterpret_cast<uint4*>(dst + i) =
+                  make_uint4(pack_bf16(f[i], f[i + 1]), pack_bf16(f[i + 2], f[i + 3]),
+                             pack_bf16(f[i + 4 < 32 ? i + 4 : 0], f[i + 5 < 32 ? i + 5 : 0]),
+                             pack_bf16(f[i + 6 < 32 ? i + 6 : 0], f[i + 7 < 32 ? i + 7 : 0]));
+            else
+              *reinterpret_cast<float4*>(dst + i) = make_float4(f[i], f[i + 1], f[i + 2], f[i + 3]);
+          } else {
+#pragma unroll
+            for (int j = 0; j < PER; ++j)
+              if (n0 + c * 32 + i + j < p.n) Elem<OUT>::store(dst + i + j, f[i + j]);
+          }
+        }
+      }
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&acc_empty[buf]);
+      ++done;
+    }
+  }
+
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem_got, 512);
+  }
+}
+
+// ----------------------------------------------------------------------------- host
+struct GgKey {
+  const void* ptr; int64_t rows, cols, stride; int box_rows;
+  bool operator==(const GgKey& o) const {
+    return ptr == o.ptr && rows == o.rows && cols == o.cols && stride == o.stride &&
+           box_rows == o.box_rows;
+  }
+};
+struct GgHash {
+  size_t operator()(const GgKey& k) const {
+    return std::hash<const void*>()(k.ptr) ^
+           std::hash<int64_t>()(k.rows * 1315423911ll + k.cols * 2654435761ll + k.stride +
+                                k.box_rows * 7919ll);
+  }
+};
+static std::mutex g_gg_mu;
+static std::unordered_map<GgKey, CUtensorMap, GgHash> g_gg_maps;
+
+// [rows, cols] bf16 with a row stride: box = 64 columns x box_rows rows, 128B swizzle
+static int gg_map(const void* ptr, int64_t rows, int64_t cols, int64_t stride, int box_rows,
+                  CUtensorMap* out) {
+  GgKey key{ptr, rows, cols, stride, box_rows};
+  std::lock_guard<std::mutex> lk(g_gg_mu);
+  auto it = g_gg_maps.find(key);
+  if (it != g_gg_maps.end()) {
+    *out = it->second;
+    return FK_OK;
+  }
+  tensormap_encode_fn enc = get_tensormap_encode();
+  FK_REQUIRE(enc != nullptr, FK_ERR_CUDA,
+             "cuTensorMapEncodeTiled not available from the driver");
+  cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
+  cuuint64_t strides[1] = {(cuuint64_t)stride * 2};
+  cuuint32_t box[2] = {GG_BK, (cuuint32_t)box_rows};
+  cuuint32_t estr[2] = {1, 1};
+  CUtensorMap m;
+  CUresult r = enc(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(ptr), dims,
+                   strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                   CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                   CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  FK_REQUIRE(r == CUDA_SUCCESS, FK_ERR_CUDA, "cuTensorMapEncodeTiled failed with code %d",
+             (int)r);
+  if (g_gg_maps.size() > 4096) g_gg_maps.clear();
+  g_gg_maps.emplace(key, m);
+  *out = m;
+  return FK_OK;
+}
+
+template <int MT, int NT, bool ACT, typename OUT>
+static int launch_skinny_one(const GroupParams& p, cudaStream_t s) {
+  const int chunks = (p.k + 31) / 32;
+  const int warps = chunks >= 16 && NT * MT <= 8 ? 8 : chunks >= 4 ? 4 : 2;
+  const size_t smem = (size_t)warps * (ACT ? 2 : 1) * MT * 16 * 8 * NT * 4;
+  static PerDeviceOnce once;
+  FK_CUDA_OK(set_max_dynamic_smem(once, group_skinny_kernel<MT, NT, ACT, OUT>,
+                                  8 * (ACT ? 2 : 1) * MT * 16 * 8 * NT * 4));
+  const dim3 grid((unsigned)((p.n + 16 * MT - 1) / (16 * MT)), (unsigned)p.groups);
+  FK_CUDA_OK(launch_kernel(group_skinny_kernel<MT, NT, ACT, OUT>, grid, dim3(32u * warps), smem,
+                           s, p));
+  count_launch();
+  return FK_OK;
+}
+template <bool ACT, typename OUT>
+static int launch_skinny(const GroupParams& p, int64_t expect, cudaStream_t s) {
+  if (expect <= 8) return launch_skinny_one<1, 1, ACT, OUT>(p, s);
+  if (expect <= 16) return launch_skinny_one<1, 2, ACT, OUT>(p, s);
+  if (expect <= 32) return launch_skinny_one<1, 4, ACT, OUT>(p, s);
+  return launch_skinny_one<1, 8, ACT, OUT>(p, s);
+}
+template <bool ACT, typename OUT>
+static int launch_large(const GroupParams& p, int64_t x_cols, cudaStream_t s) {
+  constexpr int TN = ACT ? GG_BN / 2 : GG_BN;
+  const int64_t n_tiles = (p.n + TN - 1) / TN;
+  const int64_t bound = p.offsets ? ((p.rows + GG_BM - 1) / GG_BM + p.groups) * n_tiles
+                                  : (p.rows + GG_BM - 1) / GG_BM * n_tiles * p.groups;
+  FK_REQUIRE(bound <= 0x7fffffff && p.rows < (1ll << 31) && p.groups * p.w_rows < (1ll << 31),
+             FK_ERR_UNSUPPORTED, "fk_group_gemm: too many tiles");
+  CUtensorMap mx, mw;
+  int rc = gg_map(p.x, p.x_rows, x_cols, p.x_stride, GG_BM, &mx);
+  if (rc != FK_OK) return rc;
+  rc = gg_map(p.w, p.groups * p.w_rows, p.k, p.k, TN, &mw);
+  if (rc != FK_OK) return rc;
+  static PerDeviceOnce once;
+  FK_CUDA_OK(set_max_dynamic_smem(once, group_large_kernel<ACT, OUT>, GG_SMEM_ALLOC));
+  const int ctas = (int)(bound < sm_count() ? bound : sm_count());
+  FK_CUDA_OK(launch_kernel(group_large_kernel<ACT, OUT>, dim3((unsigned)ctas), dim3(GG_THREADS),
+                           (size_t)GG_SMEM_ALLOC, s, mx, mw, p));
+  count_launch();
+  return FK_OK;
+}
+
+}  // namespace fk
+
+using namespace fk;
+
+extern "C" {
+
+int fk_group_gemm(const void* x, int64_t x_stride, int64_t x_group, int64_t x_rows,
+                  const void* w, const float* bias, void* y, int64_t y_stride, int64_t y_group,
+                  int is_f32, int y_f32, const int32_t* offsets, const int32_t* gather,
+                  int64_t rows, int64_t expect_rows, int groups, int64_t n, int64_t k, int act,
+                  int32_t* status, fk_stream_t stream) {
+  FK_REQUIRE(rows >= 0 && groups > 0 && n >= 0 && k > 0 && x_rows >= 0, FK_ERR_INVALID_ARG,
+             "fk_group_gemm: bad sizes");
+  if (rows == 0 || n == 0) return FK_OK;
+  FK_REQUIRE(x && w && y, FK_ERR_INVALID_ARG, "fk_group_gemm: null pointer");
+  FK_REQUIRE(!gather || offsets, FK_ERR_INVALID_ARG,
+             "fk_group_gemm: only row groups can be gathered");
+  FK_REQUIRE(gather || x_rows >= rows, FK_ERR_INVALID_ARG, "fk_group_gemm: x has too few rows");
+  FK_REQUIRE(act < 0 || ((act == FK_ACT_SILU || act == FK_ACT_GELU_TANH) && !bias),
+             FK_ERR_INVALID_ARG, "fk_group_gemm: unknown activation %d, or one with a bias", act);
+  const int64_t x_cols = offsets ? k : (groups - 1) * x_group + k;
+  FK_REQUIRE(x_group >= 0 && y_group >= 0 && x_stride >= x_cols &&
+                 y_stride >= (offsets ? n : (groups - 1) * y_group + n) &&
+                 (offsets || groups == 1 || y_group >= n),
+             FK_ERR_INVALID_ARG, "fk_group_gemm: row stride smaller than the row");
+  FK_REQUIRE(n < (1ll << 30) && k < (1ll << 30) && groups <= 65535, FK_ERR_UNSUPPORTED,
+             "fk_group_gemm: dimension too large");
+  const int unit = is_f32 ? 4 : 8;
+  FK_REQUIRE(k % unit == 0 && x_stride % unit == 0 && x_group % unit == 0 && aligned16(x) &&
+                 aligned16(w) && aligned16(y),
+             FK_ERR_ALIGNMENT, "fk_group_gemm: x and w need 16-byte aligned rows");
+  GroupParams p{};
+  p.x = x; p.x_stride = x_stride; p.x_group = x_group; p.x_rows = x_rows; p.w = w;
+  p.w_rows = act >= 0 ? 2 * n : n; p.bias = bias; p.y = y; p.y_stride = y_stride;
+  p.y_group = y_group; p.offsets = offsets; p.gather = gather; p.rows = rows; p.groups = groups;
+  p.n = (int)n; p.k = (int)k; p.act = act; p.status = status;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (is_f32) {
+    FK_REQUIRE(y_f32, FK_ERR_INVALID_ARG, "fk_group_gemm: fp32 operands give an fp32 result");
+    const int64_t my = (rows + GA_M - 1) / GA_M;
+    FK_REQUIRE(my <= 65535, FK_ERR_UNSUPPORTED, "fk_group_gemm: too many rows");
+    const dim3 grid((unsigned)((n + GA_N - 1) / GA_N), (unsigned)my, (unsigned)groups);
+    FK_CUDA_OK(act >= 0 ? launch_kernel(group_any_kernel<true>, grid, dim3(256), 0, s, p)
+                        : launch_kernel(group_any_kernel<false>, grid, dim3(256), 0, s, p));
+    count_launch();
+    return FK_OK;
+  }
+  FK_REQUIRE(act < 0 || !y_f32, FK_ERR_UNSUPPORTED,
+             "fk_group_gemm: an activation gives a bf16 result");
+  // 16-byte stores of the large form
+  const bool dense_y = y_stride % (y_f32 ? 4 : 8) == 0 && y_group % (y_f32 ? 4 : 8) == 0;
+  const bool large = expect_rows > 64 && !gather && dense_y && groups <= GG_MAX_GROUPS;
+  if (large) {
+    if (act >= 0) return launch_large<true, uint16_t>(p, x_cols, s);
+    return y_f32 ? launch_large<false, float>(p, x_cols, s)
+                 : launch_large<false, uint16_t>(p, x_cols, s);
+  }
+  if (act >= 0) return launch_skinny<true, uint16_t>(p, expect_rows, s);
+  return y_f32 ? launch_skinny<false, float>(p, expect_rows, s)
+               : launch_skinny<false, uint16_t>(p, expect_rows, s);
+}
+
+}  // extern "C"

@@ -1,10 +1,10 @@
 // Kernels without shape restrictions, for the number format and the head sizes the
 // tensor-core kernels do not take:
 //
-//   fk_gemm_f32         y = x w^T in true fp32 (no tensor cores, so no reduced
+//   fk_gemm_f32         y = x w^T (+ bias) in true fp32 (no tensor cores, so no reduced
 //                       precision), any m, n
 //   fk_paged_attn_any   causal attention over the paged NHD pool, bf16 or fp32, any
-//                       head size up to 512 and any query / KV head ratio; prompt
+//                       head size up to 1152 and any query / KV head ratio; prompt
 //                       portions and single decoded tokens alike
 #include "fk_types.cuh"
 
@@ -16,7 +16,8 @@ constexpr int GF_M = 64, GF_N = 64, GF_K = 16;
 
 __global__ void __launch_bounds__(256) gemm_f32_kernel(
     const float* __restrict__ x, int64_t x_stride, const float* __restrict__ w,
-    float* __restrict__ y, int64_t y_stride, int m, int n, int k) {
+    const float* __restrict__ bias, float* __restrict__ y, int64_t y_stride, int m, int n,
+    int k) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float xs[GF_K][GF_M + 4], ws[GF_K][GF_N + 4];
@@ -54,7 +55,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int c = n0 + tx * 4 + j;
-      if (c < n) y[(int64_t)r * y_stride + c] = acc[i][j];
+      if (c < n) y[(int64_t)r * y_stride + c] = acc[i][j] + (bias ? bias[c] : 0.f);
     }
   }
 }
@@ -165,7 +166,9 @@ static cudaError_t launch_any(const AnyAttnParams& p, int grid, cudaStream_t s) 
     return launch_kernel(paged_attn_any_kernel<T, 2>, dim3(grid), dim3(AA_WARPS * 32), smem, s, p);
   if (p.d <= 128)
     return launch_kernel(paged_attn_any_kernel<T, 4>, dim3(grid), dim3(AA_WARPS * 32), smem, s, p);
-  return launch_kernel(paged_attn_any_kernel<T, 16>, dim3(grid), dim3(AA_WARPS * 32), smem, s, p);
+  if (p.d <= 512)
+    return launch_kernel(paged_attn_any_kernel<T, 16>, dim3(grid), dim3(AA_WARPS * 32), smem, s, p);
+  return launch_kernel(paged_attn_any_kernel<T, 36>, dim3(grid), dim3(AA_WARPS * 32), smem, s, p);
 }
 
 }  // namespace fk
@@ -174,8 +177,8 @@ using namespace fk;
 
 extern "C" {
 
-int fk_gemm_f32(const float* x, int64_t x_stride, const float* w, float* y, int64_t y_stride,
-                int64_t m, int64_t n, int64_t k, fk_stream_t stream) {
+int fk_gemm_f32(const float* x, int64_t x_stride, const float* w, const float* bias, float* y,
+                int64_t y_stride, int64_t m, int64_t n, int64_t k, fk_stream_t stream) {
   FK_REQUIRE(m >= 0 && n >= 0 && k > 0, FK_ERR_INVALID_ARG, "fk_gemm_f32: bad sizes");
   if (m == 0 || n == 0) return FK_OK;
   FK_REQUIRE(x && w && y, FK_ERR_INVALID_ARG, "fk_gemm_f32: null pointer");
@@ -187,7 +190,7 @@ int fk_gemm_f32(const float* x, int64_t x_stride, const float* w, float* y, int6
              FK_ERR_UNSUPPORTED, "fk_gemm_f32: dimension too large");
   const dim3 grid((unsigned)((n + GF_N - 1) / GF_N), (unsigned)((m + GF_M - 1) / GF_M));
   FK_CUDA_OK(launch_kernel(gemm_f32_kernel, grid, dim3(256), 0, static_cast<cudaStream_t>(stream),
-                           x, x_stride, w, y, y_stride, (int)m, (int)n, (int)k));
+                           x, x_stride, w, bias, y, y_stride, (int)m, (int)n, (int)k));
   count_launch();
   return FK_OK;
 }
@@ -206,8 +209,8 @@ int fk_paged_attn_any(const void* q, int64_t q_stride, void* out, int64_t out_st
   FK_REQUIRE(num_q_heads % num_kv_heads == 0 && block_size > 0 && num_blocks > 0 &&
                  num_blocks < (1ll << 31) && block_table_stride > 0,
              FK_ERR_INVALID_ARG, "fk_paged_attn_any: bad sizes");
-  FK_REQUIRE(head_dim % 4 == 0 && head_dim <= 512, FK_ERR_UNSUPPORTED,
-             "fk_paged_attn_any: head_dim %d must be a multiple of 4, at most 512", head_dim);
+  FK_REQUIRE(head_dim % 4 == 0 && head_dim <= 1152, FK_ERR_UNSUPPORTED,
+             "fk_paged_attn_any: head_dim %d must be a multiple of 4, at most 1152", head_dim);
   FK_REQUIRE(aligned16(k_cache) && aligned16(v_cache), FK_ERR_ALIGNMENT,
              "fk_paged_attn_any: caches must be 16-byte aligned");
   FK_REQUIRE(q_stride >= (int64_t)num_q_heads * head_dim &&

@@ -78,6 +78,7 @@ static_assert(PF_SMEM_ALLOC <= 232448, "shared memory budget");
 
 struct PrefillParams {
   uint16_t* out; int64_t out_stride;
+  int out_head, out_packs;          // elements between heads of out, 8-channel packs stored
   float* lse; int64_t total_q;      // lse [Hq, total_q] or null
   const int32_t* cu_q; const int32_t* cu_k;
   const int32_t* block_tables; int64_t bt_stride;
@@ -457,8 +458,8 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmap_q,
           if (m0t + row < it.q_len) {
             const int64_t tok = (int64_t)it.qs + m0t + row;
             uint4* dst = reinterpret_cast<uint4*>(p.out + tok * p.out_stride +
-                                                  (int64_t)it.head * PF_D);
-            for (int c = 0; c < 16; ++c) dst[c] = make_uint4(0u, 0u, 0u, 0u);
+                                                  (int64_t)it.head * p.out_head);
+            for (int c = 0; c < p.out_packs; ++c) dst[c] = make_uint4(0u, 0u, 0u, 0u);
             if (p.lse) p.lse[(int64_t)it.head * p.total_q + tok] = -INFINITY;
           }
           kv_base += 2 * it.nkv;
@@ -587,7 +588,8 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmap_q,
       const PfItem it = pf_load_item(p, idx);
       const bool row_valid = it.m0 + t * PF_BM + row < it.q_len;
       const int64_t tok = (int64_t)it.qs + it.m0 + t * PF_BM + row;
-      uint4* dst = reinterpret_cast<uint4*>(p.out + tok * p.out_stride + (int64_t)it.head * PF_D);
+      uint4* dst = reinterpret_cast<uint4*>(p.out + tok * p.out_stride +
+                                            (int64_t)it.head * p.out_head);
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
         uint32_t o[32];
@@ -602,6 +604,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmap_q,
         if (row_valid) {
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
+            if (c * 4 + i >= p.out_packs) continue;
             dst[c * 4 + i] = make_uint4(
                 pack_bf16(__uint_as_float(o[i * 8 + 0]) * inv,
                           __uint_as_float(o[i * 8 + 1]) * inv),
@@ -761,7 +764,7 @@ using namespace fk;
 
 extern "C" {
 
-static int prefill_impl(bool split, const void* q, int64_t q_stride_token, void* out,
+static int prefill_impl(bool split, int out_head, const void* q, int64_t q_stride_token, void* out,
                     int64_t out_stride_token, float* out_lse, const void* k,
                     const void* v, int64_t kv_stride, int64_t num_blocks,
                     int block_size, int kv_layout, const int32_t* cu_seqlens_q,
@@ -786,8 +789,10 @@ static int prefill_impl(bool split, const void* q, int64_t q_stride_token, void*
              FK_ERR_ALIGNMENT,
              "fk_prefill_attn: pointers must be 16-byte aligned, strides multiples of 8");
   FK_REQUIRE(q_stride_token >= (int64_t)num_q_heads * PF_D &&
-                 out_stride_token >= (int64_t)num_q_heads * PF_D,
-             FK_ERR_INVALID_ARG, "fk_prefill_attn: token stride below heads * 128");
+                 out_stride_token >= (int64_t)num_q_heads * out_head,
+             FK_ERR_INVALID_ARG, "fk_prefill_attn: token stride below heads * head size");
+  FK_REQUIRE(out_head > 0 && out_head <= PF_D && out_head % 8 == 0, FK_ERR_UNSUPPORTED,
+             "fk_prefill_attn: %d channels per head of the result", out_head);
   const bool paged = num_blocks > 0;
   PrefillParams p{};
   CUtensorMap mq, mk, mv;
@@ -848,6 +853,8 @@ static int prefill_impl(bool split, const void* q, int64_t q_stride_token, void*
   if (rc != FK_OK) return rc;
   p.out = static_cast<uint16_t*>(out);
   p.out_stride = out_stride_token;
+  p.out_head = out_head;
+  p.out_packs = out_head / 8;
   p.lse = out_lse;
   p.total_q = total_q;
   p.cu_q = cu_seqlens_q;
@@ -901,7 +908,7 @@ int fk_prefill_attn(const void* q, int64_t q_stride_token, void* out,
                     int64_t total_k, int max_seqlen_q, int num_q_heads,
                     int num_kv_heads, int head_dim, float softmax_scale, int causal,
                     int32_t* status, fk_stream_t stream) {
-  return prefill_impl(false, q, q_stride_token, out, out_stride_token, out_lse, k, v, kv_stride,
+  return prefill_impl(false, PF_D, q, q_stride_token, out, out_stride_token, out_lse, k, v, kv_stride,
                       num_blocks, block_size, kv_layout, cu_seqlens_q, cu_seqlens_k, block_tables,
                       block_table_stride, num_seqs, total_q, total_k, max_seqlen_q, num_q_heads,
                       num_kv_heads, head_dim, softmax_scale, causal, status, stream);
@@ -914,9 +921,9 @@ int fk_prefill_attn_2p(const void* q, int64_t q_stride_token, void* out,
                     const int32_t* cu_seqlens_k, const int32_t* block_tables,
                     int64_t block_table_stride, int num_seqs, int64_t total_q,
                     int64_t total_k, int max_seqlen_q, int num_q_heads,
-                    int num_kv_heads, int head_dim, float softmax_scale, int causal,
+                    int num_kv_heads, int head_dim, int out_head_dim, float softmax_scale, int causal,
                     int32_t* status, fk_stream_t stream) {
-  return prefill_impl(true, q, q_stride_token, out, out_stride_token, out_lse, k, v, kv_stride,
+  return prefill_impl(true, out_head_dim, q, q_stride_token, out, out_stride_token, out_lse, k, v, kv_stride,
                       num_blocks, block_size, kv_layout, cu_seqlens_q, cu_seqlens_k, block_tables,
                       block_table_stride, num_seqs, total_q, total_k, max_seqlen_q, num_q_heads,
                       num_kv_heads, head_dim, softmax_scale, causal, status, stream);

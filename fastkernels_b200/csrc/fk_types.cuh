@@ -58,6 +58,12 @@ __device__ __forceinline__ float sumsq(const float4& v) {
 
 __device__ __forceinline__ float sigmoid_f32(float z) { return 1.0f / (1.0f + expf(-z)); }
 
+// Two values as a high and a low bf16 part each (16 significant bits together).
+__device__ __forceinline__ void split_bf16(float a, float b, uint32_t* hi, uint32_t* lo) {
+  *hi = pack_bf16(a, b);
+  *lo = pack_bf16(a - bf16lo(*hi), b - bf16hi(*hi));
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -317,7 +317,7 @@ class DecodeEngine:
             layout.append((put(np.concatenate(slots)), put(bt), put(kv),
                            put(np.concatenate([[0], np.cumsum(q)])),
                            put(np.concatenate([[0], np.cumsum(kv)])), int(q.max()),
-                           int(kv.max())))
+                           int(kv.max()), int(kv.sum())))
         state_shape = cu_shape = None
         if self.state_slots is not None:
             state_shape = put(np.repeat([s.state_slot for s, _, _ in portions],
@@ -334,16 +334,16 @@ class DecodeEngine:
             return v
 
         spans = []
-        for slots, bt, kv, cq, ck, max_q, max_k in layout:
-            spans.append(SpanBatch(take(slots), take(bt), take(kv), take(cq), take(ck), max_q,
-                                   max_k))
+        for slots, bt, kv, cq, ck, *sizes in layout:
+            spans.append(SpanBatch(take(slots), take(bt), take(kv), take(cq), take(ck), *sizes))
         first = spans[0]
         set_context(True, cu_seqlens_q=first.cu_seqlens_q, cu_seqlens_k=first.cu_seqlens_k,
                     max_seqlen_q=first.max_seqlen_q, max_seqlen_k=first.max_seqlen_k,
                     slot_mapping=first.slot_mapping,
                     block_tables=first.block_tables if use_block_tables else None, spans=spans,
                     state_slots=take(state_shape) if state_shape is not None else None,
-                    cu_portions=take(cu_shape) if cu_shape is not None else None)
+                    cu_portions=take(cu_shape) if cu_shape is not None else None,
+                    longest_portion=max(len(t) for _, _, t in portions))
         try:
             hidden = self.model(torch.from_numpy(ids).to(dev), torch.from_numpy(pos).to(dev))
         finally:

@@ -36,6 +36,7 @@ class SpanBatch:
     cu_seqlens_k: torch.Tensor | None = None
     max_seqlen_q: int = 1
     max_seqlen_k: int = 0
+    total_k: int = 0            # prefill: keys of all segments
 
 
 @dataclass
@@ -56,6 +57,7 @@ class Context:
     spans: list[SpanBatch] | None = None
     state_slots: torch.Tensor | None = None     # [N] int32 state slot per token, -1 padded
     cu_portions: torch.Tensor | None = None     # [portions + 1] int32: token ranges
+    longest_portion: int = 1                    # tokens of the longest one
 
 
 _CONTEXT = Context()
@@ -87,7 +89,8 @@ def reference_attn_backend():
 
 def set_context(is_prefill, cu_seqlens_q=None, cu_seqlens_k=None, max_seqlen_q=0,
                 max_seqlen_k=0, slot_mapping=None, context_lens=None, block_tables=None,
-                max_context_len=0, spans=None, state_slots=None, cu_portions=None) -> None:
+                max_context_len=0, spans=None, state_slots=None, cu_portions=None,
+                longest_portion=1) -> None:
     """Same argument order as the reference's set_context (context.py:411-440,
     the fields this path reads).  Prefill: cu_seqlens / max_seqlen, slot_mapping
     and, when a prefix is already cached, block_tables.  Decode: slot_mapping,
@@ -97,7 +100,7 @@ def set_context(is_prefill, cu_seqlens_q=None, cu_seqlens_k=None, max_seqlen_q=0
     _CONTEXT = Context(bool(is_prefill), cu_seqlens_q, cu_seqlens_k, int(max_seqlen_q),
                        int(max_seqlen_k), slot_mapping, context_lens, block_tables,
                        max_context_len, spans=spans, state_slots=state_slots,
-                       cu_portions=cu_portions)
+                       cu_portions=cu_portions, longest_portion=int(longest_portion))
 
 
 def reset_context() -> None:

@@ -140,7 +140,7 @@ def _work(name, args, kw, out):
         return 2 * _nbytes(args[0], args[1]), 0
     if name == "delta_prepare":
         return _nbytes(*args[:6], out), 0
-    if name == "delta_output":
+    if name == "head_norm_gate":
         return _nbytes(args[0], args[1], out), 0
     if name == "embed_f32":
         return 2 * _nbytes(out), 0
@@ -150,7 +150,7 @@ def _work(name, args, kw, out):
 OPS = ["gemm", "gemm_bf16", "gemm_act_mul", "gemm_silu_mul", "prefill_attn",
        "paged_decode_attn", "paged_decode_attn_plan", "rope_rms_store", "qkv_rope_store",
        "norm_shift", "branch_combine", "fused_add_rmsnorm", "rmsnorm", "delta_prepare",
-       "delta_scan", "delta_output", "act_and_mul", "silu_and_mul", "embed_f32"]
+       "delta_scan", "head_norm_gate", "act_and_mul", "silu_and_mul", "embed_f32"]
 
 
 class OpTimer:

@@ -9,6 +9,7 @@ several times in a row has one per pass.
 from __future__ import annotations
 
 import math
+from dataclasses import dataclass
 
 import torch
 
@@ -20,14 +21,43 @@ def round_up(n: int, m: int) -> int:
     return (n + m - 1) // m * m
 
 
-def rope_table(max_positions: int, rot_dims: int, base: float, device) -> torch.Tensor:
+@dataclass(frozen=True)
+class Yarn:
+    """YaRN scaling of rotary frequencies: pairs that turn fewer than `slow` times over
+    `original` positions are slowed by `factor`, those that turn more than `fast` times stay,
+    the ones between are blended; cos and sin grow by 0.1 ln(factor) + 1."""
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+    def apply(self, f: torch.Tensor, rot_dims: int, base: float) -> torch.Tensor:
+        def pair(turns):
+            return rot_dims * math.log(self.original / (2 * math.pi * turns)) \
+                / (2 * math.log(base))
+        lo = max(math.floor(pair(self.fast)), 0)
+        hi = min(math.ceil(pair(self.slow)), rot_dims - 1)
+        i = torch.arange(f.numel(), dtype=torch.float64, device=f.device)
+        ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+        return f / self.factor * ramp + f * (1.0 - ramp)
+
+    @property
+    def magnitude(self) -> float:
+        return 0.1 * math.log(self.factor) + 1.0
+
+
+def rope_table(max_positions: int, rot_dims: int, base: float, device,
+               scaling: Yarn | None = None) -> torch.Tensor:
     """[max_positions, rot_dims] fp32 = cos | sin of p * base^(-2 i / rot_dims), the
-    angles taken in 64-bit."""
+    angles taken in 64-bit; `scaling` changes the frequencies and the magnitude."""
     if rot_dims == 0:
         return torch.zeros((max_positions, 1), dtype=torch.float32, device=device)
     f = base ** (-torch.arange(0, rot_dims, 2, dtype=torch.float64, device=device) / rot_dims)
+    if scaling is not None:
+        f = scaling.apply(f, rot_dims, base)
     a = torch.arange(max_positions, dtype=torch.float64, device=device)[:, None] * f
-    return torch.cat([a.cos(), a.sin()], dim=1).float().contiguous()
+    size = 1.0 if scaling is None else scaling.magnitude
+    return (torch.cat([a.cos(), a.sin()], dim=1) * size).float().contiguous()
 
 
 class RotaryAttention:
@@ -142,4 +172,162 @@ class GeneralizedDelta:
                            ctx.is_prefill, status=self.status)
         out = torch.empty((positions.shape[0], self.out_columns), dtype=self.dtype,
                           device=positions.device)
-        return ops.delta_output(o, cols["g"], self.norm, self.heads, self.dim, self.eps, out)
+        return ops.head_norm_gate(o, cols["g"], self.norm, self.heads, self.dim, self.eps, out)
+
+
+class LatentAttention:
+    """Softmax attention over one cached row per token: a normed latent of `rank` channels,
+    from which every head makes its unrotated key and its value, and a rotated key of `rot`
+    channels that all heads share.
+
+    Two forms of the same sums.  Absorbed: a head's key projection is applied to its query and
+    its value projection to its output, so attention runs on the cached rows themselves
+    (decoding, short portions, fp32, heads above 128 channels).  Expanded: keys and values of
+    all heads are made from the cached rows by one product (the rotated part passes through
+    an identity block) and attention runs on the tcgen05 prefill kernel."""
+
+    # expanded attention makes keys and values of every visible token: worth it for portions
+    # that are not much shorter than what they see
+    EXPAND_RATIO = 8
+    MAX_TC_RANK = 512           # fk_latent_attn
+    MAX_TC_ROW = 640
+
+    def __init__(self, heads, dim, rot, vdim, rank, scale, rot_base, rot_scaling, span, eps,
+                 dtype):
+        self.heads, self.dim, self.rot, self.vdim, self.rank = heads, dim, rot, vdim, rank
+        self.scale, self.rot_base, self.rot_scaling = scale, rot_base, rot_scaling
+        self.span, self.eps, self.dtype = span, eps, dtype
+        self.q_pitch = round_up(dim + rot, 8)
+        self.row = round_up(rank + rot, 64)              # elements of a cached row
+        self.v_pitch = round_up(vdim, 8)
+        self.out_columns = round_up(heads * self.v_pitch, 64)
+        self.sections = {"q": heads * self.q_pitch, "dkv": rank + rot}
+        self.tensor_cores = dtype == torch.bfloat16 and rank <= self.MAX_TC_RANK and \
+            self.row <= self.MAX_TC_ROW
+        self.expandable = dtype == torch.bfloat16 and dim + rot <= 128 and vdim <= 128
+        self.caches = []
+        self.cos_sin = self.status = None
+
+    def load(self, w, prefix) -> dict:
+        """Packs the weights; returns the rows of the shared projection by section."""
+        h, d, r, k = self.heads, self.dim, self.rot, self.rank
+        q = w.zeros(h, self.q_pitch, w.width)
+        q[:, :d + r] = w.matrix(prefix + "q").view(h, d + r, -1)
+        uk = w.matrix(prefix + "uk").view(h, d, k)
+        uv = w.matrix(prefix + "uv").view(h, self.vdim, k)
+        self.norm = w.vector(prefix + "dkv.norm")
+        # absorbed: query [rank, dim] and value [vdim, rank] per head
+        self.w_key = w.zeros(h, k, round_up(d, 16))
+        self.w_key[:, :, :d] = uk.transpose(1, 2)
+        self.w_value = w.zeros(h, self.v_pitch, round_up(k, 16))
+        self.w_value[:, :self.vdim, :k] = uv
+        if self.expandable:
+            self.w_expand = w.zeros(2, h, 128, self.row)
+            self.w_expand[0, :, :d, :k] = uk
+            self.w_expand[0, :, d:d + r, k:k + r] = torch.eye(r, dtype=w.dtype, device=w.device)
+            self.w_expand[1, :, :self.vdim, :k] = uv
+            self.w_expand = self.w_expand.view(2 * h * 128, self.row)
+        return {"q": q.view(h * self.q_pitch, -1), "dkv": w.matrix(prefix + "dkv")}
+
+    def pack_output(self, w: torch.Tensor) -> torch.Tensor:
+        n = w.shape[0]
+        full = torch.zeros((n, self.heads, self.v_pitch), dtype=w.dtype, device=w.device)
+        full[:, :, :self.vdim] = w.view(n, self.heads, self.vdim)
+        out = torch.zeros((n, self.out_columns), dtype=w.dtype, device=w.device)
+        out[:, :self.heads * self.v_pitch] = full.view(n, -1)
+        return out
+
+    def allocate(self, passes, num_blocks, block_size, device):
+        self.caches = [torch.zeros((num_blocks, block_size, 1, self.row), dtype=self.dtype,
+                                   device=device) for _ in range(passes)]
+        return self.caches
+
+    def forward(self, h, cols, positions, run):
+        """h: input rows (not read here); cols: {section: its columns of the packed rows}."""
+        ctx = get_context()
+        span = ctx.spans[self.span]
+        t, cache = positions.shape[0], self.caches[run]
+        width = self.heads * self.v_pitch
+        alloc = torch.empty if width == self.out_columns else torch.zeros
+        out = alloc((t, self.out_columns), dtype=self.dtype, device=positions.device)
+        expand = self.expandable and ctx.is_prefill and \
+            span.total_k <= self.EXPAND_RATIO * t
+        q = torch.empty((t, self.heads, 128 if expand else self.row), dtype=self.dtype,
+                        device=positions.device)
+        ops.latent_prepare(cols["q"], cols["dkv"], self.q_pitch, self.norm, self.cos_sin,
+                           span.slot_mapping, positions, cache, q,
+                           self.dim if expand else self.rank, expand, self.dim, self.rot,
+                           self.rank, self.eps, status=self.status)
+        if expand:
+            rows = ops.latent_gather(cache, span.block_tables, span.cu_seqlens_k, span.total_k,
+                                     status=self.status)
+            kv = ops.gemm(rows, self.w_expand, status=self.status)
+            kv = kv.view(span.total_k, 2, self.heads, 128)
+            ops.prefill_attn(q, kv[:, 0], kv[:, 1], span.cu_seqlens_q, span.cu_seqlens_k,
+                             span.max_seqlen_q, self.scale,
+                             out=out[:, :width].unflatten(1, (self.heads, self.v_pitch)),
+                             status=self.status, split_weights=True)
+            return out
+        ops.group_gemm(cols["q"], self.w_key, out=q.view(t, -1), x_group=self.q_pitch,
+                       y_group=self.row, status=self.status)
+        if self.tensor_cores:
+            keys = span.max_seqlen_k if ctx.is_prefill else \
+                span.block_tables.shape[1] * cache.shape[1]
+            o = ops.latent_attn(q, cache, span.cu_seqlens_q, span.kv_lens, span.block_tables,
+                                span.max_seqlen_q, keys, self.rank, self.rot, self.scale,
+                                status=self.status)
+        else:
+            o = ops.paged_attn_any(q, cache, cache, span.cu_seqlens_q, span.kv_lens,
+                                   span.block_tables, self.scale, status=self.status)
+        ops.group_gemm(o.view(t, -1), self.w_value, out=out, x_group=o.shape[2],
+                       y_group=self.v_pitch, status=self.status)
+        return out
+
+
+class MatrixMemory:
+    """Matrix memory with exponential gating (see fk_mlstm_step): heads of dim x vdim, a
+    normalizer and a running maximum per head, per-head RMS norm and output gate."""
+
+    def __init__(self, heads, dim, vdim, gate_cap, eps, dtype):
+        self.heads, self.dim, self.vdim, self.gate_cap = heads, dim, vdim, gate_cap
+        self.eps, self.dtype = eps, dtype
+        self.sections = {"q": heads * dim, "k": heads * dim, "v": heads * vdim,
+                         "g": heads * vdim}
+        self.out_columns = round_up(heads * vdim, 64)
+        self.status = None
+        self.states = []
+
+    def load(self, w, prefix) -> dict:
+        # the gates' pre-activations stay fp32, so they are a product of their own
+        self.w_gates = w.padded(torch.cat([w.matrix(prefix + n) for n in "if"]),
+                                2 * self.heads, w.stride)
+        self.b_gates = torch.cat([w.vector(f"{prefix}{n}.b") for n in "if"])
+        self.norm = w.vector(prefix + "norm")
+        return {n: w.matrix(prefix + n) for n in "qkvg"}
+
+    def pack_output(self, w):
+        out = torch.zeros((w.shape[0], self.out_columns), dtype=w.dtype, device=w.device)
+        out[:, :w.shape[1]] = w
+        return out
+
+    def allocate(self, passes, num_slots, device):
+        shapes = ops.mlstm_state_shapes(num_slots, self.heads, self.dim, self.vdim)
+        self.states = [tuple(torch.zeros(s, dtype=torch.float32, device=device) for s in shapes)
+                       for _ in range(passes)]
+
+    def forward(self, h, cols, positions, run):
+        ctx = get_context()
+        z = ops.group_gemm(h, self.w_gates, bias=self.b_gates, out_f32=True, status=self.status)
+        out = torch.empty((positions.shape[0], self.out_columns), dtype=self.dtype,
+                          device=positions.device)
+        scale = self.dim ** -0.5
+        if not ctx.is_prefill:
+            return ops.mlstm_step(cols["q"], cols["k"], cols["v"], z, cols["g"], self.norm,
+                                  *self.states[run], ctx.state_slots, positions, self.heads,
+                                  self.dim, self.vdim, self.gate_cap, scale, self.eps, out,
+                                  status=self.status)
+        o = ops.mlstm_portions(cols["q"], cols["k"], cols["v"], z, *self.states[run],
+                               ctx.cu_portions, ctx.state_slots, positions, self.heads, self.dim,
+                               self.vdim, self.gate_cap, scale, ctx.longest_portion,
+                               status=self.status)
+        return ops.head_norm_gate(o, cols["g"], self.norm, self.heads, self.vdim, self.eps, out)

@@ -7,7 +7,7 @@ Per layer run, in launches:
   norm_shift        previous feed-forward's output normed into the residual, norm,
                     token shift
   gemm              ONE projection for everything both mixers read from the row
-  rope_rms_store / attention          delta_prepare / delta_scan / delta_output
+  rope_rms_store / attention          delta_prepare / delta_scan / head_norm_gate
   gemm x 2          the two output projections
   branch_combine    their norms, half-sum, norm, residual, norm of the feed-forward
   gemm_act_mul, gemm

@@ -13,8 +13,16 @@ from .weights import SafetensorsSource, TensorSource
 #   config_from_json(dict, source, dtype) -> config and MODEL_CLASSES {config type: class}
 _ARCHITECTURES = {
     "Pinuvik": "fastkernels_b200.models.pinuvik",
+    "Rivilix": "fastkernels_b200.models.rivilix",
     "LlamaForCausalLM": "fastkernels_b200.models.llama",
     "Qwen3ForCausalLM": "fastkernels_b200.models.llama",
+}
+
+# parts of the CUDA library (build.COMPONENT_SOURCES) that a module's models call
+_LIBRARY_PARTS = {
+    "fastkernels_b200.models.llama": ["decode_attn"],
+    "fastkernels_b200.models.pinuvik": ["decode_attn", "delta"],
+    "fastkernels_b200.models.rivilix": ["latent", "mlstm", "experts"],
 }
 
 
@@ -22,10 +30,20 @@ def architectures() -> list[str]:
     return sorted(_ARCHITECTURES)
 
 
-def _module(name: str):
+def _module_name(name: str) -> str:
     if name not in _ARCHITECTURES:
         raise ValueError(f"unknown architecture '{name}' (known: {', '.join(architectures())})")
-    return importlib.import_module(_ARCHITECTURES[name])
+    return _ARCHITECTURES[name]
+
+
+def _module(name: str):
+    return importlib.import_module(_module_name(name))
+
+
+def library_parts(folder) -> list[str]:
+    """Parts of the CUDA library that the model in a folder needs beside the core."""
+    cfg = json.loads((Path(folder) / "config.json").read_text())
+    return _LIBRARY_PARTS[_module_name(architecture_of(cfg))]
 
 
 def model_class(config):

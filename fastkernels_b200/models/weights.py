@@ -99,3 +99,31 @@ class RandomSource(TensorSource):
 
     def get(self, name):
         return self._init(name, self._shapes[name], self._gen)
+
+
+class Packer:
+    """Tensors of a source as a model's kernels take them: on the device, matrices in the
+    model's type, vectors in fp32, zero-padded where asked."""
+
+    def __init__(self, source: TensorSource, device, dtype, width: int, stride: int):
+        self.source, self.device, self.dtype = source, device, dtype
+        self.width, self.stride = width, stride      # of the residual rows
+
+    def zeros(self, *shape) -> torch.Tensor:
+        return torch.zeros(shape, dtype=self.dtype, device=self.device)
+
+    def matrix(self, name: str) -> torch.Tensor:
+        return self.source.get(name).to(device=self.device, dtype=self.dtype)
+
+    def padded(self, w, rows: int, cols: int) -> torch.Tensor:
+        if isinstance(w, str):
+            w = self.matrix(w)
+        out = self.zeros(rows, cols)
+        out[:w.shape[0], :w.shape[1]] = w
+        return out
+
+    def vector(self, name: str, pad: int | None = None, dtype=torch.float32) -> torch.Tensor:
+        v = self.source.get(name).to(device=self.device, dtype=dtype).reshape(-1)
+        out = torch.zeros(v.numel() if pad is None else pad, dtype=dtype, device=self.device)
+        out[:v.numel()] = v
+        return out

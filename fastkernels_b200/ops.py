@@ -181,7 +181,8 @@ def paged_decode_attn(q, k_cache, v_cache, context_lens, block_tables, softmax_s
 def prefill_attn(q, k, v, cu_seqlens_q, cu_seqlens_k, max_seqlen_q, softmax_scale,
                  causal=True, block_table=None, kv_layout="NHD", out=None,
                  return_lse=False, status=None, split_weights=False):
-    """Variable-length prefill attention on q [total_q, Hq, 128].
+    """Variable-length prefill attention on q [total_q, Hq, 128].  With split_weights
+    `out` may keep fewer channels per head: [total_q, Hq, a multiple of 8].
 
     Without block_table, k / v are dense [total_k, Hkv, 128] (token-strided views
     allowed) and sequence i owns rows cu_seqlens_k[i]..cu_seqlens_k[i+1].  With
@@ -205,7 +206,8 @@ def prefill_attn(q, k, v, cu_seqlens_q, cu_seqlens_k, max_seqlen_q, softmax_scal
         raise _lib.FkError("cu_seqlens_q and cu_seqlens_k must have the same length")
     if out is None:
         out = torch.empty((total_q, hq, d), dtype=BF16, device=q.device)
-    elif out.stride(2) != 1 or out.stride(1) != d:
+    elif out.stride(2) != 1 or out.stride(1) != out.shape[2] or \
+            (out.shape[2] != d and not split_weights):
         raise _lib.FkError("out heads must be dense")
     lse = torch.empty((hq, total_q), dtype=torch.float32, device=q.device) if return_lse else None
     if block_table is None:
@@ -230,11 +232,12 @@ def prefill_attn(q, k, v, cu_seqlens_q, cu_seqlens_k, max_seqlen_q, softmax_scal
             raise _lib.FkError("caches must be dense within a block")
         total_k, kv_stride, bt_stride = 0, k.stride(0), block_table.stride(0)
     fn = lib.fk_prefill_attn_2p if split_weights else lib.fk_prefill_attn
+    head = (out.shape[2],) if split_weights else ()
     check(fn(
         _ptr(q), q.stride(0) if total_q else hq * d, _ptr(out),
         out.stride(0) if total_q else hq * d, _ptr(lse), _ptr(k), _ptr(v), kv_stride, nb, bs,
         int(kv_layout == "HND"), _ptr(cu_seqlens_q), _ptr(cu_seqlens_k), _ptr(block_table),
-        bt_stride, num_seqs, total_q, total_k, int(max_seqlen_q), hq, hkv, d,
+        bt_stride, num_seqs, total_q, total_k, int(max_seqlen_q), hq, hkv, d, *head,
         float(softmax_scale), int(bool(causal)), _status_ptr(status, q), _stream()),
         "fk_prefill_attn")
     return (out, lse) if return_lse else out
@@ -505,9 +508,10 @@ def gemm_silu_mul(x, w, bias=None, out=None, workspace=None, status=None):
     return out
 
 
-def gemm_act_mul(x, w, act, out=None, workspace=None, status=None):
-    """act(x @ wg.T) * (x @ wu.T), w = [wg; wu] rows: one launch where the shape has
-    one (see gemm_silu_mul_fusable), else the projection followed by act_and_mul."""
+def gemm_act_mul(x, w, act, bias=None, out=None, workspace=None, status=None):
+    """act(x @ wg.T (+ bias)) * (x @ wu.T (+ bias)), w = [wg; wu] rows: one launch where
+    the shape has one (see gemm_silu_mul_fusable), else the projection followed by
+    act_and_mul."""
     m, k = x.shape
     half = w.shape[0] // 2
     if x.dtype == BF16 and gemm_silu_mul_fusable(m, 2 * half, k):
@@ -520,19 +524,23 @@ def gemm_act_mul(x, w, act, out=None, workspace=None, status=None):
         if workspace is None:
             workspace = gemm_workspace(x.device)
         check(lib.fk_gemm_bf16_act_mul(
-            _ptr(x), x.stride(0) if m else k, _ptr(w), None, _ptr(out),
+            _ptr(x), x.stride(0) if m else k, _ptr(w), _ptr(bias), _ptr(out),
             out.stride(0) if m else half, m, 2 * half, k, int(act), _ptr(workspace),
             workspace.numel() * workspace.element_size(), _status_ptr(status, x), _stream()),
             "fk_gemm_bf16_act_mul")
         return out
-    return act_and_mul(gemm(x, w, workspace=workspace, status=status), act, out=out)
+    return act_and_mul(gemm(x, w, bias=bias, workspace=workspace, status=status), act, out=out)
 
 
-def gemm(x, w, out=None, workspace=None, status=None):
-    """x @ w.T in the type of its operands: bf16 (tensor cores, fp32 accumulation) or
-    true fp32."""
+def gemm(x, w, bias=None, out=None, workspace=None, status=None):
+    """x @ w.T (+ bias) in the type of its operands: bf16 (tensor cores, fp32
+    accumulation) or true fp32."""
+    if bias is not None:
+        _need(bias, x.dtype, "bias")
+        if bias.shape != (w.shape[0],) or not bias.is_contiguous():
+            raise _lib.FkError("bias must have one entry per row of w")
     if x.dtype != torch.float32:
-        return gemm_bf16(x, w, out=out, workspace=workspace, status=status)
+        return gemm_bf16(x, w, bias=bias, out=out, workspace=workspace, status=status)
     _need(x, torch.float32, "x")
     _need(w, torch.float32, "w")
     if x.dim() != 2 or x.stride(1) != 1 or not w.is_contiguous():
@@ -541,7 +549,7 @@ def gemm(x, w, out=None, workspace=None, status=None):
     n = w.shape[0]
     if out is None:
         out = torch.empty((m, n), dtype=torch.float32, device=x.device)
-    check(lib.fk_gemm_f32(_ptr(x), x.stride(0) if m else k, _ptr(w), _ptr(out),
+    check(lib.fk_gemm_f32(_ptr(x), x.stride(0) if m else k, _ptr(w), _ptr(bias), _ptr(out),
                           out.stride(0) if m else n, m, n, k, _stream()), "fk_gemm_f32")
     return out
 
@@ -729,7 +737,7 @@ def delta_scan(packed, state, cu_portions, slots, positions, blocked, out=None, 
     return out
 
 
-def delta_output(o, gate, weight, heads, dim, eps, out):
+def head_norm_gate(o, gate, weight, heads, dim, eps, out):
     """out = rms(o per head) * weight * sigmoid(gate); columns of out beyond
     heads * dim are zeroed."""
     _need(o, torch.float32, "o")
@@ -738,10 +746,10 @@ def delta_output(o, gate, weight, heads, dim, eps, out):
     _need(weight, torch.float32, "weight")
     rows = o.shape[0]
     if not o.is_contiguous() or not out.is_contiguous() or gate.stride(1) != 1:
-        raise _lib.FkError("delta_output needs dense operands")
-    check(lib.fk_delta_output(_ptr(o), _ptr(gate), gate.stride(0) if rows else heads * dim,
+        raise _lib.FkError("head_norm_gate needs dense operands")
+    check(lib.fk_head_norm_gate(_ptr(o), _ptr(gate), gate.stride(0) if rows else heads * dim,
                               _ptr(weight), _ptr(out), out.shape[1], f32, rows, heads, dim,
-                              float(eps), _stream()), "fk_delta_output")
+                              float(eps), _stream()), "fk_head_norm_gate")
     return out
 
 
@@ -768,6 +776,333 @@ def paged_attn_any(q, k_cache, v_cache, cu_seqlens_q, kv_lens, block_tables, sof
         block_tables.stride(0), cu_seqlens_q.numel() - 1, rows, hq, hkv, d,
         float(softmax_scale), _status_ptr(status, q), _stream()), "fk_paged_attn_any")
     return out
+
+
+# ----------------------------- parallel sublayers, latent attention, experts, matrix memory
+def embed_pair_f32(table, ids, pairs=None, mul_prev=0, mul_cur=0, last_ids=None, slots=None,
+                   positions=None, cu_portions=None, copy=None, status=None):
+    """fp32 residual rows table[ids] (+ pairs[(previous token * mul_prev + token * mul_cur)
+    mod buckets], the last row for a sequence's first token).  last_ids [slots] int64 keeps
+    each sequence's last token; copy [T, stride]: the rows in the type of the tables too."""
+    f32 = _is_f32(table, "table")
+    _need(ids, torch.int64, "ids")
+    n, stride = ids.shape[0], table.shape[1]
+    if not table.is_contiguous():
+        raise _lib.FkError("table must be contiguous")
+    n_port = n_slots = 0
+    if pairs is not None:
+        _need(pairs, table.dtype, "pairs")
+        _need(last_ids, torch.int64, "last_ids")
+        _need(slots, torch.int32, "slots")
+        _need(positions, torch.int64, "positions")
+        _need(cu_portions, torch.int32, "cu_portions")
+        if not pairs.is_contiguous() or pairs.shape[1] != stride:
+            raise _lib.FkError("pairs must be contiguous rows of the table's width")
+        n_port, n_slots = cu_portions.numel() - 1, last_ids.numel()
+    if copy is not None:
+        _need(copy, table.dtype, "copy")
+        if copy.shape != (n, stride) or copy.stride(1) != 1:
+            raise _lib.FkError("copy must be row-dense [T, stride]")
+    x = torch.empty((n, stride), dtype=torch.float32, device=table.device)
+    check(lib.fk_embed_pair_f32(
+        _ptr(table), _ptr(pairs), f32, table.shape[0],
+        pairs.shape[0] - 1 if pairs is not None else 0, int(mul_prev), int(mul_cur), _ptr(ids),
+        _ptr(last_ids), n_slots, _ptr(slots), _ptr(positions), _ptr(cu_portions), n_port, _ptr(x),
+        _ptr(copy), copy.stride(0) if copy is not None and n else stride, n, stride,
+        _status_ptr(status, table), _stream()), "fk_embed_pair_f32")
+    return x
+
+
+def add_layernorm(x, width, eps, dtype, a=None, b=None, experts=None, norm1=None, norm2=None,
+                  out1=None, out2=None, x_out=None, status=None):
+    """x' = x + a + b + sum_j share[:, j] * rows[place[:, j]] (experts = (rows, place,
+    share)), written to x_out (default: in place where something is added);
+    norm1 / norm2 = (weight, bias) of layer norms of x', results of `dtype`.  Without norm1
+    out1 (if given) gets x' itself.  Returns (x', out1, out2)."""
+    _need(x, torch.float32, "x")
+    if x.dim() != 2 or not x.is_contiguous():
+        raise _lib.FkError("add_layernorm needs a contiguous [T, stride] residual")
+    rows, stride = x.shape
+
+    def like(t, name):
+        if t is not None:
+            _need(t, dtype, name)
+            if t.shape[1] != stride or t.stride(1) != 1:
+                raise _lib.FkError(f"{name} must be row-dense with the residual's width")
+            return t.stride(0) if t.shape[0] else stride
+        return stride
+    if norm1 is not None and out1 is None:
+        out1 = torch.empty((rows, stride), dtype=dtype, device=x.device)
+    if norm2 is not None and out2 is None:
+        out2 = torch.empty((rows, stride), dtype=dtype, device=x.device)
+    f32 = int(dtype == torch.float32)
+    if f32 == 0 and dtype != BF16:
+        raise _lib.FkError("add_layernorm: bf16 or fp32")
+    a_stride, b_stride = like(a, "a"), like(b, "b")
+    e_rows, place, share = experts if experts is not None else (None, None, None)
+    e_stride, top = like(e_rows, "experts"), 0
+    if experts is not None:
+        _need(place, torch.int32, "place")
+        _need(share, torch.float32, "share")
+        top = place.shape[1]
+        if share.shape != place.shape or place.shape[0] != rows or \
+                not place.is_contiguous() or not share.is_contiguous():
+            raise _lib.FkError("place and share must be contiguous [T, top]")
+    for name, nrm in (("norm1", norm1), ("norm2", norm2)):
+        for t in nrm or ():
+            _need(t, torch.float32, name)
+            if t.numel() < stride or not t.is_contiguous():
+                raise _lib.FkError(f"{name} must be padded to the residual's width")
+    if x_out is None and (a is not None or b is not None or experts is not None):
+        x_out = x
+    w1, b1 = norm1 if norm1 is not None else (None, None)
+    w2, b2 = norm2 if norm2 is not None else (None, None)
+    check(lib.fk_add_layernorm(
+        _ptr(x), _ptr(x_out), _ptr(a), a_stride, _ptr(b), b_stride, _ptr(e_rows), e_stride,
+        e_rows.shape[0] if e_rows is not None else 0, _ptr(place), _ptr(share), top, _ptr(w1),
+        _ptr(b1), _ptr(out1), like(out1, "out1"), _ptr(w2), _ptr(b2), _ptr(out2),
+        like(out2, "out2"), f32, rows, stride, int(width), float(eps), _status_ptr(status, x),
+        _stream()), "fk_add_layernorm")
+    return (x if x_out is None else x_out), out1, out2
+
+
+def softcap(x, cap):
+    """cap * tanh(x / cap) in place."""
+    f32 = _is_f32(x, "x")
+    if x.dim() != 2 or x.stride(1) != 1:
+        raise _lib.FkError("softcap needs a 2-D row-dense input")
+    rows, cols = x.shape
+    check(lib.fk_softcap(_ptr(x), x.stride(0) if rows else cols, f32, rows, cols, float(cap),
+                         _stream()), "fk_softcap")
+    return x
+
+
+def group_gemm(x, w, out=None, bias=None, x_group=0, y_group=0, offsets=None, gather=None,
+               rows=None, expect_rows=None, act=None, out_f32=False, status=None):
+    """x w_g^T (+ bias) for w [groups, n (2 n with act), k] (or one [n, k]): column groups
+    g take x[:, g * x_group:][:, :k] to out[:, g * y_group:][:, :n]; with offsets
+    [groups + 1] group g takes the rows between its offsets (of x, or x[gather]).
+    out_f32: fp32 result of bf16 operands.  See fk_group_gemm."""
+    f32 = _is_f32(x, "x")
+    _need(w, x.dtype, "w")
+    if w.dim() == 2:
+        w = w[None]
+    if x.dim() != 2 or x.stride(1) != 1 or not w.is_contiguous():
+        raise _lib.FkError("group_gemm needs row-dense x and contiguous w")
+    groups, wn, k = w.shape
+    n = wn if act is None else wn // 2
+    if rows is None:
+        rows = gather.shape[0] if gather is not None else x.shape[0]
+    if expect_rows is None:
+        expect_rows = rows if offsets is None else -(-rows // groups)
+    y_type = torch.float32 if f32 or out_f32 else BF16
+    if out is None:
+        out = torch.empty((rows, n if offsets is not None or groups == 1
+                           else (groups - 1) * y_group + n), dtype=y_type, device=x.device)
+    _need(out, y_type, "out")
+    for name, t in (("offsets", offsets), ("gather", gather)):
+        if t is not None:
+            _need(t, torch.int32, name)
+    if offsets is not None and offsets.numel() != groups + 1:
+        raise _lib.FkError("group_gemm: one offset per group and one more")
+    if gather is not None and gather.numel() < rows:
+        raise _lib.FkError("group_gemm: gather is shorter than the rows")
+    if bias is not None:
+        _need(bias, torch.float32, "bias")
+        if bias.numel() < n:
+            raise _lib.FkError("group_gemm: bias is shorter than the result's rows")
+    if out.dim() != 2 or out.shape[0] < rows or out.stride(1) != 1:
+        raise _lib.FkError("group_gemm: out must be row-dense with a row per row")
+    check(lib.fk_group_gemm(
+        _ptr(x), x.stride(0) if x.shape[0] else x.shape[1], x_group, x.shape[0], _ptr(w),
+        _ptr(bias), _ptr(out), out.stride(0) if rows else out.shape[1], y_group, f32,
+        int(y_type == torch.float32), _ptr(offsets), _ptr(gather), rows, int(expect_rows),
+        groups, n, k, -1 if act is None else int(act), _status_ptr(status, x), _stream()),
+        "fk_group_gemm")
+    return out
+
+
+class Routing:
+    """Which experts take which rows: chosen / share / place [T, top], source [T * top],
+    offsets [experts + 1] (see fk_moe_route)."""
+
+    def __init__(self, rows, experts, top, device):
+        def ints(*shape):
+            return torch.empty(shape, dtype=torch.int32, device=device)
+        self.chosen, self.place = ints(rows, top), ints(rows, top)
+        self.share = torch.empty((rows, top), dtype=torch.float32, device=device)
+        self.source, self.offsets = ints(rows * top), ints(experts + 1)
+
+
+def moe_route(z, top):
+    """Routing from fp32 router logits [T, experts]."""
+    _need(z, torch.float32, "z")
+    if z.dim() != 2 or z.stride(1) != 1:
+        raise _lib.FkError("moe_route needs 2-D row-dense logits")
+    rows, experts = z.shape
+    r = Routing(rows, experts, top, z.device)
+    n = int(lib.fk_moe_route_counts(rows, experts, top))
+    counts = torch.empty(n, dtype=torch.int32, device=z.device) if n else None
+    check(lib.fk_moe_route(
+        _ptr(z), z.stride(0) if rows else experts, _ptr(r.chosen), _ptr(r.share), _ptr(r.place),
+        _ptr(r.source), _ptr(r.offsets), _ptr(counts), rows, experts, top, _stream()),
+        "fk_moe_route")
+    return r
+
+
+def gather_rows(x, source, status=None):
+    """x[source], rows of x a multiple of 16 bytes."""
+    _need(source, torch.int32, "source")
+    if not x.is_cuda or x.dim() != 2 or x.stride(1) != 1:
+        raise _lib.FkError("gather_rows needs a row-dense CUDA matrix")
+    out = torch.empty((source.numel(), x.shape[1]), dtype=x.dtype, device=x.device)
+    size = x.element_size()
+    check(lib.fk_gather_rows(_ptr(x), (x.stride(0) if x.shape[0] else x.shape[1]) * size,
+                             x.shape[0], _ptr(source), _ptr(out), source.numel(),
+                             x.shape[1] * size, _status_ptr(status, x), _stream()),
+          "fk_gather_rows")
+    return out
+
+
+def latent_prepare(q, latent, q_pitch, weight, cos_sin, slots, positions, cache, q_out, q_rot_at,
+                   copy, dim, rot, rank, eps, status=None) -> None:
+    """Store the cached rows of latent attention and lay out its queries (see
+    fk_latent_prepare).  q / latent are column ranges of the packed projection rows, cache
+    [blocks, page, 1, pitch], q_out [T, heads, pitch]."""
+    f32 = _is_f32(q, "q")
+    for name, t in (("latent", latent), ("cache", cache), ("q_out", q_out)):
+        _need(t, q.dtype, name)
+    _need(weight, torch.float32, "weight")
+    _need(cos_sin, torch.float32, "cos_sin")
+    _need(slots, torch.int32, "slots")
+    _need(positions, torch.int64, "positions")
+    rows, heads = q_out.shape[:2]
+    if q.stride(1) != 1 or latent.stride(1) != 1 or (rows and q.stride(0) != latent.stride(0)):
+        raise _lib.FkError("q and latent must be column ranges of the same rows")
+    if not (cache.is_contiguous() and q_out.is_contiguous() and cos_sin.is_contiguous()) or \
+            q.shape[1] < (heads - 1) * q_pitch + dim + rot or latent.shape[1] < rank + rot or \
+            cos_sin.shape[1] != max(rot, 1) or weight.numel() < rank:
+        raise _lib.FkError("latent_prepare: shape mismatch")
+    check(lib.fk_latent_prepare(
+        _ptr(q), _ptr(latent), q.stride(0) if rows else 0, q_pitch, f32, _ptr(weight),
+        _ptr(cos_sin), cos_sin.shape[0], _ptr(slots), _ptr(positions), _ptr(cache),
+        cache.shape[0] * cache.shape[1], cache.shape[-1], _ptr(q_out), q_out.shape[2], q_rot_at,
+        int(bool(copy)), rows, heads, dim, rot, rank, float(eps), _status_ptr(status, q),
+        _stream()), "fk_latent_prepare")
+
+
+def latent_gather(cache, block_tables, cu_seqlens_k, rows, status=None):
+    """Cached rows [blocks, page, 1, pitch] of all sequences side by side: [rows, pitch]."""
+    _need(block_tables, torch.int32, "block_tables")
+    _need(cu_seqlens_k, torch.int32, "cu_seqlens_k")
+    if not cache.is_cuda or not cache.is_contiguous() or block_tables.stride(1) != 1:
+        raise _lib.FkError("latent_gather needs a contiguous CUDA pool and row-dense tables")
+    pitch = cache.shape[-1]
+    out = torch.empty((rows, pitch), dtype=cache.dtype, device=cache.device)
+    check(lib.fk_latent_gather(
+        _ptr(cache), pitch * cache.element_size(), cache.shape[0], cache.shape[1],
+        _ptr(block_tables), block_tables.stride(0), _ptr(cu_seqlens_k),
+        cu_seqlens_k.numel() - 1, _ptr(out), rows, _status_ptr(status, cache), _stream()),
+        "fk_latent_gather")
+    return out
+
+
+def latent_attn(q, cache, cu_seqlens_q, kv_lens, block_tables, max_seqlen_q, max_keys, rank, rot,
+                softmax_scale, out=None, status=None):
+    """Absorbed latent attention, bf16: q [T, heads, pitch] over cached rows
+    [blocks, page, 1, pitch] whose first `rank` channels are the values; out [T, heads,
+    pitch].  max_keys bounds the keys of any sequence (it picks the number of key ranges)."""
+    _need(q, BF16, "q")
+    _need(cache, BF16, "cache")
+    for name, t in (("cu_seqlens_q", cu_seqlens_q), ("kv_lens", kv_lens),
+                    ("block_tables", block_tables)):
+        _need(t, torch.int32, name)
+    rows, heads, pitch = q.shape
+    n_seq = cu_seqlens_q.numel() - 1
+    if not q.is_contiguous() or not cache.is_contiguous() or block_tables.stride(1) != 1:
+        raise _lib.FkError("latent_attn needs contiguous q and cache, row-dense tables")
+    if out is None:
+        out = torch.empty((rows, heads, (rank + 15) // 16 * 16), dtype=BF16, device=q.device)
+    elif not out.is_contiguous():
+        raise _lib.FkError("latent_attn: out must be contiguous")
+    splits = int(lib.fk_latent_attn_splits(n_seq, int(max_seqlen_q), heads, rank + rot,
+                                           int(max_keys)))
+    n = int(lib.fk_latent_attn_workspace_floats(rows, heads, rank, splits))
+    ws = torch.empty(n, dtype=torch.float32, device=q.device) if n else None
+    check(lib.fk_latent_attn(
+        _ptr(q), pitch, _ptr(cache), cache.shape[0], cache.shape[1], cache.shape[-1], _ptr(out),
+        out.shape[2], _ptr(cu_seqlens_q), _ptr(kv_lens), _ptr(block_tables),
+        block_tables.stride(0), n_seq, rows, int(max_seqlen_q), heads, rank, rot,
+        float(softmax_scale), splits, _ptr(ws), n, _status_ptr(status, q), _stream()),
+        "fk_latent_attn")
+    return out
+
+
+def mlstm_state_shapes(num_slots, heads, dim, vdim):
+    """Shapes of the two fp32 state tensors of a matrix memory."""
+    return ((num_slots, heads, dim, int(lib.fk_mlstm_state_cols(vdim))),
+            (num_slots, heads, int(lib.fk_mlstm_norm_cols(dim))))
+
+
+def _mlstm_args(q, k, v, z, s_state, n_state, heads, dim, vdim):
+    f32 = _is_f32(q, "q")
+    for name, t in (("k", k), ("v", v)):
+        _need(t, q.dtype, name)
+    rows = q.shape[0]
+    for name, t in (("q", q), ("k", k), ("v", v)):
+        if t.stride(1) != 1 or (rows and t.stride(0) != q.stride(0)):
+            raise _lib.FkError(f"{name} must be a column range of the packed rows")
+    for name, t in (("z", z), ("s_state", s_state), ("n_state", n_state)):
+        _need(t, torch.float32, name)
+    if z.shape[1] < 2 * heads or z.stride(1) != 1 or not s_state.is_contiguous() or \
+            not n_state.is_contiguous() or (s_state.shape, n_state.shape) != \
+            mlstm_state_shapes(s_state.shape[0], heads, dim, vdim):
+        raise _lib.FkError("matrix memory: gates or state have the wrong shape")
+    return f32, rows
+
+
+def mlstm_step(q, k, v, z, gate, weight, s_state, n_state, slots, positions, heads, dim, vdim,
+               gate_cap, q_scale, eps, out, status=None):
+    """One token per sequence: out = rms(o per head) * weight * sigmoid(gate)."""
+    f32, rows = _mlstm_args(q, k, v, z, s_state, n_state, heads, dim, vdim)
+    _need(out, q.dtype, "out")
+    _need(gate, q.dtype, "gate")
+    _need(weight, torch.float32, "weight")
+    _need(slots, torch.int32, "slots")
+    _need(positions, torch.int64, "positions")
+    if out.stride(1) != 1 or gate.stride(1) != 1:
+        raise _lib.FkError("mlstm_step needs row-dense operands")
+    check(lib.fk_mlstm_step(
+        _ptr(q), _ptr(k), _ptr(v), q.stride(0) if rows else 0, f32, _ptr(z),
+        z.stride(0) if rows else 2 * heads, _ptr(gate), gate.stride(0) if rows else heads * vdim,
+        _ptr(weight), _ptr(s_state), _ptr(n_state), s_state.shape[0], _ptr(slots),
+        _ptr(positions), _ptr(out), out.stride(0) if rows else out.shape[1], rows, heads, dim,
+        vdim, float(gate_cap), float(q_scale), float(eps), _status_ptr(status, q), _stream()),
+        "fk_mlstm_step")
+    return out
+
+
+def mlstm_portions(q, k, v, z, s_state, n_state, cu_portions, slots, positions, heads, dim, vdim,
+                   gate_cap, q_scale, longest, chunked=True, status=None):
+    """The memory over portions; o [T, heads * vdim] fp32 ahead of norm and gate.  bf16
+    goes 64 tokens at a time unless chunked is False."""
+    f32, rows = _mlstm_args(q, k, v, z, s_state, n_state, heads, dim, vdim)
+    _need(cu_portions, torch.int32, "cu_portions")
+    _need(slots, torch.int32, "slots")
+    _need(positions, torch.int64, "positions")
+    n_port = cu_portions.numel() - 1
+    o = torch.empty((rows, heads * vdim), dtype=torch.float32, device=q.device)
+    ws, n = None, 0
+    if chunked and not f32:
+        n = int(lib.fk_mlstm_workspace_floats(rows, n_port, heads, dim, vdim))
+        ws = torch.empty(n, dtype=torch.float32, device=q.device)
+    check(lib.fk_mlstm_portions(
+        _ptr(q), _ptr(k), _ptr(v), q.stride(0) if rows else 0, f32, _ptr(z),
+        z.stride(0) if rows else 2 * heads, _ptr(s_state), _ptr(n_state), s_state.shape[0],
+        _ptr(cu_portions), n_port, _ptr(slots), _ptr(positions), _ptr(o), rows, heads, dim, vdim,
+        float(gate_cap), float(q_scale), _ptr(ws), n, int(longest), _status_ptr(status, q),
+        _stream()), "fk_mlstm_portions")
+    return o
 
 
 # -------------------------------------------------------------------- decode block

@@ -644,7 +644,7 @@ int fk_gemm_bf16_act_mul(const void* x, int64_t x_stride, const void* w, const v
  * fk_delta_packed_floats: size of `packed` in floats.
  * fk_delta_scan runs the recurrence for every portion from and to
  * state [num_slots][heads][dim (value)][padded_dim (key)] fp32 and writes
- * o [rows, heads * dim] fp32.  fk_delta_output: out = rms(o per head) * weight *
+ * o [rows, heads * dim] fp32.  fk_head_norm_gate: out = rms(o per head) * weight *
  * sigmoid(gate), columns beyond heads * dim zeroed. */
 int fk_delta_padded_dim(int dim);
 int64_t fk_delta_packed_floats(int64_t rows, int num_portions, int heads, int dim, int blocked);
@@ -658,15 +658,15 @@ int fk_delta_scan(const float* packed, int blocked, float* o, float* state, int 
                   const int32_t* cu_portions, int num_portions, const int32_t* slots,
                   const int64_t* positions, int64_t rows, int heads, int dim, int32_t* status,
                   fk_stream_t stream);
-int fk_delta_output(const float* o, const void* gate, int64_t gate_stride, const float* weight,
+int fk_head_norm_gate(const float* o, const void* gate, int64_t gate_stride, const float* weight,
                     void* out, int64_t out_stride, int is_f32, int64_t rows, int heads, int dim,
                     float eps, fk_stream_t stream);
 
-/* y[m, n] = x[m, k] w[n, k]^T in fp32 (no tensor cores); k % 4 == 0. */
-int fk_gemm_f32(const float* x, int64_t x_stride, const float* w, float* y, int64_t y_stride,
-                int64_t m, int64_t n, int64_t k, fk_stream_t stream);
+/* y[m, n] = x[m, k] w[n, k]^T (+ bias) in fp32 (no tensor cores); k % 4 == 0. */
+int fk_gemm_f32(const float* x, int64_t x_stride, const float* w, const float* bias, float* y,
+                int64_t y_stride, int64_t m, int64_t n, int64_t k, fk_stream_t stream);
 
-/* Causal attention over the NHD pool for any head size up to 512 (multiple of 4), any
+/* Causal attention over the NHD pool for any head size up to 1152 (multiple of 4), any
  * query / KV head ratio, bf16 or fp32: sequence i brings query rows cu_seqlens_q[i] ..
  * cu_seqlens_q[i + 1] that end at its kv_lens[i]-th key. */
 int fk_paged_attn_any(const void* q, int64_t q_stride, void* out, int64_t out_stride,
@@ -678,7 +678,8 @@ int fk_paged_attn_any(const void* q, int64_t q_stride, void* out, int64_t out_st
 
 /* fk_paged_decode_attn (planned 0) / _planned (planned 1) and fk_prefill_attn with the
  * fp32 softmax weights taken into P V as two bf16 parts (16 significant bits) instead of
- * being rounded to one. */
+ * being rounded to one.  out_head_dim: channels stored per head of out, whose heads lie
+ * that far apart (a multiple of 8, at most head_dim). */
 int fk_paged_decode_attn_2p(int planned, const void* q, int64_t q_stride_token, void* out,
                             int64_t out_stride_token, const void* k_cache, const void* v_cache,
                             int64_t num_blocks, int block_size, int64_t kv_block_stride,
@@ -693,8 +694,127 @@ int fk_prefill_attn_2p(const void* q, int64_t q_stride_token, void* out,
                        const int32_t* cu_seqlens_q, const int32_t* cu_seqlens_k,
                        const int32_t* block_tables, int64_t block_table_stride, int num_seqs,
                        int64_t total_q, int64_t total_k, int max_seqlen_q, int num_q_heads,
-                       int num_kv_heads, int head_dim, float softmax_scale, int causal,
-                       int32_t* status, fk_stream_t stream);
+                       int num_kv_heads, int head_dim, int out_head_dim, float softmax_scale,
+                       int causal, int32_t* status, fk_stream_t stream);
+
+/* ------------------------------------------------------------------------
+ * Decoders whose mixer and feed-forward read the same residual row side by side, with
+ * latent attention, a matrix memory and mixtures of experts (conventions as above).
+ * ------------------------------------------------------------------------ */
+
+/* fk_embed_f32 plus a row of a second table: (previous token * mul_prev + token * mul_cur)
+ * mod buckets, row `buckets` for a sequence's first token.  last_ids [num_slots] int64 is
+ * each sequence's last token across calls (read and replaced).  pairs null: no second
+ * table.  copy (may be null): the row in the activation type as well. */
+int fk_embed_pair_f32(const void* table, const void* pairs, int is_f32, int64_t vocab,
+                      int64_t buckets, int64_t mul_prev, int64_t mul_cur, const int64_t* ids,
+                      int64_t* last_ids, int num_slots, const int32_t* slots,
+                      const int64_t* positions, const int32_t* cu_portions, int num_portions,
+                      float* x, void* copy, int64_t copy_stride, int64_t rows, int stride,
+                      int32_t* status, fk_stream_t stream);
+
+/* x' = x + a + b + sum_j share[t, j] * experts[place[t, j]] (each optional), stored to x_out
+ * when given (may be x_in); out1 = layernorm(x') * weight1 + bias1 and, when given, out2
+ * alike from the same statistics.  weight1 null: out1 = x'.  expert_rows bounds place. */
+int fk_add_layernorm(const float* x_in, float* x_out, const void* a, int64_t a_stride,
+                     const void* b, int64_t b_stride, const void* experts, int64_t expert_stride,
+                     int64_t expert_rows, const int32_t* place, const float* share, int top,
+                     const float* weight1, const float* bias1, void* out1, int64_t out1_stride,
+                     const float* weight2, const float* bias2, void* out2, int64_t out2_stride,
+                     int is_f32, int64_t rows, int stride, int width, float eps,
+                     int32_t* status, fk_stream_t stream);
+
+/* x = cap * tanh(x / cap) in place. */
+int fk_softcap(void* x, int64_t stride, int is_f32, int64_t rows, int64_t cols, float cap,
+               fk_stream_t stream);
+
+/* Grouped projection y = x w_g^T (+ bias), w [groups][w rows][k].
+ *   column groups (offsets null): group g takes all `rows` rows, x columns from g * x_group
+ *     and y columns from g * y_group on
+ *   row groups: group g takes rows offsets[g] .. offsets[g + 1] (device int32
+ *     [groups + 1]) of y; x rows the same, or gather[row]
+ * act >= 0 (enum fk_activation): w has 2 n rows [gate; up], y = act(gate) * up.  is_f32:
+ * fp32 operands and result; else bf16 operands, fp32 accumulation, result bf16 or (y_f32)
+ * fp32.  bias fp32 [n] (not with an activation).  expect_rows: rows a group has, roughly;
+ * picks the kernel. */
+int fk_group_gemm(const void* x, int64_t x_stride, int64_t x_group, int64_t x_rows,
+                  const void* w, const float* bias, void* y, int64_t y_stride, int64_t y_group,
+                  int is_f32, int y_f32, const int32_t* offsets, const int32_t* gather,
+                  int64_t rows, int64_t expect_rows, int groups, int64_t n, int64_t k, int act,
+                  int32_t* status, fk_stream_t stream);
+
+/* The `top` largest of every row of logits z [rows, experts] (lowest index on ties): chosen
+ * and their softmax weights share [rows, top]; place [rows, top] = position of each pair in
+ * the list sorted by expert, source [rows * top] = row of every list entry, offsets
+ * [experts + 1] = first entry of every expert.  counts: fk_moe_route_counts() int32 of
+ * scratch (0: none needed). */
+int64_t fk_moe_route_counts(int64_t rows, int experts, int top);
+int fk_moe_route(const float* z, int64_t z_stride, int32_t* chosen, float* share, int32_t* place,
+                 int32_t* source, int32_t* offsets, int32_t* counts, int64_t rows, int experts,
+                 int top, fk_stream_t stream);
+
+/* y[r] = x[source[r]], rows of row_bytes bytes. */
+int fk_gather_rows(const void* x, int64_t x_stride_bytes, int64_t x_rows, const int32_t* source,
+                   void* y, int64_t rows, int64_t row_bytes, int32_t* status,
+                   fk_stream_t stream);
+
+/* Latent attention.  A cached row is [rms(latent) * weight (rank) | rotated key (rot) | 0].
+ * fk_latent_prepare: from packed rows, heads of q [dim unrotated | rot] q_pitch apart and
+ * latent [rank | rot], store the cached row at its slot and write the rotated part of every
+ * query head to q_out [rows, heads, q_out_pitch] from column q_rot_at on (zeros behind it),
+ * with copy also the unrotated part from column 0 on.  Rotation interleaved, cos_sin
+ * [max_position, rot] = (cos | sin).
+ * fk_latent_gather: cached rows of all sequences side by side, cu_seqlens_k [num_seqs + 1].
+ * fk_latent_attn (bf16): every (token, head) row of q attends the cached rows of its
+ * sequence up to its own token (queries end at key kv_lens[i]); the value of a key is its
+ * first `rank` channels; out [rows * heads, out_pitch].  splits > 1 cuts the keys of every
+ * row into that many ranges and merges them (fk_latent_attn_splits suggests a number). */
+int fk_latent_prepare(const void* q, const void* latent, int64_t in_stride, int q_pitch,
+                      int is_f32, const float* weight, const float* cos_sin, int64_t max_position,
+                      const int32_t* slots, const int64_t* positions, void* cache,
+                      int64_t num_slots, int cache_pitch, void* q_out, int q_out_pitch,
+                      int q_rot_at, int copy, int64_t rows, int heads, int dim, int rot, int rank,
+                      float eps, int32_t* status, fk_stream_t stream);
+int fk_latent_gather(const void* cache, int64_t row_bytes, int64_t num_blocks, int block_size,
+                     const int32_t* block_tables, int64_t block_table_stride,
+                     const int32_t* cu_seqlens_k, int num_seqs, void* out, int64_t rows,
+                     int32_t* status, fk_stream_t stream);
+int fk_latent_attn_splits(int num_seqs, int64_t max_q, int heads, int row_elements,
+                          int64_t max_keys);
+int64_t fk_latent_attn_workspace_floats(int64_t rows, int heads, int rank, int splits);
+int fk_latent_attn(const void* q, int64_t q_pitch, const void* cache, int64_t num_blocks,
+                   int block_size, int cache_pitch, void* out, int64_t out_pitch,
+                   const int32_t* cu_seqlens_q, const int32_t* kv_lens,
+                   const int32_t* block_tables, int64_t block_table_stride, int num_seqs,
+                   int64_t rows, int64_t max_seqlen_q, int heads, int rank, int rot,
+                   float softmax_scale, int splits, float* workspace, int64_t workspace_floats,
+                   int32_t* status, fk_stream_t stream);
+
+/* Matrix memory, per head (equations: csrc/fk_mlstm.cu).  q, k [rows, heads * dim] and
+ * v [rows, heads * vdim] are columns of packed rows; z fp32 [rows, 2 * heads] holds the
+ * pre-activations of the input and of the forget gates.  State of a sequence: s_state
+ * [num_slots, heads, dim, fk_mlstm_state_cols(vdim)], n_state [num_slots, heads,
+ * fk_mlstm_norm_cols(dim)], fp32, read and replaced; zero at position 0.
+ * fk_mlstm_step: one token per row, out = rms(o per head) * weight * sigmoid(gate).
+ * fk_mlstm_portions: runs of tokens, o fp32 [rows, heads * vdim] before norm and gate.  With
+ * a workspace (fk_mlstm_workspace_floats) bf16 portions go 64 tokens at a time, without one
+ * token by token.  longest: tokens of the longest portion. */
+int fk_mlstm_state_cols(int vdim);
+int fk_mlstm_norm_cols(int dim);
+int fk_mlstm_step(const void* q, const void* k, const void* v, int64_t in_stride, int is_f32,
+                  const float* z, int64_t z_stride, const void* gate, int64_t gate_stride,
+                  const float* weight, float* s_state, float* n_state, int num_slots,
+                  const int32_t* slots, const int64_t* positions, void* out, int64_t out_stride,
+                  int64_t rows, int heads, int dim, int vdim, float gate_cap, float q_scale,
+                  float eps, int32_t* status, fk_stream_t stream);
+int64_t fk_mlstm_workspace_floats(int64_t rows, int num_portions, int heads, int dim, int vdim);
+int fk_mlstm_portions(const void* q, const void* k, const void* v, int64_t in_stride, int is_f32,
+                      const float* z, int64_t z_stride, float* s_state, float* n_state,
+                      int num_slots, const int32_t* cu_portions, int num_portions,
+                      const int32_t* slots, const int64_t* positions, float* o, int64_t rows,
+                      int heads, int dim, int vdim, float gate_cap, float q_scale,
+                      float* workspace, int64_t workspace_floats, int64_t longest,
+                      int32_t* status, fk_stream_t stream);
 
 /* fk_argmax_bf16 on fp32 rows. */
 int fk_argmax_f32(const float* x, int64_t x_stride, int64_t rows, int64_t cols, float* out_val,

@@ -427,7 +427,7 @@ def test_delta_rule_in_portions(heads, dim, rank, dtype):
         o = torch.zeros((len(z), hd), device="cuda")
         ops.delta_scan(packed, state, i32(cu), i32(sl), i64(pos), blocked, out=o, status=st)
         out = torch.full((len(z), (hd + 63) // 64 * 64), 9.0, dtype=dtype, device="cuda")
-        ops.delta_output(o, col["g"], dev(norm), heads, dim, eps, out)
+        ops.head_norm_gate(o, col["g"], dev(norm), heads, dim, eps, out)
         row = 0
         for i, n in portions:
             # rounding of exponentials and norms adds up over a sequence
