@@ -130,10 +130,10 @@ def causal_attention(q, k, v, scale):
     return out
 
 
-def latent_mixer(h, w, p, c, eps):
-    t, heads, dim, rot, vdim = h.shape[0], c["heads"], c["dim"], c["rot_dim"], c["vdim"]
-    q = (h @ w[p + "q"].T).reshape(t, heads, dim + rot)
-    z = h @ w[p + "dkv"].T
+def latent_attend(q, z, w, p, c, eps):
+    """Heads' outputs [T, heads * vdim] from queries [T, heads, dim + rot] and latent rows
+    [T, rank + rot]."""
+    t, heads, dim, rot, vdim = q.shape[0], c["heads"], c["dim"], c["rot_dim"], c["vdim"]
     lat = rms(z[:, :c["kv_rank"]], eps) * w[p + "dkv.norm"]
     freqs, mscale = rotary_frequencies(rot, c["rot"]["base"], c["rot"].get("scaling"))
     pos = np.arange(t, dtype=np.float64)
@@ -143,7 +143,12 @@ def latent_mixer(h, w, p, c, eps):
     v = (lat @ w[p + "uv"].T).reshape(t, heads, vdim)
     qq = np.concatenate([q[..., :dim], qr], -1)
     kk = np.concatenate([k, np.repeat(kr[:, None], heads, 1)], -1)
-    return causal_attention(qq, kk, v, c["scale"]).reshape(t, -1) @ w[p + "o"].T
+    return causal_attention(qq, kk, v, c["scale"]).reshape(t, -1)
+
+
+def latent_mixer(h, w, p, c, eps):
+    q = (h @ w[p + "q"].T).reshape(h.shape[0], c["heads"], -1)
+    return latent_attend(q, h @ w[p + "dkv"].T, w, p, c, eps) @ w[p + "o"].T
 
 
 # -------------------------------------------------------------------- feed-forward
@@ -243,3 +248,160 @@ def read_safetensors(path):
             v = np.frombuffer(data, {"F32": "<f4", "I32": "<i4"}[meta["dtype"]])
         out[name] = v.reshape(meta["shape"]).astype(np.float64)
     return out
+
+
+# ------------------------------------------------------------ small models for tests
+def memory_layer(heads=3, dim=20, vdim=28, cap=7.0, mlp=None):
+    return {"type": "mlstm", "mixer": {"heads": heads, "dim": dim, "vdim": vdim,
+                                       "gate_cap": cap}, "mlp": mlp}
+
+
+def latent_layer(heads=5, dim=24, rot=8, vdim=20, rank=40, scale=0.3, base=900.0, yarn=(4.0, 60, 8.0, 0.5),
+                 mlp=None):
+    r = {"base": base, "dims": rot}
+    if yarn:
+        r["scaling"] = dict(zip(("factor", "original", "fast", "slow"), yarn))
+    return {"type": "latent_attention",
+            "mixer": {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": vdim, "kv_rank": rank,
+                      "scale": scale, "rot": r}, "mlp": mlp}
+
+
+def dense(ff):
+    return {"kind": "dense", "ff": ff}
+
+
+def experts(n, top, ff, shared=None):
+    c = {"kind": "moe", "router": {"experts": n, "top": top}, "expert": {"ff": ff}}
+    if shared:
+        c["shared"] = {"ff": shared}
+    return c
+
+
+def model_config(layers, width=104, vocab=201, eps=1e-4, loop=None, bigram=None, softcap=None):
+    cfg = {"architecture": "Rivilix", "layers": layers, "norm": {"eps": eps}, "vocab": vocab,
+           "width": width}
+    if loop:
+        cfg["loop"] = dict(zip(("start", "stop", "times"), loop))
+    if bigram:
+        cfg["embedding"] = {"bigram": dict(zip(("buckets", "mul_prev", "mul_cur"), bigram))}
+    if softcap:
+        cfg["logit_softcap"] = softcap
+    return cfg
+
+
+MODELS = {
+    "plain": model_config([memory_layer(mlp=dense(70)),
+                           latent_layer(mlp=experts(7, 3, 36, shared=52)),
+                           latent_layer(heads=2, rot=10, dim=15, vdim=33, rank=23, yarn=None,
+                                        mlp=dense(90))],
+                          bigram=(37, 11, 5), softcap=9.0),
+    # the whole stack but its last layer repeats; a layer without feed-forward
+    "loop": model_config([memory_layer(heads=2, dim=9, vdim=7, cap=3.0, mlp=experts(5, 1, 20)),
+                          latent_layer(heads=1, dim=40, rot=40, vdim=8, rank=16, yarn=(1.0, 90, 4.0, 1.0)),
+                          memory_layer(heads=1, dim=33, vdim=65, cap=20.0, mlp=dense(30))],
+                         width=72, vocab=130, eps=1e-3, loop=(0, 2, 3), bigram=(64, 1, 3),
+                         softcap=3.0),
+    # heads beyond 128 channels, key sizes beyond 256, more heads than one tile of rows
+    "wide": model_config([latent_layer(heads=3, dim=120, rot=40, vdim=136, rank=200, scale=0.12,
+                                       mlp=experts(40, 5, 24, shared=100)),
+                          memory_layer(heads=2, dim=264, vdim=72, mlp=None),
+                          latent_layer(heads=19, dim=16, rot=2, vdim=16, rank=300, mlp=dense(64))],
+                         width=200, vocab=300, loop=(1, 3, 2)),
+    # a latent wider than the tensor-core kernels take
+    "rank": model_config([latent_layer(heads=2, dim=32, rot=64, vdim=24, rank=620, scale=0.2,
+                                       mlp=experts(2, 2, 30)),
+                          memory_layer(heads=4, dim=4, vdim=3)], width=64, vocab=90,
+                         bigram=(1, 7, 9)),
+}
+
+
+def random_weights(cfg, seed):
+    """Weights of unit-scale activations: attention that picks few keys, memories that last,
+    norms and biases away from 1 and 0."""
+    rs = np.random.RandomState(seed)
+    w, wd = {}, cfg["width"]
+
+    def mat(name, n, k, gain=1.0):
+        w[name] = bf16(rs.randn(n, k) * gain / np.sqrt(k))
+
+    def vec(name, n, lo, hi):
+        w[name] = bf16(rs.uniform(lo, hi, size=n))
+
+    def norm(name):
+        vec(name, wd, 0.6, 1.4)
+        vec(name + ".b", wd, -0.2, 0.2)
+
+    def ff(p, n, bias):
+        mat(p + "gate", n, wd, 1.5)
+        mat(p + "up", n, wd)
+        mat(p + "down", wd, n, 1.5)
+        if bias:
+            vec(p + "gate.b", n, -0.5, 0.5)
+            vec(p + "up.b", n, -0.5, 0.5)
+            vec(p + "down.b", wd, -0.3, 0.3)
+
+    w["embed"] = bf16(rs.randn(cfg["vocab"], wd))
+    big = cfg.get("embedding", {}).get("bigram")
+    if big:
+        w["bigram"] = bf16(rs.randn(big["buckets"] + 1, wd))
+    if cfg.get("loop"):
+        mat("loop.in", wd, 2 * wd)
+    mat("head", cfg["vocab"], wd, 2.0)
+    norm("final.norm")
+    for i, c in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", c["mixer"]
+        norm(p + "norm1")
+        if c["type"] == "mlstm":
+            hd, hv = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+            for n, k in (("q", hd), ("k", hd), ("v", hv), ("g", hv)):
+                mat(p + "mix." + n, k, wd, 2.0 if n == "q" else 1.0)
+            mat(p + "mix.o", wd, hv, 1.5)
+            vec(p + "mix.norm", hv, 0.5, 1.5)
+            mat(p + "mix.i", m["heads"], wd, 1.5)
+            mat(p + "mix.f", m["heads"], wd, 0.5)
+            vec(p + "mix.i.b", m["heads"], -2.0, 1.0)
+            vec(p + "mix.f.b", m["heads"], 3.0, 6.0)
+        else:
+            heads, dim, rot, vdim, rank = (m[n] for n in ("heads", "dim", "rot_dim", "vdim",
+                                                          "kv_rank"))
+            mat(p + "mix.q", heads * (dim + rot), wd, 2.0)
+            mat(p + "mix.dkv", rank + rot, wd)
+            vec(p + "mix.dkv.norm", rank, 0.5, 1.5)
+            mat(p + "mix.uk", heads * dim, rank)
+            mat(p + "mix.uv", heads * vdim, rank)
+            mat(p + "mix.o", wd, heads * vdim, 1.5)
+        f = c.get("mlp")
+        if not f:
+            continue
+        norm(p + "norm2")
+        if f["kind"] == "dense":
+            ff(p + "mlp.", f["ff"], True)
+            continue
+        n = f["router"]["experts"]
+        mat(p + "mlp.router", n, wd, 2.0)
+        vec(p + "mlp.router.b", n, -0.5, 0.5)
+        for e in range(n):
+            ff(f"{p}mlp.e{e}.", f["expert"]["ff"], False)
+            # experts resemble the first one, so that a choice which hangs on the last bits
+            # of a row does not change the row beyond recognition
+            for leaf in ("gate", "up", "down") if e else ():
+                first, own = w[f"{p}mlp.e0.{leaf}"], w[f"{p}mlp.e{e}.{leaf}"]
+                w[f"{p}mlp.e{e}.{leaf}"] = bf16(first + 0.25 * own)
+        if f.get("shared"):
+            ff(p + "mlp.shared.", f["shared"]["ff"], False)
+    return w
+
+
+def write_folder(folder, cfg, w):
+    """config.json + model.safetensors (bf16) of a small model."""
+    header, blobs, at = {}, [], 0
+    for name, a in w.items():
+        raw = (np.ascontiguousarray(a, dtype=np.float32).view(np.uint32) >> 16).astype("<u2").tobytes()
+        header[name] = {"dtype": "BF16", "shape": list(np.shape(a)),
+                        "data_offsets": [at, at + len(raw)]}
+        blobs.append(raw)
+        at += len(raw)
+    head = json.dumps(header).encode()
+    (folder / "config.json").write_text(json.dumps(cfg))
+    with open(folder / "model.safetensors", "wb") as f:
+        f.write(struct.pack("<Q", len(head)) + head + b"".join(blobs))
