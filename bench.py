@@ -2,7 +2,7 @@
 """Decode-throughput benchmark of the B200 decode hot path.
 
     python bench.py [--gpus N] [--steps K] [--warmup W] [--impl ours|reference]
-                    [--workload c3|c4|c5|pinuvik]
+                    [--workload c3|c4|c5|pinuvik|rivilix]
 
 Workload (synthetic, seeded): config "c3" = one decode step of a random-init
 Qwen3-8B-architecture decoder (36 layers, hidden 4096, FFN 12288, 32 q / 8 kv
@@ -698,12 +698,13 @@ def main():
     ap.add_argument("--steps", type=int, default=32)
     ap.add_argument("--warmup", type=int, default=4)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="c3", choices=sorted(WORKLOADS) + ["pinuvik"],
-                    help="pinuvik: that decoder's prefill and decode throughput beside the "
-                         "Llama-style decoder of equal size (1 GPU)")
-    ap.add_argument("--sizes", default="", help="pinuvik: sizes to run, with commas between")
+    ap.add_argument("--workload", default="c3", choices=sorted(WORKLOADS) + ["pinuvik", "rivilix"],
+                    help="pinuvik, rivilix: that decoder's prefill and decode throughput beside "
+                         "other decoders of equal size (1 GPU)")
+    ap.add_argument("--sizes", default="",
+                    help="pinuvik, rivilix: sizes to run, with commas between")
     ap.add_argument("--kernels", action="store_true",
-                    help="pinuvik: also time every kernel of a layer")
+                    help="pinuvik, rivilix: also time every kernel of a layer")
     ap.add_argument("--layers", type=int, default=0, help="debug only: fewer layers")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-library-points", action="store_true",
@@ -717,7 +718,7 @@ def main():
     args = ap.parse_args()
     if args.warmup < 3:
         args.warmup = 3
-    if args.workload == "pinuvik":
+    if args.workload in ("pinuvik", "rivilix"):
         if args.impl == "reference":
             print(json.dumps({"impl": "reference",
                               "unavailable": "the reference has no such model"}))

@@ -77,6 +77,20 @@ __device__ __forceinline__ bool gl_wait_warp(uint64_t* bar, uint32_t parity,
   return __all_sync(0xffffffffu, gl_wait(bar, parity, abort_flag, status) ? 1 : 0) != 0;
 }
 
+// bias of the 8 columns from `col` on
+__device__ __forceinline__ void gl_bias(const GemmLargeParams& p, int col, float (&b)[8]) {
+  if (!p.bias) return;
+  if (col + 8 <= p.n) {
+    const uint4 v = __ldg(reinterpret_cast<const uint4*>(p.bias + col));
+    b[0] = bf16lo(v.x); b[1] = bf16hi(v.x); b[2] = bf16lo(v.y); b[3] = bf16hi(v.y);
+    b[4] = bf16lo(v.z); b[5] = bf16hi(v.z); b[6] = bf16lo(v.w); b[7] = bf16hi(v.w);
+  } else {
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+      if (col + i < p.n) b[i] = bf16_bits_to_float(p.bias[col + i]);
+  }
+}
+
 __global__ void __launch_bounds__(GL_THREADS, 1)
 gemm_large_kernel(const __grid_constant__ CUtensorMap tmap_x,
                   const __grid_constant__ CUtensorMap tmap_w, const GemmLargeParams p) {
@@ -205,11 +219,7 @@ gemm_large_kernel(const __grid_constant__ CUtensorMap tmap_x,
             for (int g = 0; g < 4; ++g) {
               const int col = n0 + c * 32 + g * 8;
               float b[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-              if (p.bias) {
-#pragma unroll
-                for (int i = 0; i < 8; ++i)
-                  if (col + i < p.n) b[i] = bf16_bits_to_float(p.bias[col + i]);
-              }
+              gl_bias(p, col, b);
               float f[8];
 #pragma unroll
               for (int i = 0; i < 8; ++i) f[i] = __uint_as_float(v[g * 8 + i]) + b[i];
@@ -421,11 +431,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmap_x,
           for (int g = 0; g < 4; ++g) {
             const int col = n0 + c * 32 + g * 8;
             float b[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-            if (p.bias) {
-#pragma unroll
-              for (int i = 0; i < 8; ++i)
-                if (col + i < p.n) b[i] = bf16_bits_to_float(p.bias[col + i]);
-            }
+            gl_bias(p, col, b);
             float f[8];
 #pragma unroll
             for (int i = 0; i < 8; ++i) f[i] = __uint_as_float(v[g * 8 + i]) + b[i];
@@ -566,8 +572,8 @@ int gemm_large_launch(const void* x, int64_t x_stride, const void* w, const void
                       void* y, int64_t y_stride, int64_t m, int64_t n, int64_t k,
                       int32_t* status, cudaStream_t stream) {
   FK_REQUIRE(m < (1ll << 31), FK_ERR_UNSUPPORTED, "fk_gemm_bf16: m too large");
-  FK_REQUIRE(aligned16(y) && y_stride % 8 == 0, FK_ERR_ALIGNMENT,
-             "fk_gemm_bf16: y needs 16-byte aligned rows for m > 256");
+  FK_REQUIRE(aligned16(y) && y_stride % 8 == 0 && aligned16(bias), FK_ERR_ALIGNMENT,
+             "fk_gemm_bf16: y and bias need 16-byte aligned rows for m > 256");
   GemmLargeParams p{};
   p.bias = static_cast<const uint16_t*>(bias);
   p.y = static_cast<uint16_t*>(y);

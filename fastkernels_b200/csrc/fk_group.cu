@@ -135,36 +135,36 @@ __global__ void __launch_bounds__(256) group_any_kernel(const GroupParams p) {
 }
 
 // ------------------------------------------------------------------------- few rows
-// CTA = 16 MT weight rows (of gate and of up with ACT) of one group; its warps share the
-// k range.  Rows go 8 NT at a time.
-template <int MT, int NT, bool ACT, typename OUT>
-__global__ void __launch_bounds__(256) group_skinny_kernel(const GroupParams p) {
-  extern __shared__ float gs_red[];            // [warps][NB MT 16][8 NT]
+// A warp = 16 weight rows (of gate and of up with ACT) of one group, and every ks-th chunk
+// of 32 k's; the CTA's warps are ks parts of k by 16-row tiles.  Rows go 8 NT at a time,
+// blocks of them over grid.z.
+template <int NT, bool ACT, typename OUT>
+__global__ void __launch_bounds__(256) group_skinny_kernel(const GroupParams p, int ks) {
+  extern __shared__ float gs_red[];            // [warps][TILES 16][8 NT + 1]
   pdl_launch_dependents();
-  constexpr int NB = ACT ? 2 : 1;
-  constexpr int TILES = NB * MT;
-  constexpr int COLS = 8 * NT;
+  constexpr int TILES = ACT ? 2 : 1;
+  constexpr int COLS = 8 * NT, PITCH = COLS + 1;
   const int g = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
   const int gr = lane >> 2, tq = lane & 3;
-  const int n0 = blockIdx.x * (16 * MT);
+  const int kpart = warp % ks, fs = warps / ks;
+  const int n0 = blockIdx.x * (16 * fs);
   const uint16_t* w = static_cast<const uint16_t*>(p.w) + (int64_t)g * p.w_rows * p.k;
   const uint16_t* wr[TILES][2];
 #pragma unroll
   for (int e = 0; e < TILES; ++e)
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
-      int r = n0 + (e % MT) * 16 + h * 8 + gr;
+      int r = n0 + (warp / ks) * 16 + h * 8 + gr;
       if (r >= p.n) r = p.n - 1;               // computed, not stored
-      wr[e][h] = w + ((int64_t)(e / MT) * p.n + r) * p.k + tq * 8;
+      wr[e][h] = w + ((int64_t)e * p.n + r) * p.k + tq * 8;
     }
   pdl_wait();
   int64_t first, count;
   group_range(p, g, &first, &count);
-  if (count == 0) return;
   const uint16_t* x = static_cast<const uint16_t*>(p.x) + (p.offsets ? 0 : g * p.x_group);
   const int chunks = (p.k + 31) >> 5;
-  for (int64_t t0 = 0; t0 < count; t0 += COLS) {
+  for (int64_t t0 = (int64_t)blockIdx.z * COLS; t0 < count; t0 += (int64_t)gridDim.z * COLS) {
     const uint16_t* xr[NT];
     bool on[NT];
 #pragma unroll
@@ -180,12 +180,12 @@ __global__ void __launch_bounds__(256) group_skinny_kernel(const GroupParams p) 
       for (int j = 0; j < NT; ++j)
 #pragma unroll
         for (int i = 0; i < 4; ++i) acc[e][j][i] = 0.f;
-    constexpr int UN = TILES * 2 + NT <= 4 ? 4 : TILES * 2 + NT <= 8 ? 2 : 1;
-    for (int c0 = warp; c0 < chunks; c0 += warps * UN) {
+    constexpr int UN = TILES * 2 + NT <= 6 ? 4 : TILES * 2 + NT <= 8 ? 2 : 1;
+    for (int c0 = kpart; c0 < chunks; c0 += ks * UN) {
       uint4 a[UN][TILES][2], b[UN][NT];
 #pragma unroll
       for (int u = 0; u < UN; ++u) {
-        const int c = c0 + u * warps;
+        const int c = c0 + u * ks;
         const bool in = c * 32 + tq * 8 < p.k;
 #pragma unroll
         for (int e = 0; e < TILES; ++e)
@@ -212,24 +212,27 @@ __global__ void __launch_bounds__(256) group_skinny_kernel(const GroupParams p) 
         }
     }
     __syncthreads();
-    float* mine = gs_red + (int64_t)warp * TILES * 16 * COLS;
+    float* mine = gs_red + warp * (TILES * 16 * PITCH);
 #pragma unroll
     for (int e = 0; e < TILES; ++e)
 #pragma unroll
       for (int j = 0; j < NT; ++j)
 #pragma unroll
         for (int i = 0; i < 4; ++i)
-          mine[(e * 16 + gr + (i >> 1) * 8) * COLS + j * 8 + tq * 2 + (i & 1)] = acc[e][j][i];
+          mine[(e * 16 + gr + (i >> 1) * 8) * PITCH + j * 8 + tq * 2 + (i & 1)] = acc[e][j][i];
     __syncthreads();
     OUT* y = static_cast<OUT*>(p.y) + (p.offsets ? 0 : g * p.y_group);
-    for (int i = threadIdx.x; i < MT * 16 * COLS; i += blockDim.x) {
-      const int r = i % (MT * 16), t = i / (MT * 16);
+    const int lg = 4 + (fs > 1) + (fs > 2), feats = 16 * fs;     // fs: 1, 2 or 4
+    const int live = (int)min((int64_t)COLS, count - t0);
+    for (int i = threadIdx.x; i < feats * live; i += blockDim.x) {
+      const int r = i & (feats - 1), t = i >> lg;
       const int c = n0 + r;
-      if (c >= p.n || t0 + t >= count) continue;
+      if (c >= p.n) continue;
+      const float* part = gs_red + (r >> 4) * ks * (TILES * 16 * PITCH) + (r & 15) * PITCH + t;
       float v = p.bias ? p.bias[c] : 0.f, up = 0.f;
-      for (int q = 0; q < warps; ++q) {
-        v += gs_red[((int64_t)q * TILES * 16 + r) * COLS + t];
-        if (ACT) up += gs_red[((int64_t)q * TILES * 16 + MT * 16 + r) * COLS + t];
+      for (int q = 0; q < ks; ++q) {
+        v += part[q * (TILES * 16 * PITCH)];
+        if (ACT) up += part[q * (TILES * 16 * PITCH) + 16 * PITCH];
       }
       if (ACT) v = group_act(v, p.act) * up;
       Elem<OUT>::store(y + (first + t0 + t) * p.y_stride + c, v);
@@ -238,15 +241,21 @@ __global__ void __launch_bounds__(256) group_skinny_kernel(const GroupParams p) 
 }
 
 // ------------------------------------------------------------------------ many rows
-constexpr int GG_BM = 128, GG_BN = 256, GG_BK = 64, GG_STAGES = 4;
-constexpr int GG_A_BYTES = GG_BM * GG_BK * 2, GG_B_BYTES = GG_BN * GG_BK * 2;
-constexpr int GG_STAGE_BYTES = GG_A_BYTES + GG_B_BYTES;
+// BN weight rows a tile: 256, or 32 for narrow products (more stages of the rows' stream).
+constexpr int GG_BM = 128, GG_BK = 64;
+constexpr int GG_A_BYTES = GG_BM * GG_BK * 2;
 constexpr int GG_MAX_GROUPS = 1024;
-constexpr int GG_OFF_TILES = GG_STAGES * GG_STAGE_BYTES;       // first tile of every group
-constexpr int GG_OFF_BAR = GG_OFF_TILES + (GG_MAX_GROUPS + 8) * 4;
-constexpr int GG_SMEM_ALLOC = GG_OFF_BAR + 256 + 1024;
 constexpr int GG_THREADS = 192;
-static_assert(GG_SMEM_ALLOC <= 232448, "shared memory budget");
+template <int BN>
+struct GgCfg {
+  static constexpr int kBBytes = BN * GG_BK * 2;
+  static constexpr int kStageBytes = GG_A_BYTES + kBBytes;
+  static constexpr int kStages = BN == 256 ? 4 : 9;
+  static constexpr int kOffTiles = kStages * kStageBytes;      // first tile of every group
+  static constexpr int kOffBar = kOffTiles + (GG_MAX_GROUPS + 8) * 4;
+  static constexpr int kSmem = kOffBar + 256 + 1024;
+  static_assert(kSmem <= 232448, "shared memory budget");
+};
 
 __device__ __forceinline__ uint64_t gg_ns() {
   uint64_t t;
@@ -299,30 +308,31 @@ __device__ __forceinline__ GgTile gg_tile(const GroupParams& p, const int* first
   return t;
 }
 
-template <bool ACT, typename OUT>
+template <int BN, bool ACT, typename OUT>
 __global__ void __launch_bounds__(GG_THREADS, 1)
 group_large_kernel(const __grid_constant__ CUtensorMap tmap_x,
                    const __grid_constant__ CUtensorMap tmap_w, const GroupParams p) {
+  using Cfg = GgCfg<BN>;
   extern __shared__ uint8_t gg_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(gg_raw) + 1023) &
                                              ~uintptr_t(1023));
-  int* first_tile = reinterpret_cast<int*>(smem + GG_OFF_TILES);
-  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + GG_OFF_BAR);
+  int* first_tile = reinterpret_cast<int*>(smem + Cfg::kOffTiles);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + Cfg::kOffBar);
   uint64_t* full = bars;
-  uint64_t* empty = bars + GG_STAGES;
-  uint64_t* acc_full = bars + 2 * GG_STAGES;       // [2]
+  uint64_t* empty = bars + Cfg::kStages;
+  uint64_t* acc_full = bars + 2 * Cfg::kStages;       // [2]
   uint64_t* acc_empty = acc_full + 2;              // [2]
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(acc_empty + 2);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(acc_empty + 3);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  constexpr int TN = ACT ? GG_BN / 2 : GG_BN;      // outputs per tile
+  constexpr int TN = ACT ? BN / 2 : BN;      // outputs per tile
   const int n_tiles = (p.n + TN - 1) / TN;
   const int kb_total = (p.k + GG_BK - 1) / GG_BK;
 
   pdl_launch_dependents();
   if (threadIdx.x == 0) {
-    for (int i = 0; i < GG_STAGES; ++i) {
+    for (int i = 0; i < Cfg::kStages; ++i) {
       mbar_init(&full[i], 1);
       mbar_init(&empty[i], 1);
     }
@@ -390,23 +400,23 @@ group_large_kernel(const __grid_constant__ CUtensorMap tmap_x,
         const int wrow = (int)(t.g * p.w_rows) + t.nt * TN;
         for (int kb = 0; kb < kb_total; ++kb) {
           if (!gg_wait(&empty[stage], phase ^ 1, abort_flag, p.status)) { ok = false; break; }
-          uint8_t* dst = smem + stage * GG_STAGE_BYTES;
-          mbar_arrive_expect_tx(&full[stage], (uint32_t)GG_STAGE_BYTES);
+          uint8_t* dst = smem + stage * Cfg::kStageBytes;
+          mbar_arrive_expect_tx(&full[stage], (uint32_t)Cfg::kStageBytes);
           tma_load_2d(dst, &tmap_x, &full[stage], xc + kb * GG_BK, (int)t.row0);
           if (ACT) {
             tma_load_2d(dst + GG_A_BYTES, &tmap_w, &full[stage], kb * GG_BK, wrow);
-            tma_load_2d(dst + GG_A_BYTES + GG_B_BYTES / 2, &tmap_w, &full[stage], kb * GG_BK,
+            tma_load_2d(dst + GG_A_BYTES + Cfg::kBBytes / 2, &tmap_w, &full[stage], kb * GG_BK,
                         wrow + p.n);
           } else {
             tma_load_2d(dst + GG_A_BYTES, &tmap_w, &full[stage], kb * GG_BK, wrow);
           }
-          if (++stage == GG_STAGES) { stage = 0; phase ^= 1; }
+          if (++stage == Cfg::kStages) { stage = 0; phase ^= 1; }
         }
       }
     }
   } else if (warp == 1) {
     constexpr uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) |
-                               ((uint32_t)(GG_BN >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
+                               ((uint32_t)(BN >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
     int stage = 0;
     uint32_t phase = 0, done = 0;
     bool ok = true;
@@ -419,14 +429,14 @@ group_large_kernel(const __grid_constant__ CUtensorMap tmap_x,
         ok = gg_wait_warp(&full[stage], phase, abort_flag, p.status);
         if (!ok) break;
         tc_fence_after();
-        const uint32_t a = smem_u32(smem + stage * GG_STAGE_BYTES);
+        const uint32_t a = smem_u32(smem + stage * Cfg::kStageBytes);
         const uint32_t b = a + GG_A_BYTES;
 #pragma unroll
         for (int kk = 0; kk < GG_BK / 16; ++kk)
-          tc_mma_bf16_elect(buf * GG_BN, smem_desc_sw128(a + kk * 32),
+          tc_mma_bf16_elect(buf * BN, smem_desc_sw128(a + kk * 32),
                             smem_desc_sw128(b + kk * 32), idesc, (kb > 0 || kk > 0) ? 1u : 0u);
         tc_commit_elect(&empty[stage]);
-        if (++stage == GG_STAGES) { stage = 0; phase ^= 1; }
+        if (++stage == Cfg::kStages) { stage = 0; phase ^= 1; }
       }
       if (!ok) break;
       tc_commit_elect(&acc_full[buf]);
@@ -448,8 +458,8 @@ group_large_kernel(const __grid_constant__ CUtensorMap tmap_x,
 #pragma unroll 1
       for (int c = 0; c < TN / 32; ++c) {
         uint32_t v[32], u[ACT ? 32 : 1];
-        tc_ld32(lane_addr + buf * GG_BN + c * 32, v);
-        if (ACT) tc_ld32(lane_addr + buf * GG_BN + GG_BN / 2 + c * 32, u);
+        tc_ld32(lane_addr + buf * BN + c * 32, v);
+        if (ACT) tc_ld32(lane_addr + buf * BN + BN / 2 + c * 32, u);
         tc_wait_ld();
         if (!live || n0 + c * 32 >= p.n) continue;
         float f[32];
@@ -547,30 +557,38 @@ static int gg_map(const void* ptr, int64_t rows, int64_t cols, int64_t stride, i
   return FK_OK;
 }
 
-template <int MT, int NT, bool ACT, typename OUT>
-static int launch_skinny_one(const GroupParams& p, cudaStream_t s) {
-  const int chunks = (p.k + 31) / 32;
-  const int warps = chunks >= 16 && NT * MT <= 8 ? 8 : chunks >= 4 ? 4 : 2;
-  const size_t smem = (size_t)warps * (ACT ? 2 : 1) * MT * 16 * 8 * NT * 4;
+template <int NT, bool ACT, typename OUT>
+static int launch_skinny_one(const GroupParams& p, int ks, int fs, cudaStream_t s) {
+  constexpr int kPerWarp = (ACT ? 2 : 1) * 16 * (8 * NT + 1) * 4;
   static PerDeviceOnce once;
-  FK_CUDA_OK(set_max_dynamic_smem(once, group_skinny_kernel<MT, NT, ACT, OUT>,
-                                  8 * (ACT ? 2 : 1) * MT * 16 * 8 * NT * 4));
-  const dim3 grid((unsigned)((p.n + 16 * MT - 1) / (16 * MT)), (unsigned)p.groups);
-  FK_CUDA_OK(launch_kernel(group_skinny_kernel<MT, NT, ACT, OUT>, grid, dim3(32u * warps), smem,
-                           s, p));
+  FK_CUDA_OK(set_max_dynamic_smem(once, group_skinny_kernel<NT, ACT, OUT>, 8 * kPerWarp));
+  const int64_t blocks = p.offsets ? 1 : (p.rows + 8 * NT - 1) / (8 * NT);
+  const dim3 grid((unsigned)((p.n + 16 * fs - 1) / (16 * fs)), (unsigned)p.groups,
+                  (unsigned)(blocks < 65535 ? blocks : 65535));
+  FK_CUDA_OK(launch_kernel(group_skinny_kernel<NT, ACT, OUT>, grid, dim3(32u * ks * fs),
+                           (size_t)ks * fs * kPerWarp, s, p, ks));
   count_launch();
   return FK_OK;
 }
 template <bool ACT, typename OUT>
 static int launch_skinny(const GroupParams& p, int64_t expect, cudaStream_t s) {
-  if (expect <= 8) return launch_skinny_one<1, 1, ACT, OUT>(p, s);
-  if (expect <= 16) return launch_skinny_one<1, 2, ACT, OUT>(p, s);
-  if (expect <= 32) return launch_skinny_one<1, 4, ACT, OUT>(p, s);
-  return launch_skinny_one<1, 8, ACT, OUT>(p, s);
+  const int chunks = (p.k + 31) / 32;
+  const int ks = chunks >= 16 ? 8 : chunks >= 8 ? 4 : chunks >= 4 ? 2 : 1;
+  const int fs = ks == 8 ? 1 : ks == 1 ? 4 : 8 / ks;
+  // rows per CTA: as many as keep the machine busy (more rows read the weights once)
+  int64_t nt = expect <= 8 ? 1 : expect <= 16 ? 2 : expect <= 32 ? 4 : 8;
+  if (!p.offsets) {
+    const int64_t tiles = (int64_t)((p.n + 16 * fs - 1) / (16 * fs)) * p.groups;
+    while (nt > 1 && tiles * ((p.rows + 8 * nt - 1) / (8 * nt)) < sm_count()) nt /= 2;
+  }
+  if (nt == 1) return launch_skinny_one<1, ACT, OUT>(p, ks, fs, s);
+  if (nt == 2) return launch_skinny_one<2, ACT, OUT>(p, ks, fs, s);
+  if (nt == 4) return launch_skinny_one<4, ACT, OUT>(p, ks, fs, s);
+  return launch_skinny_one<8, ACT, OUT>(p, ks, fs, s);
 }
-template <bool ACT, typename OUT>
-static int launch_large(const GroupParams& p, int64_t x_cols, cudaStream_t s) {
-  constexpr int TN = ACT ? GG_BN / 2 : GG_BN;
+template <int BN, bool ACT, typename OUT>
+static int launch_large_one(const GroupParams& p, int64_t x_cols, cudaStream_t s) {
+  constexpr int TN = ACT ? BN / 2 : BN;
   const int64_t n_tiles = (p.n + TN - 1) / TN;
   const int64_t bound = p.offsets ? ((p.rows + GG_BM - 1) / GG_BM + p.groups) * n_tiles
                                   : (p.rows + GG_BM - 1) / GG_BM * n_tiles * p.groups;
@@ -582,12 +600,20 @@ static int launch_large(const GroupParams& p, int64_t x_cols, cudaStream_t s) {
   rc = gg_map(p.w, p.groups * p.w_rows, p.k, p.k, TN, &mw);
   if (rc != FK_OK) return rc;
   static PerDeviceOnce once;
-  FK_CUDA_OK(set_max_dynamic_smem(once, group_large_kernel<ACT, OUT>, GG_SMEM_ALLOC));
+  FK_CUDA_OK(set_max_dynamic_smem(once, group_large_kernel<BN, ACT, OUT>, GgCfg<BN>::kSmem));
   const int ctas = (int)(bound < sm_count() ? bound : sm_count());
-  FK_CUDA_OK(launch_kernel(group_large_kernel<ACT, OUT>, dim3((unsigned)ctas), dim3(GG_THREADS),
-                           (size_t)GG_SMEM_ALLOC, s, mx, mw, p));
+  FK_CUDA_OK(launch_kernel(group_large_kernel<BN, ACT, OUT>, dim3((unsigned)ctas), dim3(GG_THREADS),
+                           (size_t)GgCfg<BN>::kSmem, s, mx, mw, p));
   count_launch();
   return FK_OK;
+}
+
+template <bool ACT, typename OUT>
+static int launch_large(const GroupParams& p, int64_t x_cols, cudaStream_t s) {
+  if constexpr (!ACT) {
+    if (p.n <= 32) return launch_large_one<32, ACT, OUT>(p, x_cols, s);
+  }
+  return launch_large_one<256, ACT, OUT>(p, x_cols, s);
 }
 
 }  // namespace fk

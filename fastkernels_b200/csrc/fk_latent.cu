@@ -4,12 +4,12 @@
 // and its values the first `rank` channels of them.
 //
 //   latent_prepare_kernel   norm of the latent, rotation of the shared key, store; rotation
-//                           (and copy) of the queries
+//                           (and copy) of the queries; _vec: the same 16 bytes at a time
 //   latent_gather_kernel    cached rows of a batch's sequences side by side
 //   latent_attn_kernel      absorbed attention, bf16: portions and single tokens alike.  A
 //                           CTA owns HT (token, head) rows of one sequence and a range of
-//                           keys; key tiles of 64 rows are double-buffered and serve as K
-//                           and as V
+//                           keys; tiles of cached rows come through a ring and serve as K
+//                           and as V.  Waits are bounded
 //   latent_merge_kernel     key ranges of a row -> one result
 //
 // Scores, softmax weights and sums are fp32; the weights enter the tensor product with the
@@ -17,6 +17,8 @@
 #include "fk_types.cuh"
 
 #include <cmath>
+#include <mutex>
+#include <vector>
 
 namespace fk {
 
@@ -90,6 +92,94 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const LatentPrepPar
   }
 }
 
+// All sizes multiples of 8, bf16: 16 bytes a thread.  blockIdx.x 0: the queries of a token;
+// 1: the cached rows of 8 tokens, a warp each.
+__global__ void __launch_bounds__(256) latent_prepare_vec_kernel(const LatentPrepParams p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int half = p.rot >> 1;
+  auto rotated = [&](const uint16_t* src, int64_t pos, int pack) {
+    const uint4 x = *reinterpret_cast<const uint4*>(src + pack * 8);
+    const float* cs = p.cos_sin + pos * p.rot + pack * 4;
+    const float4 c = __ldg(reinterpret_cast<const float4*>(cs));
+    const float4 s = __ldg(reinterpret_cast<const float4*>(cs + half));
+    auto turn = [](uint32_t uv, float co, float si) {
+      const float u = bf16lo(uv), v = bf16hi(uv);
+      return pack_bf16(u * co - v * si, v * co + u * si);
+    };
+    return make_uint4(turn(x.x, c.x, s.x), turn(x.y, c.y, s.y), turn(x.z, c.z, s.z),
+                      turn(x.w, c.w, s.w));
+  };
+  auto position = [&](int64_t t) {
+    int64_t pos = p.positions[t];
+    if (pos < 0 || pos >= p.max_position) {
+      if (p.status) atomicOr(p.status, FK_DEV_BAD_POSITION);
+      pos = 0;
+    }
+    return pos;
+  };
+  if (blockIdx.x == 0) {
+    const int from = p.copy ? 0 : p.q_rot_at >> 3;       // first pack written of a head
+    const int packs = (p.q_out_pitch >> 3) - from;
+    const int r0 = (p.q_rot_at >> 3) - from, r1 = r0 + (p.rot >> 3);
+    for (int64_t t = blockIdx.y; t < p.rows; t += gridDim.y) {
+      const int64_t pos = position(t);
+      const uint16_t* q = static_cast<const uint16_t*>(p.q) + t * p.in_stride;
+      uint16_t* out = static_cast<uint16_t*>(p.q_out) + t * p.heads * p.q_out_pitch;
+      for (int i = threadIdx.x; i < p.heads * packs; i += blockDim.x) {
+        const int h = i / packs, c = i - h * packs;
+        uint4 v = make_uint4(0u, 0u, 0u, 0u);
+        if (c >= r0 && c < r1)
+          v = rotated(q + h * p.q_pitch + p.dim, pos, c - r0);
+        else if (p.copy && c * 8 < p.dim)
+          v = *reinterpret_cast<const uint4*>(q + h * p.q_pitch + c * 8);
+        *reinterpret_cast<uint4*>(out + h * p.q_out_pitch + (from + c) * 8) = v;
+      }
+    }
+    return;
+  }
+  const int lane = threadIdx.x & 31;
+  for (int64_t t = (int64_t)blockIdx.y * 8 + (threadIdx.x >> 5); t < p.rows;
+       t += (int64_t)gridDim.y * 8) {
+    const int64_t slot = p.slots[t];
+    if (slot < 0 || slot >= p.num_slots) {
+      if (slot >= p.num_slots && lane == 0 && p.status) atomicOr(p.status, FK_DEV_BAD_SLOT);
+      continue;
+    }
+    const int64_t pos = position(t);
+    const uint16_t* src = static_cast<const uint16_t*>(p.lat) + t * p.in_stride;
+    uint16_t* out = static_cast<uint16_t*>(p.cache) + slot * p.cache_pitch;
+    constexpr int VPT = 4;                               // rank up to 1024
+    uint4 x[VPT];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = (lane + i * 32) * 8;
+      x[i] = make_uint4(0u, 0u, 0u, 0u);
+      if (c < p.rank) x[i] = *reinterpret_cast<const uint4*>(src + c);
+      const uint32_t e[4] = {x[i].x, x[i].y, x[i].z, x[i].w};
+#pragma unroll
+      for (int j = 0; j < 4; ++j) ss += bf16lo(e[j]) * bf16lo(e[j]) + bf16hi(e[j]) * bf16hi(e[j]);
+    }
+    const float rs = 1.0f / sqrtf(warp_sum(ss) / (float)p.rank + p.eps);
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = (lane + i * 32) * 8;
+      if (c >= p.rank) continue;
+      const float4 a = __ldg(reinterpret_cast<const float4*>(p.weight + c));
+      const float4 b = __ldg(reinterpret_cast<const float4*>(p.weight + c + 4));
+      *reinterpret_cast<uint4*>(out + c) =
+          make_uint4(pack_bf16(bf16lo(x[i].x) * rs * a.x, bf16hi(x[i].x) * rs * a.y),
+                     pack_bf16(bf16lo(x[i].y) * rs * a.z, bf16hi(x[i].y) * rs * a.w),
+                     pack_bf16(bf16lo(x[i].z) * rs * b.x, bf16hi(x[i].z) * rs * b.y),
+                     pack_bf16(bf16lo(x[i].w) * rs * b.z, bf16hi(x[i].w) * rs * b.w));
+    }
+    for (int c = lane; c * 8 < p.cache_pitch - p.rank; c += 32)
+      *reinterpret_cast<uint4*>(out + p.rank + c * 8) =
+          c * 8 < p.rot ? rotated(src + p.rank, pos, c) : make_uint4(0u, 0u, 0u, 0u);
+  }
+}
+
 __global__ void __launch_bounds__(256) latent_gather_kernel(
     const uint4* __restrict__ cache, int block_size, int num_blocks,
     const int32_t* __restrict__ block_tables, int64_t bt_stride, const int32_t* __restrict__ cu_k,
@@ -122,33 +212,70 @@ struct LatentAttnParams {
   const int32_t* cu_q; const int32_t* kv_lens;
   const int32_t* block_tables; int64_t bt_stride;
   int64_t flat_rows;                            // rows * heads
-  int heads, lk, lo, block_size, num_blocks, splits;
+  int heads, lk, lo, block_size, num_blocks, splits, ring, run;
   float scale_log2;
   int32_t* status;
 };
 
-constexpr int LA_THREADS = 256, LA_KEYS = 64;
-constexpr int LA_SPITCH = LA_KEYS + 4, LA_PPITCH = LA_KEYS + 8;
+// Warps 0-7 make scores and softmax weights of a tile of 32 keys, warps 8-15 multiply the
+// weights of the tile before it with its values, warp 16 keeps the ring of tiles filled: a
+// tile is blocks of 64 channels, [32 rows][128 bytes] each, 128-byte swizzled by TMA.
+constexpr int LA_GROUP = 256, LA_THREADS = 2 * LA_GROUP + 32, LA_KEYS = 32;
+constexpr int LA_BLOCK = LA_KEYS * 128;
+constexpr int LA_PPITCH = LA_KEYS + 8, LA_MAX_RING = 8;
+constexpr uint32_t LA_WAIT_LIMIT = 1u << 22;
 
-__host__ __device__ constexpr int la_smem(int ht, int lk) {
-  return (ht + 2 * LA_KEYS) * (lk + 8) * 2 + 32 * LA_SPITCH * 4 + 2 * ht * LA_PPITCH * 2 +
-         ht * 4;
+// lk: channels of a row, rounded up to 16; a tile holds whole blocks of 64.
+__host__ __device__ constexpr int la_tile(int lk) { return (lk + 63) / 64 * LA_BLOCK; }
+__host__ __device__ constexpr int la_smem(int ht, int lk, int ring) {
+  return ring * la_tile(lk) + ht * (lk + 8) * 2 + 4 * ht * LA_PPITCH * 2 + 21 * ht * 4 +
+         (2 * LA_MAX_RING + 6) * 8 + 1024;
 }
-
-__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src)
-               : "memory");
+// Deepest ring that fits, 0: none.
+__host__ __device__ constexpr int la_ring(int ht, int lk) {
+  int r = LA_MAX_RING;
+  while (r >= 3 && la_smem(ht, lk, r) > 232448) --r;
+  return r >= 3 ? r : 0;
 }
 
 template <int HT, int RN>
-__global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_kernel(const LatentAttnParams p) {
-  extern __shared__ __align__(16) uint8_t la_raw[];
+__global__ void __launch_bounds__(LA_THREADS, 1)
+latent_attn_kernel(const __grid_constant__ CUtensorMap tmap, const LatentAttnParams p) {
+  extern __shared__ uint8_t la_raw[];
   pdl_launch_dependents();
-  pdl_wait();
   constexpr int MTS = HT / 16;
   const int seq = blockIdx.y, split = blockIdx.z;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int gr = lane >> 2, tq = lane & 3;
+  uint8_t* K = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(la_raw) + 1023) &
+                                          ~uintptr_t(1023));          // ring of tiles
+  const int tile_bytes = la_tile(p.lk), kp = p.lk + 8;
+  uint16_t* Q = reinterpret_cast<uint16_t*>(K + p.ring * tile_bytes); // [HT][kp]
+  uint16_t* P = Q + HT * kp;                              // [2][hi, lo][HT][LA_PPITCH]
+  float* alpha = reinterpret_cast<float*>(P + 4 * HT * LA_PPITCH);    // [2][HT]
+  float* inv_l = alpha + 2 * HT;                          // [HT]
+  float* m_run = inv_l + HT;                              // [2][HT]: running maximum
+  float* m_warp = m_run + 2 * HT;                         // [8][HT]: of a tile, per warp
+  float* l_warp = m_warp + 8 * HT;                        // [8][HT]
+  uint64_t* full = reinterpret_cast<uint64_t*>(l_warp + 8 * HT);   // [ring]: rows have come
+  uint64_t* empty = full + LA_MAX_RING;                   // [ring]: ... and are no longer read
+  uint64_t* p_full = empty + LA_MAX_RING;                 // [2]: weights of a tile written
+  uint64_t* p_empty = p_full + 2;                         // [2]: ... and read
+  uint64_t* m_full = p_empty + 2;                         // [2]: running maximum after a tile
+  if (tid == 0) {
+    for (int i = 0; i < p.ring; ++i) {
+      mbar_init(&full[i], 1);
+      mbar_init(&empty[i], LA_GROUP / 32);
+    }
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&p_full[i], 4);
+      mbar_init(&p_empty[i], LA_GROUP / 32);
+      mbar_init(&m_full[i], 4);
+    }
+    mbar_fence_init();
+    tma_prefetch_desc(&tmap);
+  }
+  pdl_wait();
   const int q0 = p.cu_q[seq], q_len = p.cu_q[seq + 1] - q0;
   const int64_t first = (int64_t)q0 * p.heads + (int64_t)blockIdx.x * HT;   // flat row
   const int64_t left = (int64_t)q_len * p.heads - (int64_t)blockIdx.x * HT;
@@ -160,50 +287,237 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_kernel(const Latent
   const int most = max(0, min(kv_len, before + (tok0 + n_rows - 1) / p.heads));
   const int per = ((most + p.splits - 1) / p.splits + LA_KEYS - 1) / LA_KEYS * LA_KEYS;
   const int k_begin = min(most, split * per), k_end = min(most, k_begin + per);
+  {
+    const int packs = p.lk >> 3;
+    for (int i = tid; i < HT * packs; i += LA_THREADS) {
+      const int r = i / packs, c = (i - r * packs) * 8;
+      uint4 v = make_uint4(0u, 0u, 0u, 0u);
+      if (r < n_rows) v = *reinterpret_cast<const uint4*>(p.q + (first + r) * p.q_pitch + c);
+      *reinterpret_cast<uint4*>(Q + r * kp + c) = v;
+    }
+  }
+  __syncthreads();
+  const int tiles = (k_end - k_begin + LA_KEYS - 1) / LA_KEYS;
+  bool ok = true;
 
-  const int kp = p.lk + 8;
-  uint16_t* Q = reinterpret_cast<uint16_t*>(la_raw);
-  uint16_t* K = Q + HT * kp;                              // two tiles
-  float* S = reinterpret_cast<float*>(K + 2 * LA_KEYS * kp);       // [32][LA_SPITCH]
-  uint16_t* Ph = reinterpret_cast<uint16_t*>(S + 32 * LA_SPITCH);
-  uint16_t* Pl = Ph + HT * LA_PPITCH;
-  float* alpha = reinterpret_cast<float*>(Pl + HT * LA_PPITCH);
-
-  const int packs = p.lk >> 3;
-  const int32_t* bt = p.block_tables + seq * p.bt_stride;
-  auto load_tile = [&](int k0, uint16_t* dst) {
-    for (int r = warp; r < LA_KEYS; r += LA_THREADS / 32) {
-      const int key = k0 + r;
-      const uint16_t* src = nullptr;
-      if (key < k_end) {
-        const int page = bt[key / p.block_size];
-        if (page >= 0 && page < p.num_blocks)
-          src = p.cache + ((int64_t)page * p.block_size + key % p.block_size) * p.cache_pitch;
-        else if (lane == 0 && p.status)
-          atomicOr(p.status, FK_DEV_BAD_PAGE);
+  if (warp == 2 * LA_GROUP / 32) {
+    // ------------------------------- cached rows ----------------------------
+    if (lane != 0) return;
+    const int32_t* bt = p.block_tables + seq * p.bt_stride;
+    const int blocks = (p.lk + 63) / 64;
+    int n = 0;
+    for (; n < tiles; ++n) {
+      const int st = n % p.ring;
+      if (n >= p.ring)
+        ok = mbar_wait(&empty[st], (uint32_t)(n / p.ring - 1) & 1u, LA_WAIT_LIMIT);
+      if (!ok) {
+        if (p.status) atomicOr(p.status, FK_DEV_WAIT_TIMEOUT);
+        break;
       }
-      for (int c = lane; c < packs; c += 32) {
-        if (src) cp_async16(dst + r * kp + c * 8, src + c * 8);
-        else *reinterpret_cast<uint4*>(dst + r * kp + c * 8) = make_uint4(0u, 0u, 0u, 0u);
+      mbar_arrive_expect_tx(&full[st], (uint32_t)tile_bytes);
+      uint8_t* dst = K + st * tile_bytes;
+      // runs of p.run keys lie in one page
+      for (int r = 0; r < LA_KEYS; r += p.run) {
+        const int key = k_begin + n * LA_KEYS + r;
+        int row = p.num_blocks * p.block_size;            // out of range: zeros
+        if (key < k_end) {
+          const int page = bt[key / p.block_size];
+          if (page >= 0 && page < p.num_blocks) row = page * p.block_size + key % p.block_size;
+          else if (p.status) atomicOr(p.status, FK_DEV_BAD_PAGE);
+        }
+        for (int c = 0; c < blocks; ++c)
+          tma_load_2d(dst + c * LA_BLOCK + r * 128, &tmap, &full[st], c * 64, row);
       }
     }
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  };
-
-  for (int i = tid; i < HT * packs; i += LA_THREADS) {
-    const int r = i / packs, c = (i - r * packs) * 8;
-    uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (r < n_rows) v = *reinterpret_cast<const uint4*>(p.q + (first + r) * p.q_pitch + c);
-    *reinterpret_cast<uint4*>(Q + r * kp + c) = v;
+    // no copy may be in flight when the CTA ends
+    if (!ok)
+      for (int i = max(0, n - p.ring); i < n; ++i)
+        (void)mbar_wait(&full[i % p.ring], (uint32_t)(i / p.ring) & 1u, LA_WAIT_LIMIT);
+    return;
   }
-  if (k_begin < k_end) load_tile(k_begin, K);
 
-  // softmax: TPR threads per row, KPT keys each
-  constexpr int TPR = LA_THREADS / HT, KPT = LA_KEYS / TPR;
-  const int srow = tid / TPR, skey = (tid % TPR) * KPT;
-  const int my_lim = srow < n_rows ? min(kv_len, before + (tok0 + srow) / p.heads) : 0;
-  float m = -INFINITY, l = 0.f;
+  // 16-byte chunk of a row's 128 bytes of a block, as the swizzle places it
+  const int sw = lane & 7;
 
+  if (warp < LA_GROUP / 32) {
+    // --------------------------- scores and weights --------------------------
+    // Four warps a tile, so that two tiles are under way; only the running maximum goes from
+    // one tile to the next.  HT = 16: a warp takes 8 keys.  HT = 32: 16 rows by 16 keys.
+    constexpr int NK = MTS;                        // 8-key groups of a warp
+    const int sub = warp >> 2, v = warp & 3;
+    const int mt = MTS == 2 ? v & 1 : 0, key0 = MTS == 2 ? (v >> 1) * 16 : v * 8;
+    const int row0 = mt * 16 + gr, row1 = row0 + 8;
+    const int lim0 = row0 < n_rows ? min(k_end, before + (tok0 + row0) / p.heads) : 0;
+    const int lim1 = row1 < n_rows ? min(k_end, before + (tok0 + row1) / p.heads) : 0;
+    const int steps = p.lk >> 4;
+    const uint32_t qa = smem_u32(Q + (mt * 16 + (lane & 15)) * kp + (lane >> 4) * 8);
+    // HT = 16: 8 keys by 32 channels a load, HT = 32: 16 keys by 16
+    const int krow = MTS == 2 ? key0 + (lane & 7) + (lane >> 4) * 8 : key0 + (lane & 7);
+    const int khi = MTS == 2 ? (lane >> 3) & 1 : lane >> 3;
+    float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
+    for (int n = sub; n < tiles; n += 2) {
+      const int k0 = k_begin + n * LA_KEYS, st = n % p.ring;
+      ok = ok && mbar_wait(&full[st], (uint32_t)(n / p.ring) & 1u, LA_WAIT_LIMIT);
+      uint8_t* tile = K + st * tile_bytes;
+      if (k0 + LA_KEYS > k_end) {
+        // rows behind the last key belong to nobody: their weights are zero, and so must
+        // the products be
+        const int per_row = tile_bytes / (LA_KEYS * 16);
+        for (int i = tid & 127; i < (k0 + LA_KEYS - k_end) * per_row; i += 128) {
+          const int r = k_end - k0 + i / per_row, c = i % per_row;
+          *reinterpret_cast<uint4*>(tile + (c >> 3) * LA_BLOCK + r * 128 + (c & 7) * 16) =
+              make_uint4(0u, 0u, 0u, 0u);
+        }
+        named_bar_sync(1 + sub, 128);
+      }
+      const uint32_t ka = smem_u32(tile) + krow * 128;
+      float s[2][NK][4] = {};                      // two chains of products
+      // fragments of UN steps come ahead of the products of the UN steps before
+      constexpr int UN = MTS == 2 ? 2 : 4, NB = MTS == 2 ? UN : UN / 2;
+      uint32_t a[2][UN][4], b[2][NB][4];
+      auto load = [&](int i0, uint32_t (&fa)[UN][4], uint32_t (&fb)[NB][4]) {
+#pragma unroll
+        for (int u = 0; u < UN; ++u) {
+          const int i = min(i0 + u, steps - 1);
+          ldmatrix_x4(qa + i * 32, fa[u][0], fa[u][1], fa[u][2], fa[u][3]);
+          if (MTS == 2 || u % 2 == 0) {
+            const int e = MTS == 2 ? i : i & ~1, f = MTS == 2 ? u : u / 2;
+            ldmatrix_x4(ka + (e >> 2) * LA_BLOCK + ((((e & 3) * 2 + khi) ^ sw) << 4), fb[f][0],
+                        fb[f][1], fb[f][2], fb[f][3]);
+          }
+        }
+      };
+      auto multiply = [&](int i0, uint32_t (&fa)[UN][4], uint32_t (&fb)[NB][4]) {
+#pragma unroll
+        for (int u = 0; u < UN; ++u)
+          if (i0 + u < steps) {
+            if (MTS == 2) {
+              mma_bf16_16816(s[u & 1][0], fa[u], fb[u % NB][0], fb[u % NB][1]);
+              mma_bf16_16816(s[u & 1][NK - 1], fa[u], fb[u % NB][2], fb[u % NB][3]);
+            } else {
+              mma_bf16_16816(s[u & 1][0], fa[u], fb[u / 2][(u & 1) * 2],
+                             fb[u / 2][(u & 1) * 2 + 1]);
+            }
+          }
+      };
+      load(0, a[0], b[0]);
+      for (int i0 = 0; i0 < steps; i0 += 2 * UN) {
+        load(i0 + UN, a[1], b[1]);
+        multiply(i0, a[0], b[0]);
+        load(i0 + 2 * UN, a[0], b[0]);
+        multiply(i0 + UN, a[1], b[1]);
+      }
+      float x[NK][4], t0 = -INFINITY, t1 = -INFINITY;
+#pragma unroll
+      for (int j = 0; j < NK; ++j)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int key = k0 + key0 + j * 8 + tq * 2 + e;
+          x[j][e] = key < lim0 ? (s[0][j][e] + s[1][j][e]) * p.scale_log2 : -INFINITY;
+          x[j][2 + e] = key < lim1 ? (s[0][j][2 + e] + s[1][j][2 + e]) * p.scale_log2 : -INFINITY;
+          t0 = fmaxf(t0, x[j][e]);
+          t1 = fmaxf(t1, x[j][2 + e]);
+        }
+#pragma unroll
+      for (int o = 1; o < 4; o <<= 1) {
+        t0 = fmaxf(t0, __shfl_xor_sync(0xffffffffu, t0, o));
+        t1 = fmaxf(t1, __shfl_xor_sync(0xffffffffu, t1, o));
+      }
+      if (tq == 0) {
+        m_warp[warp * HT + row0] = t0;
+        m_warp[warp * HT + row1] = t1;
+      }
+      named_bar_sync(1 + sub, 128);
+      // the other warps of this tile that have these rows
+#pragma unroll
+      for (int w = 0; w < (MTS == 2 ? 2 : 4); ++w) {
+        const float* mw = m_warp + (sub * 4 + (MTS == 2 ? w * 2 + mt : w)) * HT;
+        t0 = fmaxf(t0, mw[row0]);
+        t1 = fmaxf(t1, mw[row1]);
+      }
+      float p0 = -INFINITY, p1 = -INFINITY;
+      if (n > 0) {
+        ok = ok && mbar_wait(&m_full[sub ^ 1], (uint32_t)((n - 1) >> 1) & 1u, LA_WAIT_LIMIT);
+        p0 = m_run[(sub ^ 1) * HT + row0];
+        p1 = m_run[(sub ^ 1) * HT + row1];
+        t0 = fmaxf(t0, p0);
+        t1 = fmaxf(t1, p1);
+      }
+      const float z0 = t0 == -INFINITY ? 0.f : t0, z1 = t1 == -INFINITY ? 0.f : t1;
+      const bool writes = tq == 0 && key0 == 0;
+      if (writes) {
+        m_run[sub * HT + row0] = t0;
+        m_run[sub * HT + row1] = t1;
+      }
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&m_full[sub]);
+      l0 *= fast_exp2(m0 - z0);
+      l1 *= fast_exp2(m1 - z1);
+      m0 = t0;
+      m1 = t1;
+#pragma unroll
+      for (int j = 0; j < NK; ++j)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          x[j][e] = fast_exp2(x[j][e] - z0);
+          x[j][2 + e] = fast_exp2(x[j][2 + e] - z1);
+          l0 += x[j][e];
+          l1 += x[j][2 + e];
+        }
+      if (n >= 2)
+        ok = ok && mbar_wait(&p_empty[sub], (uint32_t)(n / 2 - 1) & 1u, LA_WAIT_LIMIT);
+      uint16_t* ph = P + sub * 2 * HT * LA_PPITCH + key0 + tq * 2;
+#pragma unroll
+      for (int j = 0; j < NK; ++j) {
+        uint32_t hi, lo;
+        split_bf16(x[j][0], x[j][1], &hi, &lo);
+        *reinterpret_cast<uint32_t*>(ph + row0 * LA_PPITCH + j * 8) = hi;
+        *reinterpret_cast<uint32_t*>(ph + (HT + row0) * LA_PPITCH + j * 8) = lo;
+        split_bf16(x[j][2], x[j][3], &hi, &lo);
+        *reinterpret_cast<uint32_t*>(ph + row1 * LA_PPITCH + j * 8) = hi;
+        *reinterpret_cast<uint32_t*>(ph + (HT + row1) * LA_PPITCH + j * 8) = lo;
+      }
+      if (writes) {
+        alpha[sub * HT + row0] = p0 == -INFINITY ? 1.f : fast_exp2(p0 - z0);
+        alpha[sub * HT + row1] = p1 == -INFINITY ? 1.f : fast_exp2(p1 - z1);
+      }
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&p_full[sub]);
+    }
+    if (!ok && p.status) atomicOr(p.status, FK_DEV_WAIT_TIMEOUT);
+#pragma unroll
+    for (int o = 1; o < 4; o <<= 1) {
+      l0 += __shfl_xor_sync(0xffffffffu, l0, o);
+      l1 += __shfl_xor_sync(0xffffffffu, l1, o);
+    }
+    // sums relative to the last maximum this warp has seen; rows it does not have stay out
+    for (int r = lane; r < HT; r += 32) l_warp[warp * HT + r] = 0.f;
+    __syncwarp();
+    if (tq == 0) {
+      l_warp[warp * HT + row0] = l0;
+      l_warp[warp * HT + row1] = l1;
+    }
+    if (tiles < 2 && sub == 1 && v == 0)
+      for (int r = lane; r < HT; r += 32) m_run[HT + r] = -INFINITY;
+    if (tiles < 1 && sub == 0 && v == 0)
+      for (int r = lane; r < HT; r += 32) m_run[r] = -INFINITY;
+    named_bar_sync(4, LA_GROUP);
+    if (tid < HT) {
+      const float ma = m_run[tid], mb = m_run[HT + tid], mx = fmaxf(ma, mb);
+      const float z = mx == -INFINITY ? 0.f : mx;
+      float l = 0.f;
+#pragma unroll
+      for (int w = 0; w < 8; ++w)
+        l += l_warp[w * HT + tid] * fast_exp2((w < 4 ? ma : mb) - z);
+      inv_l[tid] = l > 0.f ? 1.0f / l : 0.f;
+      if (p.splits > 1 && tid < n_rows)
+        p.ml[(int64_t)split * p.flat_rows + first + tid] = make_float2(mx, l);
+    }
+    named_bar_sync(3, 2 * LA_GROUP);
+    return;
+  }
+
+  // -------------------------------- values ---------------------------------
   float acc[MTS][RN][4];
 #pragma unroll
   for (int a = 0; a < MTS; ++a)
@@ -211,81 +525,26 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_kernel(const Latent
     for (int j = 0; j < RN; ++j)
 #pragma unroll
       for (int i = 0; i < 4; ++i) acc[a][j][i] = 0.f;
-  const int col0 = warp * RN * 8;
-  const int steps = p.lk >> 4;
-
-  int stage = 0;
-  for (int k0 = k_begin; k0 < k_end; k0 += LA_KEYS, stage ^= 1) {
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();
-    const uint16_t* Kt = K + stage * LA_KEYS * kp;
-    if (k0 + LA_KEYS < k_end) load_tile(k0 + LA_KEYS, K + (stage ^ 1) * LA_KEYS * kp);
-    {
-      // HT = 32: warps 0-3 rows 0-15, 4-7 rows 16-31.  HT = 16: each half of the channels.
-      const int kg = (warp & 3) * 16, part = warp >> 2;
-      const int mrow = MTS == 2 ? part * 16 : 0;
-      const int s0 = MTS == 2 ? 0 : part * ((steps + 1) >> 1);
-      const int s1 = MTS == 2 ? steps : part ? steps : (steps + 1) >> 1;
-      float s[2][4] = {};
-      const uint32_t qa = smem_u32(Q + (mrow + (lane & 15)) * kp + (lane >> 4) * 8);
-      const uint32_t ka = smem_u32(Kt + (kg + (lane & 7) + (lane >> 4) * 8) * kp +
-                                   ((lane >> 3) & 1) * 8);
-#pragma unroll 4
-      for (int i = s0; i < s1; ++i) {
-        uint32_t a[4], b[4];
-        ldmatrix_x4(qa + i * 32, a[0], a[1], a[2], a[3]);
-        ldmatrix_x4(ka + i * 32, b[0], b[1], b[2], b[3]);
-        mma_bf16_16816(s[0], a, b[0], b[1]);
-        mma_bf16_16816(s[1], a, b[2], b[3]);
-      }
-#pragma unroll
-      for (int j = 0; j < 2; ++j)
-#pragma unroll
-        for (int e = 0; e < 2; ++e)
-          *reinterpret_cast<float2*>(S + (part * 16 + gr + e * 8) * LA_SPITCH + kg + j * 8 +
-                                     tq * 2) = make_float2(s[j][e * 2], s[j][e * 2 + 1]);
-    }
-    __syncthreads();
-    {
-      float x[KPT], mx = m;
-#pragma unroll
-      for (int i = 0; i < KPT; ++i) {
-        float v = S[srow * LA_SPITCH + skey + i];
-        if (MTS == 1) v += S[(16 + srow) * LA_SPITCH + skey + i];
-        x[i] = k0 + skey + i < my_lim && k0 + skey + i < k_end ? v * p.scale_log2 : -INFINITY;
-        mx = fmaxf(mx, x[i]);
-      }
-#pragma unroll
-      for (int o = TPR / 2; o > 0; o >>= 1)
-        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-      const float al = mx == -INFINITY ? 1.f : exp2f(m - mx);
-      m = mx;
-      l *= al;
-#pragma unroll
-      for (int i = 0; i < KPT; ++i) {
-        x[i] = mx == -INFINITY ? 0.f : exp2f(x[i] - mx);
-        l += x[i];
-      }
-#pragma unroll
-      for (int i = 0; i < KPT; i += 2) {
-        uint32_t hi, lo;
-        split_bf16(x[i], x[i + 1], &hi, &lo);
-        *reinterpret_cast<uint32_t*>(Ph + srow * LA_PPITCH + skey + i) = hi;
-        *reinterpret_cast<uint32_t*>(Pl + srow * LA_PPITCH + skey + i) = lo;
-      }
-      if (tid % TPR == 0) alpha[srow] = al;
-    }
-    __syncthreads();
-#pragma unroll
-    for (int a = 0; a < MTS; ++a) {
-      const float a0 = alpha[a * 16 + gr], a1 = alpha[a * 16 + gr + 8];
-#pragma unroll
-      for (int j = 0; j < RN; ++j) {
-        acc[a][j][0] *= a0; acc[a][j][1] *= a0;
-        acc[a][j][2] *= a1; acc[a][j][3] *= a1;
-      }
-    }
+  const int col0 = (warp - LA_GROUP / 32) * RN * 8;
+  for (int n = 0; n < tiles; ++n) {
+    const int buf = n & 1, st = n % p.ring;
+    ok = ok && mbar_wait(&full[st], (uint32_t)(n / p.ring) & 1u, LA_WAIT_LIMIT);
+    ok = ok && mbar_wait(&p_full[buf], (uint32_t)(n >> 1) & 1u, LA_WAIT_LIMIT);
+    const uint32_t tile = smem_u32(K + st * tile_bytes) + (lane & 15) * 128;
+    const uint16_t* Ph = P + buf * 2 * HT * LA_PPITCH;
+    const uint16_t* Pl = Ph + HT * LA_PPITCH;
     if (col0 < p.lo) {
+#pragma unroll
+      for (int a = 0; a < MTS; ++a) {
+        const float a0 = alpha[buf * HT + a * 16 + gr], a1 = alpha[buf * HT + a * 16 + gr + 8];
+        if (__any_sync(0xffffffffu, a0 != 1.f || a1 != 1.f)) {
+#pragma unroll
+          for (int j = 0; j < RN; ++j) {
+            acc[a][j][0] *= a0; acc[a][j][1] *= a0;
+            acc[a][j][2] *= a1; acc[a][j][3] *= a1;
+          }
+        }
+      }
 #pragma unroll
       for (int kt = 0; kt < LA_KEYS / 16; ++kt) {
         uint32_t ph[MTS][4], pl[MTS][4];
@@ -295,35 +554,38 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_kernel(const Latent
           ldmatrix_x4(smem_u32(Ph + off), ph[a][0], ph[a][1], ph[a][2], ph[a][3]);
           ldmatrix_x4(smem_u32(Pl + off), pl[a][0], pl[a][1], pl[a][2], pl[a][3]);
         }
+        constexpr int GRP = RN / 2 < 4 / MTS ? RN / 2 : 4 / MTS;   // 16-column groups at a time
 #pragma unroll
-        for (int j = 0; j < RN; j += 2) {
-          const int c = col0 + j * 8;
-          if (c >= p.lo) break;
-          uint32_t b[4];
-          ldmatrix_x4_trans(smem_u32(Kt + (kt * 16 + (lane & 15)) * kp + c + (lane >> 4) * 8),
-                            b[0], b[1], b[2], b[3]);
+        for (int j0 = 0; j0 < RN / 2; j0 += GRP) {
+          uint32_t b[GRP][4];
 #pragma unroll
-          for (int a = 0; a < MTS; ++a) {
-            mma_bf16_16816(acc[a][j], ph[a], b[0], b[1]);
-            mma_bf16_16816(acc[a][j + 1], ph[a], b[2], b[3]);
-            mma_bf16_16816(acc[a][j], pl[a], b[0], b[1]);
-            mma_bf16_16816(acc[a][j + 1], pl[a], b[2], b[3]);
+          for (int j = 0; j < GRP; ++j) {
+            // columns beyond the latent are not stored: any column of the row will do
+            const int c = min(col0 + (j0 + j) * 16, p.lo - 16);
+            ldmatrix_x4_trans(tile + kt * 16 * 128 + (c >> 6) * LA_BLOCK +
+                                  ((((c >> 3) & 7) + (lane >> 4)) ^ sw) * 16,
+                              b[j][0], b[j][1], b[j][2], b[j][3]);
           }
+#pragma unroll
+          for (int part = 0; part < 2; ++part)
+#pragma unroll
+            for (int a = 0; a < MTS; ++a)
+#pragma unroll
+              for (int j = 0; j < GRP; ++j) {
+                mma_bf16_16816(acc[a][2 * (j0 + j)], part ? pl[a] : ph[a], b[j][0], b[j][1]);
+                mma_bf16_16816(acc[a][2 * (j0 + j) + 1], part ? pl[a] : ph[a], b[j][2], b[j][3]);
+              }
         }
       }
     }
+    __syncwarp();
+    if (lane == 0) {
+      mbar_arrive(&empty[st]);
+      mbar_arrive(&p_empty[buf]);
+    }
   }
-#pragma unroll
-  for (int o = TPR / 2; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
-  __syncthreads();
-  if (p.splits > 1) {
-    if (tid % TPR == 0 && srow < n_rows)
-      p.ml[(int64_t)split * p.flat_rows + first + srow] = make_float2(m, l);
-    if (k_begin >= k_end) return;
-  } else if (tid % TPR == 0) {
-    alpha[srow] = l > 0.f ? 1.0f / l : 0.f;
-  }
-  __syncthreads();
+  named_bar_sync(3, 2 * LA_GROUP);
+  if (p.splits > 1 && tiles == 0) return;
 #pragma unroll
   for (int a = 0; a < MTS; ++a)
 #pragma unroll
@@ -339,7 +601,7 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_kernel(const Latent
             *reinterpret_cast<float2*>(o + c) = make_float2(acc[a][j][e * 2], acc[a][j][e * 2 + 1]);
         }
       } else {
-        const float inv = alpha[r];
+        const float inv = inv_l[r];
         uint16_t* o = p.out + (first + r) * p.out_pitch;
 #pragma unroll
         for (int j = 0; j < RN; ++j) {
@@ -352,42 +614,80 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_kernel(const Latent
     }
 }
 
-// One CTA per (token, head) row.
+// One CTA per (token, head) row; at most 32 ranges, a lane each.
 __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentAttnParams p) {
   pdl_launch_dependents();
   pdl_wait();
+  __shared__ float share[32];
   const int64_t r = blockIdx.x;
-  float mx = -INFINITY;
-  for (int s = 0; s < p.splits; ++s) {
-    const float2 v = p.ml[(int64_t)s * p.flat_rows + r];
-    if (v.y > 0.f) mx = fmaxf(mx, v.x);
+  if (threadIdx.x < 32) {
+    const int s = threadIdx.x;
+    const float2 v = s < p.splits ? p.ml[(int64_t)s * p.flat_rows + r] : make_float2(0.f, 0.f);
+    const bool on = v.y > 0.f;
+    float mx = on ? v.x : -INFINITY;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+    const float w = on ? exp2f(v.x - mx) : 0.f;
+    const float l = warp_sum(w * v.y);
+    share[s] = l > 0.f ? w / l : 0.f;
   }
-  float l = 0.f;
-  for (int s = 0; s < p.splits; ++s) {
-    const float2 v = p.ml[(int64_t)s * p.flat_rows + r];
-    if (v.y > 0.f) l += v.y * exp2f(v.x - mx);
-  }
-  const float inv = l > 0.f ? 1.0f / l : 0.f;
+  __syncthreads();
   for (int c = threadIdx.x * 4; c < p.lo; c += 512) {
     float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
     for (int s = 0; s < p.splits; ++s) {
-      const float2 v = p.ml[(int64_t)s * p.flat_rows + r];
-      if (v.y > 0.f)
+      const float w = share[s];
+      if (w > 0.f)
         a = a + *reinterpret_cast<const float4*>(
-                    p.part + ((int64_t)s * p.flat_rows + r) * p.lo + c) *
-                    (exp2f(v.x - mx) * inv);
+                    p.part + ((int64_t)s * p.flat_rows + r) * p.lo + c) * w;
     }
     Elem<uint16_t>::store4(p.out + r * p.out_pitch + c, a);
   }
 }
 
+// [rows, channels] bf16 pool: box = 64 channels x `run` rows, 128B swizzle
+static int la_map(const void* ptr, int64_t rows, int64_t cols, int run, CUtensorMap* out) {
+  struct Entry { const void* ptr; int64_t rows, cols; int run; CUtensorMap map; };
+  static std::mutex mu;
+  static std::vector<Entry> maps;
+  std::lock_guard<std::mutex> lk(mu);
+  for (const Entry& e : maps)
+    if (e.ptr == ptr && e.rows == rows && e.cols == cols && e.run == run) {
+      *out = e.map;
+      return FK_OK;
+    }
+  tensormap_encode_fn enc = get_tensormap_encode();
+  FK_REQUIRE(enc != nullptr, FK_ERR_CUDA,
+             "cuTensorMapEncodeTiled not available from the driver");
+  cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
+  cuuint64_t strides[1] = {(cuuint64_t)cols * 2};
+  cuuint32_t box[2] = {64, (cuuint32_t)run};
+  cuuint32_t estr[2] = {1, 1};
+  CUresult r = enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(ptr), dims,
+                   strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                   CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                   CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  FK_REQUIRE(r == CUDA_SUCCESS, FK_ERR_CUDA, "cuTensorMapEncodeTiled failed with code %d",
+             (int)r);
+  if (maps.size() > 1024) maps.clear();
+  maps.push_back({ptr, rows, cols, run, *out});
+  return FK_OK;
+}
+
 template <int HT, int RN>
-static int launch_latent(const LatentAttnParams& p, dim3 grid, cudaStream_t s) {
-  const int smem = la_smem(HT, p.lk);
-  FK_REQUIRE(smem <= 232448, FK_ERR_UNSUPPORTED, "fk_latent_attn: rows of %d elements", p.lk);
+static int launch_latent(LatentAttnParams& p, dim3 grid, cudaStream_t s) {
+  p.ring = la_ring(HT, p.lk);
+  FK_REQUIRE(p.ring > 0, FK_ERR_UNSUPPORTED, "fk_latent_attn: rows of %d elements", p.lk);
+  const int smem = la_smem(HT, p.lk, p.ring);
   static PerDeviceOnce once;
   FK_CUDA_OK(set_max_dynamic_smem(once, latent_attn_kernel<HT, RN>, 232448));
-  FK_CUDA_OK(launch_kernel(latent_attn_kernel<HT, RN>, grid, dim3(LA_THREADS), (size_t)smem, s, p));
+  p.run = LA_KEYS;                       // keys that surely lie in one page
+  while (p.block_size % p.run) p.run /= 2;
+  CUtensorMap map;
+  const int rc = la_map(p.cache, (int64_t)p.num_blocks * p.block_size, p.cache_pitch, p.run, &map);
+  if (rc != FK_OK) return rc;
+  FK_CUDA_OK(launch_kernel(latent_attn_kernel<HT, RN>, grid, dim3(LA_THREADS), (size_t)smem, s,
+                           map, p));
   count_launch();
   return FK_OK;
 }
@@ -420,6 +720,16 @@ int fk_latent_prepare(const void* q, const void* latent, int64_t in_stride, int 
   p.heads = heads; p.dim = dim; p.rot = rot; p.rank = rank; p.eps = eps; p.status = status;
   const dim3 grid((unsigned)((heads + 1 + 7) / 8), (unsigned)(rows < 16384 ? rows : 16384));
   cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const bool vec = !is_f32 && rank <= 1024 &&
+                   (dim | rot | rank | q_pitch | cache_pitch | q_out_pitch | q_rot_at) % 8 == 0 &&
+                   in_stride % 8 == 0 && aligned16(q) && aligned16(latent) && aligned16(weight) &&
+                   aligned16(cos_sin) && aligned16(cache) && aligned16(q_out);
+  if (vec) {
+    const dim3 vgrid(2, (unsigned)(rows < 16384 ? rows : 16384));
+    FK_CUDA_OK(launch_kernel(latent_prepare_vec_kernel, vgrid, dim3(256), 0, s, p));
+    count_launch();
+    return FK_OK;
+  }
   FK_CUDA_OK(is_f32 ? launch_kernel(latent_prepare_kernel<float>, grid, dim3(256), 0, s, p)
                     : launch_kernel(latent_prepare_kernel<uint16_t>, grid, dim3(256), 0, s, p));
   count_launch();
@@ -447,14 +757,17 @@ int fk_latent_gather(const void* cache, int64_t row_bytes, int64_t num_blocks, i
   return FK_OK;
 }
 
+int fk_latent_attn_supported(int heads, int rank, int rot) {
+  return heads > 0 && rank > 0 && rank <= 512 && rot >= 0 &&
+         la_ring(heads <= 16 ? 16 : 32, (rank + rot + 15) / 16 * 16) > 0;
+}
+
 /* Key ranges a call with these sizes splits its rows into. */
-int fk_latent_attn_splits(int num_seqs, int64_t max_q, int heads, int row_elements,
-                          int64_t max_keys) {
+int fk_latent_attn_splits(int num_seqs, int64_t max_q, int heads, int64_t max_keys) {
   const int ht = heads <= 16 ? 16 : 32;
   const int64_t tiles = (max_q * heads + ht - 1) / ht * num_seqs;
   if (tiles <= 0) return 1;
-  const int per_sm = 232448 / (la_smem(ht, (row_elements + 15) / 16 * 16) + 1024);
-  int64_t s = (int64_t)sm_count() * (per_sm > 2 ? 2 : per_sm < 1 ? 1 : per_sm) / tiles;
+  int64_t s = (int64_t)sm_count() / tiles;
   const int64_t most = (max_keys + 127) / 128;
   s = s < most ? s : most;
   return (int)(s < 1 ? 1 : s > 32 ? 32 : s);
@@ -471,17 +784,21 @@ int fk_latent_attn(const void* q, int64_t q_pitch, const void* cache, int64_t nu
                    int64_t rows, int64_t max_seqlen_q, int heads, int rank, int rot,
                    float softmax_scale, int splits, float* workspace, int64_t workspace_floats,
                    int32_t* status, fk_stream_t stream) {
-  FK_REQUIRE(rows >= 0 && num_seqs >= 0 && heads > 0 && rank > 0 && rot >= 0 && splits >= 1,
+  FK_REQUIRE(rows >= 0 && num_seqs >= 0 && heads > 0 && rank > 0 && rot >= 0 && splits >= 1 &&
+                 splits <= 32,
              FK_ERR_INVALID_ARG, "fk_latent_attn: bad sizes");
   if (rows == 0 || num_seqs == 0 || max_seqlen_q <= 0) return FK_OK;
   FK_REQUIRE(q && cache && out && cu_seqlens_q && kv_lens && block_tables, FK_ERR_INVALID_ARG,
              "fk_latent_attn: null pointer");
-  FK_REQUIRE(rank <= 512, FK_ERR_UNSUPPORTED, "fk_latent_attn: rank %d above 512", rank);
+  FK_REQUIRE(fk_latent_attn_supported(heads, rank, rot), FK_ERR_UNSUPPORTED,
+             "fk_latent_attn: rank %d with %d rotated channels", rank, rot);
   const int lk = (rank + rot + 15) / 16 * 16, lo = (rank + 15) / 16 * 16;
   FK_REQUIRE(cache_pitch >= lk && q_pitch >= lk && out_pitch >= lo && block_size > 0 &&
-                 num_blocks > 0 && num_blocks < (1ll << 31),
+                 num_blocks > 0 && num_blocks * block_size < (1ll << 31),
              FK_ERR_INVALID_ARG, "fk_latent_attn: rows shorter than latent and rotated key, "
              "rounded up to 16 elements");
+  FK_REQUIRE(block_size % 8 == 0, FK_ERR_UNSUPPORTED,
+             "fk_latent_attn: block_size %d must be a multiple of 8", block_size);
   FK_REQUIRE(cache_pitch % 8 == 0 && q_pitch % 8 == 0 && out_pitch % 4 == 0 && aligned16(q) &&
                  aligned16(cache) && aligned16(out) && aligned16(workspace),
              FK_ERR_ALIGNMENT, "fk_latent_attn: rows must be 16-byte aligned");

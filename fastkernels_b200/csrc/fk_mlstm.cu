@@ -399,6 +399,21 @@ __device__ __forceinline__ uint32_t ml_tile(const uint16_t* base, int pitch, int
   return smem_u32(base + (row + (lane & 15)) * pitch + col + (lane >> 4) * 8);
 }
 
+// acc[64 columns] += a (16 x 16) times rows row .. row + 15 of B; the fragments of B come
+// ahead of the products.
+__device__ __forceinline__ void ml_products(float (&acc)[8][4], const uint32_t (&a)[4],
+                                            const uint16_t* B, int pitch, int row, int lane) {
+  uint32_t b[4][4];
+#pragma unroll
+  for (int j = 0; j < 4; ++j)
+    ldmatrix_x4_trans(ml_tile(B, pitch, row, j * 16, lane), b[j][0], b[j][1], b[j][2], b[j][3]);
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    mma_bf16_16816(acc[2 * j], a, b[j][0], b[j][1]);
+    mma_bf16_16816(acc[2 * j + 1], a, b[j][2], b[j][3]);
+  }
+}
+
 // CTA = 64 value columns of one head of one unit: inc = sum_s k_s (c_s v_s)^T with
 // c_s = e^{g_L - g_s + i_s - m_L}; the CTA of the first columns also sums c_s k_s.
 constexpr int MU_THREADS = 128, MU_COLS = 64;
@@ -426,15 +441,28 @@ __global__ void __launch_bounds__(MU_THREADS) mlstm_unit_kernel(const MlstmParam
                    p.gm[at + ML_UNIT - 1]);
   __syncthreads();
   const int cols = min(MU_COLS, p.vdim - v0);
-  for (int i = tid; i < ML_UNIT * (MU_COLS / 2); i += MU_THREADS) {
-    const int r = i / (MU_COLS / 2), c = (i % (MU_COLS / 2)) * 2;
-    float a = 0.f, b = 0.f;
-    if (r < un.count) {
-      if (c < cols) a = bf16_bits_to_float(vg[r * p.in_stride + c]) * cs[r];
-      if (c + 1 < cols) b = bf16_bits_to_float(vg[r * p.in_stride + c + 1]) * cs[r];
+  for (int i = tid; i < ML_UNIT * (MU_COLS / 8); i += MU_THREADS) {
+    const int r = i / (MU_COLS / 8), c = (i % (MU_COLS / 8)) * 8;
+    uint4 x = make_uint4(0u, 0u, 0u, 0u);
+    if (r < un.count && c < cols) {
+      if (p.vdim % 8 == 0) {
+        x = *reinterpret_cast<const uint4*>(vg + r * p.in_stride + c);
+      } else {
+        uint16_t e[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) e[j] = c + j < cols ? vg[r * p.in_stride + c + j] : (uint16_t)0;
+        x = make_uint4(e[0] | (uint32_t)e[1] << 16, e[2] | (uint32_t)e[3] << 16,
+                       e[4] | (uint32_t)e[5] << 16, e[6] | (uint32_t)e[7] << 16);
+      }
     }
-    split_bf16(a, b, reinterpret_cast<uint32_t*>(Vh + r * vpit + c),
-               reinterpret_cast<uint32_t*>(Vl + r * vpit + c));
+    const float k = cs[r];
+    uint4 hi, lo;
+    split_bf16(bf16lo(x.x) * k, bf16hi(x.x) * k, &hi.x, &lo.x);
+    split_bf16(bf16lo(x.y) * k, bf16hi(x.y) * k, &hi.y, &lo.y);
+    split_bf16(bf16lo(x.z) * k, bf16hi(x.z) * k, &hi.z, &lo.z);
+    split_bf16(bf16lo(x.w) * k, bf16hi(x.w) * k, &hi.w, &lo.w);
+    *reinterpret_cast<uint4*>(Vh + r * vpit + c) = hi;
+    *reinterpret_cast<uint4*>(Vl + r * vpit + c) = lo;
   }
   __syncthreads();
   float* inc = p.inc + (u * p.heads + h) * p.dim * p.vp;
@@ -453,16 +481,8 @@ __global__ void __launch_bounds__(MU_THREADS) mlstm_unit_kernel(const MlstmParam
       uint32_t a[4];
       ldmatrix_x4_trans(smem_u32(K + (ks + (lane & 7) + (lane >> 4) * 8) * kp + d0 +
                                  ((lane >> 3) & 1) * 8), a[0], a[1], a[2], a[3]);
-#pragma unroll
-      for (int j = 0; j < 8; j += 2) {
-        uint32_t b[4];
-        ldmatrix_x4_trans(ml_tile(Vh, vpit, ks, j * 8, lane), b[0], b[1], b[2], b[3]);
-        mma_bf16_16816(acc[j], a, b[0], b[1]);
-        mma_bf16_16816(acc[j + 1], a, b[2], b[3]);
-        ldmatrix_x4_trans(ml_tile(Vl, vpit, ks, j * 8, lane), b[0], b[1], b[2], b[3]);
-        mma_bf16_16816(acc[j], a, b[0], b[1]);
-        mma_bf16_16816(acc[j + 1], a, b[2], b[3]);
-      }
+      ml_products(acc, a, Vh, vpit, ks, lane);
+      ml_products(acc, a, Vl, vpit, ks, lane);
     }
 #pragma unroll
     for (int j = 0; j < 8; ++j)
@@ -647,16 +667,8 @@ __global__ void __launch_bounds__(MO_THREADS) mlstm_output_kernel(const MlstmPar
     for (int d = 0; d < dp; d += 16) {
       uint32_t a[4];
       ldmatrix_x4(ml_tile(Q, kp, r0, d, lane), a[0], a[1], a[2], a[3]);
-#pragma unroll
-      for (int j = 0; j < 8; j += 2) {
-        uint32_t b[4];
-        ldmatrix_x4_trans(ml_tile(Sh, vpit, d, j * 8, lane), b[0], b[1], b[2], b[3]);
-        mma_bf16_16816(acc[j], a, b[0], b[1]);
-        mma_bf16_16816(acc[j + 1], a, b[2], b[3]);
-        ldmatrix_x4_trans(ml_tile(Sl, vpit, d, j * 8, lane), b[0], b[1], b[2], b[3]);
-        mma_bf16_16816(acc[j], a, b[0], b[1]);
-        mma_bf16_16816(acc[j + 1], a, b[2], b[3]);
-      }
+      ml_products(acc, a, Sh, vpit, d, lane);
+      ml_products(acc, a, Sl, vpit, d, lane);
     }
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
@@ -666,14 +678,20 @@ __global__ void __launch_bounds__(MO_THREADS) mlstm_output_kernel(const MlstmPar
 #pragma unroll
     for (int kt = 0; kt < 4; ++kt) {
       if (kt > warp) continue;
+      uint32_t b[4][4];
 #pragma unroll
-      for (int j = 0; j < 8; j += 2) {
-        uint32_t b[4];
-        ldmatrix_x4_trans(ml_tile(V, vpit, kt * 16, j * 8, lane), b[0], b[1], b[2], b[3]);
-        mma_bf16_16816(acc[j], ph[kt], b[0], b[1]);
-        mma_bf16_16816(acc[j + 1], ph[kt], b[2], b[3]);
-        mma_bf16_16816(acc[j], pl[kt], b[0], b[1]);
-        mma_bf16_16816(acc[j + 1], pl[kt], b[2], b[3]);
+      for (int j = 0; j < 4; ++j)
+        ldmatrix_x4_trans(ml_tile(V, vpit, kt * 16, j * 16, lane), b[j][0], b[j][1], b[j][2],
+                          b[j][3]);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        mma_bf16_16816(acc[2 * j], ph[kt], b[j][0], b[j][1]);
+        mma_bf16_16816(acc[2 * j + 1], ph[kt], b[j][2], b[j][3]);
+      }
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        mma_bf16_16816(acc[2 * j], pl[kt], b[j][0], b[j][1]);
+        mma_bf16_16816(acc[2 * j + 1], pl[kt], b[j][2], b[j][3]);
       }
     }
 #pragma unroll

@@ -16,7 +16,7 @@
 namespace fk {
 
 constexpr int MR_MAX_EXPERTS = 1024;
-constexpr int MR_BLOCK_ROWS = 128;
+constexpr int MR_BLOCK_ROWS = 64;
 
 struct RouteParams {
   const float* z; int64_t z_stride;
@@ -29,36 +29,39 @@ struct RouteParams {
   int64_t rows; int experts, top, blocks;
 };
 
-// One warp: choices and weights of row t.  The chosen logits stay in the lanes below
-// `top` of rounds of 32.
+// One warp: choices and weights of row t; lane l holds the logits l, l + 32, ...
+template <int EPL>
 __device__ __forceinline__ void route_row(const RouteParams& p, int64_t t, int lane) {
   const float* z = p.z + t * p.z_stride;
-  float best_first = 0.f, total = 0.f;
-  // choice j is the largest logit below choice j - 1 in the order (value, -index)
-  float last_v = INFINITY;
-  int last_i = -1;
+  float v[EPL];
+#pragma unroll
+  for (int i = 0; i < EPL; ++i) v[i] = lane + i * 32 < p.experts ? z[lane + i * 32] : -INFINITY;
+  uint32_t taken = 0;                              // bit i: v[i] is chosen already
+  float first = 0.f, total = 0.f;
   for (int j = 0; j < p.top; ++j) {
-    float v = -INFINITY;
+    float best = -INFINITY;
     int at = 0x7fffffff;
-    for (int e = lane; e < p.experts; e += 32) {
-      const float ze = z[e];
-      const bool free_e = ze < last_v || (ze == last_v && e > last_i);
-      if (free_e && (ze > v || at == 0x7fffffff)) { v = ze; at = e; }
-    }
+#pragma unroll
+    for (int i = 0; i < EPL; ++i)
+      if (!((taken >> i) & 1u) && lane + i * 32 < p.experts && (v[i] > best || at == 0x7fffffff)) {
+        best = v[i];
+        at = lane + i * 32;
+      }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
-      const float ov = __shfl_xor_sync(0xffffffffu, v, o);
+      const float ov = __shfl_xor_sync(0xffffffffu, best, o);
       const int oi = __shfl_xor_sync(0xffffffffu, at, o);
-      if (oi != 0x7fffffff && (at == 0x7fffffff || ov > v || (ov == v && oi < at))) {
-        v = ov;
+      // a lane without candidates loses; ties go to the lowest index
+      if (oi != 0x7fffffff && (at == 0x7fffffff || ov > best || (ov == best && oi < at))) {
+        best = ov;
         at = oi;
       }
     }
-    if (at == 0x7fffffff) { at = 0; v = -INFINITY; }   // NaN logits: no choice is left
-    last_v = v;
-    last_i = at;
-    if (j == 0) best_first = v;
-    const float w = v == -INFINITY ? 0.f : expf(v - best_first);
+    at = __shfl_sync(0xffffffffu, at, 0);          // NaN logits: the lanes still agree
+    best = __shfl_sync(0xffffffffu, best, 0);
+    if ((at & 31) == lane) taken |= 1u << (at >> 5);
+    if (j == 0) first = best;
+    const float w = expf(best - first);
     total += w;
     if (lane == 0) {
       p.chosen[t * p.top + j] = at;
@@ -66,7 +69,7 @@ __device__ __forceinline__ void route_row(const RouteParams& p, int64_t t, int l
     }
   }
   __syncwarp();
-  const float inv = total > 0.f ? 1.0f / total : 0.f;
+  const float inv = 1.0f / total;
   for (int j = lane; j < p.top; j += 32) p.share[t * p.top + j] *= inv;
 }
 
@@ -93,7 +96,7 @@ __device__ __forceinline__ void warp_scan(const int* cnt, int* cursor, int32_t* 
 }
 
 // SINGLE: everything.  Otherwise choices, weights and the counts of the block's rows.
-template <bool SINGLE>
+template <bool SINGLE, int EPL>
 __global__ void __launch_bounds__(1024) moe_route_kernel(const RouteParams p) {
   pdl_launch_dependents();
   pdl_wait();
@@ -102,7 +105,7 @@ __global__ void __launch_bounds__(1024) moe_route_kernel(const RouteParams p) {
   const int64_t t0 = SINGLE ? 0 : (int64_t)blockIdx.x * MR_BLOCK_ROWS;
   const int64_t t1 = SINGLE ? p.rows : min(p.rows, t0 + MR_BLOCK_ROWS);
   for (int e = threadIdx.x; e < p.experts; e += blockDim.x) cnt[e] = 0;
-  for (int64_t t = t0 + warp; t < t1; t += warps) route_row(p, t, lane);
+  for (int64_t t = t0 + warp; t < t1; t += warps) route_row<EPL>(p, t, lane);
   __syncthreads();
   for (int64_t i = t0 * p.top + threadIdx.x; i < t1 * p.top; i += blockDim.x)
     atomicAdd(&cnt[p.chosen[i]], 1);
@@ -129,11 +132,18 @@ __global__ void __launch_bounds__(1024) moe_scan_kernel(const RouteParams p) {
   const int e = threadIdx.x;
   if (e < p.experts) {
     int run = 0;
-    for (int b = 0; b < p.blocks; ++b) {
-      int32_t* c = p.counts + (int64_t)b * p.experts + e;
-      const int mine = *c;
-      *c = run;
-      run += mine;
+    constexpr int UN = 16;
+    for (int b0 = 0; b0 < p.blocks; b0 += UN) {
+      int32_t* c = p.counts + (int64_t)b0 * p.experts + e;
+      int mine[UN];
+#pragma unroll
+      for (int i = 0; i < UN; ++i) mine[i] = b0 + i < p.blocks ? c[(int64_t)i * p.experts] : 0;
+#pragma unroll
+      for (int i = 0; i < UN; ++i)
+        if (b0 + i < p.blocks) {
+          c[(int64_t)i * p.experts] = run;
+          run += mine[i];
+        }
     }
     cnt[e] = run;
   }
@@ -175,6 +185,15 @@ __global__ void __launch_bounds__(256) gather_rows_kernel(
   }
 }
 
+template <bool SINGLE>
+static cudaError_t launch_route(const RouteParams& p, int grid, int threads, cudaStream_t s) {
+  if (p.experts <= 64)
+    return launch_kernel(moe_route_kernel<SINGLE, 2>, dim3(grid), dim3(threads), 0, s, p);
+  if (p.experts <= 256)
+    return launch_kernel(moe_route_kernel<SINGLE, 8>, dim3(grid), dim3(threads), 0, s, p);
+  return launch_kernel(moe_route_kernel<SINGLE, 32>, dim3(grid), dim3(threads), 0, s, p);
+}
+
 }  // namespace fk
 
 using namespace fk;
@@ -204,13 +223,13 @@ int fk_moe_route(const float* z, int64_t z_stride, int32_t* chosen, float* share
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (fk_moe_route_counts(rows, experts, top) == 0) {
     const int threads = rows >= 32 ? 1024 : rows >= 8 ? 512 : 256;
-    FK_CUDA_OK(launch_kernel(moe_route_kernel<true>, dim3(1), dim3(threads), 0, s, p));
+    FK_CUDA_OK(launch_route<true>(p, 1, threads, s));
     count_launch();
     return FK_OK;
   }
   FK_REQUIRE(counts, FK_ERR_WORKSPACE, "fk_moe_route: this many rows need counts");
   p.blocks = (int)((rows + MR_BLOCK_ROWS - 1) / MR_BLOCK_ROWS);
-  FK_CUDA_OK(launch_kernel(moe_route_kernel<false>, dim3((unsigned)p.blocks), dim3(1024), 0, s, p));
+  FK_CUDA_OK(launch_route<false>(p, p.blocks, 512, s));
   FK_CUDA_OK(launch_kernel(moe_scan_kernel, dim3(1), dim3(1024), 0, s, p));
   FK_CUDA_OK(launch_kernel(moe_place_kernel, dim3((unsigned)p.blocks), dim3(256), 0, s, p));
   count_launch(3);

@@ -193,14 +193,23 @@ static cudaError_t launch_add_layernorm(const AddLayerNormParams& p, cudaStream_
 
 template <typename T>
 __global__ void __launch_bounds__(256) softcap_kernel(T* __restrict__ x, int64_t stride,
-                                                      int64_t rows, int64_t cols, float cap) {
+                                                      int64_t rows, int64_t cols, float cap,
+                                                      bool vec) {
   pdl_launch_dependents();
   pdl_wait();
-  const int64_t c = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+  const int64_t c = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) * 4;
   if (c >= cols) return;
+  const float inv = 1.0f / cap;
   for (int64_t t = blockIdx.y; t < rows; t += gridDim.y) {
     T* q = x + t * stride + c;
-    Elem<T>::store(q, cap * tanhf(Elem<T>::load(q) / cap));
+    if (vec && c + 4 <= cols) {
+      const float4 v = Elem<T>::load4(q);
+      Elem<T>::store4(q, make_float4(cap * tanhf(v.x * inv), cap * tanhf(v.y * inv),
+                                     cap * tanhf(v.z * inv), cap * tanhf(v.w * inv)));
+    } else {
+      for (int i = 0; i < 4 && c + i < cols; ++i)
+        Elem<T>::store(q + i, cap * tanhf(Elem<T>::load(q + i) * inv));
+    }
   }
 }
 
@@ -403,12 +412,13 @@ int fk_softcap(void* x, int64_t stride, int is_f32, int64_t rows, int64_t cols, 
   if (rows == 0 || cols == 0) return FK_OK;
   FK_REQUIRE(x && stride >= cols, FK_ERR_INVALID_ARG, "fk_softcap: null pointer or bad stride");
   FK_REQUIRE(cols <= (1ll << 31), FK_ERR_UNSUPPORTED, "fk_softcap: row too long");
-  const dim3 grid((unsigned)((cols + 255) / 256), (unsigned)(rows < 65535 ? rows : 65535));
+  const dim3 grid((unsigned)((cols + 1023) / 1024), (unsigned)(rows < 65535 ? rows : 65535));
   cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const bool vec = stride % 4 == 0 && aligned16(x);
   FK_CUDA_OK(is_f32 ? launch_kernel(softcap_kernel<float>, grid, dim3(256), 0, s, (float*)x,
-                                    stride, rows, cols, cap)
+                                    stride, rows, cols, cap, vec)
                     : launch_kernel(softcap_kernel<uint16_t>, grid, dim3(256), 0, s, (uint16_t*)x,
-                                    stride, rows, cols, cap));
+                                    stride, rows, cols, cap, vec));
   count_launch();
   return FK_OK;
 }

@@ -1,11 +1,11 @@
-"""Prefill and decode throughput of the Pinuvik decoder beside the Llama / Qwen3-style
-decoder of the same width, depth, heads and feed-forward (random weights, bf16), and
-the time of each kernel of a layer beside its roofline.
+"""Prefill and decode throughput of the Pinuvik and Rivilix decoders beside decoders of the
+same width, depth, heads and feed-forward (random weights, bf16), and the time of each
+kernel of a layer beside its roofline.
 
-    python bench.py --workload pinuvik [--layers N] [--sizes 1b,8b]
+    python bench.py --workload pinuvik|rivilix [--layers N] [--sizes 1b,8b] [--kernels]
 
-A size is a real model's layer; the number of layers is cut (every layer is the same
-work) and the vocabulary is small.  Prefill runs whole prompts through the engine's
+pinuvik runs beside the Llama / Qwen3-style decoder, rivilix beside both.  A size is a
+real model's layer; the number of layers is cut and the vocabulary is small.  Prefill runs whole prompts through the engine's
 portion forward, decode replays the engine's CUDA graph; both are timed with CUDA
 events on the launching stream.
 """
@@ -20,7 +20,10 @@ import torch
 from . import ops
 from .candidate.L4.llama import LlamaConfig
 from .engine import DecodeEngine
+from .models.mixers import Yarn
 from .models.pinuvik import PinuvikConfig, PinuvikLayer
+from .models.rivilix import (Bigram, DenseConfig, ExpertsConfig, LatentConfig,
+                             MatrixMemoryConfig, RivilixConfig, RivilixLayer)
 
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 
@@ -30,6 +33,18 @@ SIZES = {
                    rank=64),
     "8b": dict(width=4096, ff=12288, heads=32, kv=8, dim=128, chunk=2048, delta=(64, 64),
                rank=96),
+}
+# latent: heads, unrotated, rotated, value channels, rank; memory: heads, dim, vdim;
+# experts: number, chosen, ff, shared ff
+RIVILIX_SIZES = {
+    "1b": dict(width=2048, ff=6144, latent=(16, 96, 32, 128, 512), memory=(8, 128, 256),
+               experts=(32, 4, 1024, 2048), beside=dict(SIZES["1b"])),
+    "3b-d64": dict(width=2560, ff=6400, latent=(40, 64, 32, 64, 256), memory=(10, 128, 256),
+                   experts=(16, 2, 1600, 1600),
+                   beside=dict(SIZES["3b-d64"], width=2560, ff=6400, heads=40, kv=10,
+                               delta=(20, 128))),
+    "8b": dict(width=4096, ff=12288, latent=(32, 96, 32, 128, 512), memory=(16, 128, 256),
+               experts=(64, 6, 1408, 2816), beside=dict(SIZES["8b"])),
 }
 VOCAB = 32768
 PREFILLS = [(1, 8192), (8, 1024)]
@@ -61,6 +76,25 @@ def configs(z, layers):
         head_dim=128, vocab_size=VOCAB, max_position_embeddings=16384, rope_theta=1e6,
         qk_norm=True, kv_block_size=64)
     return {"pinuvik": pin, "llama": llama}
+
+
+def rivilix_configs(z, layers):
+    """Half of the layers hold experts, every fourth a memory; the others' decoders as for
+    `configs`."""
+    h, dim, rot, vdim, rank = z["latent"]
+    latent = LatentConfig(h, dim, rot, vdim, rank, (dim + rot) ** -0.5, 1e6,
+                          Yarn(8.0, 4096, 32.0, 1.0))
+    memory = MatrixMemoryConfig(*z["memory"], 15.0)
+    dense, sparse = DenseConfig(z["ff"]), ExpertsConfig(*z["experts"])
+    pattern = [RivilixLayer(memory, dense), RivilixLayer(latent, sparse),
+               RivilixLayer(latent, dense), RivilixLayer(latent, sparse)]
+    riv = RivilixConfig(vocab_size=VOCAB, hidden_size=z["width"], eps=1e-6,
+                        layers=[pattern[i % 4] for i in range(layers)],
+                        bigram=Bigram(8192, 40503, 9973), softcap=30.0)
+    return {"rivilix": riv, **configs(z["beside"], layers)}
+
+
+WORKLOADS = {"pinuvik": (SIZES, configs), "rivilix": (RIVILIX_SIZES, rivilix_configs)}
 
 
 def _events():
@@ -112,6 +146,46 @@ def _work(name, args, kw, out):
     if name.startswith("gemm"):
         x, w = args[0], args[1]
         return _nbytes(x, w, out), 2 * x.shape[0] * w.shape[0] * w.shape[1]
+    if name == "group_gemm":
+        x, w, off = args[0], args[1], kw.get("offsets")
+        wn, k = w.shape[-2:]
+        rows, used = out.shape[0], 1 if w.dim() == 2 else w.shape[0]
+        if off is not None:
+            used = int((off[1:] > off[:-1]).sum().item())
+        read = rows * k * (1 if off is not None else used) * 2
+        return read + used * wn * k * 2 + _nbytes(out) if off is not None else \
+            read + _nbytes(w) + rows * used * wn * out.element_size(), \
+            2 * rows * wn * k * (1 if off is not None else used)
+    if name == "latent_attn":
+        q, lens, rank, rot = args[0], args[3].cpu().numpy(), args[7], args[8]
+        qn = np.diff(args[2].cpu().numpy())
+        pairs = float(sum((kv - n + 1 + kv) * n / 2 for n, kv in zip(qn, lens)))
+        return int(lens.sum()) * (rank + rot) * 2 + _nbytes(q, out), \
+            int(2 * pairs * q.shape[1] * (2 * rank + rot))
+    if name == "mlstm_step":
+        return _nbytes(*args[:3], args[4], out) + \
+            2 * args[0].shape[0] * _nbytes(args[6][0], args[7][0]), 0
+    if name == "mlstm_portions":
+        q, k, v = args[:3]
+        heads, dim, vdim = args[9:12]
+        # both products with the matrix per token
+        return _nbytes(q, k, v, out), 4 * q.shape[0] * heads * dim * vdim
+    if name == "add_layernorm":
+        ex = kw.get("experts")
+        rows = _nbytes(kw.get("a"), kw.get("b"), *out[1:])
+        gathered = ex[1].numel() * ex[0].shape[1] * ex[0].element_size() if ex else 0
+        writes = _nbytes(args[0]) if kw.get("a") is not None else 0
+        return _nbytes(args[0]) + writes + rows + gathered, 0
+    if name == "embed_pair_f32":
+        return 2 * _nbytes(out), 0
+    if name in ("moe_route", "softcap"):
+        return 2 * _nbytes(args[0]), 0
+    if name == "latent_prepare":
+        q, lat, out_q = args[0], args[1], args[8]
+        return _nbytes(q, lat, lat) + (_nbytes(out_q) if args[10] else
+                                       out_q.shape[0] * out_q.shape[1] * args[12] * 2), 0
+    if name in ("latent_gather", "gather_rows"):
+        return 2 * _nbytes(out), 0
     if name == "paged_decode_attn":
         q, k, lens = args[0], args[1], args[3]
         live = int(lens.sum().item())
@@ -150,7 +224,10 @@ def _work(name, args, kw, out):
 OPS = ["gemm", "gemm_bf16", "gemm_act_mul", "gemm_silu_mul", "prefill_attn",
        "paged_decode_attn", "paged_decode_attn_plan", "rope_rms_store", "qkv_rope_store",
        "norm_shift", "branch_combine", "fused_add_rmsnorm", "rmsnorm", "delta_prepare",
-       "delta_scan", "head_norm_gate", "act_and_mul", "silu_and_mul", "embed_f32"]
+       "delta_scan", "head_norm_gate", "act_and_mul", "silu_and_mul", "embed_f32",
+       "group_gemm", "latent_attn", "latent_prepare", "latent_gather", "gather_rows",
+       "mlstm_step", "mlstm_portions", "add_layernorm", "embed_pair_f32", "moe_route",
+       "softcap"]
 
 
 class OpTimer:
@@ -192,6 +269,8 @@ class OpTimer:
             if name.startswith("gemm"):
                 x, w = args[0], args[1]
                 label += f" {x.shape[0]}x{w.shape[0]}x{w.shape[1]}"
+            elif name == "group_gemm":
+                label += f" {out.shape[0]}x" + "x".join(map(str, args[1].shape))
             r = rows.setdefault(label, [])
             floor = max(nb / pk["hbm_gbs"] / 1e6, fl / pk["bf16_tflops"] / 1e9)
             r.append((a.elapsed_time(b), floor))
@@ -243,16 +322,17 @@ def kernel_table(eng, n, length):
 
 
 def run(args, sampler=None):
-    sizes = args.sizes.split(",") if args.sizes else list(SIZES)
+    all_sizes, make = WORKLOADS[args.workload]
+    sizes = args.sizes.split(",") if args.sizes else list(all_sizes)
     layers = args.layers or 8
-    line = {"metric": "pinuvik_decoder_tokens_per_s", "unit": "tok/s", "dtype": "bf16",
+    line = {"metric": f"{args.workload}_decoder_tokens_per_s", "unit": "tok/s", "dtype": "bf16",
             "data": "synthetic", "n_gpus": 1, "layers": layers, "vocab": VOCAB,
             "context": CONTEXT, "sizes": {}}
     if sampler:
         sampler.start()
     for name in sizes:
-        z, res = SIZES[name], {}
-        for kind, cfg in configs(z, layers).items():
+        z, res = all_sizes[name], {}
+        for kind, cfg in make(z, layers).items():
             tokens = max(n * t for n, t in PREFILLS)
             pages = max(tokens // 64 + 64, max(DECODES) * (2048 // 64 + 1) + 64)
             eng = DecodeEngine(cfg, max_num_seqs=max(DECODES), max_model_len=16384,

@@ -189,8 +189,6 @@ class LatentAttention:
     # expanded attention makes keys and values of every visible token: worth it for portions
     # that are not much shorter than what they see
     EXPAND_RATIO = 8
-    MAX_TC_RANK = 512           # fk_latent_attn
-    MAX_TC_ROW = 640
 
     def __init__(self, heads, dim, rot, vdim, rank, scale, rot_base, rot_scaling, span, eps,
                  dtype):
@@ -202,8 +200,7 @@ class LatentAttention:
         self.v_pitch = round_up(vdim, 8)
         self.out_columns = round_up(heads * self.v_pitch, 64)
         self.sections = {"q": heads * self.q_pitch, "dkv": rank + rot}
-        self.tensor_cores = dtype == torch.bfloat16 and rank <= self.MAX_TC_RANK and \
-            self.row <= self.MAX_TC_ROW
+        self.tensor_cores = dtype == torch.bfloat16 and ops.latent_attn_supported(heads, rank, rot)
         self.expandable = dtype == torch.bfloat16 and dim + rot <= 128 and vdim <= 128
         self.caches = []
         self.cos_sin = self.status = None

@@ -1007,6 +1007,11 @@ def latent_gather(cache, block_tables, cu_seqlens_k, rows, status=None):
     return out
 
 
+def latent_attn_supported(heads: int, rank: int, rot: int) -> bool:
+    """True when fk_latent_attn takes heads over rows of rank + rot channels."""
+    return bool(lib.fk_latent_attn_supported(heads, rank, rot))
+
+
 def latent_attn(q, cache, cu_seqlens_q, kv_lens, block_tables, max_seqlen_q, max_keys, rank, rot,
                 softmax_scale, out=None, status=None):
     """Absorbed latent attention, bf16: q [T, heads, pitch] over cached rows
@@ -1025,8 +1030,7 @@ def latent_attn(q, cache, cu_seqlens_q, kv_lens, block_tables, max_seqlen_q, max
         out = torch.empty((rows, heads, (rank + 15) // 16 * 16), dtype=BF16, device=q.device)
     elif not out.is_contiguous():
         raise _lib.FkError("latent_attn: out must be contiguous")
-    splits = int(lib.fk_latent_attn_splits(n_seq, int(max_seqlen_q), heads, rank + rot,
-                                           int(max_keys)))
+    splits = int(lib.fk_latent_attn_splits(n_seq, int(max_seqlen_q), heads, int(max_keys)))
     n = int(lib.fk_latent_attn_workspace_floats(rows, heads, rank, splits))
     ws = torch.empty(n, dtype=torch.float32, device=q.device) if n else None
     check(lib.fk_latent_attn(

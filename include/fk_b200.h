@@ -768,7 +768,9 @@ int fk_gather_rows(const void* x, int64_t x_stride_bytes, int64_t x_rows, const 
  * fk_latent_attn (bf16): every (token, head) row of q attends the cached rows of its
  * sequence up to its own token (queries end at key kv_lens[i]); the value of a key is its
  * first `rank` channels; out [rows * heads, out_pitch].  splits > 1 cuts the keys of every
- * row into that many ranges and merges them (fk_latent_attn_splits suggests a number). */
+ * row into that many ranges and merges them (fk_latent_attn_splits suggests a number).
+ * Rows that do not fit on an SM (fk_latent_attn_supported: rank up to 512) go through
+ * fk_paged_attn_any with one KV head. */
 int fk_latent_prepare(const void* q, const void* latent, int64_t in_stride, int q_pitch,
                       int is_f32, const float* weight, const float* cos_sin, int64_t max_position,
                       const int32_t* slots, const int64_t* positions, void* cache,
@@ -779,8 +781,8 @@ int fk_latent_gather(const void* cache, int64_t row_bytes, int64_t num_blocks, i
                      const int32_t* block_tables, int64_t block_table_stride,
                      const int32_t* cu_seqlens_k, int num_seqs, void* out, int64_t rows,
                      int32_t* status, fk_stream_t stream);
-int fk_latent_attn_splits(int num_seqs, int64_t max_q, int heads, int row_elements,
-                          int64_t max_keys);
+int fk_latent_attn_supported(int heads, int rank, int rot);
+int fk_latent_attn_splits(int num_seqs, int64_t max_q, int heads, int64_t max_keys);
 int64_t fk_latent_attn_workspace_floats(int64_t rows, int heads, int rank, int splits);
 int fk_latent_attn(const void* q, int64_t q_pitch, const void* cache, int64_t num_blocks,
                    int block_size, int cache_pitch, void* out, int64_t out_pitch,
