@@ -7,7 +7,7 @@
 //                           (and copy) of the queries; _vec: the same 16 bytes at a time
 //   latent_gather_kernel    cached rows of a batch's sequences side by side
 //   latent_attn_kernel      absorbed attention, bf16: portions and single tokens alike.  A
-//                           CTA owns HT (token, head) rows of one sequence and a range of
+//                           CTA owns 16 (token, head) rows of one sequence and a range of
 //                           keys; tiles of cached rows come through a ring and serve as K
 //                           and as V.  Waits are bounded
 //   latent_merge_kernel     key ranges of a row -> one result
@@ -218,146 +218,115 @@ struct LatentAttnParams {
 };
 
 // Warps 0-7 make scores and softmax weights of a tile of 32 keys, warps 8-15 multiply the
-// weights of the tile before it with its values, warp 16 keeps the ring of tiles filled: a
-// tile is blocks of 64 channels, [32 rows][128 bytes] each, 128-byte swizzled by TMA.
-constexpr int LA_GROUP = 256, LA_THREADS = 2 * LA_GROUP + 32, LA_KEYS = 32;
+// weights of the tile before it with its values; one lane of warp 8 keeps the ring of tiles
+// filled.  A tile is blocks of 64 channels, [32 rows][128 bytes] each, 128-byte swizzled by
+// TMA.  The steps of a tile are short, so what bounds the kernel is the latency of fragment
+// loads and of hand-overs: query fragments stay in registers, fragments are loaded several
+// steps ahead, and warps hand over through named barriers (a wait on a shared-memory barrier
+// costs several times as much; only the copies need one).
+constexpr int LA_ROWS = 16, LA_GROUP = 256, LA_THREADS = 2 * LA_GROUP, LA_KEYS = 32;
 constexpr int LA_BLOCK = LA_KEYS * 128;
-constexpr int LA_PPITCH = LA_KEYS + 8, LA_MAX_RING = 8;
+constexpr int LA_PPITCH = LA_KEYS + 8, LA_XPITCH = LA_KEYS + 8, LA_MAX_RING = 8;
 constexpr uint32_t LA_WAIT_LIMIT = 1u << 22;
+// named barriers
+constexpr int LA_BAR_SUB = 1, LA_BAR_END = 3, LA_BAR_SUM = 4, LA_BAR_FULL = 5, LA_BAR_EMPTY = 7,
+              LA_BAR_MAX = 9;
 
 // lk: channels of a row, rounded up to 16; a tile holds whole blocks of 64.
 __host__ __device__ constexpr int la_tile(int lk) { return (lk + 63) / 64 * LA_BLOCK; }
-__host__ __device__ constexpr int la_smem(int ht, int lk, int ring) {
-  return ring * la_tile(lk) + ht * (lk + 8) * 2 + 4 * ht * LA_PPITCH * 2 + 21 * ht * 4 +
-         (2 * LA_MAX_RING + 6) * 8 + 1024;
+// 8-column groups of values per warp, and 16-channel steps of scores per warp.
+__host__ __device__ constexpr int la_rn(int rank) { return rank <= 128 ? 2 : rank <= 256 ? 4 : 8; }
+__host__ __device__ constexpr int la_steps(int rn) { return rn == 8 ? 10 : rn == 4 ? 6 : 4; }
+__host__ __device__ constexpr int la_smem(int lk, int ring) {
+  return ring * la_tile(lk) + 2 * 4 * LA_ROWS * LA_XPITCH * 4 + 4 * LA_ROWS * LA_PPITCH * 2 +
+         21 * LA_ROWS * 4 + LA_MAX_RING * 8 + 1024;
 }
 // Deepest ring that fits, 0: none.
-__host__ __device__ constexpr int la_ring(int ht, int lk) {
+__host__ __device__ constexpr int la_ring(int lk) {
   int r = LA_MAX_RING;
-  while (r >= 3 && la_smem(ht, lk, r) > 232448) --r;
+  while (r >= 3 && la_smem(lk, r) > 232448) --r;
   return r >= 3 ? r : 0;
 }
 
-template <int HT, int RN>
+__device__ __forceinline__ void named_bar_arrive(int id, int nthreads) {
+  asm volatile("bar.arrive %0, %1;" ::"r"(id), "r"(nthreads) : "memory");
+}
+
+template <int RN>
 __global__ void __launch_bounds__(LA_THREADS, 1)
 latent_attn_kernel(const __grid_constant__ CUtensorMap tmap, const LatentAttnParams p) {
   extern __shared__ uint8_t la_raw[];
   pdl_launch_dependents();
-  constexpr int MTS = HT / 16;
   const int seq = blockIdx.y, split = blockIdx.z;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int gr = lane >> 2, tq = lane & 3;
-  uint8_t* K = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(la_raw) + 1023) &
-                                          ~uintptr_t(1023));          // ring of tiles
-  const int tile_bytes = la_tile(p.lk), kp = p.lk + 8;
-  uint16_t* Q = reinterpret_cast<uint16_t*>(K + p.ring * tile_bytes); // [HT][kp]
-  uint16_t* P = Q + HT * kp;                              // [2][hi, lo][HT][LA_PPITCH]
-  float* alpha = reinterpret_cast<float*>(P + 4 * HT * LA_PPITCH);    // [2][HT]
-  float* inv_l = alpha + 2 * HT;                          // [HT]
-  float* m_run = inv_l + HT;                              // [2][HT]: running maximum
-  float* m_warp = m_run + 2 * HT;                         // [8][HT]: of a tile, per warp
-  float* l_warp = m_warp + 8 * HT;                        // [8][HT]
-  uint64_t* full = reinterpret_cast<uint64_t*>(l_warp + 8 * HT);   // [ring]: rows have come
-  uint64_t* empty = full + LA_MAX_RING;                   // [ring]: ... and are no longer read
-  uint64_t* p_full = empty + LA_MAX_RING;                 // [2]: weights of a tile written
-  uint64_t* p_empty = p_full + 2;                         // [2]: ... and read
-  uint64_t* m_full = p_empty + 2;                         // [2]: running maximum after a tile
+  uint8_t* K = la_raw + ((1024u - (smem_u32(la_raw) & 1023u)) & 1023u);    // ring of tiles
+  const int tile_bytes = la_tile(p.lk);
+  float* X = reinterpret_cast<float*>(K + p.ring * tile_bytes);   // [2][4][16][LA_XPITCH]
+  uint16_t* P = reinterpret_cast<uint16_t*>(X + 8 * LA_ROWS * LA_XPITCH);  // [2][hi, lo][16][]
+  float* alpha = reinterpret_cast<float*>(P + 4 * LA_ROWS * LA_PPITCH);    // [2][16]
+  float* inv_l = alpha + 2 * LA_ROWS;                     // [16]
+  float* m_run = inv_l + LA_ROWS;                         // [2][16]: running maximum
+  float* m_warp = m_run + 2 * LA_ROWS;                    // [8][16]: of a tile, per warp
+  float* l_warp = m_warp + 8 * LA_ROWS;                   // [8][16]
+  uint64_t* full = reinterpret_cast<uint64_t*>(l_warp + 8 * LA_ROWS);      // [ring]
   if (tid == 0) {
-    for (int i = 0; i < p.ring; ++i) {
-      mbar_init(&full[i], 1);
-      mbar_init(&empty[i], LA_GROUP / 32);
-    }
-    for (int i = 0; i < 2; ++i) {
-      mbar_init(&p_full[i], 4);
-      mbar_init(&p_empty[i], LA_GROUP / 32);
-      mbar_init(&m_full[i], 4);
-    }
+    for (int i = 0; i < p.ring; ++i) mbar_init(&full[i], 1);
     mbar_fence_init();
     tma_prefetch_desc(&tmap);
   }
   pdl_wait();
   const int q0 = p.cu_q[seq], q_len = p.cu_q[seq + 1] - q0;
-  const int64_t first = (int64_t)q0 * p.heads + (int64_t)blockIdx.x * HT;   // flat row
-  const int64_t left = (int64_t)q_len * p.heads - (int64_t)blockIdx.x * HT;
-  if (left <= 0 || first + min(left, (int64_t)HT) > p.flat_rows) return;
-  const int n_rows = (int)min(left, (int64_t)HT);
+  const int64_t first = (int64_t)q0 * p.heads + (int64_t)blockIdx.x * LA_ROWS;   // flat row
+  const int64_t left = (int64_t)q_len * p.heads - (int64_t)blockIdx.x * LA_ROWS;
+  if (left <= 0 || first + min(left, (int64_t)LA_ROWS) > p.flat_rows) return;
+  const int n_rows = (int)min(left, (int64_t)LA_ROWS);
   const int kv_len = p.kv_lens[seq];
   const int before = kv_len - q_len + 1;                 // keys token 0 of the portion sees
-  const int tok0 = blockIdx.x * HT;
+  const int tok0 = blockIdx.x * LA_ROWS;
   const int most = max(0, min(kv_len, before + (tok0 + n_rows - 1) / p.heads));
   const int per = ((most + p.splits - 1) / p.splits + LA_KEYS - 1) / LA_KEYS * LA_KEYS;
   const int k_begin = min(most, split * per), k_end = min(most, k_begin + per);
-  {
-    const int packs = p.lk >> 3;
-    for (int i = tid; i < HT * packs; i += LA_THREADS) {
-      const int r = i / packs, c = (i - r * packs) * 8;
-      uint4 v = make_uint4(0u, 0u, 0u, 0u);
-      if (r < n_rows) v = *reinterpret_cast<const uint4*>(p.q + (first + r) * p.q_pitch + c);
-      *reinterpret_cast<uint4*>(Q + r * kp + c) = v;
-    }
-  }
   __syncthreads();
   const int tiles = (k_end - k_begin + LA_KEYS - 1) / LA_KEYS;
-  bool ok = true;
-
-  if (warp == 2 * LA_GROUP / 32) {
-    // ------------------------------- cached rows ----------------------------
-    if (lane != 0) return;
-    const int32_t* bt = p.block_tables + seq * p.bt_stride;
-    const int blocks = (p.lk + 63) / 64;
-    int n = 0;
-    for (; n < tiles; ++n) {
-      const int st = n % p.ring;
-      if (n >= p.ring)
-        ok = mbar_wait(&empty[st], (uint32_t)(n / p.ring - 1) & 1u, LA_WAIT_LIMIT);
-      if (!ok) {
-        if (p.status) atomicOr(p.status, FK_DEV_WAIT_TIMEOUT);
-        break;
-      }
-      mbar_arrive_expect_tx(&full[st], (uint32_t)tile_bytes);
-      uint8_t* dst = K + st * tile_bytes;
-      // runs of p.run keys lie in one page
-      for (int r = 0; r < LA_KEYS; r += p.run) {
-        const int key = k_begin + n * LA_KEYS + r;
-        int row = p.num_blocks * p.block_size;            // out of range: zeros
-        if (key < k_end) {
-          const int page = bt[key / p.block_size];
-          if (page >= 0 && page < p.num_blocks) row = page * p.block_size + key % p.block_size;
-          else if (p.status) atomicOr(p.status, FK_DEV_BAD_PAGE);
-        }
-        for (int c = 0; c < blocks; ++c)
-          tma_load_2d(dst + c * LA_BLOCK + r * 128, &tmap, &full[st], c * 64, row);
-      }
-    }
-    // no copy may be in flight when the CTA ends
-    if (!ok)
-      for (int i = max(0, n - p.ring); i < n; ++i)
-        (void)mbar_wait(&full[i % p.ring], (uint32_t)(i / p.ring) & 1u, LA_WAIT_LIMIT);
-    return;
-  }
-
   // 16-byte chunk of a row's 128 bytes of a block, as the swizzle places it
   const int sw = lane & 7;
+  const int row0 = gr, row1 = gr + 8;
 
   if (warp < LA_GROUP / 32) {
     // --------------------------- scores and weights --------------------------
     // Four warps a tile, so that two tiles are under way; only the running maximum goes from
-    // one tile to the next.  HT = 16: a warp takes 8 keys.  HT = 32: 16 rows by 16 keys.
-    constexpr int NK = MTS;                        // 8-key groups of a warp
-    const int sub = warp >> 2, v = warp & 3;
-    const int mt = MTS == 2 ? v & 1 : 0, key0 = MTS == 2 ? (v >> 1) * 16 : v * 8;
-    const int row0 = mt * 16 + gr, row1 = row0 + 8;
+    // one tile to the next.  Products: a warp has all keys and a quarter of the channels.
+    // Weights: 8 keys.
+    constexpr int QS = la_steps(RN), AHEAD = 3;
+    const int sub = warp >> 2, v = warp & 3, key0 = v * 8;
     const int lim0 = row0 < n_rows ? min(k_end, before + (tok0 + row0) / p.heads) : 0;
     const int lim1 = row1 < n_rows ? min(k_end, before + (tok0 + row1) / p.heads) : 0;
-    const int steps = p.lk >> 4;
-    const uint32_t qa = smem_u32(Q + (mt * 16 + (lane & 15)) * kp + (lane >> 4) * 8);
-    // HT = 16: 8 keys by 32 channels a load, HT = 32: 16 keys by 16
-    const int krow = MTS == 2 ? key0 + (lane & 7) + (lane >> 4) * 8 : key0 + (lane & 7);
-    const int khi = MTS == 2 ? (lane >> 3) & 1 : lane >> 3;
+    const int steps = p.lk >> 4, each = (steps + 3) >> 2;
+    const int s0 = min(steps, v * each), s1 = min(steps, s0 + each);
+    uint32_t qf[QS][4];
+    {
+      const uint16_t* r0 = p.q + (first + row0) * p.q_pitch + tq * 2;
+      const uint16_t* r1 = p.q + (first + row1) * p.q_pitch + tq * 2;
+#pragma unroll
+      for (int u = 0; u < QS; ++u) {
+        const int c = (s0 + u) * 16;
+        const bool on = s0 + u < s1;
+        qf[u][0] = on && row0 < n_rows ? *reinterpret_cast<const uint32_t*>(r0 + c) : 0u;
+        qf[u][1] = on && row1 < n_rows ? *reinterpret_cast<const uint32_t*>(r1 + c) : 0u;
+        qf[u][2] = on && row0 < n_rows ? *reinterpret_cast<const uint32_t*>(r0 + c + 8) : 0u;
+        qf[u][3] = on && row1 < n_rows ? *reinterpret_cast<const uint32_t*>(r1 + c + 8) : 0u;
+      }
+    }
+    const int krow = (lane & 7) + (lane >> 4) * 8, khi = (lane >> 3) & 1;
+    float* xs = X + sub * 4 * LA_ROWS * LA_XPITCH;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
+    bool ok = true;
+    int st = sub;
+    uint32_t phase = 0;
     for (int n = sub; n < tiles; n += 2) {
-      const int k0 = k_begin + n * LA_KEYS, st = n % p.ring;
-      ok = ok && mbar_wait(&full[st], (uint32_t)(n / p.ring) & 1u, LA_WAIT_LIMIT);
+      const int k0 = k_begin + n * LA_KEYS;
+      ok = ok && mbar_wait(&full[st], phase, LA_WAIT_LIMIT);
       uint8_t* tile = K + st * tile_bytes;
       if (k0 + LA_KEYS > k_end) {
         // rows behind the last key belong to nobody: their weights are zero, and so must
@@ -368,121 +337,113 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmap, const LatentAttnPar
           *reinterpret_cast<uint4*>(tile + (c >> 3) * LA_BLOCK + r * 128 + (c & 7) * 16) =
               make_uint4(0u, 0u, 0u, 0u);
         }
-        named_bar_sync(1 + sub, 128);
+        named_bar_sync(LA_BAR_SUB + sub, 128);
       }
       const uint32_t ka = smem_u32(tile) + krow * 128;
-      float s[2][NK][4] = {};                      // two chains of products
-      // fragments of UN steps come ahead of the products of the UN steps before
-      constexpr int UN = MTS == 2 ? 2 : 4, NB = MTS == 2 ? UN : UN / 2;
-      uint32_t a[2][UN][4], b[2][NB][4];
-      auto load = [&](int i0, uint32_t (&fa)[UN][4], uint32_t (&fb)[NB][4]) {
-#pragma unroll
-        for (int u = 0; u < UN; ++u) {
-          const int i = min(i0 + u, steps - 1);
-          ldmatrix_x4(qa + i * 32, fa[u][0], fa[u][1], fa[u][2], fa[u][3]);
-          if (MTS == 2 || u % 2 == 0) {
-            const int e = MTS == 2 ? i : i & ~1, f = MTS == 2 ? u : u / 2;
-            ldmatrix_x4(ka + (e >> 2) * LA_BLOCK + ((((e & 3) * 2 + khi) ^ sw) << 4), fb[f][0],
-                        fb[f][1], fb[f][2], fb[f][3]);
-          }
-        }
+      float s[4][4] = {};
+      uint32_t b[AHEAD + 1][2][4];
+      auto load = [&](int u, uint32_t (&fb)[2][4]) {
+        const int i = min(s0 + u, steps - 1);
+        const uint32_t at = ka + (i >> 2) * LA_BLOCK + ((((i & 3) * 2 + khi) ^ sw) << 4);
+        ldmatrix_x4(at, fb[0][0], fb[0][1], fb[0][2], fb[0][3]);
+        ldmatrix_x4(at + 16 * 128, fb[1][0], fb[1][1], fb[1][2], fb[1][3]);
       };
-      auto multiply = [&](int i0, uint32_t (&fa)[UN][4], uint32_t (&fb)[NB][4]) {
 #pragma unroll
-        for (int u = 0; u < UN; ++u)
-          if (i0 + u < steps) {
-            if (MTS == 2) {
-              mma_bf16_16816(s[u & 1][0], fa[u], fb[u % NB][0], fb[u % NB][1]);
-              mma_bf16_16816(s[u & 1][NK - 1], fa[u], fb[u % NB][2], fb[u % NB][3]);
-            } else {
-              mma_bf16_16816(s[u & 1][0], fa[u], fb[u / 2][(u & 1) * 2],
-                             fb[u / 2][(u & 1) * 2 + 1]);
-            }
-          }
-      };
-      load(0, a[0], b[0]);
-      for (int i0 = 0; i0 < steps; i0 += 2 * UN) {
-        load(i0 + UN, a[1], b[1]);
-        multiply(i0, a[0], b[0]);
-        load(i0 + 2 * UN, a[0], b[0]);
-        multiply(i0 + UN, a[1], b[1]);
+      for (int u = 0; u < AHEAD; ++u) load(u, b[u]);
+#pragma unroll
+      for (int u = 0; u < QS; ++u) {
+        if (u + AHEAD < QS) load(u + AHEAD, b[(u + AHEAD) % (AHEAD + 1)]);
+        const uint32_t (&fb)[2][4] = b[u % (AHEAD + 1)];
+        // steps beyond the part have zero queries
+        mma_bf16_16816(s[0], qf[u], fb[0][0], fb[0][1]);
+        mma_bf16_16816(s[1], qf[u], fb[0][2], fb[0][3]);
+        mma_bf16_16816(s[2], qf[u], fb[1][0], fb[1][1]);
+        mma_bf16_16816(s[3], qf[u], fb[1][2], fb[1][3]);
       }
-      float x[NK][4], t0 = -INFINITY, t1 = -INFINITY;
 #pragma unroll
-      for (int j = 0; j < NK; ++j)
+      for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int e = 0; e < 2; ++e)
+          *reinterpret_cast<float2*>(xs + (v * LA_ROWS + row0 + e * 8) * LA_XPITCH + j * 8 +
+                                     tq * 2) = make_float2(s[j][e * 2], s[j][e * 2 + 1]);
+      named_bar_sync(LA_BAR_SUB + sub, 128);
+      float x[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int q = 0; q < 4; ++q)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-          const int key = k0 + key0 + j * 8 + tq * 2 + e;
-          x[j][e] = key < lim0 ? (s[0][j][e] + s[1][j][e]) * p.scale_log2 : -INFINITY;
-          x[j][2 + e] = key < lim1 ? (s[0][j][2 + e] + s[1][j][2 + e]) * p.scale_log2 : -INFINITY;
-          t0 = fmaxf(t0, x[j][e]);
-          t1 = fmaxf(t1, x[j][2 + e]);
+          const float2 y = *reinterpret_cast<const float2*>(
+              xs + (q * LA_ROWS + row0 + e * 8) * LA_XPITCH + key0 + tq * 2);
+          x[e * 2] += y.x;
+          x[e * 2 + 1] += y.y;
         }
+      float t0 = -INFINITY, t1 = -INFINITY;
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int key = k0 + key0 + tq * 2 + e;
+        x[e] = key < lim0 ? x[e] * p.scale_log2 : -INFINITY;
+        x[2 + e] = key < lim1 ? x[2 + e] * p.scale_log2 : -INFINITY;
+        t0 = fmaxf(t0, x[e]);
+        t1 = fmaxf(t1, x[2 + e]);
+      }
 #pragma unroll
       for (int o = 1; o < 4; o <<= 1) {
         t0 = fmaxf(t0, __shfl_xor_sync(0xffffffffu, t0, o));
         t1 = fmaxf(t1, __shfl_xor_sync(0xffffffffu, t1, o));
       }
       if (tq == 0) {
-        m_warp[warp * HT + row0] = t0;
-        m_warp[warp * HT + row1] = t1;
+        m_warp[warp * LA_ROWS + row0] = t0;
+        m_warp[warp * LA_ROWS + row1] = t1;
       }
-      named_bar_sync(1 + sub, 128);
-      // the other warps of this tile that have these rows
+      named_bar_sync(LA_BAR_SUB + sub, 128);
 #pragma unroll
-      for (int w = 0; w < (MTS == 2 ? 2 : 4); ++w) {
-        const float* mw = m_warp + (sub * 4 + (MTS == 2 ? w * 2 + mt : w)) * HT;
+      for (int w = 0; w < 4; ++w) {
+        const float* mw = m_warp + (sub * 4 + w) * LA_ROWS;
         t0 = fmaxf(t0, mw[row0]);
         t1 = fmaxf(t1, mw[row1]);
       }
       float p0 = -INFINITY, p1 = -INFINITY;
       if (n > 0) {
-        ok = ok && mbar_wait(&m_full[sub ^ 1], (uint32_t)((n - 1) >> 1) & 1u, LA_WAIT_LIMIT);
-        p0 = m_run[(sub ^ 1) * HT + row0];
-        p1 = m_run[(sub ^ 1) * HT + row1];
+        named_bar_sync(LA_BAR_MAX + (sub ^ 1), 2 * 128);
+        p0 = m_run[(sub ^ 1) * LA_ROWS + row0];
+        p1 = m_run[(sub ^ 1) * LA_ROWS + row1];
         t0 = fmaxf(t0, p0);
         t1 = fmaxf(t1, p1);
       }
-      const float z0 = t0 == -INFINITY ? 0.f : t0, z1 = t1 == -INFINITY ? 0.f : t1;
-      const bool writes = tq == 0 && key0 == 0;
+      const bool writes = tq == 0 && v == 0;
       if (writes) {
-        m_run[sub * HT + row0] = t0;
-        m_run[sub * HT + row1] = t1;
+        m_run[sub * LA_ROWS + row0] = t0;
+        m_run[sub * LA_ROWS + row1] = t1;
       }
-      __syncwarp();
-      if (lane == 0) mbar_arrive(&m_full[sub]);
+      if (n + 1 < tiles) named_bar_arrive(LA_BAR_MAX + sub, 2 * 128);
+      const float z0 = t0 == -INFINITY ? 0.f : t0, z1 = t1 == -INFINITY ? 0.f : t1;
       l0 *= fast_exp2(m0 - z0);
       l1 *= fast_exp2(m1 - z1);
       m0 = t0;
       m1 = t1;
 #pragma unroll
-      for (int j = 0; j < NK; ++j)
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          x[j][e] = fast_exp2(x[j][e] - z0);
-          x[j][2 + e] = fast_exp2(x[j][2 + e] - z1);
-          l0 += x[j][e];
-          l1 += x[j][2 + e];
-        }
-      if (n >= 2)
-        ok = ok && mbar_wait(&p_empty[sub], (uint32_t)(n / 2 - 1) & 1u, LA_WAIT_LIMIT);
-      uint16_t* ph = P + sub * 2 * HT * LA_PPITCH + key0 + tq * 2;
-#pragma unroll
-      for (int j = 0; j < NK; ++j) {
-        uint32_t hi, lo;
-        split_bf16(x[j][0], x[j][1], &hi, &lo);
-        *reinterpret_cast<uint32_t*>(ph + row0 * LA_PPITCH + j * 8) = hi;
-        *reinterpret_cast<uint32_t*>(ph + (HT + row0) * LA_PPITCH + j * 8) = lo;
-        split_bf16(x[j][2], x[j][3], &hi, &lo);
-        *reinterpret_cast<uint32_t*>(ph + row1 * LA_PPITCH + j * 8) = hi;
-        *reinterpret_cast<uint32_t*>(ph + (HT + row1) * LA_PPITCH + j * 8) = lo;
+      for (int e = 0; e < 2; ++e) {
+        x[e] = fast_exp2(x[e] - z0);
+        x[2 + e] = fast_exp2(x[2 + e] - z1);
+        l0 += x[e];
+        l1 += x[2 + e];
       }
+      if (n >= 2) named_bar_sync(LA_BAR_EMPTY + sub, 128 + LA_GROUP);
+      uint16_t* ph = P + sub * 2 * LA_ROWS * LA_PPITCH + key0 + tq * 2;
+      uint32_t hi, lo;
+      split_bf16(x[0], x[1], &hi, &lo);
+      *reinterpret_cast<uint32_t*>(ph + row0 * LA_PPITCH) = hi;
+      *reinterpret_cast<uint32_t*>(ph + (LA_ROWS + row0) * LA_PPITCH) = lo;
+      split_bf16(x[2], x[3], &hi, &lo);
+      *reinterpret_cast<uint32_t*>(ph + row1 * LA_PPITCH) = hi;
+      *reinterpret_cast<uint32_t*>(ph + (LA_ROWS + row1) * LA_PPITCH) = lo;
       if (writes) {
-        alpha[sub * HT + row0] = p0 == -INFINITY ? 1.f : fast_exp2(p0 - z0);
-        alpha[sub * HT + row1] = p1 == -INFINITY ? 1.f : fast_exp2(p1 - z1);
+        alpha[sub * LA_ROWS + row0] = p0 == -INFINITY ? 1.f : fast_exp2(p0 - z0);
+        alpha[sub * LA_ROWS + row1] = p1 == -INFINITY ? 1.f : fast_exp2(p1 - z1);
       }
-      __syncwarp();
-      if (lane == 0) mbar_arrive(&p_full[sub]);
+      named_bar_arrive(LA_BAR_FULL + sub, 128 + LA_GROUP);
+      st += 2;
+      if (st >= p.ring) { st -= p.ring; phase ^= 1; }
     }
     if (!ok && p.status) atomicOr(p.status, FK_DEV_WAIT_TIMEOUT);
 #pragma unroll
@@ -490,128 +451,146 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmap, const LatentAttnPar
       l0 += __shfl_xor_sync(0xffffffffu, l0, o);
       l1 += __shfl_xor_sync(0xffffffffu, l1, o);
     }
-    // sums relative to the last maximum this warp has seen; rows it does not have stay out
-    for (int r = lane; r < HT; r += 32) l_warp[warp * HT + r] = 0.f;
-    __syncwarp();
+    // sums relative to the last maximum this warp has seen
     if (tq == 0) {
-      l_warp[warp * HT + row0] = l0;
-      l_warp[warp * HT + row1] = l1;
+      l_warp[warp * LA_ROWS + row0] = l0;
+      l_warp[warp * LA_ROWS + row1] = l1;
     }
-    if (tiles < 2 && sub == 1 && v == 0)
-      for (int r = lane; r < HT; r += 32) m_run[HT + r] = -INFINITY;
-    if (tiles < 1 && sub == 0 && v == 0)
-      for (int r = lane; r < HT; r += 32) m_run[r] = -INFINITY;
-    named_bar_sync(4, LA_GROUP);
-    if (tid < HT) {
-      const float ma = m_run[tid], mb = m_run[HT + tid], mx = fmaxf(ma, mb);
+    if (tiles <= sub && v == 0 && lane < LA_ROWS) m_run[sub * LA_ROWS + lane] = -INFINITY;
+    named_bar_sync(LA_BAR_SUM, LA_GROUP);
+    if (tid < LA_ROWS) {
+      const float ma = m_run[tid], mb = m_run[LA_ROWS + tid], mx = fmaxf(ma, mb);
       const float z = mx == -INFINITY ? 0.f : mx;
       float l = 0.f;
 #pragma unroll
       for (int w = 0; w < 8; ++w)
-        l += l_warp[w * HT + tid] * fast_exp2((w < 4 ? ma : mb) - z);
+        l += l_warp[w * LA_ROWS + tid] * fast_exp2((w < 4 ? ma : mb) - z);
       inv_l[tid] = l > 0.f ? 1.0f / l : 0.f;
       if (p.splits > 1 && tid < n_rows)
         p.ml[(int64_t)split * p.flat_rows + first + tid] = make_float2(mx, l);
     }
-    named_bar_sync(3, 2 * LA_GROUP);
+    named_bar_sync(LA_BAR_END, 2 * LA_GROUP);
     return;
   }
 
   // -------------------------------- values ---------------------------------
-  float acc[MTS][RN][4];
+  // The ring: tile n comes into slot n % ring.  When the weights of tile n have been handed
+  // over, every warp here is through with tile n - 1: its slot takes the next tile.
+  const int32_t* bt = p.block_tables + seq * p.bt_stride;
+  // row of the pool where the run of keys from `key` on begins; out of range: zeros
+  auto pool_row = [&](int key) {
+    const int none = p.num_blocks * p.block_size;
+    if (key >= k_end) return none;
+    const int page = bt[key / p.block_size];
+    if (page >= 0 && page < p.num_blocks) return page * p.block_size + key % p.block_size;
+    if (p.status) atomicOr(p.status, FK_DEV_BAD_PAGE);
+    return none;
+  };
+  auto issue = [&](int n, int slot, int first_row) {
+    mbar_arrive_expect_tx(&full[slot], (uint32_t)tile_bytes);
+    uint8_t* dst = K + slot * tile_bytes;
+    if (p.run == LA_KEYS) {
+      tma_load_3d(dst, &tmap, &full[slot], 0, first_row, 0);    // the whole tile
+    } else {
+      // runs of p.run keys lie in one page; blocks of 64 channels one by one
+      for (int r = 0; r < LA_KEYS; r += p.run) {
+        const int row = r == 0 ? first_row : pool_row(k_begin + n * LA_KEYS + r);
+        for (int c = 0; c < tile_bytes / LA_BLOCK; ++c)
+          tma_load_3d(dst + c * LA_BLOCK + r * 128, &tmap, &full[slot], 0, row, c);
+      }
+    }
+  };
+  const bool feeds = warp == LA_GROUP / 32 && lane == 0;
+  int next_row = 0;                       // of tile n - 1 + ring, looked up ahead
+  if (feeds) {
+    for (int n = 0; n < min(tiles, p.ring); ++n) issue(n, n, pool_row(k_begin + n * LA_KEYS));
+    if (tiles > p.ring) next_row = pool_row(k_begin + p.ring * LA_KEYS);
+  }
+  __syncwarp();
+  float acc[RN][4];
 #pragma unroll
-  for (int a = 0; a < MTS; ++a)
+  for (int j = 0; j < RN; ++j)
 #pragma unroll
-    for (int j = 0; j < RN; ++j)
-#pragma unroll
-      for (int i = 0; i < 4; ++i) acc[a][j][i] = 0.f;
+    for (int i = 0; i < 4; ++i) acc[j][i] = 0.f;
   const int col0 = (warp - LA_GROUP / 32) * RN * 8;
+  uint32_t at[RN / 2];                    // this lane's fragment addresses inside a tile
+#pragma unroll
+  for (int j = 0; j < RN / 2; ++j) {
+    // columns beyond the latent are not stored: any column of the row will do
+    const int c = min(col0 + j * 16, p.lo - 16);
+    at[j] = (lane & 15) * 128 + (c >> 6) * LA_BLOCK + ((((c >> 3) & 7) + (lane >> 4)) ^ sw) * 16;
+  }
+  const uint32_t pa = smem_u32(P + (lane & 15) * LA_PPITCH + (lane >> 4) * 8);
+  int st = 0;
   for (int n = 0; n < tiles; ++n) {
-    const int buf = n & 1, st = n % p.ring;
-    ok = ok && mbar_wait(&full[st], (uint32_t)(n / p.ring) & 1u, LA_WAIT_LIMIT);
-    ok = ok && mbar_wait(&p_full[buf], (uint32_t)(n >> 1) & 1u, LA_WAIT_LIMIT);
-    const uint32_t tile = smem_u32(K + st * tile_bytes) + (lane & 15) * 128;
-    const uint16_t* Ph = P + buf * 2 * HT * LA_PPITCH;
-    const uint16_t* Pl = Ph + HT * LA_PPITCH;
-    if (col0 < p.lo) {
-#pragma unroll
-      for (int a = 0; a < MTS; ++a) {
-        const float a0 = alpha[buf * HT + a * 16 + gr], a1 = alpha[buf * HT + a * 16 + gr + 8];
-        if (__any_sync(0xffffffffu, a0 != 1.f || a1 != 1.f)) {
-#pragma unroll
-          for (int j = 0; j < RN; ++j) {
-            acc[a][j][0] *= a0; acc[a][j][1] *= a0;
-            acc[a][j][2] *= a1; acc[a][j][3] *= a1;
-          }
-        }
-      }
-#pragma unroll
-      for (int kt = 0; kt < LA_KEYS / 16; ++kt) {
-        uint32_t ph[MTS][4], pl[MTS][4];
-#pragma unroll
-        for (int a = 0; a < MTS; ++a) {
-          const uint32_t off = (a * 16 + (lane & 15)) * LA_PPITCH + kt * 16 + (lane >> 4) * 8;
-          ldmatrix_x4(smem_u32(Ph + off), ph[a][0], ph[a][1], ph[a][2], ph[a][3]);
-          ldmatrix_x4(smem_u32(Pl + off), pl[a][0], pl[a][1], pl[a][2], pl[a][3]);
-        }
-        constexpr int GRP = RN / 2 < 4 / MTS ? RN / 2 : 4 / MTS;   // 16-column groups at a time
-#pragma unroll
-        for (int j0 = 0; j0 < RN / 2; j0 += GRP) {
-          uint32_t b[GRP][4];
-#pragma unroll
-          for (int j = 0; j < GRP; ++j) {
-            // columns beyond the latent are not stored: any column of the row will do
-            const int c = min(col0 + (j0 + j) * 16, p.lo - 16);
-            ldmatrix_x4_trans(tile + kt * 16 * 128 + (c >> 6) * LA_BLOCK +
-                                  ((((c >> 3) & 7) + (lane >> 4)) ^ sw) * 16,
-                              b[j][0], b[j][1], b[j][2], b[j][3]);
-          }
-#pragma unroll
-          for (int part = 0; part < 2; ++part)
-#pragma unroll
-            for (int a = 0; a < MTS; ++a)
-#pragma unroll
-              for (int j = 0; j < GRP; ++j) {
-                mma_bf16_16816(acc[a][2 * (j0 + j)], part ? pl[a] : ph[a], b[j][0], b[j][1]);
-                mma_bf16_16816(acc[a][2 * (j0 + j) + 1], part ? pl[a] : ph[a], b[j][2], b[j][3]);
-              }
-        }
-      }
+    const int buf = n & 1;
+    const uint32_t tile = smem_u32(K) + st * tile_bytes;
+    named_bar_sync(LA_BAR_FULL + buf, 128 + LA_GROUP);
+    if (feeds && n > 0 && n - 1 + p.ring < tiles) {
+      issue(n - 1 + p.ring, st == 0 ? p.ring - 1 : st - 1, next_row);
+      if (n + p.ring < tiles) next_row = pool_row(k_begin + (n + p.ring) * LA_KEYS);
     }
     __syncwarp();
-    if (lane == 0) {
-      mbar_arrive(&empty[st]);
-      mbar_arrive(&p_empty[buf]);
-    }
-  }
-  named_bar_sync(3, 2 * LA_GROUP);
-  if (p.splits > 1 && tiles == 0) return;
+    if (col0 < p.lo) {
+      uint32_t ph[2][4], pl[2][4], b[2][RN / 2][4];
+      const uint32_t pb = pa + buf * 2 * LA_ROWS * LA_PPITCH * 2;
 #pragma unroll
-  for (int a = 0; a < MTS; ++a)
+      for (int kt = 0; kt < 2; ++kt) {
+        ldmatrix_x4(pb + kt * 32, ph[kt][0], ph[kt][1], ph[kt][2], ph[kt][3]);
+        ldmatrix_x4(pb + kt * 32 + LA_ROWS * LA_PPITCH * 2, pl[kt][0], pl[kt][1], pl[kt][2],
+                    pl[kt][3]);
 #pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int r = a * 16 + gr + e * 8;
-      if (r >= n_rows) continue;
-      if (p.splits > 1) {
-        float* o = p.part + ((int64_t)split * p.flat_rows + first + r) * p.lo;
-#pragma unroll
-        for (int j = 0; j < RN; ++j) {
-          const int c = col0 + j * 8 + tq * 2;
-          if (c < p.lo)
-            *reinterpret_cast<float2*>(o + c) = make_float2(acc[a][j][e * 2], acc[a][j][e * 2 + 1]);
-        }
-      } else {
-        const float inv = inv_l[r];
-        uint16_t* o = p.out + (first + r) * p.out_pitch;
+        for (int j = 0; j < RN / 2; ++j)
+          ldmatrix_x4_trans(tile + kt * 16 * 128 + at[j], b[kt][j][0], b[kt][j][1], b[kt][j][2],
+                            b[kt][j][3]);
+      }
+      const float a0 = alpha[buf * LA_ROWS + row0], a1 = alpha[buf * LA_ROWS + row1];
+      if (__any_sync(0xffffffffu, a0 != 1.f || a1 != 1.f)) {
 #pragma unroll
         for (int j = 0; j < RN; ++j) {
-          const int c = col0 + j * 8 + tq * 2;
-          if (c < p.lo)
-            *reinterpret_cast<uint32_t*>(o + c) =
-                pack_bf16(acc[a][j][e * 2] * inv, acc[a][j][e * 2 + 1] * inv);
+          acc[j][0] *= a0; acc[j][1] *= a0;
+          acc[j][2] *= a1; acc[j][3] *= a1;
         }
       }
+#pragma unroll
+      for (int kt = 0; kt < 2; ++kt)
+#pragma unroll
+        for (int part = 0; part < 2; ++part)
+#pragma unroll
+          for (int j = 0; j < RN / 2; ++j) {
+            mma_bf16_16816(acc[2 * j], part ? pl[kt] : ph[kt], b[kt][j][0], b[kt][j][1]);
+            mma_bf16_16816(acc[2 * j + 1], part ? pl[kt] : ph[kt], b[kt][j][2], b[kt][j][3]);
+          }
     }
+    if (n + 2 < tiles) named_bar_arrive(LA_BAR_EMPTY + buf, 128 + LA_GROUP);
+    if (++st == p.ring) st = 0;
+  }
+  named_bar_sync(LA_BAR_END, 2 * LA_GROUP);
+  if (p.splits > 1 && tiles == 0) return;
+#pragma unroll
+  for (int e = 0; e < 2; ++e) {
+    const int r = gr + e * 8;
+    if (r >= n_rows) continue;
+    if (p.splits > 1) {
+      float* o = p.part + ((int64_t)split * p.flat_rows + first + r) * p.lo;
+#pragma unroll
+      for (int j = 0; j < RN; ++j) {
+        const int c = col0 + j * 8 + tq * 2;
+        if (c < p.lo)
+          *reinterpret_cast<float2*>(o + c) = make_float2(acc[j][e * 2], acc[j][e * 2 + 1]);
+      }
+    } else {
+      const float inv = inv_l[r];
+      uint16_t* o = p.out + (first + r) * p.out_pitch;
+#pragma unroll
+      for (int j = 0; j < RN; ++j) {
+        const int c = col0 + j * 8 + tq * 2;
+        if (c < p.lo)
+          *reinterpret_cast<uint32_t*>(o + c) =
+              pack_bf16(acc[j][e * 2] * inv, acc[j][e * 2 + 1] * inv);
+      }
+    }
+  }
 }
 
 // One CTA per (token, head) row; at most 32 ranges, a lane each.
@@ -645,49 +624,52 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentAttnParam
   }
 }
 
-// [rows, channels] bf16 pool: box = 64 channels x `run` rows, 128B swizzle
-static int la_map(const void* ptr, int64_t rows, int64_t cols, int run, CUtensorMap* out) {
-  struct Entry { const void* ptr; int64_t rows, cols; int run; CUtensorMap map; };
+// [rows, channels] bf16 pool as (64 channels, rows, blocks of 64 channels): box = `run` rows
+// of `blocks` blocks, 128B swizzle
+static int la_map(const void* ptr, int64_t rows, int64_t cols, int run, int blocks,
+                  CUtensorMap* out) {
+  struct Entry { const void* ptr; int64_t rows, cols; int run, blocks; CUtensorMap map; };
   static std::mutex mu;
   static std::vector<Entry> maps;
   std::lock_guard<std::mutex> lk(mu);
   for (const Entry& e : maps)
-    if (e.ptr == ptr && e.rows == rows && e.cols == cols && e.run == run) {
+    if (e.ptr == ptr && e.rows == rows && e.cols == cols && e.run == run &&
+        e.blocks == blocks) {
       *out = e.map;
       return FK_OK;
     }
   tensormap_encode_fn enc = get_tensormap_encode();
   FK_REQUIRE(enc != nullptr, FK_ERR_CUDA,
              "cuTensorMapEncodeTiled not available from the driver");
-  cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
-  cuuint64_t strides[1] = {(cuuint64_t)cols * 2};
-  cuuint32_t box[2] = {64, (cuuint32_t)run};
-  cuuint32_t estr[2] = {1, 1};
-  CUresult r = enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(ptr), dims,
+  cuuint64_t dims[3] = {64, (cuuint64_t)rows, (cuuint64_t)(cols / 64)};
+  cuuint64_t strides[2] = {(cuuint64_t)cols * 2, 128};
+  cuuint32_t box[3] = {64, (cuuint32_t)run, (cuuint32_t)blocks};
+  cuuint32_t estr[3] = {1, 1, 1};
+  CUresult r = enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(ptr), dims,
                    strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
                    CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
                    CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
   FK_REQUIRE(r == CUDA_SUCCESS, FK_ERR_CUDA, "cuTensorMapEncodeTiled failed with code %d",
              (int)r);
   if (maps.size() > 1024) maps.clear();
-  maps.push_back({ptr, rows, cols, run, *out});
+  maps.push_back({ptr, rows, cols, run, blocks, *out});
   return FK_OK;
 }
 
-template <int HT, int RN>
+template <int RN>
 static int launch_latent(LatentAttnParams& p, dim3 grid, cudaStream_t s) {
-  p.ring = la_ring(HT, p.lk);
-  FK_REQUIRE(p.ring > 0, FK_ERR_UNSUPPORTED, "fk_latent_attn: rows of %d elements", p.lk);
-  const int smem = la_smem(HT, p.lk, p.ring);
+  p.ring = la_ring(p.lk);
+  const int smem = la_smem(p.lk, p.ring);
   static PerDeviceOnce once;
-  FK_CUDA_OK(set_max_dynamic_smem(once, latent_attn_kernel<HT, RN>, 232448));
+  FK_CUDA_OK(set_max_dynamic_smem(once, latent_attn_kernel<RN>, 232448));
   p.run = LA_KEYS;                       // keys that surely lie in one page
   while (p.block_size % p.run) p.run /= 2;
   CUtensorMap map;
-  const int rc = la_map(p.cache, (int64_t)p.num_blocks * p.block_size, p.cache_pitch, p.run, &map);
+  const int rc = la_map(p.cache, (int64_t)p.num_blocks * p.block_size, p.cache_pitch, p.run,
+                        p.run == LA_KEYS ? (p.lk + 63) / 64 : 1, &map);
   if (rc != FK_OK) return rc;
-  FK_CUDA_OK(launch_kernel(latent_attn_kernel<HT, RN>, grid, dim3(LA_THREADS), (size_t)smem, s,
-                           map, p));
+  FK_CUDA_OK(launch_kernel(latent_attn_kernel<RN>, grid, dim3(LA_THREADS), (size_t)smem, s, map,
+                           p));
   count_launch();
   return FK_OK;
 }
@@ -757,15 +739,15 @@ int fk_latent_gather(const void* cache, int64_t row_bytes, int64_t num_blocks, i
   return FK_OK;
 }
 
-int fk_latent_attn_supported(int heads, int rank, int rot) {
-  return heads > 0 && rank > 0 && rank <= 512 && rot >= 0 &&
-         la_ring(heads <= 16 ? 16 : 32, (rank + rot + 15) / 16 * 16) > 0;
+int fk_latent_attn_supported(int rank, int rot) {
+  const int lk = (rank + rot + 15) / 16 * 16;
+  return rank > 0 && rank <= 512 && rot >= 0 && lk / 16 <= 4 * la_steps(la_rn(rank)) &&
+         la_ring(lk) > 0;
 }
 
 /* Key ranges a call with these sizes splits its rows into. */
 int fk_latent_attn_splits(int num_seqs, int64_t max_q, int heads, int64_t max_keys) {
-  const int ht = heads <= 16 ? 16 : 32;
-  const int64_t tiles = (max_q * heads + ht - 1) / ht * num_seqs;
+  const int64_t tiles = (max_q * heads + LA_ROWS - 1) / LA_ROWS * num_seqs;
   if (tiles <= 0) return 1;
   int64_t s = (int64_t)sm_count() / tiles;
   const int64_t most = (max_keys + 127) / 128;
@@ -790,9 +772,11 @@ int fk_latent_attn(const void* q, int64_t q_pitch, const void* cache, int64_t nu
   if (rows == 0 || num_seqs == 0 || max_seqlen_q <= 0) return FK_OK;
   FK_REQUIRE(q && cache && out && cu_seqlens_q && kv_lens && block_tables, FK_ERR_INVALID_ARG,
              "fk_latent_attn: null pointer");
-  FK_REQUIRE(fk_latent_attn_supported(heads, rank, rot), FK_ERR_UNSUPPORTED,
+  FK_REQUIRE(fk_latent_attn_supported(rank, rot), FK_ERR_UNSUPPORTED,
              "fk_latent_attn: rank %d with %d rotated channels", rank, rot);
   const int lk = (rank + rot + 15) / 16 * 16, lo = (rank + 15) / 16 * 16;
+  FK_REQUIRE(cache_pitch % 64 == 0, FK_ERR_UNSUPPORTED,
+             "fk_latent_attn: cached rows of %d elements, not a multiple of 64", cache_pitch);
   FK_REQUIRE(cache_pitch >= lk && q_pitch >= lk && out_pitch >= lo && block_size > 0 &&
                  num_blocks > 0 && num_blocks * block_size < (1ll << 31),
              FK_ERR_INVALID_ARG, "fk_latent_attn: rows shorter than latent and rotated key, "
@@ -817,20 +801,14 @@ int fk_latent_attn(const void* q, int64_t q_pitch, const void* cache, int64_t nu
   p.bt_stride = block_table_stride; p.heads = heads; p.lk = lk; p.lo = lo;
   p.block_size = block_size; p.num_blocks = (int)num_blocks; p.splits = splits;
   p.scale_log2 = softmax_scale * 1.4426950408889634f; p.status = status;
-  const int ht = heads <= 16 ? 16 : 32;
-  const int64_t tiles = (max_seqlen_q * heads + ht - 1) / ht;
-  FK_REQUIRE(tiles <= 0x7fffffff && num_seqs <= 65535 && splits <= 65535 &&
-                 p.flat_rows <= 0x7fffffff,
+  const int64_t tiles = (max_seqlen_q * heads + LA_ROWS - 1) / LA_ROWS;
+  FK_REQUIRE(tiles <= 0x7fffffff && num_seqs <= 65535 && p.flat_rows <= 0x7fffffff,
              FK_ERR_UNSUPPORTED, "fk_latent_attn: too many rows");
   const dim3 grid((unsigned)tiles, (unsigned)num_seqs, (unsigned)splits);
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  int rc;
-  if (ht == 16)
-    rc = rank <= 128 ? launch_latent<16, 2>(p, grid, s)
-         : rank <= 256 ? launch_latent<16, 4>(p, grid, s) : launch_latent<16, 8>(p, grid, s);
-  else
-    rc = rank <= 128 ? launch_latent<32, 2>(p, grid, s)
-         : rank <= 256 ? launch_latent<32, 4>(p, grid, s) : launch_latent<32, 8>(p, grid, s);
+  const int rn = la_rn(rank);
+  const int rc = rn == 2 ? launch_latent<2>(p, grid, s)
+                 : rn == 4 ? launch_latent<4>(p, grid, s) : launch_latent<8>(p, grid, s);
   if (rc != FK_OK || splits == 1) return rc;
   FK_CUDA_OK(launch_kernel(latent_merge_kernel, dim3((unsigned)p.flat_rows), dim3(128), 0, s, p));
   count_launch();

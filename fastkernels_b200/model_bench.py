@@ -121,14 +121,28 @@ def time_prefill(eng, n, length, iters=5):
 
 
 def time_decode(eng, batch, steps=32):
+    """Every step's tokens are drawn anew: random weights would soon sample one and the
+    same token in all sequences, and so visit few experts."""
+    rs = np.random.RandomState(batch)
     eng.add_sequences([CONTEXT] * batch, list(range(batch)))
+
+    def step():
+        for s, t in zip(eng.seqs, rs.randint(0, VOCAB, size=batch).tolist()):
+            s.last_token = t
+        n = eng.prepare_decode(use_host_ids=True)
+        bs = eng.graph_batch_size(n)
+        eng.stage_inputs(n, bs, True)
+        eng.run_step_device(bs)
+        eng._mark_slot_in_flight()
+        for s in eng.seqs:
+            s.num_tokens += 1
     for _ in range(4):
-        eng.step(sync=False)
+        step()
     torch.cuda.synchronize()
     a, b = _events()
     a.record()
     for _ in range(steps):
-        eng.step(sync=False)
+        step()
     b.record()
     torch.cuda.synchronize()
     for s in list(eng.seqs):
@@ -292,7 +306,7 @@ def kernel_table(eng, n, length):
     rs = np.random.RandomState(7)
     if length > 1:
         prompts = [rs.randint(0, VOCAB, size=length).tolist() for _ in range(n)]
-        for timed in (False, True):
+        for timed in (False, False, True):
             seqs = [eng.open_sequence() for _ in range(n)]
             if timed:
                 preload()
@@ -304,11 +318,13 @@ def kernel_table(eng, n, length):
                     eng.finish(s)
                 torch.cuda.synchronize()
     else:
-        eng.add_sequences([CONTEXT] * n, list(range(n)))
+        eng.add_sequences([CONTEXT] * n, rs.randint(0, VOCAB, size=n).tolist())
         eng.prepare_decode(True)
         eng.stage_inputs(n, n, True)
         eng.enforce_eager = True
-        eng.run_step_device(n)
+        for _ in range(2):           # kernels and allocations in place
+            eng.run_step_device(n)
+        eng.stage_inputs(n, n, True)
         torch.cuda.synchronize()
         preload()
         with OpTimer() as t:

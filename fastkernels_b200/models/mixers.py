@@ -200,7 +200,7 @@ class LatentAttention:
         self.v_pitch = round_up(vdim, 8)
         self.out_columns = round_up(heads * self.v_pitch, 64)
         self.sections = {"q": heads * self.q_pitch, "dkv": rank + rot}
-        self.tensor_cores = dtype == torch.bfloat16 and ops.latent_attn_supported(heads, rank, rot)
+        self.tensor_cores = dtype == torch.bfloat16 and ops.latent_attn_supported(rank, rot)
         self.expandable = dtype == torch.bfloat16 and dim + rot <= 128 and vdim <= 128
         self.caches = []
         self.cos_sin = self.status = None

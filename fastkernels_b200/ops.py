@@ -1007,9 +1007,9 @@ def latent_gather(cache, block_tables, cu_seqlens_k, rows, status=None):
     return out
 
 
-def latent_attn_supported(heads: int, rank: int, rot: int) -> bool:
-    """True when fk_latent_attn takes heads over rows of rank + rot channels."""
-    return bool(lib.fk_latent_attn_supported(heads, rank, rot))
+def latent_attn_supported(rank: int, rot: int) -> bool:
+    """True when fk_latent_attn takes rows of rank + rot channels."""
+    return bool(lib.fk_latent_attn_supported(rank, rot))
 
 
 def latent_attn(q, cache, cu_seqlens_q, kv_lens, block_tables, max_seqlen_q, max_keys, rank, rot,

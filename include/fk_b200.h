@@ -781,7 +781,7 @@ int fk_latent_gather(const void* cache, int64_t row_bytes, int64_t num_blocks, i
                      const int32_t* block_tables, int64_t block_table_stride,
                      const int32_t* cu_seqlens_k, int num_seqs, void* out, int64_t rows,
                      int32_t* status, fk_stream_t stream);
-int fk_latent_attn_supported(int heads, int rank, int rot);
+int fk_latent_attn_supported(int rank, int rot);
 int fk_latent_attn_splits(int num_seqs, int64_t max_q, int heads, int64_t max_keys);
 int64_t fk_latent_attn_workspace_floats(int64_t rows, int heads, int rank, int splits);
 int fk_latent_attn(const void* q, int64_t q_pitch, const void* cache, int64_t num_blocks,
