@@ -164,6 +164,8 @@ __global__ void __launch_bounds__(256) group_skinny_kernel(const GroupParams p, 
   group_range(p, g, &first, &count);
   const uint16_t* x = static_cast<const uint16_t*>(p.x) + (p.offsets ? 0 : g * p.x_group);
   const int chunks = (p.k + 31) >> 5;
+  constexpr int kUnit = 16 / (int)sizeof(OUT);
+  const bool vec = p.y_stride % kUnit == 0 && p.y_group % kUnit == 0;
   for (int64_t t0 = (int64_t)blockIdx.z * COLS; t0 < count; t0 += (int64_t)gridDim.z * COLS) {
     const uint16_t* xr[NT];
     bool on[NT];
@@ -224,32 +226,62 @@ __global__ void __launch_bounds__(256) group_skinny_kernel(const GroupParams p, 
     OUT* y = static_cast<OUT*>(p.y) + (p.offsets ? 0 : g * p.y_group);
     const int lg = 4 + (fs > 1) + (fs > 2), feats = 16 * fs;     // fs: 1, 2 or 4
     const int live = (int)min((int64_t)COLS, count - t0);
-    for (int i = threadIdx.x; i < feats * live; i += blockDim.x) {
-      const int r = i & (feats - 1), t = i >> lg;
+    // one output of row r, column t of this CTA's block
+    auto value = [&](int r, int t) {
       const int c = n0 + r;
-      if (c >= p.n) continue;
       const float* part = gs_red + (r >> 4) * ks * (TILES * 16 * PITCH) + (r & 15) * PITCH + t;
-      float v = p.bias ? p.bias[c] : 0.f, up = 0.f;
+      float v = p.bias && c < p.n ? p.bias[c] : 0.f, up = 0.f;
       for (int q = 0; q < ks; ++q) {
         v += part[q * (TILES * 16 * PITCH)];
         if (ACT) up += part[q * (TILES * 16 * PITCH) + 16 * PITCH];
       }
-      if (ACT) v = group_act(v, p.act) * up;
-      Elem<OUT>::store(y + (first + t0 + t) * p.y_stride + c, v);
+      return ACT ? group_act(v, p.act) * up : v;
+    };
+    // enough outputs for all threads: VEC features each, 16 bytes
+    constexpr int VEC = 16 / (int)sizeof(OUT);
+    const int step = vec && feats * live >= (int)blockDim.x * VEC ? VEC : 1;
+    for (int i = threadIdx.x * step; i < feats * live; i += blockDim.x * step) {
+      const int r = i & (feats - 1), t = i >> lg;
+      const int c = n0 + r;
+      if (c >= p.n) continue;
+      OUT* dst = y + (first + t0 + t) * p.y_stride + c;
+      if (step == 1) {
+        Elem<OUT>::store(dst, value(r, t));
+        continue;
+      }
+      float v[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v[e] = value(r + e, t);
+      if (c + VEC <= p.n) {
+        if (sizeof(OUT) == 2)
+          *reinterpret_cast<uint4*>(dst) =
+              make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]),
+                         pack_bf16(v[VEC > 4 ? 4 : 0], v[VEC > 4 ? 5 : 1]),
+                         pack_bf16(v[VEC > 4 ? 6 : 2], v[VEC > 4 ? 7 : 3]));
+        else
+          *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[1], v[2], v[3]);
+      } else {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e)
+          if (c + e < p.n) Elem<OUT>::store(dst + e, v[e]);
+      }
     }
   }
 }
 
 // ------------------------------------------------------------------------ many rows
-// BN weight rows a tile: 256, or 32 for narrow products (more stages of the rows' stream).
+// BN weight rows a tile: 256, or 32 for narrow products, which have only 64 rows a tile (the
+// instruction still multiplies 128; the others are not loaded and their results not kept).
 constexpr int GG_BM = 128, GG_BK = 64;
 constexpr int GG_A_BYTES = GG_BM * GG_BK * 2;
 constexpr int GG_MAX_GROUPS = 1024;
 constexpr int GG_THREADS = 192;
 template <int BN>
 struct GgCfg {
+  static constexpr int kRows = BN == 256 ? 128 : 64;
   static constexpr int kBBytes = BN * GG_BK * 2;
   static constexpr int kStageBytes = GG_A_BYTES + kBBytes;
+  static constexpr int kLoadBytes = kRows * GG_BK * 2 + kBBytes;
   static constexpr int kStages = BN == 256 ? 4 : 9;
   static constexpr int kOffTiles = kStages * kStageBytes;      // first tile of every group
   static constexpr int kOffBar = kOffTiles + (GG_MAX_GROUPS + 8) * 4;
@@ -288,6 +320,7 @@ struct GgTile {
 };
 
 // Tiles of a group lie together, rows fastest.
+template <int ROWS>
 __device__ __forceinline__ GgTile gg_tile(const GroupParams& p, const int* first_tile, int ti,
                                           int n_tiles) {
   int lo = 0, hi = p.groups;
@@ -303,7 +336,7 @@ __device__ __forceinline__ GgTile gg_tile(const GroupParams& p, const int* first
   t.nt = in_g / mts;
   int64_t a = 0, b = p.rows;
   if (p.offsets) { a = p.offsets[lo]; b = p.offsets[lo + 1]; }
-  t.row0 = a + (int64_t)mt * GG_BM;
+  t.row0 = a + (int64_t)mt * ROWS;
   t.rows_left = b - t.row0;
   return t;
 }
@@ -365,7 +398,7 @@ group_large_kernel(const __grid_constant__ CUtensorMap tmap_x,
           c = p.rows;
         }
       }
-      const int mine = (int)((c + GG_BM - 1) / GG_BM) * n_tiles;
+      const int mine = (int)((c + Cfg::kRows - 1) / Cfg::kRows) * n_tiles;
       int run = mine;
 #pragma unroll
       for (int o = 1; o < 32; o <<= 1) {
@@ -395,13 +428,13 @@ group_large_kernel(const __grid_constant__ CUtensorMap tmap_x,
       uint32_t phase = 0;
       bool ok = true;
       for (int ti = blockIdx.x; ti < total && ok; ti += gridDim.x) {
-        const GgTile t = gg_tile(p, first_tile, ti, n_tiles);
+        const GgTile t = gg_tile<Cfg::kRows>(p, first_tile, ti, n_tiles);
         const int xc = p.offsets ? 0 : (int)(t.g * p.x_group);
         const int wrow = (int)(t.g * p.w_rows) + t.nt * TN;
         for (int kb = 0; kb < kb_total; ++kb) {
           if (!gg_wait(&empty[stage], phase ^ 1, abort_flag, p.status)) { ok = false; break; }
           uint8_t* dst = smem + stage * Cfg::kStageBytes;
-          mbar_arrive_expect_tx(&full[stage], (uint32_t)Cfg::kStageBytes);
+          mbar_arrive_expect_tx(&full[stage], (uint32_t)Cfg::kLoadBytes);
           tma_load_2d(dst, &tmap_x, &full[stage], xc + kb * GG_BK, (int)t.row0);
           if (ACT) {
             tma_load_2d(dst + GG_A_BYTES, &tmap_w, &full[stage], kb * GG_BK, wrow);
@@ -447,11 +480,11 @@ group_large_kernel(const __grid_constant__ CUtensorMap tmap_x,
     const uint32_t lane_addr = (uint32_t)(q * 32) << 16;
     uint32_t done = 0;
     for (int ti = blockIdx.x; ti < total; ti += gridDim.x) {
-      const GgTile t = gg_tile(p, first_tile, ti, n_tiles);
+      const GgTile t = gg_tile<Cfg::kRows>(p, first_tile, ti, n_tiles);
       const uint32_t buf = done & 1u, use = done >> 1;
       if (!gg_wait(&acc_full[buf], use & 1u, abort_flag, p.status)) break;
       tc_fence_after();
-      const bool live = row < t.rows_left;
+      const bool live = row < Cfg::kRows && row < t.rows_left;
       OUT* y = static_cast<OUT*>(p.y) + (p.offsets ? 0 : t.g * p.y_group) +
                (t.row0 + (live ? row : 0)) * p.y_stride;
       const int n0 = t.nt * TN;
@@ -590,12 +623,13 @@ template <int BN, bool ACT, typename OUT>
 static int launch_large_one(const GroupParams& p, int64_t x_cols, cudaStream_t s) {
   constexpr int TN = ACT ? BN / 2 : BN;
   const int64_t n_tiles = (p.n + TN - 1) / TN;
-  const int64_t bound = p.offsets ? ((p.rows + GG_BM - 1) / GG_BM + p.groups) * n_tiles
-                                  : (p.rows + GG_BM - 1) / GG_BM * n_tiles * p.groups;
+  constexpr int kRows = GgCfg<BN>::kRows;
+  const int64_t bound = p.offsets ? ((p.rows + kRows - 1) / kRows + p.groups) * n_tiles
+                                  : (p.rows + kRows - 1) / kRows * n_tiles * p.groups;
   FK_REQUIRE(bound <= 0x7fffffff && p.rows < (1ll << 31) && p.groups * p.w_rows < (1ll << 31),
              FK_ERR_UNSUPPORTED, "fk_group_gemm: too many tiles");
   CUtensorMap mx, mw;
-  int rc = gg_map(p.x, p.x_rows, x_cols, p.x_stride, GG_BM, &mx);
+  int rc = gg_map(p.x, p.x_rows, x_cols, p.x_stride, kRows, &mx);
   if (rc != FK_OK) return rc;
   rc = gg_map(p.w, p.groups * p.w_rows, p.k, p.k, TN, &mw);
   if (rc != FK_OK) return rc;

@@ -8,7 +8,7 @@
 //   mlstm_step_kernel     one token per sequence: state streamed once, head norm and
 //                         output gate applied on the way out
 //   mlstm_scan_kernel     portions, token by token, any size, bf16 or fp32
-//   chunked form (bf16)   blocks ("units") of 64 tokens of a portion.  With g_t the sum of
+//   chunked form (bf16)   blocks ("units") of 128 tokens of a portion.  With g_t the sum of
 //                         f inside the unit up to t and S, n, m the values ahead of it,
 //     m_t   = max(g_t + m, max_{s <= t} g_t - g_s + i_s)
 //     num_t = e^{g_t + m - m_t} S^T q_t + sum_{s <= t} e^{g_t - g_s + i_s - m_t} (q_t . k_s) v_s
@@ -25,7 +25,7 @@
 
 namespace fk {
 
-constexpr int ML_UNIT = 64;
+constexpr int ML_UNIT = 128;
 constexpr float ML_EPS = 1e-6f;
 constexpr float ML_NONE = -1e30f;     // log gate of a token that is not there
 
@@ -44,7 +44,7 @@ struct MlstmParams {
   void* out; int64_t out_stride;
   // portions
   float* o;                                    // [rows, heads * vdim]
-  float* gg; float* gi; float* gm;             // [heads][units * 64]: g, i, m
+  float* gg; float* gi; float* gm;             // [heads][units * ML_UNIT]: g, i, m
   float* unit_m; float* unit_decay;            // [heads][units]
   float* inc;                                  // [units][heads][dim][vp]
   float* ninc;                                 // [units][heads][dim]
@@ -263,7 +263,7 @@ __global__ void __launch_bounds__(128) mlstm_scan_norm_kernel(const MlstmParams 
 }
 
 // ------------------------------------------------------------------------ chunked form
-// Portion that owns unit u (units cu[i] / 64 + i .. of portion i); its token range.
+// Portion that owns unit u (units cu[i] / ML_UNIT + i .. of portion i); its token range.
 struct MlUnit {
   int portion;
   int64_t t0;       // first token
@@ -288,9 +288,9 @@ __device__ __forceinline__ MlUnit ml_unit(const MlstmParams& p, int64_t u) {
   return r;
 }
 
-// CTA = one head of one portion; each warp takes units in turn, two tokens a lane.
-constexpr int MG_THREADS = 512;
-constexpr int MG_MAX_UNITS = 4096;            // per portion (262144 tokens)
+// CTA = one head of one portion; each warp takes units in turn, some tokens a lane.
+constexpr int MG_THREADS = 1024, MG_TPL = ML_UNIT / 32;
+constexpr int MG_MAX_UNITS = 4096;            // per portion (524288 tokens)
 __global__ void __launch_bounds__(MG_THREADS) mlstm_gates_kernel(const MlstmParams p) {
   extern __shared__ float mg_smem[];          // per unit: sum of f, local maximum, m ahead
   pdl_launch_dependents();
@@ -310,16 +310,23 @@ __global__ void __launch_bounds__(MG_THREADS) mlstm_gates_kernel(const MlstmPara
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = MG_THREADS >> 5;
   const int64_t row_of = (int64_t)h * p.units * ML_UNIT;
   for (int u = warp; u < n_units; u += warps) {
-    float f[2], i[2];
+    float f[MG_TPL], i[MG_TPL], m[MG_TPL];
 #pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int64_t t = a + (int64_t)u * ML_UNIT + lane * 2 + e;
+    for (int e = 0; e < MG_TPL; ++e) {
+      const int64_t t = a + (int64_t)u * ML_UNIT + lane * MG_TPL + e;
       const bool on = t < b;
       i[e] = on ? ml_input_gate(p.z[t * p.z_stride + h], p.cap) : ML_NONE;
       f[e] = on ? ml_forget_gate(p.z[t * p.z_stride + p.heads + h], p.cap) : 0.f;
     }
-    // (sum of f, maximum of the decayed i) up to and with each token
-    float F = f[0] + f[1], M = fmaxf(i[0] + f[1], i[1]);
+    // (sum of f, maximum of the decayed i) up to and with each token: of this lane's tokens,
+    // then over the lanes
+    m[0] = i[0];
+#pragma unroll
+    for (int e = 1; e < MG_TPL; ++e) {
+      m[e] = fmaxf(m[e - 1] + f[e], i[e]);
+      f[e] += f[e - 1];
+    }
+    float F = f[MG_TPL - 1], M = m[MG_TPL - 1];
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
       const float pf = __shfl_up_sync(0xffffffffu, F, o), pm = __shfl_up_sync(0xffffffffu, M, o);
@@ -327,11 +334,13 @@ __global__ void __launch_bounds__(MG_THREADS) mlstm_gates_kernel(const MlstmPara
     }
     float pf = __shfl_up_sync(0xffffffffu, F, 1), pm = __shfl_up_sync(0xffffffffu, M, 1);
     if (lane == 0) { pf = 0.f; pm = ML_NONE; }
-    const int64_t at = row_of + (u0 + u) * ML_UNIT + lane * 2;
-    const float g0 = pf + f[0];
-    *reinterpret_cast<float2*>(p.gg + at) = make_float2(g0, F);
-    *reinterpret_cast<float2*>(p.gi + at) = make_float2(i[0], i[1]);
-    *reinterpret_cast<float2*>(p.gm + at) = make_float2(fmaxf(pm + f[0], i[0]), M);
+    const int64_t at = row_of + (u0 + u) * ML_UNIT + lane * MG_TPL;
+#pragma unroll
+    for (int e = 0; e < MG_TPL; ++e) {
+      p.gg[at + e] = pf + f[e];
+      p.gi[at + e] = i[e];
+      p.gm[at + e] = fmaxf(pm + f[e], m[e]);
+    }
     if (lane == 31) { tot_f[u] = F; tot_m[u] = M; }
   }
   __syncthreads();
@@ -362,16 +371,13 @@ __global__ void __launch_bounds__(MG_THREADS) mlstm_gates_kernel(const MlstmPara
   }
   __syncthreads();
   for (int u = warp; u < n_units; u += warps) {
-    const int64_t at = row_of + (u0 + u) * ML_UNIT + lane * 2;
-    const float2 g = *reinterpret_cast<const float2*>(p.gg + at);
-    float2 m = *reinterpret_cast<const float2*>(p.gm + at);
-    m.x = fmaxf(m.x, g.x + m_in[u]);
-    m.y = fmaxf(m.y, g.y + m_in[u]);
-    *reinterpret_cast<float2*>(p.gm + at) = m;
+    const int64_t at = row_of + (u0 + u) * ML_UNIT + lane * MG_TPL;
+#pragma unroll
+    for (int e = 0; e < MG_TPL; ++e) p.gm[at + e] = fmaxf(p.gm[at + e], p.gg[at + e] + m_in[u]);
   }
 }
 
-// Rows of a unit's q, k or v columns into shared memory [64][pitch], zeros beyond `count`
+// Rows of a unit's q, k or v columns into shared memory [ML_UNIT][pitch], zeros beyond `count`
 // rows and `cols` columns up to `cols_p`.
 __device__ __forceinline__ void ml_load_rows(const uint16_t* src, int64_t stride, int count,
                                              int cols, int cols_p, uint16_t* dst, int pitch,
@@ -399,16 +405,17 @@ __device__ __forceinline__ uint32_t ml_tile(const uint16_t* base, int pitch, int
   return smem_u32(base + (row + (lane & 15)) * pitch + col + (lane >> 4) * 8);
 }
 
-// acc[64 columns] += a (16 x 16) times rows row .. row + 15 of B; the fragments of B come
+// acc[8 NT columns] += a (16 x 16) times rows row .. row + 15 of B; the fragments of B come
 // ahead of the products.
-__device__ __forceinline__ void ml_products(float (&acc)[8][4], const uint32_t (&a)[4],
+template <int NT>
+__device__ __forceinline__ void ml_products(float (&acc)[NT][4], const uint32_t (&a)[4],
                                             const uint16_t* B, int pitch, int row, int lane) {
-  uint32_t b[4][4];
+  uint32_t b[NT / 2][4];
 #pragma unroll
-  for (int j = 0; j < 4; ++j)
+  for (int j = 0; j < NT / 2; ++j)
     ldmatrix_x4_trans(ml_tile(B, pitch, row, j * 16, lane), b[j][0], b[j][1], b[j][2], b[j][3]);
 #pragma unroll
-  for (int j = 0; j < 4; ++j) {
+  for (int j = 0; j < NT / 2; ++j) {
     mma_bf16_16816(acc[2 * j], a, b[j][0], b[j][1]);
     mma_bf16_16816(acc[2 * j + 1], a, b[j][2], b[j][3]);
   }
@@ -416,9 +423,9 @@ __device__ __forceinline__ void ml_products(float (&acc)[8][4], const uint32_t (
 
 // CTA = 64 value columns of one head of one unit: inc = sum_s k_s (c_s v_s)^T with
 // c_s = e^{g_L - g_s + i_s - m_L}; the CTA of the first columns also sums c_s k_s.
-constexpr int MU_THREADS = 128, MU_COLS = 64;
+constexpr int MU_THREADS = 256, MU_COLS = 64;
 __global__ void __launch_bounds__(MU_THREADS) mlstm_unit_kernel(const MlstmParams p) {
-  extern __shared__ uint16_t mu_smem[];        // K [64][dp + 8] | V hi, lo [64][72]
+  extern __shared__ uint16_t mu_smem[];        // K [unit][dp + 8] | V hi, lo [unit][72]
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float cs[ML_UNIT];
@@ -481,8 +488,8 @@ __global__ void __launch_bounds__(MU_THREADS) mlstm_unit_kernel(const MlstmParam
       uint32_t a[4];
       ldmatrix_x4_trans(smem_u32(K + (ks + (lane & 7) + (lane >> 4) * 8) * kp + d0 +
                                  ((lane >> 3) & 1) * 8), a[0], a[1], a[2], a[3]);
-      ml_products(acc, a, Vh, vpit, ks, lane);
-      ml_products(acc, a, Vl, vpit, ks, lane);
+      ml_products<8>(acc, a, Vh, vpit, ks, lane);
+      ml_products<8>(acc, a, Vl, vpit, ks, lane);
     }
 #pragma unroll
     for (int j = 0; j < 8; ++j)
@@ -554,13 +561,13 @@ __global__ void __launch_bounds__(256) mlstm_carry_kernel(const MlstmParams p) {
   if (ok) *st = s;
 }
 
-// CTA = one head of one unit, 16 tokens a warp.  Value columns go 64 at a time.
-constexpr int MO_THREADS = 128, MO_COLS = 64;
+// CTA = one head of one unit, 16 tokens a warp.  Value columns go 32 at a time.
+constexpr int MO_THREADS = ML_UNIT / 16 * 32, MO_COLS = 32, MO_KT = ML_UNIT / 16;
 __host__ __device__ constexpr int mo_smem(int dp) {
   return (2 * ML_UNIT * (dp + 8) + ML_UNIT * (MO_COLS + 8) + 2 * dp * (MO_COLS + 8)) * 2 +
          (3 * ML_UNIT + dp) * 4;
 }
-__global__ void __launch_bounds__(MO_THREADS) mlstm_output_kernel(const MlstmParams p) {
+__global__ void __launch_bounds__(MO_THREADS, 2) mlstm_output_kernel(const MlstmParams p) {
   extern __shared__ uint16_t mo_raw[];
   pdl_launch_dependents();
   pdl_wait();
@@ -599,10 +606,10 @@ __global__ void __launch_bounds__(MO_THREADS) mlstm_output_kernel(const MlstmPar
   // scores of this warp's 16 tokens against the unit's tokens up to them, decayed
   const int r0 = warp * 16;
   const float g0 = g[r0 + gr], g1 = g[r0 + gr + 8], m0 = ms[r0 + gr], m1 = ms[r0 + gr + 8];
-  uint32_t ph[4][4], pl[4][4];                  // A fragments of the decayed scores
+  uint32_t ph[MO_KT][4], pl[MO_KT][4];          // A fragments of the decayed scores
   float sum0 = 0.f, sum1 = 0.f;
 #pragma unroll
-  for (int kt = 0; kt < 4; ++kt) {
+  for (int kt = 0; kt < MO_KT; ++kt) {
 #pragma unroll
     for (int i = 0; i < 4; ++i) ph[kt][i] = pl[kt][i] = 0u;
     if (kt > warp) continue;
@@ -663,36 +670,24 @@ __global__ void __launch_bounds__(MO_THREADS) mlstm_output_kernel(const MlstmPar
       *reinterpret_cast<uint2*>(Sl + r * vpit + c) = make_uint2(x.z, x.w);
     }
     __syncthreads();
-    float acc[8][4] = {};
+    constexpr int NT = MO_COLS / 8;
+    float acc[NT][4] = {};
     for (int d = 0; d < dp; d += 16) {
       uint32_t a[4];
       ldmatrix_x4(ml_tile(Q, kp, r0, d, lane), a[0], a[1], a[2], a[3]);
-      ml_products(acc, a, Sh, vpit, d, lane);
-      ml_products(acc, a, Sl, vpit, d, lane);
+      ml_products<NT>(acc, a, Sh, vpit, d, lane);
+      ml_products<NT>(acc, a, Sl, vpit, d, lane);
     }
 #pragma unroll
-    for (int j = 0; j < 8; ++j) {
+    for (int j = 0; j < NT; ++j) {
       acc[j][0] *= in0; acc[j][1] *= in0;
       acc[j][2] *= in1; acc[j][3] *= in1;
     }
 #pragma unroll
-    for (int kt = 0; kt < 4; ++kt) {
+    for (int kt = 0; kt < MO_KT; ++kt) {
       if (kt > warp) continue;
-      uint32_t b[4][4];
-#pragma unroll
-      for (int j = 0; j < 4; ++j)
-        ldmatrix_x4_trans(ml_tile(V, vpit, kt * 16, j * 16, lane), b[j][0], b[j][1], b[j][2],
-                          b[j][3]);
-#pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        mma_bf16_16816(acc[2 * j], ph[kt], b[j][0], b[j][1]);
-        mma_bf16_16816(acc[2 * j + 1], ph[kt], b[j][2], b[j][3]);
-      }
-#pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        mma_bf16_16816(acc[2 * j], pl[kt], b[j][0], b[j][1]);
-        mma_bf16_16816(acc[2 * j + 1], pl[kt], b[j][2], b[j][3]);
-      }
+      ml_products<NT>(acc, ph[kt], V, vpit, kt * 16, lane);
+      ml_products<NT>(acc, pl[kt], V, vpit, kt * 16, lane);
     }
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
@@ -701,7 +696,7 @@ __global__ void __launch_bounds__(MO_THREADS) mlstm_output_kernel(const MlstmPar
       float* o = p.o + (un.t0 + r) * hv + h * p.vdim + v0;
       const float inv = e ? inv1 : inv0;
 #pragma unroll
-      for (int j = 0; j < 8; ++j) {
+      for (int j = 0; j < NT; ++j) {
         const int c = j * 8 + tq * 2;
         if (c + 1 < cols && (p.vdim & 1) == 0) {
           *reinterpret_cast<float2*>(o + c) =

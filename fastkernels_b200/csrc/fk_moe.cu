@@ -29,39 +29,43 @@ struct RouteParams {
   int64_t rows; int experts, top, blocks;
 };
 
+// Unsigned numbers in the order of the logits, never 0; NaN counts as the smallest.
+__device__ __forceinline__ uint32_t route_key(float z) {
+  const uint32_t u = __float_as_uint(z);
+  if (z != z) return 1u;
+  return max(u >> 31 ? ~u : u | 0x80000000u, 1u);
+}
+__device__ __forceinline__ float route_logit(uint32_t key) {
+  return __uint_as_float(key >> 31 ? key & 0x7fffffffu : ~key);
+}
+
 // One warp: choices and weights of row t; lane l holds the logits l, l + 32, ...
 template <int EPL>
 __device__ __forceinline__ void route_row(const RouteParams& p, int64_t t, int lane) {
   const float* z = p.z + t * p.z_stride;
-  float v[EPL];
+  uint32_t key[EPL];
 #pragma unroll
-  for (int i = 0; i < EPL; ++i) v[i] = lane + i * 32 < p.experts ? z[lane + i * 32] : -INFINITY;
+  for (int i = 0; i < EPL; ++i)
+    key[i] = lane + i * 32 < p.experts ? route_key(z[lane + i * 32]) : 0u;
   uint32_t taken = 0;                              // bit i: v[i] is chosen already
   float first = 0.f, total = 0.f;
   for (int j = 0; j < p.top; ++j) {
-    float best = -INFINITY;
-    int at = 0x7fffffff;
+    // largest free logit, then the lowest index that has it; unsigned keys in the order of
+    // the logits, 0 = nothing free
+    uint32_t best = 0u;
 #pragma unroll
     for (int i = 0; i < EPL; ++i)
-      if (!((taken >> i) & 1u) && lane + i * 32 < p.experts && (v[i] > best || at == 0x7fffffff)) {
-        best = v[i];
-        at = lane + i * 32;
-      }
+      if (!((taken >> i) & 1u)) best = max(best, key[i]);
+    const uint32_t top = __reduce_max_sync(0xffffffffu, best);
+    uint32_t mine = 0xffffffffu;
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-      const int oi = __shfl_xor_sync(0xffffffffu, at, o);
-      // a lane without candidates loses; ties go to the lowest index
-      if (oi != 0x7fffffff && (at == 0x7fffffff || ov > best || (ov == best && oi < at))) {
-        best = ov;
-        at = oi;
-      }
-    }
-    at = __shfl_sync(0xffffffffu, at, 0);          // NaN logits: the lanes still agree
-    best = __shfl_sync(0xffffffffu, best, 0);
+    for (int i = EPL - 1; i >= 0; --i)
+      if (!((taken >> i) & 1u) && key[i] == top) mine = lane + i * 32;
+    const int at = (int)__reduce_min_sync(0xffffffffu, mine);
+    const float chosen = route_logit(top);
     if ((at & 31) == lane) taken |= 1u << (at >> 5);
-    if (j == 0) first = best;
-    const float w = expf(best - first);
+    if (j == 0) first = chosen;
+    const float w = expf(chosen - first);
     total += w;
     if (lane == 0) {
       p.chosen[t * p.top + j] = at;

@@ -182,8 +182,10 @@ def _work(name, args, kw, out):
     if name == "mlstm_portions":
         q, k, v = args[:3]
         heads, dim, vdim = args[9:12]
-        # both products with the matrix per token
-        return _nbytes(q, k, v, out), 4 * q.shape[0] * heads * dim * vdim
+        # what every block of 128 tokens adds to the state is written, read, replaced by the
+        # state ahead of it and read again; both products with the matrix per token
+        blocks = 4 * (q.shape[0] // 128) * heads * dim * vdim * 4
+        return _nbytes(q, k, v, out) + blocks, 4 * q.shape[0] * heads * dim * vdim
     if name == "add_layernorm":
         ex = kw.get("experts")
         rows = _nbytes(kw.get("a"), kw.get("b"), *out[1:])

@@ -1089,7 +1089,7 @@ def mlstm_step(q, k, v, z, gate, weight, s_state, n_state, slots, positions, hea
 def mlstm_portions(q, k, v, z, s_state, n_state, cu_portions, slots, positions, heads, dim, vdim,
                    gate_cap, q_scale, longest, chunked=True, status=None):
     """The memory over portions; o [T, heads * vdim] fp32 ahead of norm and gate.  bf16
-    goes 64 tokens at a time unless chunked is False."""
+    goes 128 tokens at a time unless chunked is False."""
     f32, rows = _mlstm_args(q, k, v, z, s_state, n_state, heads, dim, vdim)
     _need(cu_portions, torch.int32, "cu_portions")
     _need(slots, torch.int32, "slots")

@@ -799,7 +799,7 @@ int fk_latent_attn(const void* q, int64_t q_pitch, const void* cache, int64_t nu
  * fk_mlstm_norm_cols(dim)], fp32, read and replaced; zero at position 0.
  * fk_mlstm_step: one token per row, out = rms(o per head) * weight * sigmoid(gate).
  * fk_mlstm_portions: runs of tokens, o fp32 [rows, heads * vdim] before norm and gate.  With
- * a workspace (fk_mlstm_workspace_floats) bf16 portions go 64 tokens at a time, without one
+ * a workspace (fk_mlstm_workspace_floats) bf16 portions go 128 tokens at a time, without one
  * token by token.  longest: tokens of the longest portion. */
 int fk_mlstm_state_cols(int vdim);
 int fk_mlstm_norm_cols(int dim);

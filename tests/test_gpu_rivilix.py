@@ -457,11 +457,11 @@ MEMORY_SIZES = [(3, 20, 28), (1, 9, 7), (2, 64, 128), (2, 128, 64), (1, 264, 40)
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("heads,dim,vdim", MEMORY_SIZES)
 def test_matrix_memory_portions_and_tokens(heads, dim, vdim, dtype):
-    """Sequences of unequal length in portions of 1 to 130 tokens, 64 at a time and one by
+    """Sequences of unequal length in portions of 1 to 257 tokens, in blocks and one by
     one, steps in between; slots start with what others left; a padded row."""
     from fastkernels_b200 import ops
     rs = np.random.RandomState(dim)
-    cap, eps, total, scale = 6.0, 1e-4, 210, dim ** -0.5
+    cap, eps, total, scale = 6.0, 1e-4, 400, dim ** -0.5
     widths = {"q": heads * dim, "k": heads * dim, "v": heads * vdim, "g": heads * vdim}
     offs, at = {}, 0
     for n, c in widths.items():
@@ -523,13 +523,14 @@ def test_matrix_memory_portions_and_tokens(heads, dim, vdim, dtype):
     run([(0, 2), (2, 63)])
     run([(2, 1), (0, 64), (1, 1)])
     run([(0, 1), (1, 1), (2, 1)], step=True)
-    run([(0, 65), (2, 2)])
-    run([(1, 130), (2, 5)])
+    run([(0, 129), (2, 2)])
+    run([(1, 257), (2, 5)])
     run([(2, 17), (0, 9)], chunked=False)
     for _ in range(4):
         run([(0, 1), (2, 1)], step=True)
     run([(0, 2), (1, 2)])
-    run([(2, 60)])
+    run([(2, 128), (0, 127)])
+    run([(1, 60), (2, 100), (0, 45)])
     while at[0] < total or at[1] < total:
         run([(i, 1) for i in (0, 1) if at[i] < total], step=True)
     assert int(st.item()) == 0
@@ -554,7 +555,7 @@ def test_memory_recalls_a_far_token(chunked):
     t, dim, vdim, cap = 700, 32, 48, 10.0
     k, v = R.bf16(rs.randn(t, dim) * 0.3), R.bf16(rs.randn(t, vdim))
     q = R.bf16(rs.randn(t, dim) * 0.1)
-    for place in (0, 1, 63, 64, 127, 300):
+    for place in (0, 1, 64, 127, 128, 129, 255, 300):
         q[-1] = k[place]
         zi = np.full((t, 1), -12.0)
         zi[place] = 4.0
@@ -563,7 +564,7 @@ def test_memory_recalls_a_far_token(chunked):
         want, _ = R.mlstm_memory(q[:, None], k[:, None], v[:, None], i, f)
         assert np.corrcoef(want[-1, 0], v[place])[0, 1] > 0.95
         x = dev(np.concatenate([q, k, v], 1), BF16)
-        for cuts in ([700], [place + 1, 699 - place], [64, 1, 2, 632, 1]):
+        for cuts in ([700], [place + 1, 699 - place], [128, 1, 2, 568, 1]):
             state = [torch.zeros(s, device="cuda") for s in ops.mlstm_state_shapes(1, 1, dim, vdim)]
             at = 0
             for n in cuts:
