@@ -153,7 +153,7 @@ PROTOTYPES = {
     "fk_latent_gather": (_i32, [_vp, _i64, _i64, _i32, _vp, _i64, _vp, _i32, _vp, _i64, _vp,
                                 _vp]),
     "fk_latent_attn_supported": (_i32, [_i32, _i32]),
-    "fk_latent_attn_splits": (_i32, [_i32, _i64, _i32, _i64]),
+    "fk_latent_attn_splits": (_i32, [_i32, _i64, _i32, _i32, _i64]),
     "fk_latent_attn_workspace_floats": (_i64, [_i64, _i32, _i32, _i32]),
     "fk_latent_attn": (_i32, [_vp, _i64, _vp, _i64, _i32, _i32, _vp, _i64, _vp, _vp, _vp, _i64,
                               _i32, _i64, _i64, _i32, _i32, _i32, _f32, _i32, _vp, _i64, _vp,

@@ -6,7 +6,8 @@
 //   row groups      group g takes the rows offsets[g] .. offsets[g + 1] of y (x rows the
 //                   same, or gather[row]): experts of a mixture
 //
-// act >= 0: w_g has 2 n rows [gate; up] and y = act(x gate^T) * (x up^T).
+// act >= 0: w_g has 2 n rows [gate; up] and y = act(x gate^T) * (x up^T),
+// each with its part of the bias.
 // bf16 operands with fp32 accumulation and bf16 or fp32 results, or true fp32.
 //
 //   group_any_kernel     fp32 FMA, any sizes (fp32 operands)
@@ -27,7 +28,7 @@ namespace fk {
 struct GroupParams {
   const void* x; int64_t x_stride, x_group;
   const void* w; int64_t w_rows;               // weight rows per group (n, or 2 n)
-  const float* bias;                           // [n] or null
+  const float* bias;                           // [w_rows] or null
   void* y; int64_t y_stride, y_group;
   const int32_t* offsets; const int32_t* gather;
   int64_t rows;                                // column groups: rows; row groups: all rows
@@ -128,7 +129,7 @@ __global__ void __launch_bounds__(256) group_any_kernel(const GroupParams p) {
       const int c = n0 + tx * 4 + j;
       if (c >= p.n) continue;
       float v = acc[0][i][j] + (p.bias ? p.bias[c] : 0.f);
-      if (ACT) v = group_act(v, p.act) * acc[NB - 1][i][j];
+      if (ACT) v = group_act(v, p.act) * (acc[NB - 1][i][j] + (p.bias ? p.bias[p.n + c] : 0.f));
       y[(first + r) * p.y_stride + c] = v;
     }
   }
@@ -230,7 +231,8 @@ __global__ void __launch_bounds__(256) group_skinny_kernel(const GroupParams p, 
     auto value = [&](int r, int t) {
       const int c = n0 + r;
       const float* part = gs_red + (r >> 4) * ks * (TILES * 16 * PITCH) + (r & 15) * PITCH + t;
-      float v = p.bias && c < p.n ? p.bias[c] : 0.f, up = 0.f;
+      float v = p.bias && c < p.n ? p.bias[c] : 0.f;
+      float up = ACT && p.bias && c < p.n ? p.bias[p.n + c] : 0.f;
       for (int q = 0; q < ks; ++q) {
         v += part[q * (TILES * 16 * PITCH)];
         if (ACT) up += part[q * (TILES * 16 * PITCH) + 16 * PITCH];
@@ -282,10 +284,11 @@ struct GgCfg {
   static constexpr int kBBytes = BN * GG_BK * 2;
   static constexpr int kStageBytes = GG_A_BYTES + kBBytes;
   static constexpr int kLoadBytes = kRows * GG_BK * 2 + kBBytes;
-  static constexpr int kStages = BN == 256 ? 4 : 9;
+  static constexpr int kStages = BN == 256 ? 4 : 8;
   static constexpr int kOffTiles = kStages * kStageBytes;      // first tile of every group
   static constexpr int kOffBar = kOffTiles + (GG_MAX_GROUPS + 8) * 4;
-  static constexpr int kSmem = kOffBar + 256 + 1024;
+  static constexpr int kOffOut = kOffBar + 256;       // 4 warps x 32 rows x 128 bytes
+  static constexpr int kSmem = kOffOut + 4 * 4096 + 1024;
   static_assert(kSmem <= 232448, "shared memory budget");
 };
 
@@ -339,6 +342,21 @@ __device__ __forceinline__ GgTile gg_tile(const GroupParams& p, const int* first
   t.row0 = a + (int64_t)mt * ROWS;
   t.rows_left = b - t.row0;
   return t;
+}
+
+// Adds bias[from + c .. from + c + 3]; columns beyond n are not stored.
+__device__ __forceinline__ void gg_add_bias(const GroupParams& p, int from, int c, float& a,
+                                            float& b, float& d, float& e) {
+  const float* q = p.bias + from + c;
+  if (c + 4 <= p.n && (p.n & 3) == 0) {
+    const float4 v = __ldg(reinterpret_cast<const float4*>(q));
+    a += v.x; b += v.y; d += v.z; e += v.w;
+  } else {
+    if (c < p.n) a += q[0];
+    if (c + 1 < p.n) b += q[1];
+    if (c + 2 < p.n) d += q[2];
+    if (c + 3 < p.n) e += q[3];
+  }
 }
 
 template <int BN, bool ACT, typename OUT>
@@ -476,7 +494,7 @@ group_large_kernel(const __grid_constant__ CUtensorMap tmap_x,
       ++done;
     }
   } else {
-    const int q = warp & 3, row = q * 32 + lane;
+    const int q = warp & 3;
     const uint32_t lane_addr = (uint32_t)(q * 32) << 16;
     uint32_t done = 0;
     for (int ti = blockIdx.x; ti < total; ti += gridDim.x) {
@@ -484,46 +502,82 @@ group_large_kernel(const __grid_constant__ CUtensorMap tmap_x,
       const uint32_t buf = done & 1u, use = done >> 1;
       if (!gg_wait(&acc_full[buf], use & 1u, abort_flag, p.status)) break;
       tc_fence_after();
-      const bool live = row < Cfg::kRows && row < t.rows_left;
+      // rows of this warp that exist
+      const int rows = (int)max((int64_t)0, min((int64_t)32, min((int64_t)Cfg::kRows,
+                                                                 t.rows_left) - q * 32));
       OUT* y = static_cast<OUT*>(p.y) + (p.offsets ? 0 : t.g * p.y_group) +
-               (t.row0 + (live ? row : 0)) * p.y_stride;
+               (t.row0 + q * 32) * p.y_stride;
       const int n0 = t.nt * TN;
+      // 128 bytes of every row at a time, through shared memory: a warp then stores whole
+      // lines.  16-byte piece c of a row lies at c ^ (row & 7).
+      constexpr int CH = 128 / (int)sizeof(OUT) < TN ? 128 / (int)sizeof(OUT) : TN;   // columns
+      uint8_t* stage_out = smem + Cfg::kOffOut + q * 4096;
 #pragma unroll 1
-      for (int c = 0; c < TN / 32; ++c) {
-        uint32_t v[32], u[ACT ? 32 : 1];
-        tc_ld32(lane_addr + buf * BN + c * 32, v);
-        if (ACT) tc_ld32(lane_addr + buf * BN + BN / 2 + c * 32, u);
-        tc_wait_ld();
-        if (!live || n0 + c * 32 >= p.n) continue;
-        float f[32];
+      for (int c0 = 0; c0 < TN; c0 += CH) {
+        if (n0 + c0 >= p.n) break;
+        __syncwarp();
 #pragma unroll
-        for (int i = 0; i < 32; ++i) {
-          f[i] = __uint_as_float(v[i]);
-          if (ACT) {
-            const float up = __uint_as_float(u[ACT ? i : 0]);
-            f[i] = (p.act == FK_ACT_SILU ? silu_f32(f[i])
-                                         : __fdividef(f[i], 1.0f + __expf(-gelu_tanh_arg(f[i])))) *
-                   up;
-          } else if (p.bias && n0 + c * 32 + i < p.n) {
-            f[i] += p.bias[n0 + c * 32 + i];
+        for (int c = 0; c < CH; c += 32) {
+          uint32_t v[32], u[ACT ? 32 : 1];
+          tc_ld32(lane_addr + buf * BN + c0 + c, v);
+          if (ACT) tc_ld32(lane_addr + buf * BN + BN / 2 + c0 + c, u);
+          tc_wait_ld();
+          float f[32];
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            f[i] = __uint_as_float(v[i]);
           }
-        }
-        OUT* dst = y + n0 + c * 32;
-        constexpr int PER = 16 / (int)sizeof(OUT);
+          if (p.bias) {
 #pragma unroll
-        for (int i = 0; i < 32; i += PER) {
-          if (n0 + c * 32 + i + PER <= p.n) {
+            for (int i = 0; i < 32; i += 4)
+              gg_add_bias(p, 0, n0 + c0 + c + i, f[i], f[i + 1], f[i + 2], f[i + 3]);
+          }
+          if (ACT) {
+#pragma unroll
+            for (int i = 0; i < 32; i += 4) {
+              float up[4];
+#pragma unroll
+              for (int j = 0; j < 4; ++j) up[j] = __uint_as_float(u[ACT ? i + j : 0]);
+              if (p.bias) gg_add_bias(p, p.n, n0 + c0 + c + i, up[0], up[1], up[2], up[3]);
+#pragma unroll
+              for (int j = 0; j < 4; ++j) {
+                const float g = f[i + j];
+                f[i + j] = (p.act == FK_ACT_SILU
+                                ? silu_f32(g) : __fdividef(g, 1.0f + __expf(-gelu_tanh_arg(g)))) *
+                           up[j];
+              }
+            }
+          }
+          constexpr int PER = 16 / (int)sizeof(OUT);
+#pragma unroll
+          for (int i = 0; i < 32; i += PER) {
+            uint4 w;
             if (sizeof(OUT) == 2)
-              *reinterpret_cast<uint4*>(dst + i) =
-                  make_uint4(pack_bf16(f[i], f[i + 1]), pack_bf16(f[i + 2], f[i + 3]),
+              w = make_uint4(pack_bf16(f[i], f[i + 1]), pack_bf16(f[i + 2], f[i + 3]),
                              pack_bf16(f[i + 4 < 32 ? i + 4 : 0], f[i + 5 < 32 ? i + 5 : 0]),
                              pack_bf16(f[i + 6 < 32 ? i + 6 : 0], f[i + 7 < 32 ? i + 7 : 0]));
             else
-              *reinterpret_cast<float4*>(dst + i) = make_float4(f[i], f[i + 1], f[i + 2], f[i + 3]);
-          } else {
+              w = make_uint4(__float_as_uint(f[i]), __float_as_uint(f[i + 1]),
+                             __float_as_uint(f[i + 2]), __float_as_uint(f[i + 3]));
+            const int piece = (c + i) / PER;
+            *reinterpret_cast<uint4*>(stage_out + lane * 128 + ((piece ^ (lane & 7)) << 4)) = w;
+          }
+        }
+        __syncwarp();
+        const int piece = lane & 7;
+        const int col = n0 + c0 + piece * (16 / (int)sizeof(OUT));
 #pragma unroll
-            for (int j = 0; j < PER; ++j)
-              if (n0 + c * 32 + i + j < p.n) Elem<OUT>::store(dst + i + j, f[i + j]);
+        for (int r = lane >> 3; r < 32; r += 4) {
+          if (r >= rows || col >= p.n) continue;
+          const uint4 w = *reinterpret_cast<const uint4*>(stage_out + r * 128 +
+                                                          ((piece ^ (r & 7)) << 4));
+          OUT* dst = y + r * p.y_stride + col;
+          if (col + 16 / (int)sizeof(OUT) <= p.n) {
+            *reinterpret_cast<uint4*>(dst) = w;
+          } else {
+            const OUT* e = reinterpret_cast<const OUT*>(&w);
+            for (int j = 0; j < 16 / (int)sizeof(OUT); ++j)
+              if (col + j < p.n) dst[j] = e[j];
           }
         }
       }
@@ -668,8 +722,8 @@ int fk_group_gemm(const void* x, int64_t x_stride, int64_t x_group, int64_t x_ro
   FK_REQUIRE(!gather || offsets, FK_ERR_INVALID_ARG,
              "fk_group_gemm: only row groups can be gathered");
   FK_REQUIRE(gather || x_rows >= rows, FK_ERR_INVALID_ARG, "fk_group_gemm: x has too few rows");
-  FK_REQUIRE(act < 0 || ((act == FK_ACT_SILU || act == FK_ACT_GELU_TANH) && !bias),
-             FK_ERR_INVALID_ARG, "fk_group_gemm: unknown activation %d, or one with a bias", act);
+  FK_REQUIRE(act < 0 || act == FK_ACT_SILU || act == FK_ACT_GELU_TANH, FK_ERR_INVALID_ARG,
+             "fk_group_gemm: unknown activation %d", act);
   const int64_t x_cols = offsets ? k : (groups - 1) * x_group + k;
   FK_REQUIRE(x_group >= 0 && y_group >= 0 && x_stride >= x_cols &&
                  y_stride >= (offsets ? n : (groups - 1) * y_group + n) &&
@@ -679,7 +733,7 @@ int fk_group_gemm(const void* x, int64_t x_stride, int64_t x_group, int64_t x_ro
              "fk_group_gemm: dimension too large");
   const int unit = is_f32 ? 4 : 8;
   FK_REQUIRE(k % unit == 0 && x_stride % unit == 0 && x_group % unit == 0 && aligned16(x) &&
-                 aligned16(w) && aligned16(y),
+                 aligned16(w) && aligned16(y) && aligned16(bias),
              FK_ERR_ALIGNMENT, "fk_group_gemm: x and w need 16-byte aligned rows");
   GroupParams p{};
   p.x = x; p.x_stride = x_stride; p.x_group = x_group; p.x_rows = x_rows; p.w = w;

@@ -217,14 +217,15 @@ struct LatentAttnParams {
   int32_t* status;
 };
 
-// Warps 0-7 make scores and softmax weights of a tile of 32 keys, warps 8-15 multiply the
-// weights of the tile before it with its values; one lane of warp 8 keeps the ring of tiles
-// filled.  A tile is blocks of 64 channels, [32 rows][128 bytes] each, 128-byte swizzled by
+// Half of the warps make scores and softmax weights of a tile of 32 keys, the others multiply
+// the weights of the tile before it with its values; one lane of them keeps the ring of tiles
+// filled.  Latents up to 256 channels: 4 + 4 warps and two CTAs on an SM; above: 8 + 8 warps,
+// scores of two tiles under way at once (SUBS = 2).  A tile is blocks of 64 channels, [32 rows][128 bytes] each, 128-byte swizzled by
 // TMA.  The steps of a tile are short, so what bounds the kernel is the latency of fragment
 // loads and of hand-overs: query fragments stay in registers, fragments are loaded several
 // steps ahead, and warps hand over through named barriers (a wait on a shared-memory barrier
 // costs several times as much; only the copies need one).
-constexpr int LA_ROWS = 16, LA_GROUP = 256, LA_THREADS = 2 * LA_GROUP, LA_KEYS = 32;
+constexpr int LA_ROWS = 16, LA_KEYS = 32;
 constexpr int LA_BLOCK = LA_KEYS * 128;
 constexpr int LA_PPITCH = LA_KEYS + 8, LA_XPITCH = LA_KEYS + 8, LA_MAX_RING = 8;
 constexpr uint32_t LA_WAIT_LIMIT = 1u << 22;
@@ -234,17 +235,17 @@ constexpr int LA_BAR_SUB = 1, LA_BAR_END = 3, LA_BAR_SUM = 4, LA_BAR_FULL = 5, L
 
 // lk: channels of a row, rounded up to 16; a tile holds whole blocks of 64.
 __host__ __device__ constexpr int la_tile(int lk) { return (lk + 63) / 64 * LA_BLOCK; }
-// 8-column groups of values per warp, and 16-channel steps of scores per warp.
-__host__ __device__ constexpr int la_rn(int rank) { return rank <= 128 ? 2 : rank <= 256 ? 4 : 8; }
-__host__ __device__ constexpr int la_steps(int rn) { return rn == 8 ? 10 : rn == 4 ? 6 : 4; }
-__host__ __device__ constexpr int la_smem(int lk, int ring) {
-  return ring * la_tile(lk) + 2 * 4 * LA_ROWS * LA_XPITCH * 4 + 4 * LA_ROWS * LA_PPITCH * 2 +
+__host__ __device__ constexpr int la_subs(int rank) { return rank <= 256 ? 1 : 2; }
+// 16-channel steps of scores per warp: registers for its part of the queries.
+__host__ __device__ constexpr int la_steps(int rank) { return rank <= 128 ? 4 : rank <= 256 ? 6 : 10; }
+__host__ __device__ constexpr int la_smem(int subs, int lk, int ring) {
+  return ring * la_tile(lk) + subs * 4 * LA_ROWS * LA_XPITCH * 4 + 4 * LA_ROWS * LA_PPITCH * 2 +
          21 * LA_ROWS * 4 + LA_MAX_RING * 8 + 1024;
 }
 // Deepest ring that fits, 0: none.
-__host__ __device__ constexpr int la_ring(int lk) {
+__host__ __device__ constexpr int la_ring(int subs, int lk) {
   int r = LA_MAX_RING;
-  while (r >= 3 && la_smem(lk, r) > 232448) --r;
+  while (r >= 3 && la_smem(subs, lk, r) > (subs == 1 ? 115712 : 232448)) --r;
   return r >= 3 ? r : 0;
 }
 
@@ -252,18 +253,19 @@ __device__ __forceinline__ void named_bar_arrive(int id, int nthreads) {
   asm volatile("bar.arrive %0, %1;" ::"r"(id), "r"(nthreads) : "memory");
 }
 
-template <int RN>
-__global__ void __launch_bounds__(LA_THREADS, 1)
+template <int RN, int QS, int SUBS>
+__global__ void __launch_bounds__(SUBS * 256, 3 - SUBS)
 latent_attn_kernel(const __grid_constant__ CUtensorMap tmap, const LatentAttnParams p) {
   extern __shared__ uint8_t la_raw[];
+  constexpr int GROUP = SUBS * 128;                      // threads of either half
   pdl_launch_dependents();
   const int seq = blockIdx.y, split = blockIdx.z;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int gr = lane >> 2, tq = lane & 3;
   uint8_t* K = la_raw + ((1024u - (smem_u32(la_raw) & 1023u)) & 1023u);    // ring of tiles
   const int tile_bytes = la_tile(p.lk);
-  float* X = reinterpret_cast<float*>(K + p.ring * tile_bytes);   // [2][4][16][LA_XPITCH]
-  uint16_t* P = reinterpret_cast<uint16_t*>(X + 8 * LA_ROWS * LA_XPITCH);  // [2][hi, lo][16][]
+  float* X = reinterpret_cast<float*>(K + p.ring * tile_bytes);   // [SUBS][4][16][LA_XPITCH]
+  uint16_t* P = reinterpret_cast<uint16_t*>(X + SUBS * 4 * LA_ROWS * LA_XPITCH);  // [2][hi, lo][16][]
   float* alpha = reinterpret_cast<float*>(P + 4 * LA_ROWS * LA_PPITCH);    // [2][16]
   float* inv_l = alpha + 2 * LA_ROWS;                     // [16]
   float* m_run = inv_l + LA_ROWS;                         // [2][16]: running maximum
@@ -293,12 +295,12 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmap, const LatentAttnPar
   const int sw = lane & 7;
   const int row0 = gr, row1 = gr + 8;
 
-  if (warp < LA_GROUP / 32) {
+  if (warp < GROUP / 32) {
     // --------------------------- scores and weights --------------------------
-    // Four warps a tile, so that two tiles are under way; only the running maximum goes from
-    // one tile to the next.  Products: a warp has all keys and a quarter of the channels.
+    // Four warps a tile.  With two tiles under way only the running maximum goes from one
+    // tile to the next.  Products: a warp has all keys and a quarter of the channels.
     // Weights: 8 keys.
-    constexpr int QS = la_steps(RN), AHEAD = 3;
+    constexpr int AHEAD = 3;
     const int sub = warp >> 2, v = warp & 3, key0 = v * 8;
     const int lim0 = row0 < n_rows ? min(k_end, before + (tok0 + row0) / p.heads) : 0;
     const int lim1 = row1 < n_rows ? min(k_end, before + (tok0 + row1) / p.heads) : 0;
@@ -324,7 +326,8 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmap, const LatentAttnPar
     bool ok = true;
     int st = sub;
     uint32_t phase = 0;
-    for (int n = sub; n < tiles; n += 2) {
+    for (int n = sub; n < tiles; n += SUBS) {
+      const int buf = n & 1;
       const int k0 = k_begin + n * LA_KEYS;
       ok = ok && mbar_wait(&full[st], phase, LA_WAIT_LIMIT);
       uint8_t* tile = K + st * tile_bytes;
@@ -402,20 +405,20 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmap, const LatentAttnPar
         t0 = fmaxf(t0, mw[row0]);
         t1 = fmaxf(t1, mw[row1]);
       }
-      float p0 = -INFINITY, p1 = -INFINITY;
-      if (n > 0) {
+      float p0 = m0, p1 = m1;
+      if (SUBS == 2 && n > 0) {
         named_bar_sync(LA_BAR_MAX + (sub ^ 1), 2 * 128);
         p0 = m_run[(sub ^ 1) * LA_ROWS + row0];
         p1 = m_run[(sub ^ 1) * LA_ROWS + row1];
-        t0 = fmaxf(t0, p0);
-        t1 = fmaxf(t1, p1);
       }
+      t0 = fmaxf(t0, p0);
+      t1 = fmaxf(t1, p1);
       const bool writes = tq == 0 && v == 0;
       if (writes) {
         m_run[sub * LA_ROWS + row0] = t0;
         m_run[sub * LA_ROWS + row1] = t1;
       }
-      if (n + 1 < tiles) named_bar_arrive(LA_BAR_MAX + sub, 2 * 128);
+      if (SUBS == 2 && n + 1 < tiles) named_bar_arrive(LA_BAR_MAX + sub, 2 * 128);
       const float z0 = t0 == -INFINITY ? 0.f : t0, z1 = t1 == -INFINITY ? 0.f : t1;
       l0 *= fast_exp2(m0 - z0);
       l1 *= fast_exp2(m1 - z1);
@@ -428,8 +431,8 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmap, const LatentAttnPar
         l0 += x[e];
         l1 += x[2 + e];
       }
-      if (n >= 2) named_bar_sync(LA_BAR_EMPTY + sub, 128 + LA_GROUP);
-      uint16_t* ph = P + sub * 2 * LA_ROWS * LA_PPITCH + key0 + tq * 2;
+      if (n >= 2) named_bar_sync(LA_BAR_EMPTY + buf, 128 + GROUP);
+      uint16_t* ph = P + buf * 2 * LA_ROWS * LA_PPITCH + key0 + tq * 2;
       uint32_t hi, lo;
       split_bf16(x[0], x[1], &hi, &lo);
       *reinterpret_cast<uint32_t*>(ph + row0 * LA_PPITCH) = hi;
@@ -438,11 +441,11 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmap, const LatentAttnPar
       *reinterpret_cast<uint32_t*>(ph + row1 * LA_PPITCH) = hi;
       *reinterpret_cast<uint32_t*>(ph + (LA_ROWS + row1) * LA_PPITCH) = lo;
       if (writes) {
-        alpha[sub * LA_ROWS + row0] = p0 == -INFINITY ? 1.f : fast_exp2(p0 - z0);
-        alpha[sub * LA_ROWS + row1] = p1 == -INFINITY ? 1.f : fast_exp2(p1 - z1);
+        alpha[buf * LA_ROWS + row0] = p0 == -INFINITY ? 1.f : fast_exp2(p0 - z0);
+        alpha[buf * LA_ROWS + row1] = p1 == -INFINITY ? 1.f : fast_exp2(p1 - z1);
       }
-      named_bar_arrive(LA_BAR_FULL + sub, 128 + LA_GROUP);
-      st += 2;
+      named_bar_arrive(LA_BAR_FULL + buf, 128 + GROUP);
+      st += SUBS;
       if (st >= p.ring) { st -= p.ring; phase ^= 1; }
     }
     if (!ok && p.status) atomicOr(p.status, FK_DEV_WAIT_TIMEOUT);
@@ -457,19 +460,20 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmap, const LatentAttnPar
       l_warp[warp * LA_ROWS + row1] = l1;
     }
     if (tiles <= sub && v == 0 && lane < LA_ROWS) m_run[sub * LA_ROWS + lane] = -INFINITY;
-    named_bar_sync(LA_BAR_SUM, LA_GROUP);
+    named_bar_sync(LA_BAR_SUM, GROUP);
     if (tid < LA_ROWS) {
-      const float ma = m_run[tid], mb = m_run[LA_ROWS + tid], mx = fmaxf(ma, mb);
+      const float ma = m_run[tid], mb = SUBS == 2 ? m_run[LA_ROWS + tid] : ma;
+      const float mx = fmaxf(ma, mb);
       const float z = mx == -INFINITY ? 0.f : mx;
       float l = 0.f;
 #pragma unroll
-      for (int w = 0; w < 8; ++w)
+      for (int w = 0; w < 4 * SUBS; ++w)
         l += l_warp[w * LA_ROWS + tid] * fast_exp2((w < 4 ? ma : mb) - z);
       inv_l[tid] = l > 0.f ? 1.0f / l : 0.f;
       if (p.splits > 1 && tid < n_rows)
         p.ml[(int64_t)split * p.flat_rows + first + tid] = make_float2(mx, l);
     }
-    named_bar_sync(LA_BAR_END, 2 * LA_GROUP);
+    named_bar_sync(LA_BAR_END, 2 * GROUP);
     return;
   }
 
@@ -500,7 +504,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmap, const LatentAttnPar
       }
     }
   };
-  const bool feeds = warp == LA_GROUP / 32 && lane == 0;
+  const bool feeds = warp == GROUP / 32 && lane == 0;
   int next_row = 0;                       // of tile n - 1 + ring, looked up ahead
   if (feeds) {
     for (int n = 0; n < min(tiles, p.ring); ++n) issue(n, n, pool_row(k_begin + n * LA_KEYS));
@@ -512,7 +516,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmap, const LatentAttnPar
   for (int j = 0; j < RN; ++j)
 #pragma unroll
     for (int i = 0; i < 4; ++i) acc[j][i] = 0.f;
-  const int col0 = (warp - LA_GROUP / 32) * RN * 8;
+  const int col0 = (warp - GROUP / 32) * RN * 8;
   uint32_t at[RN / 2];                    // this lane's fragment addresses inside a tile
 #pragma unroll
   for (int j = 0; j < RN / 2; ++j) {
@@ -525,7 +529,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmap, const LatentAttnPar
   for (int n = 0; n < tiles; ++n) {
     const int buf = n & 1;
     const uint32_t tile = smem_u32(K) + st * tile_bytes;
-    named_bar_sync(LA_BAR_FULL + buf, 128 + LA_GROUP);
+    named_bar_sync(LA_BAR_FULL + buf, 128 + GROUP);
     if (feeds && n > 0 && n - 1 + p.ring < tiles) {
       issue(n - 1 + p.ring, st == 0 ? p.ring - 1 : st - 1, next_row);
       if (n + p.ring < tiles) next_row = pool_row(k_begin + (n + p.ring) * LA_KEYS);
@@ -562,10 +566,10 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmap, const LatentAttnPar
             mma_bf16_16816(acc[2 * j + 1], part ? pl[kt] : ph[kt], b[kt][j][2], b[kt][j][3]);
           }
     }
-    if (n + 2 < tiles) named_bar_arrive(LA_BAR_EMPTY + buf, 128 + LA_GROUP);
+    if (n + 2 < tiles) named_bar_arrive(LA_BAR_EMPTY + buf, 128 + GROUP);
     if (++st == p.ring) st = 0;
   }
-  named_bar_sync(LA_BAR_END, 2 * LA_GROUP);
+  named_bar_sync(LA_BAR_END, 2 * GROUP);
   if (p.splits > 1 && tiles == 0) return;
 #pragma unroll
   for (int e = 0; e < 2; ++e) {
@@ -656,20 +660,21 @@ static int la_map(const void* ptr, int64_t rows, int64_t cols, int run, int bloc
   return FK_OK;
 }
 
-template <int RN>
+template <int RN, int QS, int SUBS>
 static int launch_latent(LatentAttnParams& p, dim3 grid, cudaStream_t s) {
-  p.ring = la_ring(p.lk);
-  const int smem = la_smem(p.lk, p.ring);
+  p.ring = la_ring(SUBS, p.lk);
+  const int smem = la_smem(SUBS, p.lk, p.ring);
   static PerDeviceOnce once;
-  FK_CUDA_OK(set_max_dynamic_smem(once, latent_attn_kernel<RN>, 232448));
+  FK_CUDA_OK(set_max_dynamic_smem(once, latent_attn_kernel<RN, QS, SUBS>,
+                                  SUBS == 1 ? 115712 : 232448));
   p.run = LA_KEYS;                       // keys that surely lie in one page
   while (p.block_size % p.run) p.run /= 2;
   CUtensorMap map;
   const int rc = la_map(p.cache, (int64_t)p.num_blocks * p.block_size, p.cache_pitch, p.run,
                         p.run == LA_KEYS ? (p.lk + 63) / 64 : 1, &map);
   if (rc != FK_OK) return rc;
-  FK_CUDA_OK(launch_kernel(latent_attn_kernel<RN>, grid, dim3(LA_THREADS), (size_t)smem, s, map,
-                           p));
+  FK_CUDA_OK(launch_kernel(latent_attn_kernel<RN, QS, SUBS>, grid, dim3(SUBS * 256),
+                           (size_t)smem, s, map, p));
   count_launch();
   return FK_OK;
 }
@@ -741,18 +746,24 @@ int fk_latent_gather(const void* cache, int64_t row_bytes, int64_t num_blocks, i
 
 int fk_latent_attn_supported(int rank, int rot) {
   const int lk = (rank + rot + 15) / 16 * 16;
-  return rank > 0 && rank <= 512 && rot >= 0 && lk / 16 <= 4 * la_steps(la_rn(rank)) &&
-         la_ring(lk) > 0;
+  return rank > 0 && rank <= 512 && rot >= 0 && lk / 16 <= 4 * la_steps(rank) &&
+         la_ring(la_subs(rank), lk) > 0;
 }
 
-/* Key ranges a call with these sizes splits its rows into. */
-int fk_latent_attn_splits(int num_seqs, int64_t max_q, int heads, int64_t max_keys) {
+/* Key ranges a call with these sizes splits its rows into.  The lengths are on the device, so
+ * 2048 keys stand for them: the number with the shortest rounds of CTAs, each with its share
+ * of the keys and a start that costs as much as about 256. */
+int fk_latent_attn_splits(int num_seqs, int64_t max_q, int heads, int rank, int64_t max_keys) {
   const int64_t tiles = (max_q * heads + LA_ROWS - 1) / LA_ROWS * num_seqs;
-  if (tiles <= 0) return 1;
-  int64_t s = (int64_t)sm_count() / tiles;
-  const int64_t most = (max_keys + 127) / 128;
-  s = s < most ? s : most;
-  return (int)(s < 1 ? 1 : s > 32 ? 32 : s);
+  const int64_t slots = (int64_t)sm_count() * (la_subs(rank) == 1 ? 2 : 1);
+  const int64_t keys = max_keys < 2048 ? max_keys : 2048;
+  int best = 1;
+  int64_t best_cost = INT64_MAX;
+  for (int s = 1; s <= 32 && (s == 1 || s * 128 <= max_keys + 127); ++s) {
+    const int64_t cost = (tiles * s + slots - 1) / slots * ((keys + s - 1) / s + 256);
+    if (cost < best_cost) { best = s; best_cost = cost; }
+  }
+  return best;
 }
 
 int64_t fk_latent_attn_workspace_floats(int64_t rows, int heads, int rank, int splits) {
@@ -806,9 +817,9 @@ int fk_latent_attn(const void* q, int64_t q_pitch, const void* cache, int64_t nu
              FK_ERR_UNSUPPORTED, "fk_latent_attn: too many rows");
   const dim3 grid((unsigned)tiles, (unsigned)num_seqs, (unsigned)splits);
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const int rn = la_rn(rank);
-  const int rc = rn == 2 ? launch_latent<2>(p, grid, s)
-                 : rn == 4 ? launch_latent<4>(p, grid, s) : launch_latent<8>(p, grid, s);
+  const int rc = rank <= 128   ? launch_latent<4, la_steps(128), 1>(p, grid, s)
+                 : rank <= 256 ? launch_latent<8, la_steps(256), 1>(p, grid, s)
+                               : launch_latent<8, la_steps(512), 2>(p, grid, s);
   if (rc != FK_OK || splits == 1) return rc;
   FK_CUDA_OK(launch_kernel(latent_merge_kernel, dim3((unsigned)p.flat_rows), dim3(128), 0, s, p));
   count_launch();

@@ -15,6 +15,10 @@ from .mixers import round_up
 class GatedFeedForward:
     """down(act(gate h) * (up h)), with or without biases."""
 
+    # rows from which the many-row grouped product (activation in its epilogue) takes over
+    # from the projection with a kernel for the activation behind it
+    MANY_ROWS = 256
+
     def __init__(self, ff: int, bias: bool, act: int = _lib.ACT_SILU):
         self.ff, self.bias, self.act = ff, bias, act
         self.status = None
@@ -31,15 +35,20 @@ class GatedFeedForward:
         ff = round_up(self.ff, 64)
         self.w_gate_up = torch.cat([w.padded(prefix + n, ff, w.stride) for n in ("gate", "up")])
         self.w_down = w.padded(prefix + "down", w.stride, ff)
-        self.b_gate_up = self.b_down = None
+        self.b_gate_up = self.b_down = self.b_gate_up_f32 = None
         if self.bias:
             self.b_gate_up = torch.cat([w.vector(f"{prefix}{n}.b", ff, w.dtype)
                                         for n in ("gate", "up")])
+            self.b_gate_up_f32 = self.b_gate_up.float()
             self.b_down = w.vector(prefix + "down.b", w.stride, w.dtype)
 
     def forward(self, h):
-        a = ops.gemm_act_mul(h, self.w_gate_up, self.act, bias=self.b_gate_up,
-                             status=self.status)
+        if h.dtype != torch.float32 and h.shape[0] > self.MANY_ROWS:
+            a = ops.group_gemm(h, self.w_gate_up, bias=self.b_gate_up_f32, act=self.act,
+                               status=self.status)
+        else:
+            a = ops.gemm_act_mul(h, self.w_gate_up, self.act, bias=self.b_gate_up,
+                                 status=self.status)
         return ops.gemm(a, self.w_down, bias=self.b_down, status=self.status), None
 
 

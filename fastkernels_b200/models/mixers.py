@@ -258,7 +258,7 @@ class LatentAttention:
         if expand:
             rows = ops.latent_gather(cache, span.block_tables, span.cu_seqlens_k, span.total_k,
                                      status=self.status)
-            kv = ops.gemm(rows, self.w_expand, status=self.status)
+            kv = ops.group_gemm(rows, self.w_expand, status=self.status)
             kv = kv.view(span.total_k, 2, self.heads, 128)
             ops.prefill_attn(q, kv[:, 0], kv[:, 1], span.cu_seqlens_q, span.cu_seqlens_k,
                              span.max_seqlen_q, self.scale,

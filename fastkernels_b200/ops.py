@@ -909,8 +909,8 @@ def group_gemm(x, w, out=None, bias=None, x_group=0, y_group=0, offsets=None, ga
         raise _lib.FkError("group_gemm: gather is shorter than the rows")
     if bias is not None:
         _need(bias, torch.float32, "bias")
-        if bias.numel() < n:
-            raise _lib.FkError("group_gemm: bias is shorter than the result's rows")
+        if bias.numel() < wn or not bias.is_contiguous():
+            raise _lib.FkError("group_gemm: bias must have one entry per weight row")
     if out.dim() != 2 or out.shape[0] < rows or out.stride(1) != 1:
         raise _lib.FkError("group_gemm: out must be row-dense with a row per row")
     check(lib.fk_group_gemm(
@@ -1030,7 +1030,8 @@ def latent_attn(q, cache, cu_seqlens_q, kv_lens, block_tables, max_seqlen_q, max
         out = torch.empty((rows, heads, (rank + 15) // 16 * 16), dtype=BF16, device=q.device)
     elif not out.is_contiguous():
         raise _lib.FkError("latent_attn: out must be contiguous")
-    splits = int(lib.fk_latent_attn_splits(n_seq, int(max_seqlen_q), heads, int(max_keys)))
+    splits = int(lib.fk_latent_attn_splits(n_seq, int(max_seqlen_q), heads, rank,
+                                           int(max_keys)))
     n = int(lib.fk_latent_attn_workspace_floats(rows, heads, rank, splits))
     ws = torch.empty(n, dtype=torch.float32, device=q.device) if n else None
     check(lib.fk_latent_attn(

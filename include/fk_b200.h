@@ -733,9 +733,9 @@ int fk_softcap(void* x, int64_t stride, int is_f32, int64_t rows, int64_t cols, 
  *     and y columns from g * y_group on
  *   row groups: group g takes rows offsets[g] .. offsets[g + 1] (device int32
  *     [groups + 1]) of y; x rows the same, or gather[row]
- * act >= 0 (enum fk_activation): w has 2 n rows [gate; up], y = act(gate) * up.  is_f32:
+ * act >= 0 (enum fk_activation): w_g has 2 n rows [gate; up], y = act(gate) * up.  is_f32:
  * fp32 operands and result; else bf16 operands, fp32 accumulation, result bf16 or (y_f32)
- * fp32.  bias fp32 [n] (not with an activation).  expect_rows: rows a group has, roughly;
+ * fp32.  bias fp32, one per row of w_g, the same for all groups.  expect_rows: rows a group has, roughly;
  * picks the kernel. */
 int fk_group_gemm(const void* x, int64_t x_stride, int64_t x_group, int64_t x_rows,
                   const void* w, const float* bias, void* y, int64_t y_stride, int64_t y_group,
@@ -782,7 +782,7 @@ int fk_latent_gather(const void* cache, int64_t row_bytes, int64_t num_blocks, i
                      const int32_t* cu_seqlens_k, int num_seqs, void* out, int64_t rows,
                      int32_t* status, fk_stream_t stream);
 int fk_latent_attn_supported(int rank, int rot);
-int fk_latent_attn_splits(int num_seqs, int64_t max_q, int heads, int64_t max_keys);
+int fk_latent_attn_splits(int num_seqs, int64_t max_q, int heads, int rank, int64_t max_keys);
 int64_t fk_latent_attn_workspace_floats(int64_t rows, int heads, int rank, int splits);
 int fk_latent_attn(const void* q, int64_t q_pitch, const void* cache, int64_t num_blocks,
                    int block_size, int cache_pitch, void* out, int64_t out_pitch,

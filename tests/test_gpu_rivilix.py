@@ -159,7 +159,7 @@ def test_column_groups(rows, groups, n, k, dtype):
     rs = np.random.RandomState(rows + n)
     x = values(rs, rows, groups, k + 8, dtype=dtype)
     w = values(rs, groups, n, k, dtype=dtype) / 8
-    bias = values(rs, n) if groups == 1 else None
+    bias = values(rs, n) if groups != 3 else None
     pitch = (n + 7) // 8 * 8
     want = np.einsum("tgk,gnk->tgn", x[:, :, :k], w) + (bias if bias is not None else 0)
     xd, wd = dev(x.reshape(rows, -1), dtype), dev(w, dtype)
@@ -203,6 +203,28 @@ def test_row_groups(counts, act, dtype):
             got = ops.group_gemm(xs, wd, offsets=i32(off), gather=sd if gather else None, act=act,
                                  expect_rows=expect)
             close(got, z, dtype, scale=np.abs(z).max())
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("rows", [1, 37, 64, 300])
+@pytest.mark.parametrize("ff,bias", [(56, True), (200, False), (333, True)])
+def test_gated_feed_forward(rows, ff, bias, dtype):
+    """Few and many rows; a width of the feed-forward that is no multiple of anything."""
+    from fastkernels_b200.models.feedforward import GatedFeedForward
+    from fastkernels_b200.models.weights import DictSource, Packer
+    rs = np.random.RandomState(rows)
+    width, stride = 88, 128
+    w = {k[len("l0."):]: v for k, v in R.random_weights(
+        R.model_config([R.memory_layer(mlp=R.dense(ff))], width=width), ff).items()
+        if k.startswith("l0.mlp.")}
+    m = GatedFeedForward(ff, bias)
+    m.load(Packer(DictSource({n: torch.from_numpy(a) for n, a in w.items()}), "cuda", dtype, width,
+                  stride), "mlp.")
+    h = values(rs, rows, width, dtype=dtype)
+    y, none = m.forward(dev(padded(h, stride), dtype))
+    want = R.gated(h, w, "mlp.", bias)
+    assert none is None and torch.count_nonzero(y[:, width:]) == 0
+    close(y[:, :width], want, dtype, scale=2 * np.abs(want).max())
 
 
 @pytest.mark.parametrize("rows,experts,top", [(1, 1, 1), (1, 9, 9), (5, 40, 5), (70, 7, 3),
