@@ -383,12 +383,22 @@ __device__ __forceinline__ void ml_load_rows(const uint16_t* src, int64_t stride
                                              int cols, int cols_p, uint16_t* dst, int pitch,
                                              bool vec) {
   if (vec) {
-    const int packs = cols_p >> 3;
-    for (int i = threadIdx.x; i < ML_UNIT * packs; i += blockDim.x) {
-      const int r = i / packs, c = (i - r * packs) * 8;
-      uint4 v = make_uint4(0u, 0u, 0u, 0u);
-      if (r < count && c < cols) v = *reinterpret_cast<const uint4*>(src + r * stride + c);
-      *reinterpret_cast<uint4*>(dst + r * pitch + c) = v;
+    const int packs = cols_p >> 3, total = ML_UNIT * packs;
+    constexpr int UN = 8;                      // loads under way
+    for (int i0 = threadIdx.x; i0 < total; i0 += UN * blockDim.x) {
+      uint4 v[UN];
+#pragma unroll
+      for (int u = 0; u < UN; ++u) {
+        const int i = i0 + u * blockDim.x, r = i / packs, c = (i - r * packs) * 8;
+        v[u] = make_uint4(0u, 0u, 0u, 0u);
+        if (i < total && r < count && c < cols)
+          v[u] = *reinterpret_cast<const uint4*>(src + r * stride + c);
+      }
+#pragma unroll
+      for (int u = 0; u < UN; ++u) {
+        const int i = i0 + u * blockDim.x, r = i / packs, c = (i - r * packs) * 8;
+        if (i < total) *reinterpret_cast<uint4*>(dst + r * pitch + c) = v[u];
+      }
     }
   } else {
     for (int i = threadIdx.x; i < ML_UNIT * cols_p; i += blockDim.x) {
@@ -441,28 +451,37 @@ __global__ void __launch_bounds__(MU_THREADS) mlstm_unit_kernel(const MlstmParam
   const int v0 = blockIdx.x * MU_COLS;
   const uint16_t* kg = static_cast<const uint16_t*>(p.k) + un.t0 * p.in_stride + h * p.dim;
   const uint16_t* vg = static_cast<const uint16_t*>(p.v) + un.t0 * p.in_stride + h * p.vdim + v0;
-  ml_load_rows(kg, p.in_stride, un.count, p.dim, dp, K, kp, p.dim % 8 == 0);
+  // this thread's pieces of v come while the others are brought in
+  constexpr int VN = ML_UNIT * (MU_COLS / 8) / MU_THREADS;
+  const int cols = min(MU_COLS, p.vdim - v0);
+  uint4 vx[VN];
+#pragma unroll
+  for (int j = 0; j < VN; ++j) {
+    const int i = tid + j * MU_THREADS, r = i / (MU_COLS / 8), c = (i % (MU_COLS / 8)) * 8;
+    vx[j] = make_uint4(0u, 0u, 0u, 0u);
+    if (r < un.count && c < cols) {
+      if (p.vdim % 8 == 0) {
+        vx[j] = *reinterpret_cast<const uint4*>(vg + r * p.in_stride + c);
+      } else {
+        uint16_t e[8];
+#pragma unroll
+        for (int x = 0; x < 8; ++x) e[x] = c + x < cols ? vg[r * p.in_stride + c + x] : (uint16_t)0;
+        vx[j] = make_uint4(e[0] | (uint32_t)e[1] << 16, e[2] | (uint32_t)e[3] << 16,
+                           e[4] | (uint32_t)e[5] << 16, e[6] | (uint32_t)e[7] << 16);
+      }
+    }
+  }
   const int64_t at = (int64_t)h * p.units * ML_UNIT + u * ML_UNIT;
   if (tid < ML_UNIT)
     cs[tid] = expf(p.gg[at + ML_UNIT - 1] - p.gg[at + tid] + p.gi[at + tid] -
                    p.gm[at + ML_UNIT - 1]);
+  ml_load_rows(kg, p.in_stride, un.count, p.dim, dp, K, kp, p.dim % 8 == 0);
   __syncthreads();
-  const int cols = min(MU_COLS, p.vdim - v0);
-  for (int i = tid; i < ML_UNIT * (MU_COLS / 8); i += MU_THREADS) {
-    const int r = i / (MU_COLS / 8), c = (i % (MU_COLS / 8)) * 8;
-    uint4 x = make_uint4(0u, 0u, 0u, 0u);
-    if (r < un.count && c < cols) {
-      if (p.vdim % 8 == 0) {
-        x = *reinterpret_cast<const uint4*>(vg + r * p.in_stride + c);
-      } else {
-        uint16_t e[8];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) e[j] = c + j < cols ? vg[r * p.in_stride + c + j] : (uint16_t)0;
-        x = make_uint4(e[0] | (uint32_t)e[1] << 16, e[2] | (uint32_t)e[3] << 16,
-                       e[4] | (uint32_t)e[5] << 16, e[6] | (uint32_t)e[7] << 16);
-      }
-    }
+  for (int j = 0; j < VN; ++j) {
+    const int i = tid + j * MU_THREADS, r = i / (MU_COLS / 8), c = (i % (MU_COLS / 8)) * 8;
     const float k = cs[r];
+    const uint4 x = vx[j];
     uint4 hi, lo;
     split_bf16(bf16lo(x.x) * k, bf16hi(x.x) * k, &hi.x, &lo.x);
     split_bf16(bf16lo(x.y) * k, bf16hi(x.y) * k, &hi.y, &lo.y);
@@ -475,8 +494,9 @@ __global__ void __launch_bounds__(MU_THREADS) mlstm_unit_kernel(const MlstmParam
   float* inc = p.inc + (u * p.heads + h) * p.dim * p.vp;
   if (blockIdx.x == 0)
     for (int r = tid; r < p.dim; r += MU_THREADS) {
-      float s = 0.f;
-      for (int t = 0; t < un.count; ++t) s = fmaf(cs[t], bf16_bits_to_float(K[t * kp + r]), s);
+      float s = 0.f;                              // rows beyond the count are zeros
+#pragma unroll 16
+      for (int t = 0; t < ML_UNIT; ++t) s = fmaf(cs[t], bf16_bits_to_float(K[t * kp + r]), s);
       p.ninc[(u * p.heads + h) * p.dim + r] = s;
     }
   const int gr = lane >> 2, tq = lane & 3;
@@ -661,13 +681,23 @@ __global__ void __launch_bounds__(MO_THREADS, 2) mlstm_output_kernel(const Mlstm
     __syncthreads();
     ml_load_rows(vg + v0, p.in_stride, un.count, cols, MO_COLS, V, vpit,
                  p.vdim % 8 == 0);
-    for (int i = tid; i < dp * (MO_COLS / 4); i += MO_THREADS) {
-      const int r = i / (MO_COLS / 4), c = (i % (MO_COLS / 4)) * 4;
-      uint4 x = make_uint4(0u, 0u, 0u, 0u);
-      if (r < p.dim && v0 + c < p.vp)
-        x = *reinterpret_cast<const uint4*>(st + ((int64_t)r * p.vp + v0 + c) / 2);
-      *reinterpret_cast<uint2*>(Sh + r * vpit + c) = make_uint2(x.x, x.y);
-      *reinterpret_cast<uint2*>(Sl + r * vpit + c) = make_uint2(x.z, x.w);
+    constexpr int SN = 4;                      // loads under way
+    for (int i0 = tid; i0 < dp * (MO_COLS / 4); i0 += SN * MO_THREADS) {
+      uint4 x[SN];
+#pragma unroll
+      for (int j = 0; j < SN; ++j) {
+        const int i = i0 + j * MO_THREADS, r = i / (MO_COLS / 4), c = (i % (MO_COLS / 4)) * 4;
+        x[j] = make_uint4(0u, 0u, 0u, 0u);
+        if (r < p.dim && v0 + c < p.vp)
+          x[j] = *reinterpret_cast<const uint4*>(st + ((int64_t)r * p.vp + v0 + c) / 2);
+      }
+#pragma unroll
+      for (int j = 0; j < SN; ++j) {
+        const int i = i0 + j * MO_THREADS, r = i / (MO_COLS / 4), c = (i % (MO_COLS / 4)) * 4;
+        if (r >= dp) continue;
+        *reinterpret_cast<uint2*>(Sh + r * vpit + c) = make_uint2(x[j].x, x[j].y);
+        *reinterpret_cast<uint2*>(Sl + r * vpit + c) = make_uint2(x[j].z, x[j].w);
+      }
     }
     __syncthreads();
     constexpr int NT = MO_COLS / 8;
